@@ -10,6 +10,7 @@ way the reference's ``check_and_update_config`` does
 from __future__ import annotations
 
 import json
+import math
 import os
 from dataclasses import dataclass, field, asdict
 from typing import Any, Optional
@@ -29,9 +30,61 @@ def parse_dtype(d) -> torch.dtype:
     return _DTYPES[str(d).replace("torch.", "")]
 
 
+@dataclass(frozen=True)
+class RotarySpec:
+    """Rotary embedding of one mixer: the first ``dims`` dimensions of the rotated vector turn by
+    ``position * base^(-2i / dims)``, optionally with YaRN ``scaling`` ({factor, original, fast, slow})."""
+    dims: int
+    base: float
+    scaling: Optional[dict] = None
+
+    @property
+    def rope_scaling(self) -> Optional[dict]:
+        """The same scaling under the names ``ops.reference.rope_inv_freq`` reads."""
+        if not self.scaling:
+            return None
+        s = self.scaling
+        return {"rope_type": "yarn", "factor": float(s["factor"]),
+                "original_max_position_embeddings": float(s["original"]), "beta_fast": float(s["fast"]),
+                "beta_slow": float(s["slow"]), "attention_factor": 0.1 * math.log(float(s["factor"])) + 1.0}
+
+
+@dataclass(frozen=True)
+class LatentMixerSpec:
+    """Sizes of one latent-attention mixer (multi-head latent attention with a query latent)."""
+    heads: int
+    dim: int                             # unrotated query / key dimensions per head
+    rot_dim: int                         # rotated ones (the key's are shared by all heads)
+    vdim: int
+    q_rank: int
+    kv_rank: int
+    scale: float
+    rot: RotarySpec
+    kv_from: Optional[int] = None        # layer whose cached latent and rotated key this layer reads
+    output_gate: bool = True             # heads times sigmoid(W_g x) in front of the output projection
+
+    @staticmethod
+    def from_dict(d: dict) -> "LatentMixerSpec":
+        r = d["rot"]
+        rot = RotarySpec(int(r["dims"]), float(r["base"]), r.get("scaling") or None)
+        src = d.get("kv_from")
+        if rot.dims > d["rot_dim"] or rot.dims % 2:
+            raise ValueError(f"rot.dims {rot.dims} must be even and at most rot_dim {d['rot_dim']}")
+        return LatentMixerSpec(int(d["heads"]), int(d["dim"]), int(d["rot_dim"]), int(d["vdim"]), int(d["q_rank"]),
+                               int(d["kv_rank"]), float(d["scale"]), rot, None if src is None else int(src))
+
+
+@dataclass(frozen=True)
+class LayerSpec:
+    """One entry of a checkpoint configuration that lists its layers one by one."""
+    mixer: LatentMixerSpec
+    ff: int = 0                          # width of the dense feed-forward, 0 = the layer has none
+    act: str = "gelu"
+
+
 @dataclass
 class ModelConfig:
-    architecture: str = "llama"          # llama | qwen3_moe | deepseek_v3 | qwen3_next
+    architecture: str = "llama"          # llama | qwen3_moe | gpt_oss | deepseek_v3 | qwen3_next | kimi_linear | mazivik
     name: str = "tiny-llama"
     num_layers: int = 2
     hidden_size: int = 256
@@ -78,6 +131,8 @@ class ModelConfig:
     qk_rope_head_dim: int = 0
     v_head_dim: int = 0
     mla_use_nope: bool = False           # latent attention without rotary embeddings (Kimi-Linear: positions come from the KDA layers)
+    layer_specs: tuple = ()              # models configured layer by layer (LayerSpec); the scalars above are maxima
+    final_logit_softcap: Optional[float] = None    # logits = cap * tanh(logits / cap)
     # sparse MLA (DSA indexer)
     index_topk: int = 0
     index_n_heads: int = 0
@@ -130,7 +185,13 @@ class ModelConfig:
     def num_params(self) -> int:
         h, L = self.hidden_size, self.num_layers
         n = 2 * self.vocab_size * h if not self.tie_word_embeddings else self.vocab_size * h
-        for i in range(L):
+        for s in self.layer_specs:
+            m = s.mixer
+            n += h * m.q_rank + m.q_rank * m.heads * (m.dim + m.rot_dim) + m.kv_rank * m.heads * (m.dim + m.vdim)
+            n += m.heads * m.vdim * h * (2 if m.output_gate else 1) + 2 * h * s.ff
+            if m.kv_from is None:
+                n += h * (m.kv_rank + m.rot_dim)
+        for i in range(0 if self.layer_specs else L):
             if self.is_mla:
                 qk = self.qk_nope_head_dim + self.qk_rope_head_dim
                 n += h * self.q_lora_rank + self.q_lora_rank * self.num_q_heads * qk if self.q_lora_rank else h * self.num_q_heads * qk
@@ -150,6 +211,8 @@ class ModelConfig:
     @staticmethod
     def from_hf_dict(cfg: dict, name: str = "") -> "ModelConfig":
         """Map a Hugging Face ``config.json`` dictionary to ModelConfig."""
+        if "architectures" not in cfg and cfg.get("architecture") == "Mazivik":
+            return ModelConfig.from_layer_list(cfg, name)
         arch = (cfg.get("architectures") or ["LlamaForCausalLM"])[0]
         mc = ModelConfig(name=name or cfg.get("_name_or_path", arch))
         mc.num_layers = cfg["num_hidden_layers"]
@@ -302,6 +365,46 @@ class ModelConfig:
         return mc
 
     @staticmethod
+    def from_layer_list(cfg: dict, name: str = "") -> "ModelConfig":
+        """Map a ``config.json`` that lists its layers one by one (``{"architecture": "Mazivik", "layers": [...],
+        "norm": {"eps"}, "vocab", "width", "logit_softcap"}``) to ModelConfig."""
+        specs = []
+        for i, layer in enumerate(cfg["layers"]):
+            if layer["type"] != "latent_attention":
+                raise ValueError(f"layer {i}: unknown mixer type {layer['type']!r}")
+            mlp = layer.get("mlp")
+            if mlp and mlp.get("kind") != "dense":
+                raise ValueError(f"layer {i}: unknown feed-forward kind {mlp.get('kind')!r}")
+            m = LatentMixerSpec.from_dict(layer["mixer"])
+            if m.kv_from is not None:
+                src = specs[m.kv_from].mixer if 0 <= m.kv_from < i else None
+                if src is None or src.kv_from is not None:
+                    raise ValueError(f"layer {i}: kv_from {m.kv_from} must name an earlier layer with a latent of its own")
+                if (src.kv_rank, src.rot_dim, src.rot) != (m.kv_rank, m.rot_dim, m.rot):
+                    raise ValueError(f"layer {i}: kv_rank, rot_dim and rotation differ from layer {m.kv_from}'s")
+            specs.append(LayerSpec(m, int(mlp["ff"]) if mlp else 0))
+        mixers = [s.mixer for s in specs]
+        mc = ModelConfig(architecture="mazivik", name=name or "mazivik", num_layers=len(specs),
+                         hidden_size=int(cfg["width"]), vocab_size=int(cfg["vocab"]), layer_specs=tuple(specs))
+        mc.num_q_heads = mc.num_kv_heads = max(m.heads for m in mixers)
+        mc.head_dim = max(m.dim + m.rot_dim for m in mixers)
+        mc.q_lora_rank, mc.kv_lora_rank = max(m.q_rank for m in mixers), max(m.kv_rank for m in mixers)
+        mc.qk_nope_head_dim, mc.qk_rope_head_dim = max(m.dim for m in mixers), max(m.rot_dim for m in mixers)
+        mc.v_head_dim = max(m.vdim for m in mixers)
+        mc.intermediate_size = max(s.ff for s in specs)
+        mc.hidden_act = "gelu"
+        mc.rms_norm_eps = float(cfg["norm"]["eps"])
+        mc.rope_theta, mc.rope_interleaved = mixers[0].rot.base, True
+        mc.rope_scaling = mixers[0].rot.rope_scaling
+        cap = cfg.get("logit_softcap")
+        mc.final_logit_softcap = float(cap) if cap else None
+        mc.dtype = parse_dtype(cfg.get("torch_dtype", "bfloat16"))
+        # nothing in the configuration bounds a sequence: the range the rotation was scaled for is the default
+        spans = [m.rot.scaling["original"] * m.rot.scaling["factor"] for m in mixers if m.rot.scaling]
+        mc.max_model_len = int(max(spans)) if spans else 4096
+        return mc
+
+    @staticmethod
     def from_pretrained(path: str) -> "ModelConfig":
         with open(os.path.join(path, "config.json")) as f:
             return ModelConfig.from_hf_dict(json.load(f), name=os.path.basename(path.rstrip("/")))
@@ -341,6 +444,20 @@ def model_preset(name: str) -> ModelConfig:
                        moe_n_group=2, moe_topk_group=1, moe_routed_scaling=2.5,
                        q_lora_rank=96, kv_lora_rank=64, qk_nope_head_dim=32, qk_rope_head_dim=16,
                        v_head_dim=32, rope_interleaved=True, max_model_len=256)
+    if n in ("tiny-mazivik",):
+        # two latents of which the first serves two layers, unequal layers, one without a feed-forward
+        rot = {"base": 10000.0, "dims": 16, "scaling": {"factor": 2.0, "original": 64, "fast": 16.0, "slow": 1.0}}
+        mix = {"heads": 3, "dim": 24, "rot_dim": 16, "vdim": 40, "q_rank": 48, "kv_rank": 56, "scale": 0.17, "rot": rot}
+        ff = {"kind": "dense", "ff": 144}
+        mc = ModelConfig.from_layer_list({
+            "architecture": "Mazivik", "width": 112, "vocab": 320, "norm": {"eps": 1e-5}, "logit_softcap": 20.0,
+            "torch_dtype": "float32", "layers": [
+                {"type": "latent_attention", "mixer": mix, "mlp": ff},
+                {"type": "latent_attention", "mixer": dict(mix, heads=5, vdim=24, q_rank=32, kv_from=0), "mlp": None},
+                {"type": "latent_attention", "mixer": dict(mix, heads=2, dim=40, kv_rank=72), "mlp": ff}]},
+            name="tiny-mazivik")
+        mc.max_model_len, mc.init_std = 256, 0.1
+        return mc
     if n in ("tiny-odd-heads",):
         return _preset(name="tiny-odd-heads", dtype=torch.float32, num_q_heads=3, num_kv_heads=1, head_dim=64,
                        hidden_size=256, max_model_len=256)

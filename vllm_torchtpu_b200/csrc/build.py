@@ -71,13 +71,42 @@ def _headers_mtime() -> float:
     return max(hs) if hs else 0.0
 
 
-def build(verbose: bool = False, force: bool = False, extra_flags: tuple = ()) -> str:
+# sources whose kernels a model family launches on one GPU (families not listed need the full library)
+FAMILY_SOURCES = {
+    "mazivik": ("attention_mla.cu", "elementwise.cu", "gemm_2sm_tcgen05.cu", "gemm_simt.cu", "gemm_tcgen05.cu",
+                "layer_norm.cu", "runtime.cu", "sample.cu"),
+}
+
+
+def _fresh(lib: str, sources) -> bool:
+    newest = max([_headers_mtime()] + [os.path.getmtime(os.path.join(HERE, s)) for s in sources])
+    return os.path.exists(lib) and os.path.getmtime(lib) >= newest
+
+
+def ensure_built(architecture: str) -> str:
+    """Path of a library with the kernels of this model family: the full one when it is up to date, otherwise one
+    made of the family's sources only (objects are shared with the full build).  Safe to call from several
+    processes."""
+    import fcntl
+    if _fresh(lib_path(), _sources()):
+        return lib_path()
+    sources = FAMILY_SOURCES.get(architecture)
+    os.makedirs(os.path.join(HERE, "build"), exist_ok=True)
+    with open(os.path.join(HERE, "build", ".lock"), "w") as lock:
+        fcntl.flock(lock, fcntl.LOCK_EX)
+        if sources is None:
+            return build()
+        out = os.path.join(HERE, f"libb200_kernels_{architecture}.so")
+        return out if _fresh(out, sources) else build(sources=sources, out=out)
+
+
+def build(verbose: bool = False, force: bool = False, extra_flags: tuple = (), sources=None, out=None) -> str:
     objdir = os.path.join(HERE, "build")
     os.makedirs(objdir, exist_ok=True)
     hdr = _headers_mtime()
     jobs = []
     objs = []
-    for src in _sources():
+    for src in sources or _sources():
         obj = os.path.join(objdir, os.path.splitext(src)[0] + ".o")
         objs.append(obj)
         sp = os.path.join(HERE, src)
@@ -99,8 +128,8 @@ def build(verbose: bool = False, force: bool = False, extra_flags: tuple = ()) -
             failed |= r.returncode != 0
     if failed:
         raise RuntimeError("nvcc failed")
-    out = lib_path()
-    if jobs or not os.path.exists(out):
+    out = out or lib_path()
+    if jobs or not _fresh(out, sources or _sources()):
         cmd = [NVCC, *ARCH, "-shared", "-o", out, *objs, "-lcudart_static", "-lpthread", "-ldl", "-lrt"]
         r = subprocess.run(cmd, capture_output=True, text=True)
         if r.returncode != 0:

@@ -377,6 +377,8 @@ __device__ __forceinline__ T warp_max(T v) {
   return v;
 }
 
+__device__ __forceinline__ float gelu_erf(float v) { return 0.5f * v * (1.f + erff(v * 0.70710678118654752f)); }
+
 struct alignas(16) bf16x8 {
   __nv_bfloat162 v[4];
 };

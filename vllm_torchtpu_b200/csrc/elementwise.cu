@@ -126,9 +126,11 @@ __global__ void gated_act_kernel(const __nv_bfloat16* __restrict__ x, __nv_bfloa
 }
 
 // out[t] = table[ token_src[t] >= 0 ? last_tokens[token_src[t]] : ids[t] ]
+// (rows of n pieces of type V: 16 bytes, or 2 where a row is no multiple of that)
+template <typename V>
 __global__ void embedding_kernel(const int* __restrict__ ids, const int* __restrict__ token_src,
-                                 const int* __restrict__ last_tokens, const __nv_bfloat16* __restrict__ table,
-                                 __nv_bfloat16* __restrict__ out, int H, int vocab) {
+                                 const int* __restrict__ last_tokens, const V* __restrict__ table,
+                                 V* __restrict__ out, int n, int vocab) {
   const int t = blockIdx.x;
   int id = ids[t];
   if (token_src != nullptr) {
@@ -136,25 +138,25 @@ __global__ void embedding_kernel(const int* __restrict__ ids, const int* __restr
     if (src >= 0) id = last_tokens[src];
   }
   id = min(max(id, 0), vocab - 1);
-  const bf16x8* srcp = reinterpret_cast<const bf16x8*>(table + (size_t)id * H);
-  bf16x8* dst = reinterpret_cast<bf16x8*>(out + (size_t)t * H);
-  for (int i = threadIdx.x; i < (H >> 3); i += blockDim.x) dst[i] = srcp[i];
+  const V* srcp = table + (size_t)id * n;
+  V* dst = out + (size_t)t * n;
+  for (int i = threadIdx.x; i < n; i += blockDim.x) dst[i] = srcp[i];
 }
 
 // out_h[r] = hidden[idx[r]], out_r[r] = residual[idx[r]]
-__global__ void gather_rows_kernel(const __nv_bfloat16* __restrict__ hidden,
-                                   const __nv_bfloat16* __restrict__ residual, const int* __restrict__ idx,
-                                   __nv_bfloat16* __restrict__ out_h, __nv_bfloat16* __restrict__ out_r, int H,
+template <typename V>
+__global__ void gather_rows_kernel(const V* __restrict__ hidden, const V* __restrict__ residual,
+                                   const int* __restrict__ idx, V* __restrict__ out_h, V* __restrict__ out_r, int n,
                                    int T) {
   const int r = blockIdx.x;
   const int t = min(max(idx[r], 0), T - 1);
-  const bf16x8* h = reinterpret_cast<const bf16x8*>(hidden + (size_t)t * H);
-  bf16x8* oh = reinterpret_cast<bf16x8*>(out_h + (size_t)r * H);
-  for (int i = threadIdx.x; i < (H >> 3); i += blockDim.x) oh[i] = h[i];
+  const V* h = hidden + (size_t)t * n;
+  V* oh = out_h + (size_t)r * n;
+  for (int i = threadIdx.x; i < n; i += blockDim.x) oh[i] = h[i];
   if (residual != nullptr) {
-    const bf16x8* rr = reinterpret_cast<const bf16x8*>(residual + (size_t)t * H);
-    bf16x8* orr = reinterpret_cast<bf16x8*>(out_r + (size_t)r * H);
-    for (int i = threadIdx.x; i < (H >> 3); i += blockDim.x) orr[i] = rr[i];
+    const V* rr = residual + (size_t)t * n;
+    V* orr = out_r + (size_t)r * n;
+    for (int i = threadIdx.x; i < n; i += blockDim.x) orr[i] = rr[i];
   }
 }
 
@@ -324,20 +326,30 @@ extern "C" int b200_gated_act(const void* x, void* y, int T, int I, int act, flo
   return 0;
 }
 
+// rows of row_bytes bytes (a multiple of 2)
 extern "C" int b200_embedding(const int* ids, const int* token_src, const int* last_tokens, const void* table,
-                              void* out, int T, int H, int vocab, cudaStream_t stream) {
+                              void* out, int T, int row_bytes, int vocab, cudaStream_t stream) {
   if (T == 0) return 0;
-  embedding_kernel<<<T, 128, 0, stream>>>(ids, token_src, last_tokens, (const __nv_bfloat16*)table,
-                                          (__nv_bfloat16*)out, H, vocab);
+  if (row_bytes % 16 == 0 && (((uintptr_t)table | (uintptr_t)out) & 15) == 0)
+    embedding_kernel<uint4><<<T, 128, 0, stream>>>(ids, token_src, last_tokens, (const uint4*)table, (uint4*)out,
+                                                   row_bytes / 16, vocab);
+  else
+    embedding_kernel<uint16_t><<<T, 128, 0, stream>>>(ids, token_src, last_tokens, (const uint16_t*)table,
+                                                      (uint16_t*)out, row_bytes / 2, vocab);
   B200_CUDA_CHECK(cudaGetLastError());
   return 0;
 }
 
 extern "C" int b200_gather_rows(const void* hidden, const void* residual, const int* idx, void* out_h,
-                                void* out_r, int R, int H, int T, cudaStream_t stream) {
+                                void* out_r, int R, int row_bytes, int T, cudaStream_t stream) {
   if (R == 0) return 0;
-  gather_rows_kernel<<<R, 128, 0, stream>>>((const __nv_bfloat16*)hidden, (const __nv_bfloat16*)residual, idx,
-                                            (__nv_bfloat16*)out_h, (__nv_bfloat16*)out_r, H, T);
+  const uintptr_t a = (uintptr_t)hidden | (uintptr_t)residual | (uintptr_t)out_h | (uintptr_t)out_r;
+  if (row_bytes % 16 == 0 && (a & 15) == 0)
+    gather_rows_kernel<uint4><<<R, 128, 0, stream>>>((const uint4*)hidden, (const uint4*)residual, idx, (uint4*)out_h,
+                                                     (uint4*)out_r, row_bytes / 16, T);
+  else
+    gather_rows_kernel<uint16_t><<<R, 128, 0, stream>>>((const uint16_t*)hidden, (const uint16_t*)residual, idx,
+                                                        (uint16_t*)out_h, (uint16_t*)out_r, row_bytes / 2, T);
   B200_CUDA_CHECK(cudaGetLastError());
   return 0;
 }

@@ -120,10 +120,12 @@ __device__ __forceinline__ void decode_work(int w, const Params& p, int& n_pair,
   n_pair = first + rem - t_tile * gsize;
 }
 
-template <bool SWIGLU>
+// EPI 0: bias, 1: SwiGLU, 2: gelu (erf)
+template <int EPI>
 __global__ void __cluster_dims__(2, 1, 1) __launch_bounds__(THREADS, 1)
 gemm_bf16_2sm_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant__ CUtensorMap tmX,
                      const Params p) {
+  constexpr bool SWIGLU = EPI == 1;
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
   uint64_t* bars = reinterpret_cast<uint64_t*>(smem + STAGES * STAGE_BYTES);
@@ -308,7 +310,10 @@ gemm_bf16_2sm_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_const
           __nv_bfloat16* yp = p.Y + (size_t)(t0 + c0) * p.ldy + n;
 #pragma unroll
           for (int j = 0; j < 32; ++j)
-            if (c0 + j < t_valid) yp[(size_t)j * p.ldy] = __float2bfloat16(__uint_as_float(r[j]) + bias);
+            if (c0 + j < t_valid) {
+              const float v = __uint_as_float(r[j]) + bias;
+              yp[(size_t)j * p.ldy] = __float2bfloat16(EPI == 2 ? gelu_erf(v) : v);
+            }
         }
       }
       tc_fence_before();
@@ -375,19 +380,19 @@ static int operand_map(CUtensorMap* out, const void* ptr, uint64_t rows, uint64_
 
 // persistent grid: exactly as many SM pairs as can be resident at once (a cluster needs both SMs of a
 // pair, so this can be fewer than num_sms / 2)
-template <bool SWIGLU>
+template <int EPI>
 static int launch_pairs(const CUtensorMap& tmW, const CUtensorMap& tmX, const Params& p, int num_sms,
                         cudaStream_t stream) {
   static int max_pairs = 0;
   static unsigned long long attr_seen = 0;
-  B200_CUDA_CHECK(ensure_dynamic_smem(gemm_bf16_2sm_kernel<SWIGLU>, SMEM, &attr_seen));
+  B200_CUDA_CHECK(ensure_dynamic_smem(gemm_bf16_2sm_kernel<EPI>, SMEM, &attr_seen));
   if (max_pairs == 0) {
     cudaLaunchConfig_t cfg = {};
     cfg.gridDim = dim3(2 * (num_sms / 2));
     cfg.blockDim = dim3(THREADS);
     cfg.dynamicSmemBytes = SMEM;
     int n = 0;
-    if (cudaOccupancyMaxActiveClusters(&n, gemm_bf16_2sm_kernel<SWIGLU>, &cfg) != cudaSuccess || n < 1) {
+    if (cudaOccupancyMaxActiveClusters(&n, gemm_bf16_2sm_kernel<EPI>, &cfg) != cudaSuccess || n < 1) {
       cudaGetLastError();
       n = num_sms / 2;
     }
@@ -397,7 +402,7 @@ static int launch_pairs(const CUtensorMap& tmW, const CUtensorMap& tmX, const Pa
   int pairs = max_pairs < num_sms / 2 ? max_pairs : num_sms / 2;
   if (pairs > total) pairs = total;
   if (pairs < 1) pairs = 1;
-  B200_CUDA_CHECK(launch_pdl(gemm_bf16_2sm_kernel<SWIGLU>, dim3(2 * pairs), dim3(THREADS), SMEM, stream, tmW, tmX,
+  B200_CUDA_CHECK(launch_pdl(gemm_bf16_2sm_kernel<EPI>, dim3(2 * pairs), dim3(THREADS), SMEM, stream, tmW, tmX,
                              p));
   B200_CUDA_CHECK(cudaGetLastError());
   return 0;
@@ -408,8 +413,9 @@ static int launch_pairs(const CUtensorMap& tmW, const CUtensorMap& tmX, const Pa
 
 // X [T,K] row stride ldx, W [N,K] row stride ldw, Y [T,N] row stride ldy (elements); status: device int
 // that receives a time-out code (common.cuh) if a wait inside the kernel gives up.
-extern "C" int b200_gemm_bf16_2sm(const void* X, const void* W, void* Y, const void* bias, int T, int N, int K,
-                                  int ldx, int ldw, int ldy, int* status, int num_sms, cudaStream_t stream) {
+static int gemm_bf16_2sm(const void* X, const void* W, void* Y, const void* bias, int T, int N, int K,
+                         int ldx, int ldw, int ldy, int* status, int num_sms, int act,
+                         cudaStream_t stream) {
   using namespace b200;
   using namespace b200::g2;
   if (T <= 0 || N <= 0 || K <= 0) return 0;
@@ -431,7 +437,17 @@ extern "C" int b200_gemm_bf16_2sm(const void* X, const void* W, void* Y, const v
   if (rc) return rc;
   rc = operand_map(&tmX, X, (uint64_t)T, (uint64_t)K, (uint64_t)ldx * 2);
   if (rc) return rc;
-  return launch_pairs<false>(tmW, tmX, p, num_sms, stream);
+  return act == 1 ? launch_pairs<2>(tmW, tmX, p, num_sms, stream) : launch_pairs<0>(tmW, tmX, p, num_sms, stream);
+}
+
+extern "C" int b200_gemm_bf16_2sm(const void* X, const void* W, void* Y, const void* bias, int T, int N, int K,
+                                  int ldx, int ldw, int ldy, int* status, int num_sms, cudaStream_t stream) {
+  return gemm_bf16_2sm(X, W, Y, bias, T, N, K, ldx, ldw, ldy, status, num_sms, 0, stream);
+}
+// Y = gelu(X * W^T), gelu in its erf form
+extern "C" int b200_gemm_bf16_gelu_2sm(const void* X, const void* W, void* Y, int T, int N, int K, int ldx, int ldw,
+                                       int ldy, int* status, int num_sms, cudaStream_t stream) {
+  return gemm_bf16_2sm(X, W, Y, nullptr, T, N, K, ldx, ldw, ldy, status, num_sms, 1, stream);
 }
 
 // Y[T, I] = silu(X * W[0:I]^T) * (X * W[I:2I]^T); W [2I, K] row stride ldw.
@@ -458,5 +474,5 @@ extern "C" int b200_gemm_bf16_swiglu_2sm(const void* X, const void* W, void* Y, 
   if (rc) return rc;
   rc = operand_map(&tmX, X, (uint64_t)T, (uint64_t)K, (uint64_t)ldx * 2);
   if (rc) return rc;
-  return launch_pairs<true>(tmW, tmX, p, num_sms, stream);
+  return launch_pairs<1>(tmW, tmX, p, num_sms, stream);
 }

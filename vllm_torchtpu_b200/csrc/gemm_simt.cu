@@ -1,0 +1,102 @@
+// CUDA-core GEMM for what the tensor-core kernels do not take: 32-bit activations and weights (full fp32
+// products and sums, no reduced-precision mode), and bf16 operands whose sizes or strides are no multiple of
+// the TMA granule.  Batched over heads, with the epilogues the tcgen05 kernels have:
+//
+//   Y[t, b * ys + n] = act( sum_k X[t, b * xs + k] * W[b * N + n, k] + bias[n] ) [ * sigmoid(G[t, b * N + n]) ]
+//
+// act: 0 none, 1 gelu (erf).  64 x 64 output tile per CTA, 4 x 4 per thread, 16-wide K slices in shared memory.
+#include "common.cuh"
+
+namespace b200 {
+namespace simt {
+
+__device__ __forceinline__ float to_f(float v) { return v; }
+__device__ __forceinline__ float to_f(__nv_bfloat16 v) { return __bfloat162float(v); }
+template <typename T> __device__ __forceinline__ T from_f(float v);
+template <> __device__ __forceinline__ float from_f<float>(float v) { return v; }
+template <> __device__ __forceinline__ __nv_bfloat16 from_f<__nv_bfloat16>(float v) { return __float2bfloat16(v); }
+
+struct Params {
+  const void *x, *w, *bias, *gate;
+  void* y;
+  int T, N, K, batch, act;
+  long long ldx, ldw, ldy, ldg, xs, ys;
+};
+
+constexpr int TM = 64, TN = 64, TK = 16;
+
+template <typename E>
+__global__ void __launch_bounds__(256) gemm_kernel(const Params p) {
+  __shared__ float sx[TK][TM + 4];
+  __shared__ float sw[TK][TN + 4];
+  pdl_launch_dependents();
+  pdl_wait();
+  const int n_tiles = (p.N + TN - 1) / TN;
+  const int b = blockIdx.x / n_tiles, n0 = (blockIdx.x - b * n_tiles) * TN;
+  const int tx = threadIdx.x & 15, ty = threadIdx.x >> 4;
+  const E* w = reinterpret_cast<const E*>(p.w) + (size_t)b * p.N * p.ldw;
+  for (int t0 = blockIdx.y * TM; t0 < p.T; t0 += gridDim.y * TM) {
+    const E* x = reinterpret_cast<const E*>(p.x) + (size_t)b * p.xs;
+    float acc[4][4] = {};
+    for (int k0 = 0; k0 < p.K; k0 += TK) {
+#pragma unroll
+      for (int i = 0; i < TM * TK / 256; ++i) {
+        const int idx = threadIdx.x + i * 256, k = idx & (TK - 1), r = idx / TK;
+        const bool kin = k0 + k < p.K;
+        sx[k][r] = (kin && t0 + r < p.T) ? to_f(x[(size_t)(t0 + r) * p.ldx + k0 + k]) : 0.f;
+        sw[k][r] = (kin && n0 + r < p.N) ? to_f(w[(size_t)(n0 + r) * p.ldw + k0 + k]) : 0.f;
+      }
+      __syncthreads();
+#pragma unroll
+      for (int k = 0; k < TK; ++k) {
+        const float4 a = *reinterpret_cast<const float4*>(&sx[k][ty * 4]);
+        const float4 c = *reinterpret_cast<const float4*>(&sw[k][tx * 4]);
+        const float av[4] = {a.x, a.y, a.z, a.w}, cv[4] = {c.x, c.y, c.z, c.w};
+#pragma unroll
+        for (int i = 0; i < 4; ++i)
+#pragma unroll
+          for (int j = 0; j < 4; ++j) acc[i][j] = fmaf(av[i], cv[j], acc[i][j]);
+      }
+      __syncthreads();
+    }
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+      const int t = t0 + ty * 4 + i;
+      if (t >= p.T) continue;
+#pragma unroll
+      for (int j = 0; j < 4; ++j) {
+        const int n = n0 + tx * 4 + j;
+        if (n >= p.N) continue;
+        float v = acc[i][j];
+        if (p.bias) v += to_f(reinterpret_cast<const E*>(p.bias)[n]);
+        if (p.act == 1) v = gelu_erf(v);
+        if (p.gate) {
+          const float g = to_f(reinterpret_cast<const E*>(p.gate)[(size_t)t * p.ldg + (size_t)b * p.N + n]);
+          v *= 1.f / (1.f + expf(-g));
+        }
+        reinterpret_cast<E*>(p.y)[(size_t)t * p.ldy + (size_t)b * p.ys + n] = from_f<E>(v);
+      }
+    }
+  }
+}
+
+}  // namespace simt
+}  // namespace b200
+
+// elem: 2 = bf16, 4 = fp32 (all operands alike); strides in elements.
+extern "C" int b200_gemm_simt(const void* x, const void* w, void* y, const void* bias, const void* gate, int T, int N,
+                              int K, int batch, long long ldx, long long ldw, long long ldy, long long ldg,
+                              long long xs, long long ys, int act, int elem, cudaStream_t stream) {
+  using namespace b200;
+  if (T <= 0 || N <= 0 || batch <= 0) return 0;
+  simt::Params p{x, w, bias, gate, y, T, N, K, batch, act, ldx, ldw, ldy, ldg, xs, ys};
+  const long long gx = (long long)batch * ((N + simt::TN - 1) / simt::TN);
+  int gy = (T + simt::TM - 1) / simt::TM;
+  if (gy > 65535) gy = 65535;
+  const dim3 grid((unsigned)gx, gy);
+  if (elem == 4)
+    B200_CUDA_CHECK(launch_pdl(simt::gemm_kernel<float>, grid, dim3(256), (size_t)0, stream, p));
+  else
+    B200_CUDA_CHECK(launch_pdl(simt::gemm_kernel<__nv_bfloat16>, grid, dim3(256), (size_t)0, stream, p));
+  return 0;
+}

@@ -99,6 +99,11 @@ struct GemmParams {
   unsigned long long ag_done_off;
   int ag_flip;
   unsigned long long* dbg;               // optional: per-CTA phase timestamps (ns), 16 slots per CTA
+  // ---- MODE 3: epilogue (act 0 none / 1 gelu; optional gate: y *= sigmoid(gate[t, b * N + n])) and batch over
+  // heads: head b reads activation columns from b * x_head_cols, weight rows from b * N and writes output
+  // columns from b * y_head_cols
+  int act, batch, x_head_cols, y_head_cols, ldg;
+  const __nv_bfloat16* gate;
   int* epoch_ptr;                        // local: epoch of the last completed fused launch
   int* cta_done;                         // local: CTA exit counter
   unsigned int spin_limit;
@@ -131,6 +136,7 @@ __device__ __forceinline__ void decode_work(int w, const GemmParams& p, int& n_t
 
 struct Work {
   int w_row, t_row, t_valid, n0, kb0, kb1, tile, split;
+  int head;                              // MODE 3 only
 };
 
 // dense: tiles rastered in groups of GROUP_N weight tiles; grouped: work = (token tile of an expert, n tile)
@@ -138,7 +144,18 @@ template <int BN, int MODE = 2>
 __device__ __forceinline__ Work get_work(int w, const GemmParams& p, const int* s_prefix) {
   constexpr bool FULL = MODE == 2;
   Work k;
-  if (!FULL || p.group_off == nullptr) {
+  if (MODE == 3) {
+    const int per = p.n_tiles * p.t_tiles * p.splits;
+    int n_tile, t_tile;
+    k.head = w / per;
+    decode_work(w - k.head * per, p, n_tile, t_tile, k.split, k.tile);
+    k.w_row = k.head * p.N + n_tile * BM;
+    k.n0 = n_tile * BM;
+    k.t_row = t_tile * BN;
+    k.t_valid = min(BN, p.T - k.t_row);
+    k.kb0 = k.split * p.kb_per_split;
+    k.kb1 = min(p.kb_total, k.kb0 + p.kb_per_split);
+  } else if (!FULL || p.group_off == nullptr) {
     int n_tile, t_tile;
     decode_work(w, p, n_tile, t_tile, k.split, k.tile);
     if (FULL && p.ar_mode == 5) {  // start with the token blocks of this rank's own shard
@@ -190,6 +207,9 @@ __device__ __forceinline__ TileDst tile_dst(const GemmParams& p, const Work& wk,
     t.base = reinterpret_cast<__nv_bfloat16*>(p.peer[d] + p.part_off + (size_t)p.rank * p.part_src_stride) +
              (size_t)wk.t_row * p.N + wk.n0;
     t.cs = p.N;
+  } else if (MODE == 3) {
+    t.base = p.Y + (size_t)wk.t_row * p.ldy + (size_t)wk.head * p.y_head_cols + wk.n0;
+    t.cs = p.ldy;
   } else if (!FULL || p.world == 1 || p.ar_mode == 5) {
     t.base = p.Y + (size_t)wk.t_row * p.ldy + wk.n0;
     t.cs = p.ldy;
@@ -324,6 +344,9 @@ __device__ __forceinline__ void cluster_reduce_cols(const GemmParams& p, const W
           a.z = a.z / (1.f + __expf(-a.z)) * u.z;
           a.w = a.w / (1.f + __expf(-a.w)) * u.w;
         }
+        if (MODE == 3 && p.act == 1) {           // (no bias in this mode)
+          a.x = gelu_erf(a.x); a.y = gelu_erf(a.y); a.z = gelu_erf(a.z); a.w = gelu_erf(a.w);
+        }
         for (int d = 0; d < ndst; ++d) {
           const TileDst td = tile_dst<BN, MODE>(p, wk, d);
           __nv_bfloat16* yp = td.base + (size_t)c * td.cs + 4 * lane;
@@ -366,6 +389,7 @@ __device__ __forceinline__ void dbg_stamp(const GemmParams& p, int slot) {
 // misses in the short decode GEMMs even when they are never taken.
 // MODE 1 is the equally compact instantiation of the decode push plane (ar_mode 3): a dense GEMM whose
 // output rows go to every rank's receive slab, flags raised per tile, nothing else.
+// MODE 3 is MODE 0 with the epilogues and the batch over heads described at GemmParams.
 template <int BN, int NACC, int MODE>
 __global__ void __launch_bounds__(MODE == 2 ? NUM_THREADS_FUSED : NUM_THREADS, 1)
 gemm_bf16_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant__ CUtensorMap tmX,
@@ -443,7 +467,7 @@ gemm_bf16_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant_
   tc_fence_after();
   const uint32_t tmem_base = *tmem_slot;
   const int total_work = (FULL && p.group_off != nullptr) ? s_prefix[p.num_groups] * p.n_tiles
-                                                : p.n_tiles * p.t_tiles * p.splits;
+                                                : p.n_tiles * p.t_tiles * p.splits * (MODE == 3 ? p.batch : 1);
   if (threadIdx.x == 0) dbg_stamp(p, 1);
 
   if (warp == 0) {
@@ -490,7 +514,8 @@ gemm_bf16_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant_
           uint8_t* a = smem + s * Cfg::STAGE_BYTES;
           if (issued < npre) {
             // barrier already armed and the weight tile already requested: add the activation tile
-            tma_load_2d(a + NACC * Cfg::A_BYTES, &tmX, &full[s], kb * BK, k.t_row);
+            tma_load_2d(a + NACC * Cfg::A_BYTES, &tmX, &full[s],
+                        kb * BK + (MODE == 3 ? k.head * p.x_head_cols : 0), k.t_row);
             armed |= 1u << s;
             if (++s == STAGES) { s = 0; ph ^= 1; }
             continue;
@@ -505,7 +530,8 @@ gemm_bf16_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant_
             tma_load_2d(a, &tmW, &full[s], kb * BK, k.w_row);
             if (NACC == 2) tma_load_2d(a + Cfg::A_BYTES, &tmW, &full[s], kb * BK, k.w_row + p.up_row_off);
           }
-          tma_load_2d(a + NACC * Cfg::A_BYTES, &tmX, &full[s], kb * BK, k.t_row);
+          tma_load_2d(a + NACC * Cfg::A_BYTES, &tmX, &full[s],
+                      kb * BK + (MODE == 3 ? k.head * p.x_head_cols : 0), k.t_row);
           armed |= 1u << s;
           if (++s == STAGES) { s = 0; ph ^= 1; }
         }
@@ -701,6 +727,27 @@ gemm_bf16_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant_
             for (int d = 0; d < ndst; ++d) {
               const TileDst td = tile_dst<BN, MODE>(p, wk, d);
               __nv_bfloat16* yp = td.base + (size_t)c0 * td.cs + row;
+              if constexpr (MODE == 3) {
+                if (p.gate != nullptr) {
+                  const __nv_bfloat16* gp = p.gate + (size_t)(t0 + c0) * p.ldg + (size_t)wk.head * p.N + n;
+                  float gv[32];
+#pragma unroll
+                  for (int j = 0; j < 32; ++j)
+                    gv[j] = c0 + j < t_valid ? __bfloat162float(gp[(size_t)j * p.ldg]) : 0.f;
+#pragma unroll
+                  for (int j = 0; j < 32; ++j)
+                    if (c0 + j < t_valid)
+                      yp[(size_t)j * td.cs] =
+                          __float2bfloat16(__fdividef(__uint_as_float(r[j]), 1.f + __expf(-gv[j])));
+                  continue;
+                }
+                if (p.act == 1) {
+#pragma unroll
+                  for (int j = 0; j < 32; ++j)
+                    if (c0 + j < t_valid) yp[(size_t)j * td.cs] = __float2bfloat16(gelu_erf(__uint_as_float(r[j])));
+                  continue;
+                }
+              }
 #pragma unroll
               for (int j = 0; j < 32; ++j) {
                 if (c0 + j < t_valid) yp[(size_t)j * td.cs] = __float2bfloat16(__uint_as_float(r[j]) + bias);
@@ -1228,8 +1275,9 @@ static int fit_cluster_splits(int want, int tiles, int bn, int threads) {
 }
 
 // 0: compact kernel (dense single-rank launches without split-K or with cluster split-K),
-// 1: compact push kernel (ar_mode 3), 2: the full kernel
+// 1: compact push kernel (ar_mode 3), 2: the full kernel, 3: epilogue / head-batched kernel
 static int kernel_mode(const GemmParams& p) {
+  if (p.batch > 0) return 3;
   const bool simple = p.group_off == nullptr && p.row_route == nullptr && (p.splits == 1 || p.cluster_splitk);
   if (simple && p.world == 1) return 0;
   if (simple && p.world > 1 && p.ar_mode == 3) return 1;
@@ -1246,6 +1294,7 @@ static int launch_gemm(const CUtensorMap& tmW, const CUtensorMap& tmX, const Gem
   const int mode = kernel_mode(p);
   if (mode == 0) return launch_gemm_v<BN, NACC, 0>(tmW, tmX, p, grid, stream);
   if (mode == 1 && NACC == 1) return launch_gemm_v<BN, 1, 1>(tmW, tmX, p, grid, stream);
+  if (mode == 3 && NACC == 1) return launch_gemm_v<BN, 1, 3>(tmW, tmX, p, grid, stream);
   return launch_gemm_v<BN, NACC, 2>(tmW, tmX, p, grid, stream);
 }
 
@@ -1367,6 +1416,60 @@ extern "C" int b200_gemm_bf16(const void* X, const void* W, void* Y, const void*
   if (rc) return rc;
   int total = tiles * p.splits;
   int grid = p.cluster_splitk ? total : (total < num_sms ? total : num_sms);
+  switch (bn) {
+    case 32: return launch_gemm<32>(tmW, tmX, p, grid, stream);
+    case 64: return launch_gemm<64>(tmW, tmX, p, grid, stream);
+    case 128: return launch_gemm<128>(tmW, tmX, p, grid, stream);
+    default: return launch_gemm<256>(tmW, tmX, p, grid, stream);
+  }
+}
+
+// Y[t, b * ys + n] = act(X[t, b * xs : b * xs + K] . W[b * N + n, :]) [* sigmoid(gate[t, b * N + n])] for b < batch
+// (heads), act 0 none / 1 gelu (erf).  X row stride ldx, W [batch * N, K] row stride ldw, Y row stride ldy.  A head
+// whose K is no multiple of the 64-wide K block reads into its neighbour's columns; those meet the zero fill
+// behind the weight's K columns.
+extern "C" int b200_gemm_bf16_heads(const void* X, const void* W, void* Y, const void* gate, int T, int N, int K,
+                                    int batch, int ldx, int ldw, int ldy, int ldg, int xs, int ys, int act,
+                                    int* status, int num_sms, cudaStream_t stream) {
+  using namespace b200;
+  if (T <= 0 || N <= 0 || K <= 0 || batch <= 0) return 0;
+  if (ldx % 8 || ldw % 8 || xs % 8) {
+    b200_set_last_error("gemm_heads: row and head strides must be multiples of 8 elements", __FILE__, __LINE__);
+    return -3;
+  }
+  GemmParams p;
+  memset(&p, 0, sizeof(p));
+  p.world = 1;
+  p.Y = reinterpret_cast<__nv_bfloat16*>(Y);
+  p.gate = reinterpret_cast<const __nv_bfloat16*>(gate);
+  p.status = status;
+  p.T = T; p.N = N; p.K = K; p.ldy = ldy; p.ldg = ldg;
+  p.batch = batch; p.x_head_cols = xs; p.y_head_cols = ys; p.act = act;
+  int bn, splits, cneed;
+  size_t need;
+  b200_gemm_plan(T, N, K, num_sms, &bn, &splits, &need, &cneed);
+  p.n_tiles = (N + BM - 1) / BM;
+  p.t_tiles = (T + bn - 1) / bn;
+  p.kb_total = (K + BK - 1) / BK;
+  const int tiles = p.n_tiles * p.t_tiles;
+  if (batch > 1 || gate != nullptr) splits = 1;
+  if (splits > p.kb_total) splits = p.kb_total;
+  if (splits > 1) splits = fit_cluster_splits(splits, tiles, bn, NUM_THREADS);
+  p.splits = splits;
+  p.kb_per_split = (p.kb_total + splits - 1) / splits;
+  while (p.splits > 1 && (p.splits - 1) * p.kb_per_split >= p.kb_total) {      // every split owns a K block
+    --p.splits;
+    p.kb_per_split = (p.kb_total + p.splits - 1) / p.splits;
+  }
+  p.w_evict_first = (p.t_tiles == 1) ? 1 : 0;
+  p.cluster_splitk = p.splits > 1 ? 1 : 0;
+  CUtensorMap tmW, tmX;
+  int rc = cached_tmap(&tmW, W, (uint64_t)batch * N, (uint64_t)K, (uint64_t)ldw * 2, BM);
+  if (rc) return rc;
+  rc = cached_tmap(&tmX, X, (uint64_t)T, (uint64_t)(batch - 1) * xs + K, (uint64_t)ldx * 2, (uint32_t)bn);
+  if (rc) return rc;
+  const int total = tiles * p.splits * batch;
+  const int grid = p.cluster_splitk ? total : (total < num_sms ? total : num_sms);
   switch (bn) {
     case 32: return launch_gemm<32>(tmW, tmX, p, grid, stream);
     case 64: return launch_gemm<64>(tmW, tmX, p, grid, stream);

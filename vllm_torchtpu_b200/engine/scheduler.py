@@ -43,6 +43,7 @@ class SchedulerOutput:
     preempted_ids: list
     total_num_tokens: int
     kv_connector_metadata: object = None
+    logit_places: Optional[dict] = None     # request id -> places among its tokens of this step: logits wanted
 
     @property
     def num_reqs(self) -> int:

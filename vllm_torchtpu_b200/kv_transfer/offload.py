@@ -228,7 +228,9 @@ class OffloadWorkerHalf(WorkerConnectorBase):
 
 def create_offloading_connector(cfg, runner, **kw) -> Connector:
     extra = (cfg.kv_transfer or {}).get("kv_connector_extra_config", {})
-    layers = runner.kv_caches
+    layers = runner.distinct_kv_caches
+    if any(l.shape[1:] != layers[0].shape[1:] for l in layers):
+        raise ValueError("KV offload needs cache rows of one width in all layers")
     block_shape = tuple(layers[0].shape[1:])
     per_block = layers[0][0].numel() * layers[0].element_size() * len(layers)
     gb = float(extra.get("dram_gb", envs.B200_OFFLOAD_DRAM_GB or 1.0))

@@ -288,7 +288,10 @@ def create_p2p_connector(cfg, runner, *, transport=None, channel_factory=None) -
     if transport is None:
         kind = extra.get("transport", "ipc" if str(runner.device).startswith("cuda") else "local")
         transport = IpcTransport(engine_id) if kind == "ipc" else LocalTransport(engine_id)
-    transport.register_pool(runner.kv_caches)
+    layers = runner.distinct_kv_caches
+    if geometry is not None and any(l.shape[1:] != first.shape[1:] for l in layers):
+        raise ValueError("KV transfer needs cache rows of one width in all layers")
+    transport.register_pool(layers)
     if channel_factory is None:
         if extra.get("channel", "tcp") == "inproc":
             channel_factory = lambda h: InProcessChannel(engine_id, h)

@@ -147,10 +147,40 @@ def _load_oss_experts(moe, parts: dict) -> None:
             moe.load_expert_bias(e - lo, b[0::2], b[1::2], parts["down_proj_bias"][e])
 
 
+def load_grouped_tensors(model, tensors, names: set, source: str = "memory") -> None:
+    """Models that list their checkpoint tensors themselves (``checkpoint_groups``): every group is handed to its
+    loader once all of its tensors have been read.  A directory must hold exactly the listed tensors; tensors handed
+    over in memory may cover a part of the groups."""
+    of: dict = {}
+    for gid, (members, done) in enumerate(model.checkpoint_groups()):
+        c = _Collector(set(members), lambda parts, members=members, done=done: done(*(parts[m] for m in members)))
+        for m in members:
+            of[m] = (gid, c)
+    unknown = sorted(set(names) - set(of))
+    if unknown:
+        raise ValueError(f"{source}: tensors the model does not have: {unknown[:8]}")
+    open_groups, seen = {gid: c for gid, c in of.values()}, 0
+    touched = set()
+    for name, t in tensors:
+        seen += 1
+        gid, c = of[name]
+        touched.add(gid)
+        if c.add(name, t):
+            del open_groups[gid]
+    partial = source == "update_weights"
+    short = {g: c for g, c in open_groups.items() if g in touched or not partial}
+    if short:
+        raise ValueError(f"checkpoint {source} is incomplete; missing tensors: "
+                         f"{sorted(set().union(*(c.need - set(c.parts) for c in short.values())))[:8]}")
+    logger.info("loaded %d tensors from %s on rank %d", seen, source, get_state().rank)
+
+
 def load_named_tensors(model, tensors, names: set, source: str = "memory") -> None:
     """Load checkpoint-named tensors (Hugging Face layout) from any iterator of (name, tensor): a directory
     of safetensors files, or tensors handed over in memory by a trainer (``LLMEngine.update_weights``).
     ``names`` is the set of all names the iterator will yield (fused parameters wait for their pieces)."""
+    if hasattr(model, "checkpoint_groups"):
+        return load_grouped_tensors(model, tensors, names, source)
     path = source
     cfg = model.cfg
     st = get_state()

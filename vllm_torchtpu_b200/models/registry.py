@@ -24,8 +24,11 @@ def get_model_class(cfg: ModelConfig):
     if a == "kimi_linear":
         from .kimi_linear import KimiLinearForCausalLM
         return KimiLinearForCausalLM
+    if a == "mazivik":
+        from .mazivik import MazivikForCausalLM
+        return MazivikForCausalLM
     raise ValueError(f"no model class for architecture {a!r}")
 
 
 def supported_architectures() -> list[str]:
-    return ["llama", "qwen3_moe", "gpt_oss", "deepseek_v3", "qwen3_next", "kimi_linear"]
+    return ["llama", "qwen3_moe", "gpt_oss", "deepseek_v3", "qwen3_next", "kimi_linear", "mazivik"]

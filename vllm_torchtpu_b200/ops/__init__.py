@@ -30,6 +30,20 @@ def rms_norm(x, weight, eps):
     return cuda_ops().rms_norm(x, weight, eps) if _on_gpu(x) else ref.rms_norm(x, weight, eps)
 
 
+def layer_norm(x, weight, eps):
+    return cuda_ops().layer_norm(x, weight, eps) if _on_gpu(x) else ref.layer_norm(x, weight, eps)
+
+
+def layer_norm_add(y, residual, weight, eps):
+    """(rounded r', fp32 r') of r' = residual + LN(y) * weight; an fp32 residual is updated in place on a GPU."""
+    return cuda_ops().layer_norm_add(y, residual, weight, eps) if _on_gpu(y) else \
+        ref.layer_norm_add(y, residual, weight, eps)
+
+
+def softcap(x, cap):
+    return cuda_ops().softcap(x, cap) if _on_gpu(x) else ref.softcap(x, cap)
+
+
 def materialize(x):
     """A row-parallel output whose cross-rank sum is still pending becomes a tensor."""
     return x.materialize() if hasattr(x, "materialize") else x
@@ -55,6 +69,24 @@ def silu_and_mul(x):
 
 def gemm(x, w, bias=None, out=None):
     return cuda_ops().gemm(x, w, bias, out=out) if _on_gpu(x) else ref.gemm(x, w, bias)
+
+
+def gemm_gelu(x, w):
+    """gelu(x @ w.T) with gelu in its erf form, in the GEMM's epilogue on a GPU."""
+    return cuda_ops().gemm_gelu(x, w) if _on_gpu(x) else ref.gemm_gelu(x, w)
+
+
+def gemm_heads(x, w, gate=None, out=None):
+    """Per-head product x [T, H, >= K] with w [H, N, K] -> [T, H, N]; see ``ops.reference.gemm_heads``."""
+    return cuda_ops().gemm_heads(x, w, gate, out) if _on_gpu(x) else ref.gemm_heads(x, w, gate, out)
+
+
+def latent_prep(*a, **kw):
+    return cuda_ops().latent_prep(*a, **kw) if _on_gpu(a[0]) else ref.latent_prep(*a, **kw)
+
+
+def rope_heads_into(q, out, *a, **kw):
+    return cuda_ops().rope_heads_into(q, out, *a, **kw) if _on_gpu(q) else ref.rope_heads_into(q, out, *a, **kw)
 
 
 def embedding(ids, table):

@@ -70,17 +70,26 @@ def reload_lib(path: Optional[str] = None) -> str:
     return src
 
 
-def lib():
+def load_lib(path: str) -> None:
+    """Load this kernel library: the full one, or one that holds the sources of a model family only."""
     global _lib, _sms
+    _lib = ctypes.CDLL(path, mode=ctypes.RTLD_GLOBAL)
+    _lib.b200_get_last_error.restype = ctypes.c_char_p
+    if hasattr(_lib, "b200_attn_decode_scratch_bytes"):
+        _lib.b200_attn_decode_scratch_bytes.restype = c_size_t
+    if torch.cuda.is_available():
+        _sms = torch.cuda.get_device_properties(torch.cuda.current_device()).multi_processor_count
+
+
+def lib():
+    global _lib
     if _lib is not None:
         return _lib
     from ..csrc import build as _build
     path = envs.B200_KERNEL_LIB or _build.lib_path()
     if not os.path.exists(path):
         raise RuntimeError(f"kernel library {path} is missing; run `python -m vllm_torchtpu_b200.csrc.build`")
-    _lib = ctypes.CDLL(path, mode=ctypes.RTLD_GLOBAL)
-    _lib.b200_get_last_error.restype = ctypes.c_char_p
-    _lib.b200_attn_decode_scratch_bytes.restype = c_size_t
+    load_lib(path)
     if envs.B200_BOUNDS_CHECK:
         # the attention kernels from the bounds-checked library, everything else from the main one
         checked = _build.checked_lib_path()
@@ -89,8 +98,6 @@ def lib():
         over = ctypes.CDLL(checked)
         over.b200_attn_decode_scratch_bytes.restype = c_size_t
         _lib = _Overlay(_lib, over)
-    if torch.cuda.is_available():
-        _sms = torch.cuda.get_device_properties(torch.cuda.current_device()).multi_processor_count
     return _lib
 
 
@@ -211,13 +218,59 @@ def silu_and_mul(x):
     return y
 
 
+def _mixed(t) -> int:
+    """Element bytes of a tensor the 32-bit-capable kernels take."""
+    if t.dtype == torch.bfloat16:
+        return 2
+    if t.dtype == torch.float32:
+        return 4
+    raise TypeError(f"bfloat16 or float32 expected, got {t.dtype}")
+
+
+def layer_norm(x, weight, eps):
+    """LN(x) * weight (no bias), fp32 inside; the output has the weight's dtype."""
+    x = x.contiguous()
+    H = x.shape[-1]
+    out = torch.empty(x.shape, dtype=weight.dtype, device=x.device)
+    _check(lib().b200_layer_norm(_p(x), c_int(_mixed(x)), _p(weight), c_int(_mixed(weight)), _p(out),
+                                 c_int(x.numel() // H), c_int(H), c_float(eps), _stream()), "layer_norm")
+    count_launch()
+    return out
+
+
+def layer_norm_add(y, residual, weight, eps):
+    """r' = residual + LN(y) * weight.  Returns (r' in the weight's dtype, r' fp32); an fp32 residual is
+    updated in place, a bf16 one (the embedding rows) starts the 32-bit stream."""
+    y = y.contiguous()
+    assert residual.is_contiguous()
+    H = y.shape[-1]
+    r = residual if residual.dtype == torch.float32 else torch.empty(y.shape, dtype=torch.float32, device=y.device)
+    h = torch.empty(y.shape, dtype=weight.dtype, device=y.device) if weight.dtype != torch.float32 else None
+    _check(lib().b200_layer_norm_add(_p(y), c_int(_mixed(y)), _p(residual), c_int(_mixed(residual)), _p(weight),
+                                     c_int(_mixed(weight)), _p(r), _p(h), c_int(y.numel() // H), c_int(H),
+                                     c_float(eps), _stream()), "layer_norm_add")
+    count_launch()
+    return (r if h is None else h), r
+
+
+def softcap(x, cap: float):
+    """cap * tanh(x / cap) in fp32 (in place when x is fp32)."""
+    x = x.contiguous()
+    y = x if x.dtype == torch.float32 else torch.empty(x.shape, dtype=torch.float32, device=x.device)
+    _check(lib().b200_softcap(_p(x), c_int(_mixed(x)), _p(y), c_longlong(x.numel()), c_float(cap), _stream()),
+           "softcap")
+    count_launch()
+    return y
+
+
 def embedding(ids, table, token_src=None, last_tokens=None):
-    _require_bf16(table)
+    _mixed(table)
     T = ids.numel()
     out = torch.empty((T, table.shape[1]), dtype=table.dtype, device=table.device)
     assert ids.dtype == torch.int32
     _check(lib().b200_embedding(_p(ids), _p(token_src), _p(last_tokens), _p(table), _p(out), c_int(T),
-                                c_int(table.shape[1]), c_int(table.shape[0]), _stream()), "embedding")
+                                c_int(table.shape[1] * table.element_size()), c_int(table.shape[0]), _stream()),
+           "embedding")
     count_launch()
     return out
 
@@ -226,8 +279,8 @@ def gather_rows(hidden, residual, idx):
     R, H = idx.numel(), hidden.shape[1]
     oh = torch.empty((R, H), dtype=hidden.dtype, device=hidden.device)
     orr = torch.empty_like(oh) if residual is not None else None
-    _check(lib().b200_gather_rows(_p(hidden), _p(residual), _p(idx), _p(oh), _p(orr), c_int(R), c_int(H),
-                                  c_int(hidden.shape[0]), _stream()), "gather_rows")
+    _check(lib().b200_gather_rows(_p(hidden), _p(residual), _p(idx), _p(oh), _p(orr), c_int(R),
+                                  c_int(H * hidden.element_size()), c_int(hidden.shape[0]), _stream()), "gather_rows")
     count_launch()
     return oh, orr
 
@@ -264,8 +317,82 @@ def rope_and_cache(qkv, positions, inv_freq, kv_cache, slot_mapping, num_q_heads
 
 
 # ------------------------------------------------------------------------ GEMM
+def _tma_ready(t, stride: int) -> bool:
+    """bf16 operand that a TMA tensor map can describe: 16-byte rows and base."""
+    return t.dtype == torch.bfloat16 and stride % 8 == 0 and t.data_ptr() % 16 == 0
+
+
+def gemm_simt(x, w, y, T, N, K, ldx, ldy, *, bias=None, gate=None, ldg=0, batch=1, xs=0, ys=0, act=0):
+    """CUDA-core GEMM (``csrc/gemm_simt.cu``): fp32 operands, or bf16 ones without the TMA's alignment."""
+    elem = _mixed(x)
+    assert all(t is None or t.dtype == x.dtype for t in (w, y, bias, gate)), "operands of one dtype"
+    _check(lib().b200_gemm_simt(_p(x), _p(w), _p(y), _p(bias), _p(gate), c_int(T), c_int(N), c_int(K), c_int(batch),
+                                c_longlong(ldx), c_longlong(K), c_longlong(ldy), c_longlong(ldg), c_longlong(xs),
+                                c_longlong(ys), c_int(act), c_int(elem), _stream()), "gemm_simt")
+    count_launch()
+    return y
+
+
+def gemm_gelu(x, w):
+    """gelu(x @ w.T), erf form, applied in the epilogue."""
+    lead, (N, K) = x.shape[:-1], w.shape
+    x2 = x.reshape(-1, K)
+    if x2.stride(-1) != 1:
+        x2 = x2.contiguous()
+    T = x2.shape[0]
+    y = torch.empty((T, N), dtype=x.dtype, device=x.device)
+    if T == 0:
+        return y.reshape(*lead, N)
+    if not (_tma_ready(x2, x2.stride(0)) and _tma_ready(w, K)):
+        return gemm_simt(x2, w, y, T, N, K, x2.stride(0), N, act=1).reshape(*lead, N)
+    ws = Workspace.get(x.device)
+    if 0 < envs.B200_GEMM_2SM_MIN_T <= T:
+        _check(lib().b200_gemm_bf16_gelu_2sm(_p(x2), _p(w), _p(y), c_int(T), c_int(N), c_int(K), c_int(x2.stride(0)),
+                                             c_int(K), c_int(N), _p(ws.status), c_int(_sms), _stream()), "gemm_gelu_2sm")
+    else:
+        _check(lib().b200_gemm_bf16_heads(_p(x2), _p(w), _p(y), c_void_p(0), c_int(T), c_int(N), c_int(K), c_int(1),
+                                          c_int(x2.stride(0)), c_int(K), c_int(N), c_int(0), c_int(0), c_int(0),
+                                          c_int(1), _p(ws.status), c_int(_sms), _stream()), "gemm_gelu")
+    count_launch()
+    return y.reshape(*lead, N)
+
+
+def gemm_heads(x, w, gate=None, out=None):
+    """Per head h: x[:, h, :K] @ w[h].T -> [T, H, N] (w [H, N, K]), times sigmoid(gate) with gate [T, H * N] (rows may
+    be strided) when given, as one launch over the heads; into the first N columns of ``out`` [T, H, >= N] if given."""
+    H, N, K = w.shape
+    T = x.shape[0]
+    assert x.shape[1] == H and x.shape[2] >= K and x.stride(2) == 1 and w.is_contiguous()
+    y = out if out is not None else torch.empty((T, H, N), dtype=x.dtype, device=x.device)
+    assert y.stride(2) == 1
+    if T == 0:
+        return y
+    ldg = 0
+    if gate is not None:
+        assert gate.stride(1) == 1 and gate.shape[1] == H * N
+        ldg = gate.stride(0)
+    ldx, xs, ldy, ys = x.stride(0), x.stride(1), y.stride(0), y.stride(1)
+    if not (_tma_ready(x, ldx) and xs % 8 == 0 and _tma_ready(w, K)):
+        return gemm_simt(x, w, y, T, N, K, ldx, ldy, gate=gate, ldg=ldg, batch=H, xs=xs, ys=ys)
+    ws = Workspace.get(x.device)
+    _check(lib().b200_gemm_bf16_heads(_p(x), _p(w), _p(y), _p(gate), c_int(T), c_int(N), c_int(K), c_int(H), c_int(ldx),
+                                      c_int(K), c_int(ldy), c_int(ldg), c_int(xs), c_int(ys), c_int(0), _p(ws.status),
+                                      c_int(_sms), _stream()), "gemm_heads")
+    count_launch()
+    return y
+
+
 def gemm(x, w, bias=None, out=None, force_splits: int = 0):
-    """y[T,N] = x[T,K] @ w[N,K]^T (+bias) on the tcgen05 kernel."""
+    """y[T,N] = x[T,K] @ w[N,K]^T (+bias) on the tcgen05 kernel; fp32 operands, and bf16 ones a tensor map
+    cannot describe, run on the CUDA cores."""
+    if x.dtype == torch.float32 or x.shape[-1] % 8:
+        x2 = x.reshape(-1, x.shape[-1])
+        x2 = x2 if x2.stride(-1) == 1 else x2.contiguous()
+        T, N = x2.shape[0], w.shape[0]
+        assert w.is_contiguous()
+        y = out if out is not None else torch.empty((T, N), dtype=x.dtype, device=x.device)
+        gemm_simt(x2, w, y, T, N, x2.shape[1], x2.stride(0), y.stride(0), bias=bias)
+        return y.reshape(*x.shape[:-1], N)
     _require_bf16(x, w, bias)
     if envs.B200_GEMM_IMPL == "cublas":
         y = torch.nn.functional.linear(x, w, bias)
@@ -736,7 +863,8 @@ _SUBMODULE_EXPORTS = {
                  "moe_experts_fp8", "quant_act_1x128", "quant_act_int8", "quant_rows_1x128"),
     "cuda_fp4": ("grouped_w4a16_gemm", "moe_experts_w4a16", "w4a16_gemm", "w4a16_int4_gemm", "dequant_w4", "dequant_int4"),
     "cuda_gdn": ("gdn_forward", "kda_forward", "short_conv"),
-    "cuda_mla": ("mla_absorb", "mla_paged_attention", "mla_unabsorb", "mla_write_cache", "permute_rows", "rope_rows"),
+    "cuda_mla": ("latent_prep", "mla_absorb", "mla_paged_attention", "mla_unabsorb", "mla_write_cache", "permute_rows", "rope_heads_into",
+                 "rope_rows"),
 }
 _EXPORT_HOME = {name: mod for mod, names in _SUBMODULE_EXPORTS.items() for name in names}
 

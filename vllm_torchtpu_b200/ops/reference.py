@@ -39,6 +39,42 @@ def fused_add_rms_norm(x, residual, weight, eps):
     return rms_norm(r, weight, eps), r
 
 
+def layer_norm(x: torch.Tensor, weight: torch.Tensor, eps: float) -> torch.Tensor:
+    """Layer norm with a weight and no bias, fp32; the result has the weight's dtype."""
+    xf = x.float()
+    d = xf - xf.mean(-1, keepdim=True)
+    return (d * torch.rsqrt(d.pow(2).mean(-1, keepdim=True) + eps) * weight.float()).to(weight.dtype)
+
+
+def layer_norm_add(y: torch.Tensor, residual: torch.Tensor, weight: torch.Tensor, eps: float):
+    """Sublayer output normalised and added to a 32-bit residual stream: r' = r + LN(y) * w.
+    Returns (r' rounded to the weight's dtype, r' fp32)."""
+    r = residual.float() + layer_norm(y, weight.float(), eps)
+    return r.to(weight.dtype), r
+
+
+def softcap(x: torch.Tensor, cap: float) -> torch.Tensor:
+    return cap * torch.tanh(x.float() / cap)
+
+
+def gemm_gelu(x: torch.Tensor, w: torch.Tensor) -> torch.Tensor:
+    return F.gelu(x.float() @ w.float().t()).to(x.dtype)
+
+
+def gemm_heads(x: torch.Tensor, w: torch.Tensor, gate: Optional[torch.Tensor] = None,
+               out: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """Per head h: x[:, h, :K] (K = w.shape[2]) times w[h] [N, K] transposed -> [T, H, N], optionally times
+    sigmoid(gate) with gate [T, H * N]; written into the first N columns of ``out`` when given."""
+    H, N, K = w.shape
+    y = torch.einsum("thk,hnk->thn", x[..., :K].float(), w.float())
+    if gate is not None:
+        y = y * torch.sigmoid(gate.float()).reshape(y.shape)
+    if out is None:
+        return y.to(x.dtype).contiguous()
+    out[..., :N] = y.to(out.dtype)
+    return out
+
+
 GATED_ACTS = ("silu", "gelu", "gelu_tanh", "swigluoai", "silu_clamp", "situ")
 
 
@@ -128,9 +164,7 @@ def rope_inv_freq(head_dim: int, theta: float, scaling: Optional[dict] = None,
         if scaling.get("truncate", True):
             lo, hi = math.floor(lo), math.ceil(hi)
         lo, hi = max(lo, 0), min(hi, rd - 1)
-        if lo == hi:
-            hi += 0.001
-        ramp = ((torch.arange(rd // 2, dtype=torch.float64) - lo) / (hi - lo)).clamp(0, 1)
+        ramp = ((torch.arange(rd // 2, dtype=torch.float64) - lo) / max(hi - lo, 0.001)).clamp(0, 1)
         keep = 1.0 - ramp
         inv = inv / factor * (1.0 - keep) + inv * keep
     return inv.float()
@@ -418,6 +452,38 @@ def moe_experts(x, w13, w2, topk_ids, topk_w, expert_offset: int = 0, act: str =
 
 
 # ---- MLA -------------------------------------------------------------------------
+def rope_scaled(x: torch.Tensor, positions: torch.Tensor, inv_freq: torch.Tensor, mult: float,
+                interleaved: bool) -> torch.Tensor:
+    """``apply_rope`` of x [T, H, D] with cos and sin times ``mult`` (YaRN); dims behind the rotated ones pass."""
+    n = 2 * inv_freq.numel()
+    out = apply_rope(x.float(), positions, inv_freq, interleaved)
+    out[..., :n] *= mult
+    return out.to(x.dtype)
+
+
+def latent_prep(row, cq_norm, c_norm, cache, slot_mapping, positions, inv_freq, mult, eps, kv_rank, rot_dim,
+                interleaved=True):
+    """row [T, Q + L + R + ...] = query latent ‖ latent ‖ shared rotated key of a packed input projection.
+    Returns the RMS-normed query latent [T, Q]; when ``c_norm`` is given the normed latent and the rotated key
+    go to the cache rows of ``slot_mapping``."""
+    Q = cq_norm.shape[0]
+    if c_norm is not None:
+        c = rms_norm(row[:, Q:Q + kv_rank], c_norm, eps)
+        k = rope_scaled(row[:, None, Q + kv_rank:Q + kv_rank + rot_dim], positions, inv_freq, mult, interleaved)[:, 0]
+        valid = slot_mapping >= 0
+        slots = slot_mapping[valid].long()
+        bs = cache.shape[1]
+        cache[slots // bs, slots % bs, :kv_rank + rot_dim] = torch.cat([c, k], -1)[valid].to(cache.dtype)
+    return rms_norm(row[:, :Q], cq_norm, eps)
+
+
+def rope_heads_into(q, out, nope: int, rot_dim: int, col: int, positions, inv_freq, mult, interleaved=True):
+    """out[t, h, col : col + rot_dim] = rotated q[t, h, nope : nope + rot_dim]; columns behind are zeroed."""
+    out[..., col:col + rot_dim] = rope_scaled(q[..., nope:nope + rot_dim], positions, inv_freq, mult, interleaved)
+    out[..., col + rot_dim:] = 0
+    return out
+
+
 def mla_write_cache(cache: torch.Tensor, kv_c: torch.Tensor, k_pe: torch.Tensor,
                     slot_mapping: torch.Tensor) -> None:
     """cache: [num_blocks, block_size, kv_lora + rope]; row = kv_c_normed ‖ k_pe

@@ -205,6 +205,17 @@ class B200Platform:
             m.num_q_heads_unpadded = m.num_q_heads
             m.num_q_heads = m.num_kv_heads * gp
             logger.info("query heads padded %d -> %d for tp=%d", m.num_q_heads_unpadded, m.num_q_heads, tp)
+        if m.layer_specs:
+            if m.quantization:
+                raise ValueError(f"quantised weights are not built for {m.architecture}")
+            if p.pipeline_parallel_size > 1:
+                raise ValueError(f"pipeline parallelism is not built for {m.architecture}: its 32-bit residual stream "
+                                 "and shared caches do not cross the stage hand-off")
+            bad = [i for i, l in enumerate(m.layer_specs) if l.mixer.heads % tp]
+            if bad:
+                raise ValueError(f"the query heads of layers {bad[:8]} do not divide over tp={tp}")
+            if cfg.speculative and cfg.speculative.get("method") not in ("ngram", "suffix", "medusa"):
+                raise ValueError(f"drafters that run a layer of the target are not built for {m.architecture}")
         if p.enable_expert_parallel and not m.is_moe:
             logger.warning("--enable-expert-parallel ignored: %s has no experts", m.name)
             p.enable_expert_parallel = False

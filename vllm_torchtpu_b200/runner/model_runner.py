@@ -67,6 +67,7 @@ class StepResult:
     hidden: Optional[torch.Tensor] = None   # final-norm hidden state of every sampled row (draft heads)
     hidden_all: Optional[torch.Tensor] = None   # ... of every row of the step (drafters with their own KV cache)
     rows: Optional[dict] = None     # row layout of the step: query_start_loc, first position, batch slot per request
+    place_logits: Optional[dict] = None     # request id -> fp32 [places, vocab] (host) of the wanted positions
     status_host: Optional[torch.Tensor] = None   # copy of the device status word taken after the step
 
     def take_logprobs(self):
@@ -172,6 +173,8 @@ class ModelRunner:
         self._last_h_all = None
         self.extra_kv_layers = 0         # KV layers a drafter allocates beside the model's (HBM budget)
         self._pool_plan = None           # pooling requests of the current step: (id, row lo, row hi, mode, last chunk)
+        self._want_rows = None           # token rows of the current step whose logits the caller reads (host list)
+        self._want_logits = None
         self._pool_acc: dict = {}        # request id -> [sum or last row, count]
         if envs.B200_STAGE_TIMING and self.is_cuda:
             from ..tracing.stage_timing import RunnerStageTiming
@@ -278,6 +281,8 @@ class ModelRunner:
             if hasattr(self.model, "allocate_kv_caches") else [
                 torch.zeros(self.model.kv_cache_shape(num_blocks, self.block_size), dtype=kv_dtype,
                             device=self.device) for _ in self.model.layers]
+        # layers may share one cache tensor: what moves blocks between pools handles each tensor once
+        self.distinct_kv_caches = list({id(c): c for c in self.kv_caches}.values())
         if not hasattr(self, "bufs_prefill"):
             self._alloc_step_buffers()
         if self.is_cuda and hasattr(self.model, "setup_decode_fusion"):
@@ -444,6 +449,9 @@ class ModelRunner:
         ex = self._step_extras
         if ex is not None and ex["prompt"]:
             self._prompt_logprobs(hidden, residual, ex)
+        if self._want_rows:
+            idx = torch.tensor(self._want_rows, dtype=torch.int32, device=hidden.device)
+            self._want_logits = self.model.compute_logits(self.model.finalize(*self._select_rows(hidden, residual, idx)))
         rows = self._select_rows(hidden, residual, meta.logits_indices)
         h = self.model.finalize(*rows)
         if getattr(meta, "pcp", None) is not None:
@@ -564,6 +572,23 @@ class ModelRunner:
             return None
         return {"lp_rows": lp_rows, "lp_ks": lp_ks, "mask_rows": mask_rows, "mask_ids": mask_ids,
                 "prompt": prompt, "adjust": adjust, "out": {}}
+
+    @staticmethod
+    def _plan_places(out, p):
+        """([(request id, first, last + 1)], token rows) of the positions whose logits the caller wants."""
+        want = getattr(out, "logit_places", None)
+        if not want:
+            return None
+        spans, rows = [], []
+        for i, s in enumerate(p["scheds"]):
+            places = want.get(s.request.request_id)
+            if places:
+                if min(places) < 0 or max(places) >= s.num_new_tokens:
+                    raise ValueError(f"request {s.request.request_id}: logits wanted at a place outside its tokens")
+                lo = int(p["qsl_np"][i])
+                spans.append((s.request.request_id, len(rows), len(rows) + len(places)))
+                rows += [lo + k for k in places]
+        return (spans, rows) if rows else None
 
     def _pp_handoff(self):
         if getattr(self, "_pp", None) is None:
@@ -812,6 +837,9 @@ class ModelRunner:
                      and self._step_extras is None and not self.keep_hidden and self.dcp_size == 1
                      and getattr(self.model, "dp_vocab", None) is None
                      and get_state().pp.size == 1)          # pipeline stages hand off through host threads
+        places, self._want_rows = self._plan_places(out, p), None
+        if places and not use_graph:
+            self._want_rows = places[1]
         if use_graph:
             key = (R, p["all_greedy"])
             g = self.graphs.get(key)
@@ -821,6 +849,8 @@ class ModelRunner:
                 g = self._capture(key, bufs, meta, T, R, p["all_greedy"])
             g["graph"].replay()
             tokens = g["tokens"]
+            if places:                   # a decode step's rows are its sampled rows, in order
+                self._want_logits = g["logits"][torch.tensor(places[1], device=self.device)]
             self.stats["graph_steps"] += 1
             self.launch_counter += g["launches"]
         else:
@@ -864,6 +894,9 @@ class ModelRunner:
         self.stats["d2h_bytes"] += rows * 4 + 4
         res = StepResult([s.request.request_id for s in p["scheds"]], [s.samples for s in p["scheds"]],
                          host, ev, n, rows * 4 + 4, status_host=st_host)
+        if places:
+            got, self._want_logits = self._want_logits.float().cpu(), None
+            res.place_logits = {rid: got[lo:hi] for rid, lo, hi in places[0]}
         if self.keep_hidden:
             res.hidden, self._last_h = self._last_h, None
         if self.keep_all_hidden:
@@ -910,10 +943,10 @@ class ModelRunner:
         g = torch.cuda.CUDAGraph()
         c0 = launch_count()
         with torch.cuda.graph(g, pool=self.graph_pool):
-            tokens, _ = self._forward_and_sample(bufs, meta, T, R, all_greedy)
+            tokens, logits = self._forward_and_sample(bufs, meta, T, R, all_greedy)
         if self.graph_pool is None:
             self.graph_pool = g.pool()
-        entry = {"graph": g, "tokens": tokens, "launches": launch_count() - c0}
+        entry = {"graph": g, "tokens": tokens, "logits": logits, "launches": launch_count() - c0}
         self.graphs[key] = entry
         return entry
 

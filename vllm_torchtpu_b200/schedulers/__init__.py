@@ -23,4 +23,7 @@ def get_scheduler_class(name: str):
     if name == "priority":
         from .priority import PriorityScheduler
         return PriorityScheduler
+    if name == "replay":
+        from .replay import ReplayScheduler
+        return ReplayScheduler
     raise ValueError(f"unknown scheduler {name!r}")
