@@ -49,12 +49,13 @@ def rotate_pairs(x, positions, rot):
     """x [S, ..., d]: dimensions (2i, 2i + 1) turned by position * frequency_i; dims beyond rot.dims pass."""
     freqs, mult = rotary_frequencies(rot)
     out = x.clone()
-    for s, p in enumerate(positions):
-        for i, f in enumerate(freqs):
-            c, n = mult * math.cos(p * f), mult * math.sin(p * f)
-            u, v = x[s, ..., 2 * i], x[s, ..., 2 * i + 1]
-            out[s, ..., 2 * i] = u * c - v * n
-            out[s, ..., 2 * i + 1] = v * c + u * n
+    for i, f in enumerate(freqs):
+        c = torch.tensor([mult * math.cos(p * f) for p in positions], dtype=x.dtype)
+        n = torch.tensor([mult * math.sin(p * f) for p in positions], dtype=x.dtype)
+        u, v = x[..., 2 * i], x[..., 2 * i + 1]
+        c, n = (t.reshape(-1, *[1] * (u.dim() - 1)) for t in (c, n))
+        out[..., 2 * i] = u * c - v * n
+        out[..., 2 * i + 1] = v * c + u * n
     return out
 
 
@@ -66,15 +67,18 @@ def latent_of(h, w, p, m, eps):
     return c, k_rot
 
 
-def causal_softmax(scores):
+def causal_softmax(scores, hidden_keys=()):
+    """Softmax over the keys j <= i; ``hidden_keys`` leaves out a key that should be seen (a planted mistake)."""
     S = scores.shape[-1]
-    future = torch.ones(S, S, dtype=torch.bool).triu(1)
-    scores = scores.masked_fill(future, float("-inf"))
+    masked = torch.ones(S, S, dtype=torch.bool).triu(1)
+    for k in hidden_keys:
+        masked[k + 1:, k] = True
+    scores = scores.masked_fill(masked, float("-inf"))
     e = torch.exp(scores - scores.max(-1, keepdim=True).values)
     return e / e.sum(-1, keepdim=True)
 
 
-def latent_attention(h, w, p, m, eps, c, k_rot):
+def latent_attention(h, w, p, m, eps, c, k_rot, hidden_keys=()):
     """Mixer output [S, width].  c, k_rot: this layer's latent, or the one of the layer it shares."""
     S, H, dn, dr, dv = h.shape[0], m["heads"], m["dim"], m["rot_dim"], m["vdim"]
     q = rms_norm(h @ w[p + "dq"].t(), w[p + "dq.norm"], eps) @ w[p + "uq"].t()
@@ -83,7 +87,7 @@ def latent_attention(h, w, p, m, eps, c, k_rot):
     k = (c @ w[p + "uk"].t()).reshape(S, H, dn)
     v = (c @ w[p + "uv"].t()).reshape(S, H, dv)
     scores = torch.einsum("qhd,khd->hqk", q[..., :dn], k) + torch.einsum("qhd,kd->hqk", q_rot, k_rot)
-    o = torch.einsum("hqk,khd->qhd", causal_softmax(scores * m["scale"]), v).reshape(S, H * dv)
+    o = torch.einsum("hqk,khd->qhd", causal_softmax(scores * m["scale"], hidden_keys), v).reshape(S, H * dv)
     return (o * torch.sigmoid(h @ w[p + "g"].t())) @ w[p + "o"].t()
 
 
@@ -91,7 +95,7 @@ def feed_forward(x, w, p):
     return gelu_erf(x @ w[p + "up"].t()) @ w[p + "down"].t()
 
 
-def forward(cfg, w, tokens, *, layers_out=None, dtype=torch.float64):
+def forward(cfg, w, tokens, *, layers_out=None, dtype=torch.float64, hidden_keys=()):
     """Logits [S, vocab] of one sequence; appends the residual stream after every layer to ``layers_out``."""
     w = {k: v.to(dtype) for k, v in w.items()}
     eps = cfg["norm"]["eps"]
@@ -102,7 +106,7 @@ def forward(cfg, w, tokens, *, layers_out=None, dtype=torch.float64):
         src = m.get("kv_from")
         if src is None:
             latents[i] = latent_of(x, w, p, m, eps)
-        y = latent_attention(x, w, p, m, eps, *latents[i if src is None else src])
+        y = latent_attention(x, w, p, m, eps, *latents[i if src is None else src], hidden_keys)
         x = x + layer_norm(y, w[f"l{i}.norm1"], eps)
         if layer.get("mlp"):
             x = x + layer_norm(feed_forward(x, w, f"l{i}.mlp."), w[f"l{i}.norm2"], eps)

@@ -447,13 +447,13 @@ def model_preset(name: str) -> ModelConfig:
     if n in ("tiny-mazivik",):
         # two latents of which the first serves two layers, unequal layers, one without a feed-forward
         rot = {"base": 10000.0, "dims": 16, "scaling": {"factor": 2.0, "original": 64, "fast": 16.0, "slow": 1.0}}
-        mix = {"heads": 3, "dim": 24, "rot_dim": 16, "vdim": 40, "q_rank": 48, "kv_rank": 56, "scale": 0.17, "rot": rot}
+        mix = {"heads": 4, "dim": 24, "rot_dim": 16, "vdim": 40, "q_rank": 48, "kv_rank": 56, "scale": 0.17, "rot": rot}
         ff = {"kind": "dense", "ff": 144}
         mc = ModelConfig.from_layer_list({
             "architecture": "Mazivik", "width": 112, "vocab": 320, "norm": {"eps": 1e-5}, "logit_softcap": 20.0,
             "torch_dtype": "float32", "layers": [
                 {"type": "latent_attention", "mixer": mix, "mlp": ff},
-                {"type": "latent_attention", "mixer": dict(mix, heads=5, vdim=24, q_rank=32, kv_from=0), "mlp": None},
+                {"type": "latent_attention", "mixer": dict(mix, heads=6, vdim=24, q_rank=32, kv_from=0), "mlp": None},
                 {"type": "latent_attention", "mixer": dict(mix, heads=2, dim=40, kv_rank=72), "mlp": ff}]},
             name="tiny-mazivik")
         mc.max_model_len, mc.init_std = 256, 0.1

@@ -379,6 +379,8 @@ __device__ __forceinline__ T warp_max(T v) {
 
 __device__ __forceinline__ float gelu_erf(float v) { return 0.5f * v * (1.f + erff(v * 0.70710678118654752f)); }
 
+__device__ __forceinline__ float soft_cap(float v, float cap) { return cap > 0.f ? cap * tanhf(v / cap) : v; }
+
 struct alignas(16) bf16x8 {
   __nv_bfloat162 v[4];
 };

@@ -99,11 +99,13 @@ struct GemmParams {
   unsigned long long ag_done_off;
   int ag_flip;
   unsigned long long* dbg;               // optional: per-CTA phase timestamps (ns), 16 slots per CTA
-  // ---- MODE 3: epilogue (act 0 none / 1 gelu; optional gate: y *= sigmoid(gate[t, b * N + n])) and batch over
-  // heads: head b reads activation columns from b * x_head_cols, weight rows from b * N and writes output
-  // columns from b * y_head_cols
+  // ---- MODE 3: epilogue (act 0 none / 1 gelu / 2 fp32 output Yf with the soft cap cap * tanh(y / cap), cap 0: none;
+  // optional gate: y *= sigmoid(gate[t, b * N + n])) and batch over heads: head b reads activation columns from
+  // b * x_head_cols, weight rows from b * N and writes output columns from b * y_head_cols
   int act, batch, x_head_cols, y_head_cols, ldg;
+  float cap;
   const __nv_bfloat16* gate;
+  float* Yf;
   int* epoch_ptr;                        // local: epoch of the last completed fused launch
   int* cta_done;                         // local: CTA exit counter
   unsigned int spin_limit;
@@ -346,6 +348,13 @@ __device__ __forceinline__ void cluster_reduce_cols(const GemmParams& p, const W
         }
         if (MODE == 3 && p.act == 1) {           // (no bias in this mode)
           a.x = gelu_erf(a.x); a.y = gelu_erf(a.y); a.z = gelu_erf(a.z); a.w = gelu_erf(a.w);
+        }
+        if (MODE == 3 && p.act == 2) {
+          const float vals[4] = {a.x, a.y, a.z, a.w};
+#pragma unroll
+          for (int j = 0; j < 4; ++j)
+            if (n4 + j < p.N) p.Yf[(size_t)(wk.t_row + c) * p.ldy + n4 + j] = soft_cap(vals[j], p.cap);
+          continue;
         }
         for (int d = 0; d < ndst; ++d) {
           const TileDst td = tile_dst<BN, MODE>(p, wk, d);
@@ -739,6 +748,13 @@ gemm_bf16_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant_
                     if (c0 + j < t_valid)
                       yp[(size_t)j * td.cs] =
                           __float2bfloat16(__fdividef(__uint_as_float(r[j]), 1.f + __expf(-gv[j])));
+                  continue;
+                }
+                if (p.act == 2) {
+                  float* yf = p.Yf + (size_t)(t0 + c0) * p.ldy + n;
+#pragma unroll
+                  for (int j = 0; j < 32; ++j)
+                    if (c0 + j < t_valid) yf[(size_t)j * p.ldy] = soft_cap(__uint_as_float(r[j]), p.cap);
                   continue;
                 }
                 if (p.act == 1) {
@@ -1428,8 +1444,9 @@ extern "C" int b200_gemm_bf16(const void* X, const void* W, void* Y, const void*
 // (heads), act 0 none / 1 gelu (erf).  X row stride ldx, W [batch * N, K] row stride ldw, Y row stride ldy.  A head
 // whose K is no multiple of the 64-wide K block reads into its neighbour's columns; those meet the zero fill
 // behind the weight's K columns.
+// act 2: Y is fp32 and holds cap * tanh(. / cap) (cap 0: the products themselves).
 extern "C" int b200_gemm_bf16_heads(const void* X, const void* W, void* Y, const void* gate, int T, int N, int K,
-                                    int batch, int ldx, int ldw, int ldy, int ldg, int xs, int ys, int act,
+                                    int batch, int ldx, int ldw, int ldy, int ldg, int xs, int ys, int act, float cap,
                                     int* status, int num_sms, cudaStream_t stream) {
   using namespace b200;
   if (T <= 0 || N <= 0 || K <= 0 || batch <= 0) return 0;
@@ -1441,6 +1458,12 @@ extern "C" int b200_gemm_bf16_heads(const void* X, const void* W, void* Y, const
   memset(&p, 0, sizeof(p));
   p.world = 1;
   p.Y = reinterpret_cast<__nv_bfloat16*>(Y);
+  p.Yf = reinterpret_cast<float*>(Y);
+  p.cap = cap;
+  if (act == 2 && (batch > 1 || gate != nullptr)) {
+    b200_set_last_error("gemm_heads: fp32 output is for one ungated product", __FILE__, __LINE__);
+    return -3;
+  }
   p.gate = reinterpret_cast<const __nv_bfloat16*>(gate);
   p.status = status;
   p.T = T; p.N = N; p.K = K; p.ldy = ldy; p.ldg = ldg;

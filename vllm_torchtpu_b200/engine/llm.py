@@ -79,7 +79,8 @@ class LLM:
             additional=additional_config or {})
         self.engine = LLMEngine(cfg, init_dist=init_dist)
         self.tokenizer = tokenizer
-        if tokenizer is None and model_path:
+        files = os.listdir(tokenizer_path or model_path) if tokenizer is None and model_path else []
+        if any(f.startswith("tokenizer") or f.endswith((".model", ".tiktoken")) or f == "vocab.json" for f in files):
             try:
                 from transformers import AutoTokenizer
                 self.tokenizer = AutoTokenizer.from_pretrained(tokenizer_path or model_path)

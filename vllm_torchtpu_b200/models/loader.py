@@ -149,8 +149,8 @@ def _load_oss_experts(moe, parts: dict) -> None:
 
 def load_grouped_tensors(model, tensors, names: set, source: str = "memory") -> None:
     """Models that list their checkpoint tensors themselves (``checkpoint_groups``): every group is handed to its
-    loader once all of its tensors have been read.  A directory must hold exactly the listed tensors; tensors handed
-    over in memory may cover a part of the groups."""
+    loader once all of its tensors have been read.  A directory must hold all listed tensors; tensors handed over in
+    memory may cover a part of the groups."""
     of: dict = {}
     for gid, (members, done) in enumerate(model.checkpoint_groups()):
         c = _Collector(set(members), lambda parts, members=members, done=done: done(*(parts[m] for m in members)))
@@ -158,10 +158,12 @@ def load_grouped_tensors(model, tensors, names: set, source: str = "memory") -> 
             of[m] = (gid, c)
     unknown = sorted(set(names) - set(of))
     if unknown:
-        raise ValueError(f"{source}: tensors the model does not have: {unknown[:8]}")
+        logger.warning("%s: %d tensors the model does not have are ignored: %s", source, len(unknown), unknown[:8])
     open_groups, seen = {gid: c for gid, c in of.values()}, 0
     touched = set()
     for name, t in tensors:
+        if name not in of:
+            continue
         seen += 1
         gid, c = of[name]
         touched.add(gid)

@@ -21,6 +21,7 @@ from ..config import ModelConfig
 from ..layers.latent_attention import LatentAttention
 from ..layers.linear import seeded_normal
 from ..layers.mlp import DenseMLP
+from ..parallel.communicator import get_tp_comm
 from .llama import LlamaForCausalLM
 
 
@@ -124,15 +125,18 @@ class MazivikForCausalLM(LlamaForCausalLM):
     def finalize(self, hidden, residual):
         return ops.layer_norm(hidden, self.norm, self.cfg.rms_norm_eps)
 
-    def _cap(self, logits):
-        cap = self.cfg.final_logit_softcap
-        return ops.softcap(logits, cap) if cap else logits
-
     def compute_logits(self, hidden_rows):
-        return self._cap(super().compute_logits(hidden_rows))
+        """fp32, soft-capped."""
+        cap = self.cfg.final_logit_softcap or 0.0
+        if getattr(self, "dp_vocab", None) is not None:
+            logits = self.dp_vocab.logits(hidden_rows, self.lm_head)
+            return ops.softcap(logits, cap) if cap else logits
+        logits = self.local_logits(hidden_rows)
+        comm = get_tp_comm()
+        return comm.all_gather(logits, dim=-1) if comm.size > 1 and self.vocab_shard is not None else logits
 
     def local_logits(self, hidden_rows):
-        return self._cap(super().local_logits(hidden_rows))
+        return ops.gemm_softcap(hidden_rows, self.lm_head, self.cfg.final_logit_softcap or 0.0)
 
     # ---- KV geometry -----------------------------------------------------------
     def _cache_owners(self) -> list:

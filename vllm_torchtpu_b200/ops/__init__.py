@@ -76,6 +76,11 @@ def gemm_gelu(x, w):
     return cuda_ops().gemm_gelu(x, w) if _on_gpu(x) else ref.gemm_gelu(x, w)
 
 
+def gemm_softcap(x, w, cap=0.0):
+    """fp32 logits with the tanh soft cap in the GEMM's epilogue on a GPU; see ``ops.reference.gemm_softcap``."""
+    return cuda_ops().gemm_softcap(x, w, cap) if _on_gpu(x) else ref.gemm_softcap(x, w, cap)
+
+
 def gemm_heads(x, w, gate=None, out=None):
     """Per-head product x [T, H, >= K] with w [H, N, K] -> [T, H, N]; see ``ops.reference.gemm_heads``."""
     return cuda_ops().gemm_heads(x, w, gate, out) if _on_gpu(x) else ref.gemm_heads(x, w, gate, out)

@@ -322,13 +322,14 @@ def _tma_ready(t, stride: int) -> bool:
     return t.dtype == torch.bfloat16 and stride % 8 == 0 and t.data_ptr() % 16 == 0
 
 
-def gemm_simt(x, w, y, T, N, K, ldx, ldy, *, bias=None, gate=None, ldg=0, batch=1, xs=0, ys=0, act=0):
+def gemm_simt(x, w, y, T, N, K, ldx, ldy, *, bias=None, gate=None, ldg=0, batch=1, xs=0, ys=0, act=0, cap=0.0):
     """CUDA-core GEMM (``csrc/gemm_simt.cu``): fp32 operands, or bf16 ones without the TMA's alignment."""
     elem = _mixed(x)
-    assert all(t is None or t.dtype == x.dtype for t in (w, y, bias, gate)), "operands of one dtype"
+    assert all(t is None or t.dtype == x.dtype for t in (w, bias, gate)), "operands of one dtype"
+    assert y.dtype == (torch.float32 if act == 2 else x.dtype)
     _check(lib().b200_gemm_simt(_p(x), _p(w), _p(y), _p(bias), _p(gate), c_int(T), c_int(N), c_int(K), c_int(batch),
                                 c_longlong(ldx), c_longlong(K), c_longlong(ldy), c_longlong(ldg), c_longlong(xs),
-                                c_longlong(ys), c_int(act), c_int(elem), _stream()), "gemm_simt")
+                                c_longlong(ys), c_int(act), c_float(cap), c_int(elem), _stream()), "gemm_simt")
     count_launch()
     return y
 
@@ -352,9 +353,25 @@ def gemm_gelu(x, w):
     else:
         _check(lib().b200_gemm_bf16_heads(_p(x2), _p(w), _p(y), c_void_p(0), c_int(T), c_int(N), c_int(K), c_int(1),
                                           c_int(x2.stride(0)), c_int(K), c_int(N), c_int(0), c_int(0), c_int(0),
-                                          c_int(1), _p(ws.status), c_int(_sms), _stream()), "gemm_gelu")
+                                          c_int(1), c_float(0), _p(ws.status), c_int(_sms), _stream()), "gemm_gelu")
     count_launch()
     return y.reshape(*lead, N)
+
+
+def gemm_softcap(x, w, cap: float = 0.0):
+    """fp32 cap * tanh((x @ w.T) / cap) straight from the accumulator (cap 0: x @ w.T): logits."""
+    (T, K), N = x.shape, w.shape[0]
+    y = torch.empty((T, N), dtype=torch.float32, device=x.device)
+    if T == 0:
+        return y
+    if not (_tma_ready(x, x.stride(0)) and _tma_ready(w, K)):
+        return gemm_simt(x, w, y, T, N, K, x.stride(0), N, act=2, cap=cap)
+    ws = Workspace.get(x.device)
+    _check(lib().b200_gemm_bf16_heads(_p(x), _p(w), _p(y), c_void_p(0), c_int(T), c_int(N), c_int(K), c_int(1),
+                                      c_int(x.stride(0)), c_int(K), c_int(N), c_int(0), c_int(0), c_int(0), c_int(2),
+                                      c_float(cap), _p(ws.status), c_int(_sms), _stream()), "gemm_softcap")
+    count_launch()
+    return y
 
 
 def gemm_heads(x, w, gate=None, out=None):
@@ -376,8 +393,8 @@ def gemm_heads(x, w, gate=None, out=None):
         return gemm_simt(x, w, y, T, N, K, ldx, ldy, gate=gate, ldg=ldg, batch=H, xs=xs, ys=ys)
     ws = Workspace.get(x.device)
     _check(lib().b200_gemm_bf16_heads(_p(x), _p(w), _p(y), _p(gate), c_int(T), c_int(N), c_int(K), c_int(H), c_int(ldx),
-                                      c_int(K), c_int(ldy), c_int(ldg), c_int(xs), c_int(ys), c_int(0), _p(ws.status),
-                                      c_int(_sms), _stream()), "gemm_heads")
+                                      c_int(K), c_int(ldy), c_int(ldg), c_int(xs), c_int(ys), c_int(0), c_float(0),
+                                      _p(ws.status), c_int(_sms), _stream()), "gemm_heads")
     count_launch()
     return y
 

@@ -61,6 +61,12 @@ def gemm_gelu(x: torch.Tensor, w: torch.Tensor) -> torch.Tensor:
     return F.gelu(x.float() @ w.float().t()).to(x.dtype)
 
 
+def gemm_softcap(x: torch.Tensor, w: torch.Tensor, cap: float = 0.0) -> torch.Tensor:
+    """fp32 logits cap * tanh((x @ w.T) / cap); cap 0: x @ w.T."""
+    y = x.float() @ w.float().t()
+    return softcap(y, cap) if cap else y
+
+
 def gemm_heads(x: torch.Tensor, w: torch.Tensor, gate: Optional[torch.Tensor] = None,
                out: Optional[torch.Tensor] = None) -> torch.Tensor:
     """Per head h: x[:, h, :K] (K = w.shape[2]) times w[h] [N, K] transposed -> [T, H, N], optionally times
