@@ -72,6 +72,11 @@ def parse_args():
     ap.add_argument("--enforce-eager", action="store_true")
     ap.add_argument("--warmup-requests", type=int, default=0,
                     help="requests per warm-up serve (0 = the full workload)")
+    ap.add_argument("--layer-bench", default="", choices=["", "mazivik"],
+                    help="instead of the serving workload: layer throughput and kernels of this model beside its "
+                         "closest neighbour, one JSON line per measurement")
+    ap.add_argument("--layer-size", default="2048x16,4096x32,7168x128", help="--layer-bench: width x heads, ...")
+    ap.add_argument("--layer-parts", default="layers,steps", help="--layer-bench: layers, steps or both")
     a = ap.parse_args()
     # request shapes of the target configurations
     shapes = {"llama-3.1-8b": (512, 1024, 128, 64, "tp"), "llama-3.1-70b-fp8": (512, 2048, 256, 128, "tp"),
@@ -166,6 +171,11 @@ def main():
     args = parse_args()
     if args.impl == "reference":
         print(json.dumps({"impl": "reference", "unavailable": REFERENCE_UNAVAILABLE}))
+        return 0
+    if args.layer_bench:
+        from vllm_torchtpu_b200.ops.bench_latent import run
+        for row in run(args.layer_size, args.layer_parts):
+            print(json.dumps(row))
         return 0
     import torch
     import torch.distributed as dist
