@@ -10,12 +10,13 @@ way the reference's ``check_and_update_config`` does
 from __future__ import annotations
 
 import json
-import math
 import os
 from dataclasses import dataclass, field, asdict
 from typing import Any, Optional
 
 import torch
+
+from .layer_specs import LatentMixerSpec, LayerSpec, RotarySpec, layer_specs  # noqa: F401
 
 _DTYPES = {
     "float32": torch.float32, "fp32": torch.float32, "float": torch.float32,
@@ -30,61 +31,9 @@ def parse_dtype(d) -> torch.dtype:
     return _DTYPES[str(d).replace("torch.", "")]
 
 
-@dataclass(frozen=True)
-class RotarySpec:
-    """Rotary embedding of one mixer: the first ``dims`` dimensions of the rotated vector turn by
-    ``position * base^(-2i / dims)``, optionally with YaRN ``scaling`` ({factor, original, fast, slow})."""
-    dims: int
-    base: float
-    scaling: Optional[dict] = None
-
-    @property
-    def rope_scaling(self) -> Optional[dict]:
-        """The same scaling under the names ``ops.reference.rope_inv_freq`` reads."""
-        if not self.scaling:
-            return None
-        s = self.scaling
-        return {"rope_type": "yarn", "factor": float(s["factor"]),
-                "original_max_position_embeddings": float(s["original"]), "beta_fast": float(s["fast"]),
-                "beta_slow": float(s["slow"]), "attention_factor": 0.1 * math.log(float(s["factor"])) + 1.0}
-
-
-@dataclass(frozen=True)
-class LatentMixerSpec:
-    """Sizes of one latent-attention mixer (multi-head latent attention with a query latent)."""
-    heads: int
-    dim: int                             # unrotated query / key dimensions per head
-    rot_dim: int                         # rotated ones (the key's are shared by all heads)
-    vdim: int
-    q_rank: int
-    kv_rank: int
-    scale: float
-    rot: RotarySpec
-    kv_from: Optional[int] = None        # layer whose cached latent and rotated key this layer reads
-    output_gate: bool = True             # heads times sigmoid(W_g x) in front of the output projection
-
-    @staticmethod
-    def from_dict(d: dict) -> "LatentMixerSpec":
-        r = d["rot"]
-        rot = RotarySpec(int(r["dims"]), float(r["base"]), r.get("scaling") or None)
-        src = d.get("kv_from")
-        if rot.dims > d["rot_dim"] or rot.dims % 2:
-            raise ValueError(f"rot.dims {rot.dims} must be even and at most rot_dim {d['rot_dim']}")
-        return LatentMixerSpec(int(d["heads"]), int(d["dim"]), int(d["rot_dim"]), int(d["vdim"]), int(d["q_rank"]),
-                               int(d["kv_rank"]), float(d["scale"]), rot, None if src is None else int(src))
-
-
-@dataclass(frozen=True)
-class LayerSpec:
-    """One entry of a checkpoint configuration that lists its layers one by one."""
-    mixer: LatentMixerSpec
-    ff: int = 0                          # width of the dense feed-forward, 0 = the layer has none
-    act: str = "gelu"
-
-
 @dataclass
 class ModelConfig:
-    architecture: str = "llama"          # llama | qwen3_moe | gpt_oss | deepseek_v3 | qwen3_next | kimi_linear | mazivik
+    architecture: str = "llama"          # llama | qwen3_moe | gpt_oss | deepseek_v3 | qwen3_next | kimi_linear | mazivik | popanex
     name: str = "tiny-llama"
     num_layers: int = 2
     hidden_size: int = 256
@@ -133,6 +82,7 @@ class ModelConfig:
     mla_use_nope: bool = False           # latent attention without rotary embeddings (Kimi-Linear: positions come from the KDA layers)
     layer_specs: tuple = ()              # models configured layer by layer (LayerSpec); the scalars above are maxima
     final_logit_softcap: Optional[float] = None    # logits = cap * tanh(logits / cap)
+    logit_scale: float = 1.0             # logits = scale * (head x)
     # sparse MLA (DSA indexer)
     index_topk: int = 0
     index_n_heads: int = 0
@@ -163,14 +113,17 @@ class ModelConfig:
         return self.kv_lora_rank > 0
 
     @property
-    def is_hybrid_gdn(self) -> bool:
-        return self.full_attention_interval > 0
+    def has_recurrent_state(self) -> bool:
+        """Some layers carry a state per request instead of a KV cache."""
+        return self.full_attention_interval > 0 or any(s.mixer.recurrent for s in self.layer_specs)
 
     def layer_is_moe(self, i: int) -> bool:
         return self.is_moe and i >= self.first_dense_layers
 
     def layer_is_full_attention(self, i: int) -> bool:
-        if not self.is_hybrid_gdn:
+        if self.layer_specs:
+            return not self.layer_specs[i].mixer.recurrent
+        if not self.full_attention_interval:
             return True
         return (i + 1) % self.full_attention_interval == 0
 
@@ -185,12 +138,7 @@ class ModelConfig:
     def num_params(self) -> int:
         h, L = self.hidden_size, self.num_layers
         n = 2 * self.vocab_size * h if not self.tie_word_embeddings else self.vocab_size * h
-        for s in self.layer_specs:
-            m = s.mixer
-            n += h * m.q_rank + m.q_rank * m.heads * (m.dim + m.rot_dim) + m.kv_rank * m.heads * (m.dim + m.vdim)
-            n += m.heads * m.vdim * h * (2 if m.output_gate else 1) + 2 * h * s.ff
-            if m.kv_from is None:
-                n += h * (m.kv_rank + m.rot_dim)
+        n += sum(s.num_params(h) for s in self.layer_specs)
         for i in range(0 if self.layer_specs else L):
             if self.is_mla:
                 qk = self.qk_nope_head_dim + self.qk_rope_head_dim
@@ -211,7 +159,7 @@ class ModelConfig:
     @staticmethod
     def from_hf_dict(cfg: dict, name: str = "") -> "ModelConfig":
         """Map a Hugging Face ``config.json`` dictionary to ModelConfig."""
-        if "architectures" not in cfg and cfg.get("architecture") == "Mazivik":
+        if "architectures" not in cfg and cfg.get("architecture") in ("Mazivik", "Popanex"):
             return ModelConfig.from_layer_list(cfg, name)
         arch = (cfg.get("architectures") or ["LlamaForCausalLM"])[0]
         mc = ModelConfig(name=name or cfg.get("_name_or_path", arch))
@@ -366,48 +314,64 @@ class ModelConfig:
 
     @staticmethod
     def from_layer_list(cfg: dict, name: str = "") -> "ModelConfig":
-        """Map a ``config.json`` that lists its layers one by one (``{"architecture": "Mazivik", "layers": [...],
-        "norm": {"eps"}, "vocab", "width", "logit_softcap"}``) to ModelConfig."""
-        specs = []
-        for i, layer in enumerate(cfg["layers"]):
-            if layer["type"] != "latent_attention":
-                raise ValueError(f"layer {i}: unknown mixer type {layer['type']!r}")
-            mlp = layer.get("mlp")
-            if mlp and mlp.get("kind") != "dense":
-                raise ValueError(f"layer {i}: unknown feed-forward kind {mlp.get('kind')!r}")
-            m = LatentMixerSpec.from_dict(layer["mixer"])
-            if m.kv_from is not None:
-                src = specs[m.kv_from].mixer if 0 <= m.kv_from < i else None
-                if src is None or src.kv_from is not None:
-                    raise ValueError(f"layer {i}: kv_from {m.kv_from} must name an earlier layer with a latent of its own")
-                if (src.kv_rank, src.rot_dim, src.rot) != (m.kv_rank, m.rot_dim, m.rot):
-                    raise ValueError(f"layer {i}: kv_rank, rot_dim and rotation differ from layer {m.kv_from}'s")
-            specs.append(LayerSpec(m, int(mlp["ff"]) if mlp else 0))
-        mixers = [s.mixer for s in specs]
-        mc = ModelConfig(architecture="mazivik", name=name or "mazivik", num_layers=len(specs),
-                         hidden_size=int(cfg["width"]), vocab_size=int(cfg["vocab"]), layer_specs=tuple(specs))
-        mc.num_q_heads = mc.num_kv_heads = max(m.heads for m in mixers)
-        mc.head_dim = max(m.dim + m.rot_dim for m in mixers)
-        mc.q_lora_rank, mc.kv_lora_rank = max(m.q_rank for m in mixers), max(m.kv_rank for m in mixers)
-        mc.qk_nope_head_dim, mc.qk_rope_head_dim = max(m.dim for m in mixers), max(m.rot_dim for m in mixers)
-        mc.v_head_dim = max(m.vdim for m in mixers)
-        mc.intermediate_size = max(s.ff for s in specs)
-        mc.hidden_act = "gelu"
+        """Map a ``config.json`` that lists its layers one by one (``{"architecture": "Mazivik" | "Popanex",
+        "layers": [...], "norm": {"eps"}, "vocab", "width", ...}``) to ModelConfig."""
+        arch = cfg["architecture"].lower()
+        build = {"mazivik": _mazivik_layers, "popanex": _popanex_layers}[arch]
+        mc = ModelConfig(architecture=arch, name=name or arch, num_layers=len(cfg["layers"]),
+                         hidden_size=int(cfg["width"]), vocab_size=int(cfg["vocab"]))
         mc.rms_norm_eps = float(cfg["norm"]["eps"])
-        mc.rope_theta, mc.rope_interleaved = mixers[0].rot.base, True
-        mc.rope_scaling = mixers[0].rot.rope_scaling
-        cap = cfg.get("logit_softcap")
-        mc.final_logit_softcap = float(cap) if cap else None
         mc.dtype = parse_dtype(cfg.get("torch_dtype", "bfloat16"))
-        # nothing in the configuration bounds a sequence: the range the rotation was scaled for is the default
-        spans = [m.rot.scaling["original"] * m.rot.scaling["factor"] for m in mixers if m.rot.scaling]
-        mc.max_model_len = int(max(spans)) if spans else 4096
+        mc.max_model_len = 4096          # nothing in such a configuration bounds a sequence
+        build(mc, cfg)
+        mc.intermediate_size = max(s.ff for s in mc.layer_specs)
         return mc
 
     @staticmethod
     def from_pretrained(path: str) -> "ModelConfig":
         with open(os.path.join(path, "config.json")) as f:
             return ModelConfig.from_hf_dict(json.load(f), name=os.path.basename(path.rstrip("/")))
+
+
+def _mazivik_layers(mc: ModelConfig, cfg: dict) -> None:
+    specs = layer_specs(cfg["layers"], ("latent_attention",), act="gelu", gated=False)
+    for i, s in enumerate(specs):
+        m = s.mixer
+        if m.kv_from is not None:
+            src = specs[m.kv_from].mixer if 0 <= m.kv_from < i else None
+            if src is None or src.kv_from is not None:
+                raise ValueError(f"layer {i}: kv_from {m.kv_from} must name an earlier layer with a latent of its own")
+            if (src.kv_rank, src.rot_dim, src.rot) != (m.kv_rank, m.rot_dim, m.rot):
+                raise ValueError(f"layer {i}: kv_rank, rot_dim and rotation differ from layer {m.kv_from}'s")
+    mc.layer_specs = tuple(specs)
+    mixers = [s.mixer for s in specs]
+    mc.num_q_heads = mc.num_kv_heads = max(m.heads for m in mixers)
+    mc.head_dim = max(m.dim + m.rot_dim for m in mixers)
+    mc.q_lora_rank, mc.kv_lora_rank = max(m.q_rank for m in mixers), max(m.kv_rank for m in mixers)
+    mc.qk_nope_head_dim, mc.qk_rope_head_dim = max(m.dim for m in mixers), max(m.rot_dim for m in mixers)
+    mc.v_head_dim = max(m.vdim for m in mixers)
+    mc.hidden_act = "gelu"
+    mc.rope_theta, mc.rope_interleaved = mixers[0].rot.base, True
+    mc.rope_scaling = mixers[0].rot.rope_scaling
+    cap = cfg.get("logit_softcap")
+    mc.final_logit_softcap = float(cap) if cap else None
+    # the range the rotation was scaled for
+    spans = [m.rot.scaling["original"] * m.rot.scaling["factor"] for m in mixers if m.rot.scaling]
+    if spans:
+        mc.max_model_len = int(max(spans))
+
+
+def _popanex_layers(mc: ModelConfig, cfg: dict) -> None:
+    specs = layer_specs(cfg["layers"], ("attention", "retention", "channel_delta"), act="gelu_tanh", gated=True)
+    mc.layer_specs = tuple(specs)
+    mc.hidden_act = "gelu_tanh"
+    mc.logit_scale = float(cfg.get("logit_scale", 1.0))
+    mixers = [s.mixer for s in specs]
+    att = [m for m in mixers if not m.recurrent]
+    mc.num_q_heads = max(m.heads for m in mixers)
+    mc.num_kv_heads = max((m.kv_heads for m in att), default=1)
+    mc.head_dim = max(max(m.dim, m.vdim) for m in att or mixers)
+    mc.attn_sinks = bool(att)
 
 
 def _preset(**kw) -> ModelConfig:
@@ -456,6 +420,22 @@ def model_preset(name: str) -> ModelConfig:
                 {"type": "latent_attention", "mixer": dict(mix, heads=6, vdim=24, q_rank=32, kv_from=0), "mlp": None},
                 {"type": "latent_attention", "mixer": dict(mix, heads=2, dim=40, kv_rank=72), "mlp": ff}]},
             name="tiny-mazivik")
+        mc.max_model_len, mc.init_std = 256, 0.1
+        return mc
+    if n in ("tiny-popanex",):
+        # every mixer, unequal sizes, a layer that runs a second time with a state of its own, layers without an MLP
+        ret = {"heads": 3, "dim": 24, "vdim": 40, "rot": {"base": 5000.0, "dims": 16}, "decay": [0.9, 0.97, 0.995]}
+        att = {"heads": 6, "kv_heads": 2, "dim": 24, "vdim": 32, "scale": 0.2, "q_temp": {"coef": 0.3, "every": 48}}
+        delta = {"heads": 4, "kv_heads": 2, "dim": 16, "vdim": 24, "conv": 3, "gate_rank": 12}
+        ff = {"kind": "dense", "ff": 136}
+        mc = ModelConfig.from_layer_list({
+            "architecture": "Popanex", "width": 96, "vocab": 320, "norm": {"eps": 1e-5}, "logit_scale": 1.5,
+            "torch_dtype": "float32", "layers": [
+                {"type": "channel_delta", "mixer": delta, "mlp": ff}, {"type": "attention", "mixer": att, "mlp": ff},
+                {"type": "retention", "mixer": ret, "mlp": None},
+                {"type": "retention", "mixer": ret, "mlp": None, "weights_of": 2},
+                {"type": "attention", "mixer": dict(att, heads=4, kv_heads=1, vdim=24), "mlp": None}]},
+            name="tiny-popanex")
         mc.max_model_len, mc.init_std = 256, 0.1
         return mc
     if n in ("tiny-odd-heads",):

@@ -19,23 +19,8 @@ import torch
 from .. import ops
 from ..config import ModelConfig
 from ..layers.latent_attention import LatentAttention
-from ..layers.linear import seeded_normal
 from ..layers.mlp import DenseMLP
-from ..parallel.communicator import get_tp_comm
-from .llama import LlamaForCausalLM
-
-
-class NoMLP:
-    """Stands for the feed-forward of a layer that has none."""
-
-    def linears(self):
-        return []
-
-    def init_dummy(self, std, seed):
-        pass
-
-    def weight_bytes(self):
-        return 0
+from .layer_list import LayerListForCausalLM, NoMLP, packed_loader, vector_loader
 
 
 class MazivikDecoderLayer:
@@ -61,59 +46,30 @@ class MazivikDecoderLayer:
         return hidden, residual
 
 
-class MazivikForCausalLM(LlamaForCausalLM):
+class MazivikForCausalLM(LayerListForCausalLM):
     layer_cls = MazivikDecoderLayer
-    float32_kernels = True              # every op of this model has a 32-bit CUDA kernel
+    fusion_reason = "latent attention with normalised sublayer outputs"
 
     # ---- weights -------------------------------------------------------------
-    def init_dummy(self) -> None:
-        cfg = self.cfg
-        std, seed = cfg.init_std, cfg.seed
-        self.embed = seeded_normal("model.embed_tokens", (cfg.vocab_size, cfg.hidden_size), std, cfg.dtype, self.device,
-                                   seed)
-        self.lm_head = self._shard_vocab(seeded_normal("lm_head", (cfg.vocab_size, cfg.hidden_size), std, cfg.dtype,
-                                                       self.device, seed))
-        for l in self.layers:
-            l.self_attn.init_dummy(std, seed)
-            l.mlp.init_dummy(std, seed)
-
-    def weight_bytes(self) -> int:
-        n = sum(t.numel() * t.element_size() for t in (self.embed, self.lm_head) if t is not None)
-        return n + sum(l.self_attn.weight_bytes() + l.mlp.weight_bytes() for l in self.layers)
-
     def checkpoint_groups(self) -> list:
         """[(checkpoint tensors that make up one parameter, loader of these tensors)] for ``models/loader.py``."""
-        def vector(t):
-            return lambda src: t.copy_(src.to(device=t.device, dtype=t.dtype))
-
-        def packed(lin):
-            return lambda *parts: lin.load_weight(torch.cat(parts, 0) if len(parts) > 1 else parts[0])
-
-        def embed(t):
-            self.embed = t.to(device=self.device, dtype=self.cfg.dtype).contiguous()
-
-        def head(t):
-            self.lm_head = self._shard_vocab(t.to(device=self.device, dtype=self.cfg.dtype).contiguous())
-        groups = [(("embed",), embed), (("head",), head), (("final.norm",), vector(self.norm))]
+        groups = self.embedding_groups()
         for l in self.layers:
             a, p = l.self_attn, f"l{l.idx}."
             m = p + "mix."
             own = a.dkv_norm is not None
-            groups += [((m + "dq",) + ((m + "dkv",) if own else ()) + (m + "g",), packed(a.inp)),
-                       ((m + "uq",), packed(a.uq)), ((m + "o",), packed(a.o)), ((m + "uk",), a.load_uk),
-                       ((m + "uv",), a.load_uv), ((m + "dq.norm",), vector(a.dq_norm)),
-                       ((p + "norm1",), vector(l.norm1))]
+            groups += [((m + "dq",) + ((m + "dkv",) if own else ()) + (m + "g",), packed_loader(a.inp)),
+                       ((m + "uq",), packed_loader(a.uq)), ((m + "o",), packed_loader(a.o)), ((m + "uk",), a.load_uk),
+                       ((m + "uv",), a.load_uv), ((m + "dq.norm",), vector_loader(a.dq_norm)),
+                       ((p + "norm1",), vector_loader(l.norm1))]
             if own:
-                groups.append(((m + "dkv.norm",), vector(a.dkv_norm)))
+                groups.append(((m + "dkv.norm",), vector_loader(a.dkv_norm)))
             if l.norm2 is not None:
-                groups += [((p + "norm2",), vector(l.norm2)), ((p + "mlp.up",), packed(l.mlp.up)),
-                           ((p + "mlp.down",), packed(l.mlp.down))]
+                groups += [((p + "norm2",), vector_loader(l.norm2)), ((p + "mlp.up",), packed_loader(l.mlp.up)),
+                           ((p + "mlp.down",), packed_loader(l.mlp.down))]
         return groups
 
     # ---- forward -------------------------------------------------------------
-    def setup_decode_fusion(self, kv_caches) -> None:
-        self.decode_mega, self.decode_mega_reason = None, "latent attention with normalised sublayer outputs"
-
     def forward(self, input_ids, meta, kv_caches, *, hidden=None, residual=None):
         """Returns (32-bit residual stream, None)."""
         if hidden is None:
@@ -124,19 +80,6 @@ class MazivikForCausalLM(LlamaForCausalLM):
 
     def finalize(self, hidden, residual):
         return ops.layer_norm(hidden, self.norm, self.cfg.rms_norm_eps)
-
-    def compute_logits(self, hidden_rows):
-        """fp32, soft-capped."""
-        cap = self.cfg.final_logit_softcap or 0.0
-        if getattr(self, "dp_vocab", None) is not None:
-            logits = self.dp_vocab.logits(hidden_rows, self.lm_head)
-            return ops.softcap(logits, cap) if cap else logits
-        logits = self.local_logits(hidden_rows)
-        comm = get_tp_comm()
-        return comm.all_gather(logits, dim=-1) if comm.size > 1 and self.vocab_shard is not None else logits
-
-    def local_logits(self, hidden_rows):
-        return ops.gemm_softcap(hidden_rows, self.lm_head, self.cfg.final_logit_softcap or 0.0)
 
     # ---- KV geometry -----------------------------------------------------------
     def _cache_owners(self) -> list:

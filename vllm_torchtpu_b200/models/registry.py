@@ -27,8 +27,11 @@ def get_model_class(cfg: ModelConfig):
     if a == "mazivik":
         from .mazivik import MazivikForCausalLM
         return MazivikForCausalLM
+    if a == "popanex":
+        from .popanex import PopanexForCausalLM
+        return PopanexForCausalLM
     raise ValueError(f"no model class for architecture {a!r}")
 
 
 def supported_architectures() -> list[str]:
-    return ["llama", "qwen3_moe", "gpt_oss", "deepseek_v3", "qwen3_next", "kimi_linear", "mazivik"]
+    return ["llama", "qwen3_moe", "gpt_oss", "deepseek_v3", "qwen3_next", "kimi_linear", "mazivik", "popanex"]

@@ -40,6 +40,14 @@ def layer_norm_add(y, residual, weight, eps):
         ref.layer_norm_add(y, residual, weight, eps)
 
 
+def add_rms_norm(y, residual, weight, eps, offset=0.0, update=True):
+    """(h, fp32 r) of r = residual (+ y), h = RMS norm of r times (offset + weight); an fp32 residual is updated in
+    place on a GPU.  ``y`` None: r = residual.  Without ``update`` the stream is only read and r is None."""
+    y = materialize(y)
+    return cuda_ops().add_rms_norm(y, residual, weight, eps, offset, update) if _on_gpu(residual) else \
+        ref.add_rms_norm(y, residual, weight, eps, offset, update)
+
+
 def softcap(x, cap):
     return cuda_ops().softcap(x, cap) if _on_gpu(x) else ref.softcap(x, cap)
 
@@ -76,9 +84,23 @@ def gemm_gelu(x, w):
     return cuda_ops().gemm_gelu(x, w) if _on_gpu(x) else ref.gemm_gelu(x, w)
 
 
-def gemm_softcap(x, w, cap=0.0):
-    """fp32 logits with the tanh soft cap in the GEMM's epilogue on a GPU; see ``ops.reference.gemm_softcap``."""
-    return cuda_ops().gemm_softcap(x, w, cap) if _on_gpu(x) else ref.gemm_softcap(x, w, cap)
+def gemm_softcap(x, w, cap=0.0, scale=1.0):
+    """fp32 logits with a factor and the tanh soft cap in the GEMM's epilogue on a GPU; see
+    ``ops.reference.gemm_softcap``."""
+    return cuda_ops().gemm_softcap(x, w, cap, scale) if _on_gpu(x) else ref.gemm_softcap(x, w, cap, scale)
+
+
+def gemm_gated(x, w, act):
+    """act(x @ w[:I].T, x @ w[I:].T), in the GEMM's epilogue where it has the activation (silu, gelu_tanh)."""
+    return cuda_ops().gemm_gated(x, w, act) if _on_gpu(x) else ref.gated_act_and_mul(ref.gemm(x, w), act)
+
+
+def carried_state_attention(plan, row, decay_in, gate, meta, cache):
+    """Linear attention with a carried state; see ``ops.linear_attention``."""
+    if _on_gpu(row):
+        return cuda_ops().carried_state_attention(plan, row, decay_in, gate, meta, cache)
+    from .linear_attention import linear_attention_reference
+    return linear_attention_reference(plan, row, decay_in, gate, meta, cache)
 
 
 def gemm_heads(x, w, gate=None, out=None):
@@ -104,6 +126,11 @@ def rope_and_cache(qkv, positions, inv_freq, kv_cache, slot_mapping, num_q_heads
     f = cuda_ops().rope_and_cache if _on_gpu(qkv) else ref.rope_and_cache
     return f(qkv, positions, inv_freq, kv_cache, slot_mapping, num_q_heads, num_kv_heads, head_dim,
              interleaved, q_norm_w, k_norm_w, eps, k_scale, v_scale)
+
+
+def norm_and_cache(qkv, positions, kv_cache, slot_mapping, *a, **kw):
+    f = cuda_ops().norm_and_cache if _on_gpu(qkv) else ref.norm_and_cache
+    return f(qkv, positions, kv_cache, slot_mapping, *a, **kw)
 
 
 def paged_attention(q, kv_cache, meta, scale, *, sliding_window=None, softcap=None, sinks=None,

@@ -53,6 +53,15 @@ def layer_norm_add(y: torch.Tensor, residual: torch.Tensor, weight: torch.Tensor
     return r.to(weight.dtype), r
 
 
+def add_rms_norm(y: Optional[torch.Tensor], residual: torch.Tensor, weight: torch.Tensor, eps: float,
+                 offset: float = 0.0, update: bool = True):
+    """32-bit residual stream in front of a sublayer: r = residual (+ y); h = r / rms(r) * (offset + w).
+    Returns (h in the weight's dtype, r fp32 or None without ``update``)."""
+    r = residual.float() if y is None else residual.float() + y.float()
+    h = r * torch.rsqrt(r.pow(2).mean(-1, keepdim=True) + eps) * (offset + weight.float())
+    return h.to(weight.dtype), (r if update else None)
+
+
 def softcap(x: torch.Tensor, cap: float) -> torch.Tensor:
     return cap * torch.tanh(x.float() / cap)
 
@@ -61,9 +70,9 @@ def gemm_gelu(x: torch.Tensor, w: torch.Tensor) -> torch.Tensor:
     return F.gelu(x.float() @ w.float().t()).to(x.dtype)
 
 
-def gemm_softcap(x: torch.Tensor, w: torch.Tensor, cap: float = 0.0) -> torch.Tensor:
-    """fp32 logits cap * tanh((x @ w.T) / cap); cap 0: x @ w.T."""
-    y = x.float() @ w.float().t()
+def gemm_softcap(x: torch.Tensor, w: torch.Tensor, cap: float = 0.0, scale: float = 1.0) -> torch.Tensor:
+    """fp32 logits cap * tanh(scale * (x @ w.T) / cap); cap 0: scale * (x @ w.T)."""
+    y = scale * (x.float() @ w.float().t())
     return softcap(y, cap) if cap else y
 
 
@@ -248,6 +257,35 @@ def rope_and_cache(qkv, positions, inv_freq, kv_cache, slot_mapping, num_q_heads
         else:
             write_kv_cache(kv_cache, k, v, slot_mapping)
     return q.contiguous()
+
+
+def query_temperature(positions: torch.Tensor, coef: float, every: int) -> torch.Tensor:
+    """1 + coef * ln(floor((p + 1) / every) + 1) of every position, fp32."""
+    return 1.0 + coef * torch.log(torch.div(positions + 1, every, rounding_mode="floor").float() + 1.0)
+
+
+def norm_and_cache(qkv, positions, kv_cache, slot_mapping, num_q_heads, num_kv_heads, dim, vdim, q_norm_w=None,
+                   k_norm_w=None, eps: float = 1e-6, q_temp=None, q_sumsq=None, k_sumsq=None, norm_sizes=None,
+                   offsets=None):
+    """Split packed q|k|v (k and v from columns ``offsets`` on) without rotation: RMS norm over the whole q and k rows (weights of their full length), the
+    query temperature ``q_temp`` = (coef, every), k and v written to the pages.  Heads are zero-padded to the head
+    size D of the cache; returns q [T, Hq, D].  ``q_sumsq`` / ``k_sumsq`` [T] with ``norm_sizes``: squared sums
+    over rows that are sharded (this rank holds a part of them)."""
+    T, D = qkv.shape[0], kv_cache.shape[4]
+    nq, nk = num_q_heads * dim, num_kv_heads * dim
+    k0, v0 = offsets or (nq, nq + nk)
+    q, k, v = qkv[:, :nq].float(), qkv[:, k0:k0 + nk].float(), qkv[:, v0:v0 + num_kv_heads * vdim]
+    if q_norm_w is not None:
+        sizes = norm_sizes or (nq, nk)
+        ssq = q.pow(2).sum(-1) if q_sumsq is None else q_sumsq
+        ssk = k.pow(2).sum(-1) if k_sumsq is None else k_sumsq
+        q = q * torch.rsqrt(ssq / sizes[0] + eps)[:, None] * q_norm_w.float()
+        k = k * torch.rsqrt(ssk / sizes[1] + eps)[:, None] * k_norm_w.float()
+    if q_temp is not None:
+        q = q * query_temperature(positions, *q_temp)[:, None]
+    pad = lambda t, h, d: F.pad(t.reshape(T, h, d), (0, D - d)).to(qkv.dtype)         # noqa: E731
+    write_kv_cache(kv_cache, pad(k, num_kv_heads, dim), pad(v, num_kv_heads, vdim), slot_mapping)
+    return pad(q, num_q_heads, dim).contiguous()
 
 
 def paged_attention(q, kv_cache, block_tables, seq_lens, query_start_loc, scale, *,

@@ -43,7 +43,7 @@ class PcpStaticSupportValidator:
             raise ValueError("sliding-window models are not supported under PCP")
         if self.cfg.speculative:
             raise ValueError("speculative decoding is not supported under PCP")
-        if m.is_mla or getattr(m, "is_hybrid_gdn", False):
+        if m.is_mla or getattr(m, "has_recurrent_state", False):
             raise ValueError("PCP in the engine splits GQA attention layers; latent-attention and linear-attention "
                              "models are not supported")
         if p.enable_expert_parallel or p.data_parallel_size > 1:

@@ -59,7 +59,7 @@ def validate_pipeline_parallel_config(cfg) -> None:
     for lo, hi in partition_layers(m.num_layers, pp):
         if hi <= lo:
             raise ValueError("a pipeline stage would hold no layer")
-        if m.is_hybrid_gdn and not any(m.layer_is_full_attention(i) for i in range(lo, hi)):
+        if m.has_recurrent_state and not any(m.layer_is_full_attention(i) for i in range(lo, hi)):
             raise ValueError(f"pipeline stage with layers [{lo},{hi}) holds no full-attention layer")
     if cfg.kv_transfer and cfg.kv_transfer.get("kv_connector") not in (
             "B200P2PConnector", "B200HostConnector", "B200MultiConnector", "B200OffloadingConnector"):

@@ -239,7 +239,7 @@ class B200Platform:
             method = cfg.speculative.get("method")
             if method not in cls.supported_spec_methods:
                 raise ValueError(f"speculative method {method!r} not in {cls.supported_spec_methods}")
-            if m.is_hybrid_gdn and s.async_scheduling:
+            if m.has_recurrent_state and s.async_scheduling:
                 # rejected drafts advance the recurrent state; it is rebuilt (snapshot + replay of the accepted
                 # rows, runner/spec_boundary_state.py) when the host has the step's tokens, before the next launch
                 logger.info("speculative decoding on a linear-attention hybrid: async scheduling switched off")

@@ -250,6 +250,8 @@ class ModelRunner:
         per_block = self.model.kv_bytes_per_block(self.block_size, kv_dtype)
         if self.extra_kv_layers:
             per_block += self.extra_kv_layers * per_block // max(1, len(self.model.layers))
+        if not per_block:
+            return self.max_reqs * self.batch.max_blocks + 1      # no layer has a KV cache: blocks are only counted
         if c.kv_cache_memory_bytes:
             return max(2, c.kv_cache_memory_bytes // per_block)
         if not self.is_cuda:
@@ -786,7 +788,7 @@ class ModelRunner:
         meta = self._make_meta(p)
         meta.pcp = self._pcp_plan
         self._pending_rollback = None
-        if p.get("has_spec") and self.mcfg.is_hybrid_gdn:
+        if p.get("has_spec") and self.mcfg.has_recurrent_state:
             # recurrent layers fold all k + 1 rows into their state: keep what it takes to undo rejected ones
             from .spec_boundary_state import StateRollback
             k_, qsl_ = p["spec_k"], p["qsl_np"]

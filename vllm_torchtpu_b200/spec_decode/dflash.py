@@ -46,7 +46,7 @@ class DFlashProposer:
         self.runner, self.cfg = runner, cfg
         m = self.m = cfg.model
         self.device, self.dtype, self.eps = runner.device, m.dtype, m.rms_norm_eps
-        if runner.dcp_size > 1 or m.is_hybrid_gdn or m.is_mla:
+        if runner.dcp_size > 1 or m.has_recurrent_state or m.is_mla:
             raise ValueError("block drafting is built for GQA attention targets without context parallelism")
         model = runner.model
         if not hasattr(model, "aux_layers"):

@@ -74,7 +74,7 @@ class DraftLayerProposer:
         # on a linear-attention hybrid the module is a full-attention layer: build it at the index of the
         # target's last full-attention layer and give it a cache of that layer's shape
         self.build_idx = L
-        if m.is_hybrid_gdn:
+        if m.has_recurrent_state:
             self.build_idx = max(i for i in range(L) if m.layer_is_full_attention(i))
         self.layer = model.layer_cls(self.build_idx, m, self.device, quant)
         H = m.hidden_size
@@ -111,7 +111,7 @@ class DraftLayerProposer:
         def blank(c):
             return torch.zeros_like(c) if torch.is_tensor(c) else type(c)(blank(x) for x in c)
         # the draft layer has the shape of the target layer it was modelled on
-        self.kv_cache = blank(runner.kv_caches[self.build_idx - model.layer_range[0]] if m.is_hybrid_gdn
+        self.kv_cache = blank(runner.kv_caches[self.build_idx - model.layer_range[0]] if m.has_recurrent_state
                               else runner.kv_caches[-1])
         self._res = None
         self.last_confidences: dict = {}
