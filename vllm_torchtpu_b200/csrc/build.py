@@ -75,6 +75,9 @@ def _headers_mtime() -> float:
 FAMILY_SOURCES = {
     "mazivik": ("attention_mla.cu", "elementwise.cu", "gemm_2sm_tcgen05.cu", "gemm_simt.cu", "gemm_tcgen05.cu",
                 "layer_norm.cu", "runtime.cu", "sample.cu"),
+    "popanex": ("attention.cu", "attention_simt.cu", "attention_tc.cu", "elementwise.cu", "gemm_2sm_tcgen05.cu",
+                "gemm_simt.cu", "gemm_tcgen05.cu", "layer_norm.cu", "linear_attention.cu", "norm_cache.cu", "runtime.cu",
+                "sample.cu"),
 }
 
 

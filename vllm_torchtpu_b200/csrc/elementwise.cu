@@ -125,6 +125,30 @@ __global__ void gated_act_kernel(const __nv_bfloat16* __restrict__ x, __nv_bfloa
   }
 }
 
+// the same activation, element by element: 32-bit rows, and bf16 rows that are no multiple of 8 wide
+__device__ __forceinline__ float act_load(float v) { return v; }
+__device__ __forceinline__ float act_load(__nv_bfloat16 v) { return __bfloat162float(v); }
+__device__ __forceinline__ void act_store(float* p, float v) { *p = v; }
+__device__ __forceinline__ void act_store(__nv_bfloat16* p, float v) { *p = __float2bfloat16(v); }
+template <typename E>
+__global__ void gated_act_any_kernel(const E* __restrict__ x, E* __restrict__ y, int T, int I, int act, float a, float b) {
+  const size_t total = (size_t)T * I;
+  for (size_t idx = (size_t)blockIdx.x * blockDim.x + threadIdx.x; idx < total; idx += (size_t)gridDim.x * blockDim.x) {
+    const size_t t = idx / I;
+    const float g = act_load(x[t * I + idx]), u = act_load(x[t * I + idx + I]);
+    float v;
+    switch (act) {
+      case 0: v = g / (1.f + expf(-g)) * u; break;
+      case 1: v = gated_act<1>(g, u, a, b); break;
+      case 2: v = gated_act<2>(g, u, a, b); break;
+      case 3: v = gated_act<3>(g, u, a, b); break;
+      case 4: v = gated_act<4>(g, u, a, b); break;
+      default: v = gated_act<5>(g, u, a, b); break;
+    }
+    act_store(y + idx, v);
+  }
+}
+
 // out[t] = table[ token_src[t] >= 0 ? last_tokens[token_src[t]] : ids[t] ]
 // (rows of n pieces of type V: 16 bytes, or 2 where a row is no multiple of that)
 template <typename V>
@@ -302,12 +326,24 @@ extern "C" int b200_silu_and_mul(const void* x, void* y, int T, int I, cudaStrea
 }
 
 // x [T, 2I] (gate columns first) -> y [T, I]; act and its parameters a, b as listed at gated_act.
-extern "C" int b200_gated_act(const void* x, void* y, int T, int I, int act, float a, float b,
+// elem: 2 = bf16, 4 = fp32
+extern "C" int b200_gated_act(const void* x, void* y, int T, int I, int act, float a, float b, int elem,
                               cudaStream_t stream) {
   if (T == 0) return 0;
-  if (I % 8 || act < 0 || act > 5) {
-    b200_set_last_error("gated_act: width must be a multiple of 8, activation 0..5", __FILE__, __LINE__);
+  if (act < 0 || act > 5) {
+    b200_set_last_error("gated_act: activation 0..5", __FILE__, __LINE__);
     return -1;
+  }
+  if (elem == 4 || I % 8 || ((uintptr_t)x | (uintptr_t)y) % 16) {
+    size_t n = ((size_t)T * I + 255) / 256;
+    const int grid = n > 148 * 16 ? 148 * 16 : (int)n;
+    if (elem == 4)
+      gated_act_any_kernel<float><<<grid, 256, 0, stream>>>((const float*)x, (float*)y, T, I, act, a, b);
+    else
+      gated_act_any_kernel<__nv_bfloat16><<<grid, 256, 0, stream>>>((const __nv_bfloat16*)x, (__nv_bfloat16*)y, T, I,
+                                                                    act, a, b);
+    B200_CUDA_CHECK(cudaGetLastError());
+    return 0;
   }
   size_t total = (size_t)T * (I / 8);
   int blocks = (int)((total + 255) / 256);

@@ -120,12 +120,12 @@ __device__ __forceinline__ void decode_work(int w, const Params& p, int& n_pair,
   n_pair = first + rem - t_tile * gsize;
 }
 
-// EPI 0: bias, 1: SwiGLU, 2: gelu (erf)
+// EPI 0: bias, 1: SwiGLU, 2: gelu (erf), 3: gate and up as in 1 with gelu in its tanh form
 template <int EPI>
 __global__ void __cluster_dims__(2, 1, 1) __launch_bounds__(THREADS, 1)
 gemm_bf16_2sm_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant__ CUtensorMap tmX,
                      const Params p) {
-  constexpr bool SWIGLU = EPI == 1;
+  constexpr bool SWIGLU = EPI == 1 || EPI == 3;
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
   uint64_t* bars = reinterpret_cast<uint64_t*>(smem + STAGES * STAGE_BYTES);
@@ -278,7 +278,7 @@ gemm_bf16_2sm_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_const
               for (int j = 0; j < 16; ++j) {
                 if (c0 + 16 + j < t_valid) {
                   const float gv = buf[(16 + j) * 32 + lane], uv = __uint_as_float(r[16 + j]);
-                  yp[(size_t)j * p.ldy] = __float2bfloat16(__fdividef(gv, 1.f + __expf(-gv)) * uv);
+                  yp[(size_t)j * p.ldy] = __float2bfloat16(EPI == 3 ? gated_pair<true>(gv, uv) : __fdividef(gv, 1.f + __expf(-gv)) * uv);
                 }
               }
             } else {             // gate warp: columns 0-15, up values from the partner
@@ -287,7 +287,7 @@ gemm_bf16_2sm_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_const
               for (int j = 0; j < 16; ++j) {
                 if (c0 + j < t_valid) {
                   const float gv = __uint_as_float(r[j]), uv = buf[j * 32 + lane];
-                  yp[(size_t)j * p.ldy] = __float2bfloat16(__fdividef(gv, 1.f + __expf(-gv)) * uv);
+                  yp[(size_t)j * p.ldy] = __float2bfloat16(EPI == 3 ? gated_pair<true>(gv, uv) : __fdividef(gv, 1.f + __expf(-gv)) * uv);
                 }
               }
             }
@@ -450,9 +450,10 @@ extern "C" int b200_gemm_bf16_gelu_2sm(const void* X, const void* W, void* Y, in
   return gemm_bf16_2sm(X, W, Y, nullptr, T, N, K, ldx, ldw, ldy, status, num_sms, 1, stream);
 }
 
-// Y[T, I] = silu(X * W[0:I]^T) * (X * W[I:2I]^T); W [2I, K] row stride ldw.
+// Y[T, I] = act(X * W[0:I]^T) * (X * W[I:2I]^T), act silu or gelu (tanh form); W [2I, K] row stride ldw.
 extern "C" int b200_gemm_bf16_swiglu_2sm(const void* X, const void* W, void* Y, int T, int I, int K, int ldx,
-                                         int ldw, int ldy, int* status, int num_sms, cudaStream_t stream) {
+                                         int ldw, int ldy, int gelu_tanh, int* status, int num_sms,
+                                         cudaStream_t stream) {
   using namespace b200;
   using namespace b200::g2;
   if (T <= 0 || I <= 0 || K <= 0) return 0;
@@ -474,5 +475,5 @@ extern "C" int b200_gemm_bf16_swiglu_2sm(const void* X, const void* W, void* Y, 
   if (rc) return rc;
   rc = operand_map(&tmX, X, (uint64_t)T, (uint64_t)K, (uint64_t)ldx * 2);
   if (rc) return rc;
-  return launch_pairs<1>(tmW, tmX, p, num_sms, stream);
+  return gelu_tanh ? launch_pairs<3>(tmW, tmX, p, num_sms, stream) : launch_pairs<1>(tmW, tmX, p, num_sms, stream);
 }

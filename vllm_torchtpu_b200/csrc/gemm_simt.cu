@@ -4,7 +4,7 @@
 //
 //   Y[t, b * ys + n] = act( sum_k X[t, b * xs + k] * W[b * N + n, k] + bias[n] ) [ * sigmoid(G[t, b * N + n]) ]
 //
-// act: 0 none, 1 gelu (erf), 2 soft cap (cap * tanh(. / cap), cap 0: none) with fp32 output.  64 x 64 output tile per CTA, 4 x 4 per thread, 16-wide K slices in shared memory.
+// act: 0 none, 1 gelu (erf), 2 out_scale and soft cap (cap * tanh(. / cap), cap 0: none) with fp32 output.  64 x 64 output tile per CTA, 4 x 4 per thread, 16-wide K slices in shared memory.
 #include "common.cuh"
 
 namespace b200 {
@@ -20,7 +20,7 @@ struct Params {
   const void *x, *w, *bias, *gate;
   void* y;
   int T, N, K, batch, act, y_f32;
-  float cap;
+  float cap, out_scale;
   long long ldx, ldw, ldy, ldg, xs, ys;
 };
 
@@ -71,7 +71,7 @@ __global__ void __launch_bounds__(256) gemm_kernel(const Params p) {
         float v = acc[i][j];
         if (p.bias) v += to_f(reinterpret_cast<const E*>(p.bias)[n]);
         if (p.act == 1) v = gelu_erf(v);
-        if (p.act == 2) v = soft_cap(v, p.cap);
+        if (p.act == 2) v = soft_cap(v * p.out_scale, p.cap);
         if (p.gate) {
           const float g = to_f(reinterpret_cast<const E*>(p.gate)[(size_t)t * p.ldg + (size_t)b * p.N + n]);
           v *= 1.f / (1.f + expf(-g));
@@ -91,10 +91,10 @@ __global__ void __launch_bounds__(256) gemm_kernel(const Params p) {
 // elem: 2 = bf16, 4 = fp32 (all operands alike); strides in elements.
 extern "C" int b200_gemm_simt(const void* x, const void* w, void* y, const void* bias, const void* gate, int T, int N,
                               int K, int batch, long long ldx, long long ldw, long long ldy, long long ldg,
-                              long long xs, long long ys, int act, float cap, int elem, cudaStream_t stream) {
+                              long long xs, long long ys, int act, float cap, float out_scale, int elem, cudaStream_t stream) {
   using namespace b200;
   if (T <= 0 || N <= 0 || batch <= 0) return 0;
-  simt::Params p{x, w, bias, gate, y, T, N, K, batch, act, act == 2 ? 1 : 0, cap, ldx, ldw, ldy, ldg, xs, ys};
+  simt::Params p{x, w, bias, gate, y, T, N, K, batch, act, act == 2 ? 1 : 0, cap, out_scale, ldx, ldw, ldy, ldg, xs, ys};
   const long long gx = (long long)batch * ((N + simt::TN - 1) / simt::TN);
   int gy = (T + simt::TM - 1) / simt::TM;
   if (gy > 65535) gy = 65535;

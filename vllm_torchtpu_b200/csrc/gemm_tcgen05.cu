@@ -99,11 +99,12 @@ struct GemmParams {
   unsigned long long ag_done_off;
   int ag_flip;
   unsigned long long* dbg;               // optional: per-CTA phase timestamps (ns), 16 slots per CTA
-  // ---- MODE 3: epilogue (act 0 none / 1 gelu / 2 fp32 output Yf with the soft cap cap * tanh(y / cap), cap 0: none;
+  // ---- gate / up pairs: act 0 silu, 3 gelu (tanh form)
+  // ---- MODE 3: epilogue (act 0 none / 1 gelu / 2 fp32 output Yf: out_scale * y, then the soft cap (cap 0: none);
   // optional gate: y *= sigmoid(gate[t, b * N + n])) and batch over heads: head b reads activation columns from
   // b * x_head_cols, weight rows from b * N and writes output columns from b * y_head_cols
   int act, batch, x_head_cols, y_head_cols, ldg;
-  float cap;
+  float cap, out_scale;
   const __nv_bfloat16* gate;
   float* Yf;
   int* epoch_ptr;                        // local: epoch of the last completed fused launch
@@ -341,10 +342,13 @@ __device__ __forceinline__ void cluster_reduce_cols(const GemmParams& p, const W
 #pragma unroll
           for (int r2 = 0; r2 < SMAX; ++r2)
             if (r2 < S) { u.x += vu[ci][r2].x; u.y += vu[ci][r2].y; u.z += vu[ci][r2].z; u.w += vu[ci][r2].w; }
-          a.x = a.x / (1.f + __expf(-a.x)) * u.x;
-          a.y = a.y / (1.f + __expf(-a.y)) * u.y;
-          a.z = a.z / (1.f + __expf(-a.z)) * u.z;
-          a.w = a.w / (1.f + __expf(-a.w)) * u.w;
+          if (p.act == 3) {
+            a.x = gated_pair<true>(a.x, u.x); a.y = gated_pair<true>(a.y, u.y);
+            a.z = gated_pair<true>(a.z, u.z); a.w = gated_pair<true>(a.w, u.w);
+          } else {
+            a.x = gated_pair<false>(a.x, u.x); a.y = gated_pair<false>(a.y, u.y);
+            a.z = gated_pair<false>(a.z, u.z); a.w = gated_pair<false>(a.w, u.w);
+          }
         }
         if (MODE == 3 && p.act == 1) {           // (no bias in this mode)
           a.x = gelu_erf(a.x); a.y = gelu_erf(a.y); a.z = gelu_erf(a.z); a.w = gelu_erf(a.w);
@@ -353,7 +357,7 @@ __device__ __forceinline__ void cluster_reduce_cols(const GemmParams& p, const W
           const float vals[4] = {a.x, a.y, a.z, a.w};
 #pragma unroll
           for (int j = 0; j < 4; ++j)
-            if (n4 + j < p.N) p.Yf[(size_t)(wk.t_row + c) * p.ldy + n4 + j] = soft_cap(vals[j], p.cap);
+            if (n4 + j < p.N) p.Yf[(size_t)(wk.t_row + c) * p.ldy + n4 + j] = soft_cap(vals[j] * p.out_scale, p.cap);
           continue;
         }
         for (int d = 0; d < ndst; ++d) {
@@ -618,12 +622,18 @@ gemm_bf16_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant_
           tmem_ld_wait();
           if (n < p.N) {
             __nv_bfloat16* yp = dst_base + (size_t)(t0 + c0) * p.ldy + n;
+            if (p.act == 3) {
 #pragma unroll
-            for (int j = 0; j < 32; ++j) {
-              if (c0 + j < t_valid) {
-                const float gv = __uint_as_float(g[j]), uv = __uint_as_float(u[j]);
-                yp[(size_t)j * p.ldy] = __float2bfloat16(gv / (1.f + __expf(-gv)) * uv);
-              }
+              for (int j = 0; j < 32; ++j)
+                if (c0 + j < t_valid)
+                  yp[(size_t)j * p.ldy] =
+                      __float2bfloat16(gated_pair<true>(__uint_as_float(g[j]), __uint_as_float(u[j])));
+            } else {
+#pragma unroll
+              for (int j = 0; j < 32; ++j)
+                if (c0 + j < t_valid)
+                  yp[(size_t)j * p.ldy] =
+                      __float2bfloat16(gated_pair<false>(__uint_as_float(g[j]), __uint_as_float(u[j])));
             }
           }
         }
@@ -754,7 +764,7 @@ gemm_bf16_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant_
                   float* yf = p.Yf + (size_t)(t0 + c0) * p.ldy + n;
 #pragma unroll
                   for (int j = 0; j < 32; ++j)
-                    if (c0 + j < t_valid) yf[(size_t)j * p.ldy] = soft_cap(__uint_as_float(r[j]), p.cap);
+                    if (c0 + j < t_valid) yf[(size_t)j * p.ldy] = soft_cap(__uint_as_float(r[j]) * p.out_scale, p.cap);
                   continue;
                 }
                 if (p.act == 1) {
@@ -1444,10 +1454,10 @@ extern "C" int b200_gemm_bf16(const void* X, const void* W, void* Y, const void*
 // (heads), act 0 none / 1 gelu (erf).  X row stride ldx, W [batch * N, K] row stride ldw, Y row stride ldy.  A head
 // whose K is no multiple of the 64-wide K block reads into its neighbour's columns; those meet the zero fill
 // behind the weight's K columns.
-// act 2: Y is fp32 and holds cap * tanh(. / cap) (cap 0: the products themselves).
+// act 2: Y is fp32 and holds cap * tanh(out_scale * . / cap) (cap 0: out_scale * the products).
 extern "C" int b200_gemm_bf16_heads(const void* X, const void* W, void* Y, const void* gate, int T, int N, int K,
                                     int batch, int ldx, int ldw, int ldy, int ldg, int xs, int ys, int act, float cap,
-                                    int* status, int num_sms, cudaStream_t stream) {
+                                    float out_scale, int* status, int num_sms, cudaStream_t stream) {
   using namespace b200;
   if (T <= 0 || N <= 0 || K <= 0 || batch <= 0) return 0;
   if (ldx % 8 || ldw % 8 || xs % 8) {
@@ -1460,6 +1470,7 @@ extern "C" int b200_gemm_bf16_heads(const void* X, const void* W, void* Y, const
   p.Y = reinterpret_cast<__nv_bfloat16*>(Y);
   p.Yf = reinterpret_cast<float*>(Y);
   p.cap = cap;
+  p.out_scale = out_scale;
   if (act == 2 && (batch > 1 || gate != nullptr)) {
     b200_set_last_error("gemm_heads: fp32 output is for one ungated product", __FILE__, __LINE__);
     return -3;
@@ -1610,9 +1621,10 @@ static void init_params(GemmParams& p, void* Y, int T, int N, int K, int ldy, in
 }
 }  // namespace b200
 
-// Y[T, I] = silu(X * Wg^T) * (X * Wu^T) with W = [gate rows (I) ; up rows (I)] x K packed as [2I, K].
+// Y[T, I] = act(X * Wg^T) * (X * Wu^T) with W = [gate rows (I) ; up rows (I)] x K packed as [2I, K]; act: silu, or
+// gelu in its tanh form.
 extern "C" int b200_gemm_bf16_swiglu(const void* X, const void* W, void* Y, int T, int I, int K, int ldx,
-                                     int ldw, int ldy, int* status, int num_sms, cudaStream_t stream) {
+                                     int ldw, int ldy, int gelu_tanh, int* status, int num_sms, cudaStream_t stream) {
   using namespace b200;
   if (T <= 0 || I <= 0 || K <= 0) return 0;
   if (K % 8 || ldx % 8 || ldw % 8) {
@@ -1623,6 +1635,7 @@ extern "C" int b200_gemm_bf16_swiglu(const void* X, const void* W, void* Y, int 
   GemmParams p;
   init_params(p, Y, T, I, K, ldy, bn, status);
   p.up_row_off = I;
+  p.act = gelu_tanh ? 3 : 0;
   p.w_evict_first = (p.t_tiles == 1) ? 1 : 0;
   {
     // few output tiles (small I per rank under tensor parallelism): split K over a cluster so that

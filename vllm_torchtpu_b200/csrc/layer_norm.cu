@@ -4,6 +4,10 @@
 //   ADD:    r' = r + LN(y) * w     (r' fp32, also stored rounded as the next projection's input)
 //   plain:  o  = LN(x) * w
 //
+// and of blocks that normalise the INPUT of a sublayer (RMS norm, weight stored with an offset):
+//
+//   add_rms: r' = r (+ y),  o = r' / rms(r') * (offset + w)     (r' fp32)
+//
 // mean and variance (mean of the squared deviations) in fp32 over the row, which stays in shared memory between
 // the passes.  Also the tanh soft cap of the logits.
 #include "common.cuh"
@@ -114,6 +118,65 @@ static int launch_v(const void* x, const void* res, const void* w, void* res_out
   return launch<1, TX, TR, TO, ADD>(x, res, w, res_out, out, T, H, eps, stream);
 }
 
+// One CTA per row.  TY: type of the sublayer output y (null: nothing is added), TR: of the stream that comes in, TO: of
+// w and of the normalised output; res_out (fp32, may be res itself) is written when given.
+template <int V, typename TY, typename TR, typename TO>
+__global__ void add_rms_norm_kernel(const TY* __restrict__ y, const TR* res, const TO* __restrict__ w, float* res_out,
+                                    TO* __restrict__ out, int H, float eps, float offset) {
+  pdl_launch_dependents();
+  pdl_wait();
+  extern __shared__ __align__(16) float row[];
+  __shared__ float red[32];
+  const size_t base = (size_t)blockIdx.x * H;
+  float ss = 0.f;
+  for (int i = threadIdx.x * V; i < H; i += blockDim.x * V) {
+    float v[V];
+    load<V>(res + base + i, v);
+    if (y != nullptr) {
+      float a[V];
+      load<V>(y + base + i, a);
+#pragma unroll
+      for (int j = 0; j < V; ++j) v[j] += a[j];
+    }
+    if (res_out != nullptr) store<V>(res_out + base + i, v);
+#pragma unroll
+    for (int j = 0; j < V; ++j) ss += v[j] * v[j];
+    store<V>(row + i, v);
+  }
+  const float inv = 1.f / sqrtf(block_sum(ss, red) / (float)H + eps);
+  for (int i = threadIdx.x * V; i < H; i += blockDim.x * V) {
+    float v[V], g[V];
+    load<V>(row + i, v);
+    load<V>(w + i, g);
+#pragma unroll
+    for (int j = 0; j < V; ++j) v[j] = v[j] * inv * (offset + g[j]);
+    store<V>(out + base + i, v);
+  }
+}
+
+template <typename TY, typename TR, typename TO>
+static int launch_add_rms(const void* y, const void* res, const void* w, void* res_out, void* out, int T, int H,
+                          float eps, float offset, cudaStream_t stream) {
+  const uintptr_t a = (uintptr_t)y | (uintptr_t)res | (uintptr_t)w | (uintptr_t)res_out | (uintptr_t)out;
+  const bool vec = H % 8 == 0 && a % 16 == 0;
+  int threads = (H / (vec ? 8 : 1) + 31) / 32 * 32;
+  threads = threads < 32 ? 32 : (threads > 512 ? 512 : threads);
+  const int smem = H * (int)sizeof(float);
+  static unsigned long long seen8 = 0, seen1 = 0;
+  if (vec) {
+    if (smem > 48 * 1024)
+      B200_CUDA_CHECK(ensure_dynamic_smem(add_rms_norm_kernel<8, TY, TR, TO>, 200 * 1024, &seen8));
+    B200_CUDA_CHECK(launch_pdl(add_rms_norm_kernel<8, TY, TR, TO>, dim3(T), dim3(threads), (size_t)smem, stream,
+                               (const TY*)y, (const TR*)res, (const TO*)w, (float*)res_out, (TO*)out, H, eps, offset));
+  } else {
+    if (smem > 48 * 1024)
+      B200_CUDA_CHECK(ensure_dynamic_smem(add_rms_norm_kernel<1, TY, TR, TO>, 200 * 1024, &seen1));
+    B200_CUDA_CHECK(launch_pdl(add_rms_norm_kernel<1, TY, TR, TO>, dim3(T), dim3(threads), (size_t)smem, stream,
+                               (const TY*)y, (const TR*)res, (const TO*)w, (float*)res_out, (TO*)out, H, eps, offset));
+  }
+  return 0;
+}
+
 template <typename T>
 __global__ void softcap_kernel(const T* __restrict__ x, float* __restrict__ y, size_t n, float cap, float inv_cap) {
   pdl_launch_dependents();
@@ -161,6 +224,24 @@ extern "C" int b200_layer_norm(const void* x, int x_elem, const void* w, int w_e
   if (x_elem == 4 && w_elem == 4)
     return ln::launch_v<float, float, float, false>(x, nullptr, w, nullptr, out, T, H, eps, stream);
   b200_set_last_error("layer_norm: unsupported combination of types", __FILE__, __LINE__);
+  return -1;
+}
+
+// y (or null): type of w; res: element bytes res_elem; w and out: w_elem (2 = bf16, 4 = fp32); res_out fp32 or null.
+extern "C" int b200_add_rms_norm(const void* y, const void* res, int res_elem, const void* w, int w_elem, void* res_out,
+                                 void* out, int T, int H, float eps, float offset, cudaStream_t stream) {
+  if (T <= 0 || H <= 0) return 0;
+  if (H > 50000) {
+    b200_set_last_error("add_rms_norm: rows of at most 50000 elements", __FILE__, __LINE__);
+    return -1;
+  }
+  if (res_elem == 2 && w_elem == 2)
+    return ln::launch_add_rms<bf16, bf16, bf16>(y, res, w, res_out, out, T, H, eps, offset, stream);
+  if (res_elem == 4 && w_elem == 2)
+    return ln::launch_add_rms<bf16, float, bf16>(y, res, w, res_out, out, T, H, eps, offset, stream);
+  if (res_elem == 4 && w_elem == 4)
+    return ln::launch_add_rms<float, float, float>(y, res, w, res_out, out, T, H, eps, offset, stream);
+  b200_set_last_error("add_rms_norm: unsupported combination of types", __FILE__, __LINE__);
   return -1;
 }
 

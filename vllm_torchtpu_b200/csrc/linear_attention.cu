@@ -1,0 +1,817 @@
+// Linear attention with a carried state per request and head (S is [dk, dv], fp32), two rules:
+//
+//   fixed decay per head:           S <- decay_h S + k v^T
+//   delta rule, decay per channel:  S <- g S (rows);  u = beta (v - S^T k);  S <- S + k u^T
+//
+//   o = S^T q;   y = o / rms(o) [* norm] * act(gate)
+//
+// q, k, v are columns of a packed projection, optionally behind a causal short convolution with silu, a rotation of
+// half-split pairs and unit length.  Decays, step sizes, norms, angles and the state are fp32 throughout.
+//
+// State pools are indexed by the request's slot.  The convolution's inputs live in a ring of `taps` rows (the input of
+// position p in row p % taps): the row that a single token writes is none of those it reads.  A request whose first
+// token of the step has position 0 starts from zeros.
+//
+// Kernels:
+//  * lin_step_kernel: one CTA per (head, request), token by token, everything fused (convolution to gate).  The state
+//    is held in registers, so a decoded token reads and writes it once.  Decoding, and prompts in 32-bit.
+//  * prompts in bf16, chunks of 16 tokens:
+//      lin_chunk_kernel (parallel over chunks): with G_i the decays accumulated up to token i of the chunk (log2),
+//        A_ij = beta_i sum_c k_ic k_jc 2^(G_ic - G_jc) (i > j),  Q_ij the same with q_i and i >= j;
+//        (I + A) U = beta v,  (I + A) W = beta k 2^G  by forward substitution;  q' = q 2^G,  k' = k 2^(G_last - G).
+//        Decay factors only ever appear as 2^(difference <= 0).
+//      lin_scan_kernel (sequential over chunks, one warp per 16 value columns, no exchange between warps):
+//        U' = U - W S,  O = q' S + Q U',  S <- 2^G_last S + k'^T U'.
+//        The warp keeps S^T as mma accumulators: they are at the same time the A operand of the two products with S
+//        (the contraction index is permuted alike in the B operand), and U'^T comes out in the layout that the update
+//        and Q U' take.  tf32 operands, fp32 accumulation and state.
+//      lin_finish_kernel: norm and gate.
+//    The scratch of a slab of chunks stays within the L2.
+#include <cstring>
+
+#include "common.cuh"
+
+namespace b200 {
+namespace lin {
+
+__device__ __forceinline__ float to_f(float v) { return v; }
+__device__ __forceinline__ float to_f(__nv_bfloat16 v) { return __bfloat162float(v); }
+__device__ __forceinline__ void put(float* p, float v) { *p = v; }
+__device__ __forceinline__ void put(__nv_bfloat16* p, float v) { *p = __float2bfloat16(v); }
+__device__ __forceinline__ float silu(float v) { return v / (1.f + expf(-v)); }
+__device__ __forceinline__ float sigmoid(float v) { return 1.f / (1.f + expf(-v)); }
+__device__ __forceinline__ float softplus(float v) { return fmaxf(v, 0.f) + log1pf(expf(-fabsf(v))); }
+__device__ __forceinline__ float ex2(float x) {
+  float y;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
+__device__ __forceinline__ uint32_t tf32(float v) {
+  uint32_t r;
+  asm("cvt.rna.tf32.f32 %0, %1;" : "=r"(r) : "f"(v));
+  return r;
+}
+__device__ __forceinline__ float tf32f(float v) { return __uint_as_float(tf32(v)); }
+__device__ __forceinline__ void mma_tf32(float* c, const uint32_t* a, uint32_t b0, uint32_t b1) {
+  asm volatile(
+      "mma.sync.aligned.m16n8k8.row.col.f32.tf32.tf32.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
+      : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
+      : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
+}
+__device__ __forceinline__ void cp_async16(uint32_t dst, const void* src) {
+  asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(dst), "l"(src) : "memory");
+}
+
+constexpr int C = 16;                 // tokens per chunk
+constexpr float UNIT_EPS = 1e-6f;
+constexpr float LOG2E = 1.4426950408889634f;
+constexpr int AQ_LD = 24;             // row stride of Q in the scratch
+
+struct Params {
+  const void *row, *a, *gate, *conv_w;
+  void *ring, *y;
+  float* state;
+  const float *inv_freq, *decay, *A_log, *dt_bias, *norm_w;
+  const int *qsl, *seq_lens, *slots;
+  int ldr, q_off, k_off, v_off, beta_off, lda, ldg, taps, pairs, unit, gate_silu;
+  int T, H, Hk, dk, dv, req_begin, zero_rows;
+  float eps, q_mult, k_mult;
+  // ---- chunked prompts
+  float *qd, *w, *kd, *u, *aq, *gl, *o;
+  int dkp, dvp, slab, chunk_begin;
+};
+
+struct Req {
+  int qs, len, start, slot;           // first row, rows, position of the first, state slot
+};
+__device__ __forceinline__ Req request(const Params& p, int r) {
+  Req q;
+  q.qs = p.qsl[r];
+  q.len = p.qsl[r + 1] - q.qs;
+  q.start = p.seq_lens[r] - q.len;
+  q.slot = p.slots[r];
+  return q;
+}
+// column of channel c (q | k | v) in the packed row
+__device__ __forceinline__ int column(const Params& p, int c) {
+  const int n = p.Hk * p.dk;
+  return c < n ? p.q_off + c : (c < 2 * n ? p.k_off + c - n : p.v_off + c - 2 * n);
+}
+// input of channel c at position pos (zero in front of the sequence): from this step's rows or from the ring
+template <typename E>
+__device__ __forceinline__ float input_at(const Params& p, const Req& q, int pos, int c, int col) {
+  if (pos < 0) return 0.f;
+  if (pos >= q.start) return to_f(reinterpret_cast<const E*>(p.row)[(size_t)(q.qs + pos - q.start) * p.ldr + col]);
+  const int ch = 2 * p.Hk * p.dk + p.H * p.dv;
+  return to_f(reinterpret_cast<const E*>(p.ring)[((size_t)q.slot * p.taps + pos % p.taps) * ch + c]);
+}
+
+// ------------------------------------------------------------------------------------------- token by token
+// Thread (row group rg, column group cg) owns columns VEC * cg .. of rows rg, rg + RG, ... of the state.
+// HOLD: they stay in registers (at most RPT rows); otherwise the pool is read twice and written once per token.
+template <typename E, bool DELTA, int VEC, int RPT, bool HOLD>
+__global__ void __launch_bounds__(HOLD ? 512 : 1024) lin_step_kernel(const Params p) {
+  pdl_launch_dependents();
+  pdl_wait();
+  extern __shared__ __align__(16) float sm[];
+  __shared__ float red[32];
+  __shared__ float sc[3];
+  const int h = blockIdx.x, r = p.req_begin + blockIdx.y, tid = threadIdx.x, NT = blockDim.x;
+  const Req q = request(p, r);
+  if (q.len <= 0 || q.slot < 0) {
+    if (p.zero_rows && r < p.T)
+      for (int j = tid; j < p.dv; j += NT) put(reinterpret_cast<E*>(p.y) + (size_t)r * p.H * p.dv + h * p.dv + j, 0.f);
+    return;
+  }
+  const int dk = p.dk, dv = p.dv, n = p.Hk * dk, group = p.H / p.Hk, hk = h / group;
+  const int ncg = dv / VEC, RG = NT / ncg, cg = tid % ncg, rg = tid / ncg;
+  const bool act = rg < RG;
+  float* sq = sm;                       // [dk]
+  float* sk = sq + dk;                  // [dk]
+  float* sg = sk + dk;                  // [dk]
+  float* sv = sg + dk;                  // [dv]
+  float* su = sv + dv;                  // [dv]
+  float* pm = su + dv;                  // [RG][dv]
+  float* po = pm + RG * dv;             // [RG][dv]
+  float* st = p.state + ((size_t)q.slot * p.H + h) * dk * dv + VEC * cg;
+  const bool fresh = q.start == 0;
+  const int rows = act ? (dk - rg + RG - 1) / RG : 0;
+  auto load_row = [&](int i, float (&s)[VEC]) {
+    if constexpr (VEC == 4) {
+      const float4 f = *reinterpret_cast<const float4*>(st + (size_t)i * dv);
+      s[0] = f.x; s[1] = f.y; s[2] = f.z; s[3] = f.w;
+    } else {
+      s[0] = st[(size_t)i * dv];
+    }
+  };
+  auto store_row = [&](int i, const float (&s)[VEC]) {
+    if constexpr (VEC == 4) *reinterpret_cast<float4*>(st + (size_t)i * dv) = make_float4(s[0], s[1], s[2], s[3]);
+    else st[(size_t)i * dv] = s[0];
+  };
+  float S[HOLD ? RPT : 1][VEC];
+  if constexpr (HOLD) {
+#pragma unroll
+    for (int x = 0; x < RPT; ++x) {
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) S[x][e] = 0.f;
+      if (!fresh && x < rows) load_row(rg + x * RG, S[x]);
+    }
+  }
+  const float a_log = DELTA ? expf(p.A_log[h]) : 0.f;
+  const float decay = DELTA ? 0.f : p.decay[h];
+  for (int t = q.qs; t < q.qs + q.len; ++t) {
+    const int pos = q.start + t - q.qs;
+    for (int x = tid; x < 2 * dk + dv; x += NT) {
+      const int c = x < dk ? hk * dk + x : (x < 2 * dk ? n + hk * dk + x - dk : 2 * n + h * dv + x - 2 * dk);
+      const int col = column(p, c);
+      float v;
+      if (p.taps > 0) {
+        const E* w = reinterpret_cast<const E*>(p.conv_w) + (size_t)c * p.taps;
+        v = 0.f;
+        for (int j = 0; j < p.taps; ++j) v += to_f(w[j]) * input_at<E>(p, q, pos - p.taps + 1 + j, c, col);
+        v = silu(v);
+        // a single token enters the ring here; longer portions once all of their readers are done
+        if (q.len == 1 && (x >= 2 * dk || h % group == 0))
+          reinterpret_cast<E*>(p.ring)[((size_t)q.slot * p.taps + pos % p.taps) * (2 * n + p.H * dv) + c] =
+              reinterpret_cast<const E*>(p.row)[(size_t)t * p.ldr + col];
+      } else {
+        v = to_f(reinterpret_cast<const E*>(p.row)[(size_t)t * p.ldr + col]);
+      }
+      if (x < dk) sq[x] = v;
+      else if (x < 2 * dk) sk[x - dk] = v;
+      else sv[x - 2 * dk] = v;
+    }
+    if constexpr (DELTA) {
+      for (int i = tid; i < dk; i += NT) {
+        const float z = to_f(reinterpret_cast<const E*>(p.a)[(size_t)t * p.lda + h * dk + i]) + p.dt_bias[h * dk + i];
+        sg[i] = expf(-a_log * softplus(z));
+      }
+    }
+    __syncthreads();
+    if (p.pairs > 0) {
+      for (int i = tid; i < 2 * p.pairs; i += NT) {
+        const int f = i < p.pairs ? i : i - p.pairs;
+        float* x = i < p.pairs ? sq : sk;
+        float sn, cs;
+        sincosf((float)pos * p.inv_freq[f], &sn, &cs);
+        const float a = x[f], b = x[f + p.pairs];
+        x[f] = a * cs - b * sn;
+        x[f + p.pairs] = b * cs + a * sn;
+      }
+      __syncthreads();
+    }
+    if (tid < 96) {
+      const int wq = tid >> 5, lane = tid & 31;
+      const float* x = wq == 1 ? sk : sq;
+      const float* y = wq == 0 ? sq : sk;
+      float s = 0.f;
+      for (int i = lane; i < dk; i += 32) s += x[i] * y[i];
+      s = warp_sum(s);
+      if (lane == 0) sc[wq] = s;
+    }
+    __syncthreads();
+    const float iq = p.q_mult * (p.unit ? 1.f / sqrtf(sc[0] + UNIT_EPS) : 1.f);
+    const float ik = p.k_mult * (p.unit ? 1.f / sqrtf(sc[1] + UNIT_EPS) : 1.f);
+    const float qk = sc[2] * iq * ik;
+    float mem[VEC], os[VEC];
+#pragma unroll
+    for (int e = 0; e < VEC; ++e) mem[e] = os[e] = 0.f;
+    const bool zero = !HOLD && fresh && t == q.qs;
+    auto pass = [&](int i, float (&s)[VEC]) {
+      const float g = DELTA ? sg[i] : decay, kk = sk[i] * ik, qq = sq[i] * iq;
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) {
+        s[e] *= g;
+        if (DELTA) mem[e] = fmaf(kk, s[e], mem[e]);
+        os[e] = fmaf(qq, s[e], os[e]);
+      }
+    };
+    if constexpr (HOLD) {
+#pragma unroll
+      for (int x = 0; x < RPT; ++x)
+        if (x < rows) pass(rg + x * RG, S[x]);
+    } else if (!zero) {
+      for (int x = 0; x < rows; ++x) {
+        float s[VEC];
+        load_row(rg + x * RG, s);
+        pass(rg + x * RG, s);
+      }
+    }
+    if (act) {
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) {
+        if (DELTA) pm[rg * dv + VEC * cg + e] = mem[e];
+        po[rg * dv + VEC * cg + e] = os[e];
+      }
+    }
+    __syncthreads();
+    const float beta =
+        DELTA ? sigmoid(to_f(reinterpret_cast<const E*>(p.row)[(size_t)t * p.ldr + p.beta_off + h])) : 1.f;
+    float ss = 0.f;
+    for (int j = tid; j < dv; j += NT) {
+      float m = 0.f, o = 0.f;
+      for (int x = 0; x < RG; ++x) {
+        if (DELTA) m += pm[x * dv + j];
+        o += po[x * dv + j];
+      }
+      const float u = DELTA ? beta * (sv[j] - m) : sv[j];
+      o = fmaf(qk, u, o);
+      su[j] = u;
+      po[j] = o;                        // (row group 0; only this thread reads column j)
+      ss += o * o;
+    }
+    ss = block_sum(ss, red);            // also orders su for the update
+    const float inv = 1.f / sqrtf(ss / (float)dv + p.eps);
+    for (int j = tid; j < dv; j += NT) {
+      float v = po[j] * inv;
+      if (p.norm_w != nullptr) v *= p.norm_w[j];
+      const float g = to_f(reinterpret_cast<const E*>(p.gate)[(size_t)t * p.ldg + h * dv + j]);
+      v *= p.gate_silu ? silu(g) : sigmoid(g);
+      put(reinterpret_cast<E*>(p.y) + (size_t)t * p.H * dv + h * dv + j, v);
+    }
+    float u[VEC];
+#pragma unroll
+    for (int e = 0; e < VEC; ++e) u[e] = act ? su[VEC * cg + e] : 0.f;
+    if constexpr (HOLD) {
+#pragma unroll
+      for (int x = 0; x < RPT; ++x)
+        if (x < rows) {
+          const float kk = sk[rg + x * RG] * ik;
+#pragma unroll
+          for (int e = 0; e < VEC; ++e) S[x][e] = fmaf(kk, u[e], S[x][e]);
+        }
+    } else {
+      for (int x = 0; x < rows; ++x) {
+        const int i = rg + x * RG;
+        const float g = DELTA ? sg[i] : decay, kk = sk[i] * ik;
+        float s[VEC];
+        if (zero) {
+#pragma unroll
+          for (int e = 0; e < VEC; ++e) s[e] = kk * u[e];
+        } else {
+          load_row(i, s);
+#pragma unroll
+          for (int e = 0; e < VEC; ++e) s[e] = fmaf(kk, u[e], s[e] * g);
+        }
+        store_row(i, s);
+      }
+    }
+    __syncthreads();                    // before the next token's q, k, v
+  }
+  if constexpr (HOLD) {
+#pragma unroll
+    for (int x = 0; x < RPT; ++x)
+      if (x < rows) store_row(rg + x * RG, S[x]);
+  }
+}
+
+// The last inputs of a prompt's portion, once the convolutions have run.  grid (channels / 256, requests)
+template <typename E>
+__global__ void lin_ring_kernel(const Params p) {
+  pdl_launch_dependents();
+  pdl_wait();
+  const Req q = request(p, p.req_begin + blockIdx.y);
+  const int ch = 2 * p.Hk * p.dk + p.H * p.dv, c = blockIdx.x * blockDim.x + threadIdx.x;
+  if (q.len <= 0 || q.slot < 0 || c >= ch) return;
+  const int col = column(p, c), end = q.start + q.len;
+  for (int pos = max(q.start, end - p.taps); pos < end; ++pos)
+    reinterpret_cast<E*>(p.ring)[((size_t)q.slot * p.taps + pos % p.taps) * ch + c] =
+        reinterpret_cast<const E*>(p.row)[(size_t)(q.qs + pos - q.start) * p.ldr + col];
+}
+
+// ------------------------------------------------------------------------------------------- chunks of 16 tokens
+typedef __nv_bfloat16 bf16;
+
+// The 16 values of channel c in a chunk that begins at position pos0 (n of them exist; zeros behind).  KM: taps the
+// window is unrolled for (0: no convolution).
+template <int KM>
+__device__ __forceinline__ void chunk_column(const Params& p, const Req& q, int pos0, int n, int c, float (&v)[C]) {
+  const int col = column(p, c);
+  if constexpr (KM == 0) {
+    const bf16* x = reinterpret_cast<const bf16*>(p.row) + (size_t)(q.qs + pos0 - q.start) * p.ldr + col;
+#pragma unroll
+    for (int i = 0; i < C; ++i) v[i] = i < n ? to_f(x[(size_t)i * p.ldr]) : 0.f;
+  } else {
+    float x[C + KM - 1], w[KM];
+    const bf16* wp = reinterpret_cast<const bf16*>(p.conv_w) + (size_t)c * p.taps;
+#pragma unroll
+    for (int j = 0; j < KM; ++j) w[j] = j >= KM - p.taps ? to_f(wp[j - (KM - p.taps)]) : 0.f;
+#pragma unroll
+    for (int m = 0; m < C + KM - 1; ++m) {
+      const int i = m - (KM - 1);
+      x[m] = (i > -p.taps && i < n) ? input_at<bf16>(p, q, pos0 + i, c, col) : 0.f;
+    }
+#pragma unroll
+    for (int i = 0; i < C; ++i) {
+      float s = 0.f;
+#pragma unroll
+      for (int j = 0; j < KM; ++j) s = fmaf(w[j], x[i + j], s);
+      v[i] = i < n ? silu(s) : 0.f;
+    }
+  }
+}
+
+// grid (requests * slab, H), 256 threads
+template <bool DELTA, int KM>
+__global__ void __launch_bounds__(256, 2) lin_chunk_kernel(const Params p) {
+  pdl_launch_dependents();
+  pdl_wait();
+  extern __shared__ __align__(16) float sm[];
+  __shared__ float beta[C], sa[C][C + 4], norm[2][C];
+  const int slot = blockIdx.x, h = blockIdx.y, tid = threadIdx.x;
+  const Req q = request(p, p.req_begin + slot / p.slab);
+  const int t0 = (p.chunk_begin + slot % p.slab) * C, n = min(C, q.len - t0);
+  if (n <= 0 || q.slot < 0) return;
+  const int pos0 = q.start + t0, row0 = q.qs + t0;
+  const int dk = p.dk, dv = p.dv, dkp = p.dkp, ds = dkp + 4, nk = p.Hk * dk, hk = h / (p.H / p.Hk);
+  float* sq = sm;                       // [C][ds]
+  float* sk = sq + C * ds;
+  float* sg = sk + C * ds;              // decays accumulated from the chunk's first token on, log2 (delta rule)
+  // ---- q, k and the accumulated decays
+  for (int x = tid; x < 2 * dkp; x += 256) {
+    const int i0 = x < dkp ? x : x - dkp;
+    float v[C];
+    if (i0 < dk) {
+      chunk_column<KM>(p, q, pos0, n, (x < dkp ? 0 : nk) + hk * dk + i0, v);
+    } else {
+#pragma unroll
+      for (int i = 0; i < C; ++i) v[i] = 0.f;
+    }
+    float* d = x < dkp ? sq : sk;
+#pragma unroll
+    for (int i = 0; i < C; ++i) d[i * ds + i0] = v[i];
+  }
+  if constexpr (DELTA) {
+    const float a_log = expf(p.A_log[h]) * LOG2E;
+    for (int c = tid; c < dkp; c += 256) {
+      float g = 0.f;
+      const float b = c < dk ? p.dt_bias[h * dk + c] : 0.f;
+      const bf16* a = reinterpret_cast<const bf16*>(p.a) + (size_t)row0 * p.lda + h * dk + c;
+#pragma unroll
+      for (int i = 0; i < C; ++i) {
+        // a factor below 2^-64 leaves nothing of the state in fp32: the sum keeps its digits
+        if (c < dk && i < n) g -= fminf(a_log * softplus(to_f(a[(size_t)i * p.lda]) + b), 64.f);
+        sg[i * ds + c] = g;
+      }
+    }
+    if (tid < C)
+      beta[tid] = tid < n ? sigmoid(to_f(reinterpret_cast<const bf16*>(p.row)[(size_t)(row0 + tid) * p.ldr + p.beta_off + h]))
+                          : 0.f;
+  }
+  __syncthreads();
+  if (p.pairs > 0) {
+    for (int x = tid; x < C * p.pairs; x += 256) {
+      const int i = x / p.pairs, f = x - i * p.pairs;
+      float sn, cs;
+      sincosf((float)(pos0 + i) * p.inv_freq[f], &sn, &cs);
+#pragma unroll
+      for (int s = 0; s < 2; ++s) {
+        float* d = (s ? sk : sq) + i * ds + f;
+        const float a = d[0], b = d[p.pairs];
+        d[0] = a * cs - b * sn;
+        d[p.pairs] = b * cs + a * sn;
+      }
+    }
+    __syncthreads();
+  }
+  {
+    const int warp = tid >> 5, lane = tid & 31;
+    for (int x = warp; x < 2 * C; x += 8) {
+      float* d = (x < C ? sq : sk) + (x & (C - 1)) * ds;
+      float m = x < C ? p.q_mult : p.k_mult;
+      if (p.unit) {
+        float s = 0.f;
+        for (int i = lane; i < dk; i += 32) s += d[i] * d[i];
+        m /= sqrtf(warp_sum(s) + UNIT_EPS);
+      }
+      if (lane == 0) norm[x >= C][x & (C - 1)] = m;
+    }
+  }
+  __syncthreads();
+  const size_t unit = (size_t)slot * p.H + h;
+  const float ld = DELTA ? 0.f : fmaxf(log2f(p.decay[h]), -64.f);
+  // ---- products of the tokens of the chunk
+  {
+    const int i = tid >> 4, j = tid & 15;
+    float qk = 0.f, kk = 0.f;
+    if (j <= i) {
+      const float *qi = sq + i * ds, *ki = sk + i * ds, *kj = sk + j * ds, *gi = sg + i * ds, *gj = sg + j * ds;
+      for (int c = 0; c < dkp; c += 4) {
+        const float4 a = *reinterpret_cast<const float4*>(qi + c), b = *reinterpret_cast<const float4*>(kj + c);
+        if constexpr (DELTA) {
+          const float4 e = *reinterpret_cast<const float4*>(ki + c), x = *reinterpret_cast<const float4*>(gi + c),
+                       y = *reinterpret_cast<const float4*>(gj + c);
+          const float d0 = b.x * ex2(x.x - y.x), d1 = b.y * ex2(x.y - y.y), d2 = b.z * ex2(x.z - y.z),
+                      d3 = b.w * ex2(x.w - y.w);
+          qk = fmaf(a.x, d0, qk); qk = fmaf(a.y, d1, qk); qk = fmaf(a.z, d2, qk); qk = fmaf(a.w, d3, qk);
+          kk = fmaf(e.x, d0, kk); kk = fmaf(e.y, d1, kk); kk = fmaf(e.z, d2, kk); kk = fmaf(e.w, d3, kk);
+        } else {
+          qk = fmaf(a.x, b.x, qk); qk = fmaf(a.y, b.y, qk); qk = fmaf(a.z, b.z, qk); qk = fmaf(a.w, b.w, qk);
+        }
+      }
+      qk *= norm[0][i] * norm[1][j];
+      if constexpr (!DELTA) qk *= exp2f(ld * (float)(i - j));
+      kk *= norm[1][i] * norm[1][j];
+    }
+    p.aq[(unit * C + i) * AQ_LD + j] = tf32f(qk);
+    if constexpr (DELTA) sa[i][j] = j < i ? beta[i] * kk : 0.f;
+  }
+  if constexpr (DELTA) __syncthreads();
+  // ---- columns of W and U (forward substitution), q', k', last decay
+  for (int x = tid; x < dkp + p.dvp; x += 256) {
+    float v[C];
+    if (x < dkp) {
+      float *qd = p.qd + unit * C * (dkp + 8) + x, *kd = p.kd + unit * C * (dkp + 4) + x;
+      if constexpr (DELTA) {
+        const float last = sg[(C - 1) * ds + x];
+#pragma unroll
+        for (int i = 0; i < C; ++i) {
+          const float g = sg[i * ds + x], e = ex2(g), k = sk[i * ds + x] * norm[1][i];
+          qd[i * (dkp + 8)] = tf32f(sq[i * ds + x] * norm[0][i] * e);
+          kd[i * (dkp + 4)] = tf32f(k * ex2(last - g));
+          v[i] = beta[i] * k * e;
+        }
+        p.gl[unit * dkp + x] = ex2(last);
+      } else {
+#pragma unroll
+        for (int i = 0; i < C; ++i) {
+          qd[i * (dkp + 8)] = tf32f(sq[i * ds + x] * norm[0][i] * exp2f(ld * (float)(i + 1)));
+          kd[i * (dkp + 4)] = i < n ? tf32f(sk[i * ds + x] * norm[1][i] * exp2f(ld * (float)(n - 1 - i))) : 0.f;
+        }
+        p.gl[unit * dkp + x] = exp2f(ld * (float)n);
+      }
+    } else {
+      const int j = x - dkp;
+      if (j < dv) {
+        chunk_column<KM>(p, q, pos0, n, 2 * nk + h * dv + j, v);
+      } else {
+#pragma unroll
+        for (int i = 0; i < C; ++i) v[i] = 0.f;
+      }
+      if constexpr (DELTA) {
+#pragma unroll
+        for (int i = 0; i < C; ++i) v[i] *= beta[i];
+      }
+    }
+    if constexpr (DELTA) {
+#pragma unroll
+      for (int i = 1; i < C; ++i) {
+#pragma unroll
+        for (int j = 0; j < i; ++j) v[i] = fmaf(-sa[i][j], v[j], v[i]);
+      }
+      if (x < dkp) {
+        float* w = p.w + unit * C * (dkp + 8) + x;
+#pragma unroll
+        for (int i = 0; i < C; ++i) w[i * (dkp + 8)] = tf32f(-v[i]);
+      }
+    }
+    if (x >= dkp) {
+      float* u = p.u + unit * C * p.dvp + x - dkp;
+#pragma unroll
+      for (int i = 0; i < C; ++i) u[i * p.dvp] = v[i];
+    }
+  }
+}
+
+// grid (H * dvp / 64, requests), 128 threads: warp w owns value columns 16 w .. 16 w + 15 of the CTA's 64
+template <bool DELTA, int NT>
+struct Scan {
+  static constexpr int DKP = 8 * NT;
+  static constexpr int QD = 0, W = C * (DKP + 8), KD = W + (DELTA ? C * (DKP + 8) : 0), U = KD + C * (DKP + 4);
+  static constexpr int U_LD = 68, AQ = U + C * U_LD, GL = AQ + C * AQ_LD, WORDS = GL + DKP;
+  static constexpr int STAGES = 3;
+  static constexpr int BYTES = STAGES * WORDS * 4;
+};
+
+template <bool DELTA, int NT>
+__global__ void __launch_bounds__(128) lin_scan_kernel(const Params p) {
+  pdl_launch_dependents();
+  pdl_wait();
+  using L = Scan<DELTA, NT>;
+  constexpr int DKP = L::DKP;
+  extern __shared__ __align__(16) float sm[];
+  const int splits = p.dvp / 64, h = blockIdx.x / splits, col0 = (blockIdx.x % splits) * 64;
+  const Req q = request(p, p.req_begin + blockIdx.y);
+  const int chunks = min(p.slab, (q.len + C - 1) / C - p.chunk_begin);
+  if (chunks <= 0 || q.slot < 0) return;
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, t = lane & 3;
+  const int dk = p.dk, dv = p.dv;
+  const uint32_t base = smem_u32(sm);
+  auto issue = [&](int c, int stage) {
+    const size_t unit = ((size_t)blockIdx.y * p.slab + c) * p.H + h;
+    const uint32_t d = base + stage * L::WORDS * 4;
+    auto copy = [&](int word, const float* src, int words) {
+      for (int i = tid * 4; i < words; i += 128 * 4) cp_async16(d + (word + i) * 4, src + i);
+    };
+    copy(L::QD, p.qd + unit * C * (DKP + 8), C * (DKP + 8));
+    if constexpr (DELTA) copy(L::W, p.w + unit * C * (DKP + 8), C * (DKP + 8));
+    copy(L::KD, p.kd + unit * C * (DKP + 4), C * (DKP + 4));
+    copy(L::AQ, p.aq + unit * C * AQ_LD, C * AQ_LD);
+    copy(L::GL, p.gl + unit * DKP, DKP);
+#pragma unroll
+    for (int i = tid; i < C * 16; i += 128) {
+      const int r = i >> 4, s = (i & 15) * 4;
+      cp_async16(d + (L::U + r * L::U_LD + s) * 4, p.u + (unit * C + r) * p.dvp + col0 + s);
+    }
+  };
+  float* st = p.state + ((size_t)q.slot * p.H + h) * dk * dv;
+  const int j0 = col0 + warp * 16 + g, j1 = j0 + 8;          // value columns of this thread
+  const bool fresh = q.start == 0 && p.chunk_begin == 0;
+  float S[NT][4];
+#pragma unroll
+  for (int x = 0; x < NT; ++x) {
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      const int i = 8 * x + 2 * t + (e & 1), j = e < 2 ? j0 : j1;
+      S[x][e] = (!fresh && i < dk && j < dv) ? st[(size_t)i * dv + j] : 0.f;
+    }
+  }
+#pragma unroll
+  for (int s = 0; s < L::STAGES - 1; ++s) {
+    if (s < chunks) issue(s, s);
+    asm volatile("cp.async.commit_group;" ::: "memory");
+  }
+  for (int c = 0; c < chunks; ++c) {
+    asm volatile("cp.async.wait_group %0;" ::"n"(L::STAGES - 2) : "memory");
+    __syncthreads();
+    if (c + L::STAGES - 1 < chunks) issue(c + L::STAGES - 1, (c + L::STAGES - 1) % L::STAGES);
+    asm volatile("cp.async.commit_group;" ::: "memory");
+    const float* b = sm + (c % L::STAGES) * L::WORDS;
+    float U[2][4], O[2][4];              // transposed: rows value columns, columns tokens 8 x + 2 t, + 1
+#pragma unroll
+    for (int x = 0; x < 2; ++x) {
+      const float* u = b + L::U + (8 * x + 2 * t) * L::U_LD + warp * 16 + g;
+      U[x][0] = u[0]; U[x][1] = u[L::U_LD]; U[x][2] = u[8]; U[x][3] = u[L::U_LD + 8];
+      O[x][0] = O[x][1] = O[x][2] = O[x][3] = 0.f;
+    }
+    const float* qd = b + L::QD + g * (DKP + 8) + 2 * t;
+    const float* w = b + L::W + g * (DKP + 8) + 2 * t;
+#pragma unroll
+    for (int x = 0; x < NT; ++x) {
+      const uint32_t a[4] = {tf32(S[x][0]), tf32(S[x][2]), tf32(S[x][1]), tf32(S[x][3])};
+#pragma unroll
+      for (int y = 0; y < 2; ++y) {
+        const uint2 bq = *reinterpret_cast<const uint2*>(qd + 8 * y * (DKP + 8) + 8 * x);
+        mma_tf32(O[y], a, bq.x, bq.y);
+        if constexpr (DELTA) {
+          const uint2 bw = *reinterpret_cast<const uint2*>(w + 8 * y * (DKP + 8) + 8 * x);
+          mma_tf32(U[y], a, bw.x, bw.y);
+        }
+      }
+    }
+    uint32_t ua[2][4];
+#pragma unroll
+    for (int x = 0; x < 2; ++x) {
+      ua[x][0] = tf32(U[x][0]); ua[x][1] = tf32(U[x][2]); ua[x][2] = tf32(U[x][1]); ua[x][3] = tf32(U[x][3]);
+    }
+#pragma unroll
+    for (int y = 0; y < 2; ++y) {
+#pragma unroll
+      for (int x = 0; x < 2; ++x) {
+        if (x > y) continue;             // Q is lower triangular
+        const uint2 bq = *reinterpret_cast<const uint2*>(b + L::AQ + (8 * y + g) * AQ_LD + 8 * x + 2 * t);
+        mma_tf32(O[y], ua[x], bq.x, bq.y);
+      }
+    }
+    const float* kd = b + L::KD + 2 * t * (DKP + 4) + g;
+    const float* gl = b + L::GL + 2 * t;
+#pragma unroll
+    for (int x = 0; x < NT; ++x) {
+      const float2 e = *reinterpret_cast<const float2*>(gl + 8 * x);
+      S[x][0] *= e.x; S[x][1] *= e.y; S[x][2] *= e.x; S[x][3] *= e.y;
+#pragma unroll
+      for (int y = 0; y < 2; ++y) {
+        const float* k = kd + 8 * y * (DKP + 4) + 8 * x;
+        mma_tf32(S[x], ua[y], __float_as_uint(k[0]), __float_as_uint(k[DKP + 4]));
+      }
+    }
+    const int rows = min(C, q.len - (p.chunk_begin + c) * C);
+    float* o = p.o + ((((size_t)blockIdx.y * p.slab + c) * C) * p.H + h) * dv;
+#pragma unroll
+    for (int x = 0; x < 2; ++x) {
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        const int i = 8 * x + 2 * t + (e & 1), j = e < 2 ? j0 : j1;
+        if (i < rows && j < dv) o[(size_t)i * p.H * dv + j] = O[x][e];
+      }
+    }
+  }
+#pragma unroll
+  for (int x = 0; x < NT; ++x) {
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      const int i = 8 * x + 2 * t + (e & 1), j = e < 2 ? j0 : j1;
+      if (i < dk && j < dv) st[(size_t)i * dv + j] = S[x][e];
+    }
+  }
+}
+
+// One warp per (token of the slab, head).
+__global__ void __launch_bounds__(256) lin_finish_kernel(const Params p) {
+  pdl_launch_dependents();
+  pdl_wait();
+  const int idx = blockIdx.x, h = blockIdx.y * 8 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+  if (h >= p.H) return;
+  const Req q = request(p, p.req_begin + idx / (p.slab * C));
+  const int i = p.chunk_begin * C + idx % (p.slab * C);
+  if (i >= q.len || q.slot < 0) return;
+  const int dv = p.dv;
+  const float* o = p.o + ((size_t)idx * p.H + h) * dv;
+  float ss = 0.f;
+  for (int j = lane; j < dv; j += 32) ss += o[j] * o[j];
+  const float inv = 1.f / sqrtf(warp_sum(ss) / (float)dv + p.eps);
+  const size_t t = q.qs + i;
+  const bf16* gate = reinterpret_cast<const bf16*>(p.gate) + t * p.ldg + h * dv;
+  bf16* y = reinterpret_cast<bf16*>(p.y) + t * p.H * dv + h * dv;
+  for (int j = lane; j < dv; j += 32) {
+    float v = o[j] * inv;
+    if (p.norm_w != nullptr) v *= p.norm_w[j];
+    const float g = to_f(gate[j]);
+    put(y + j, v * (p.gate_silu ? silu(g) : sigmoid(g)));
+  }
+}
+
+// ------------------------------------------------------------------------------------------- host
+template <typename E, bool DELTA, int VEC, int RPT, bool HOLD>
+static int launch_step_as(const Params& p, int R, int threads, cudaStream_t stream) {
+  const int RG = threads / (p.dv / VEC);
+  const int smem = (3 * p.dk + 2 * p.dv + 2 * RG * p.dv) * (int)sizeof(float);
+  static unsigned long long seen = 0;
+  if (smem > 48 * 1024)
+    B200_CUDA_CHECK(ensure_dynamic_smem(lin_step_kernel<E, DELTA, VEC, RPT, HOLD>, 200 * 1024, &seen));
+  B200_CUDA_CHECK(launch_pdl(lin_step_kernel<E, DELTA, VEC, RPT, HOLD>, dim3(p.H, R), dim3(threads), (size_t)smem,
+                             stream, p));
+  return 0;
+}
+
+template <typename E, bool DELTA, int VEC>
+static int launch_step_v(const Params& p, int R, cudaStream_t stream) {
+  const int ncg = p.dv / VEC;
+  for (int threads = 128; threads <= 512; threads *= 2) {
+    if (threads < ncg) continue;
+    const int RG = threads / ncg, rows = (p.dk + RG - 1) / RG;
+    if (rows <= 4) return launch_step_as<E, DELTA, VEC, 4, true>(p, R, threads, stream);
+    if (rows <= 16) return launch_step_as<E, DELTA, VEC, 16, true>(p, R, threads, stream);
+  }
+  int threads = 512;
+  while (threads < ncg) threads *= 2;
+  if (threads > 1024) {
+    b200_set_last_error("linear attention: at most 1024 value columns per thread group", __FILE__, __LINE__);
+    return -1;
+  }
+  return launch_step_as<E, DELTA, VEC, 1, false>(p, R, threads, stream);
+}
+
+template <typename E>
+static int launch_step(const Params& p, int R, cudaStream_t stream) {
+  const bool delta = p.decay == nullptr;
+  if (p.dv % 4 == 0)
+    return delta ? launch_step_v<E, true, 4>(p, R, stream) : launch_step_v<E, false, 4>(p, R, stream);
+  return delta ? launch_step_v<E, true, 1>(p, R, stream) : launch_step_v<E, false, 1>(p, R, stream);
+}
+
+template <bool DELTA, int NT>
+static int launch_scan(const Params& p, int R, cudaStream_t stream) {
+  static unsigned long long seen = 0;
+  using L = Scan<DELTA, NT>;
+  B200_CUDA_CHECK(ensure_dynamic_smem(lin_scan_kernel<DELTA, NT>, L::BYTES, &seen));
+  B200_CUDA_CHECK(launch_pdl(lin_scan_kernel<DELTA, NT>, dim3(p.H * (p.dvp / 64), R), dim3(128), (size_t)L::BYTES,
+                             stream, p));
+  return 0;
+}
+
+template <bool DELTA, int KM>
+static int launch_chunk(const Params& p, int R, cudaStream_t stream) {
+  const int smem = (DELTA ? 3 : 2) * C * (p.dkp + 4) * (int)sizeof(float);
+  static unsigned long long seen = 0;
+  if (smem > 44 * 1024) B200_CUDA_CHECK(ensure_dynamic_smem(lin_chunk_kernel<DELTA, KM>, 100 * 1024, &seen));
+  B200_CUDA_CHECK(launch_pdl(lin_chunk_kernel<DELTA, KM>, dim3(R * p.slab, p.H), dim3(256), (size_t)smem, stream, p));
+  return 0;
+}
+
+static int padded_dk(int dk) { return dk <= 32 ? 32 : (dk <= 64 ? 64 : (dk <= 128 ? 128 : 256)); }
+
+// floats of scratch per chunk and head
+static size_t chunk_words(int dk, int dv, bool delta) {
+  const int dkp = padded_dk(dk), dvp = (dv + 63) / 64 * 64;
+  return (size_t)C * ((delta ? 2 : 1) * (dkp + 8) + dkp + 4 + dvp + AQ_LD + dv) + dkp;
+}
+
+template <bool DELTA>
+static int launch_chunks(Params& p, int R, float* scratch, cudaStream_t stream) {
+  const size_t units = (size_t)R * p.slab * p.H;
+  p.qd = scratch;
+  p.w = p.qd + units * C * (p.dkp + 8);
+  p.kd = p.w + (DELTA ? units * C * (p.dkp + 8) : 0);
+  p.u = p.kd + units * C * (p.dkp + 4);
+  p.aq = p.u + units * C * p.dvp;
+  p.gl = p.aq + units * C * AQ_LD;
+  p.o = p.gl + units * p.dkp;
+  int rc = p.taps == 0 ? launch_chunk<DELTA, 0>(p, R, stream)
+                       : (p.taps <= 4 ? launch_chunk<DELTA, 4>(p, R, stream) : launch_chunk<DELTA, 8>(p, R, stream));
+  if (rc) return rc;
+  switch (p.dkp) {
+    case 32: rc = launch_scan<DELTA, 4>(p, R, stream); break;
+    case 64: rc = launch_scan<DELTA, 8>(p, R, stream); break;
+    case 128: rc = launch_scan<DELTA, 16>(p, R, stream); break;
+    default: rc = launch_scan<DELTA, 32>(p, R, stream); break;
+  }
+  if (rc) return rc;
+  B200_CUDA_CHECK(launch_pdl(lin_finish_kernel, dim3(R * p.slab * C, (p.H + 7) / 8), dim3(256), (size_t)0, stream, p));
+  return 0;
+}
+
+}  // namespace lin
+}  // namespace b200
+
+// Bytes of scratch per (chunk of 16 tokens, head) of b200_linear_attention in mode 1.
+extern "C" size_t b200_linear_attention_chunk_bytes(int dk, int dv, int delta) {
+  return b200::lin::chunk_words(dk, dv, delta != 0) * sizeof(float);
+}
+
+// Requests [req_begin, req_end) of the batch.  mode 0: token by token (any sizes; the ring takes portions of more than
+// one token when ring_update is set); mode 1: chunks [chunk_begin, chunk_begin + slab) of every request (bf16,
+// dk <= 256, taps <= 8; scratch for (req_end - req_begin) * slab * H chunks); mode 2: the ring of a prompt that ran in
+// mode 1.  decay != null: fixed decay per head, otherwise the delta rule with a, A_log, dt_bias and the step sizes in
+// column beta_off of the row.  elem: 2 = bf16, 4 = fp32.
+extern "C" int b200_linear_attention(int mode, const void* row, int ldr, int q_off, int k_off, int v_off, int beta_off,
+                                     const void* a, int lda, const void* gate, int ldg, const void* conv_w, void* ring,
+                                     int taps, const float* inv_freq, int pairs, const float* decay, const float* A_log,
+                                     const float* dt_bias, const float* norm_w, float* state, void* y, const int* qsl,
+                                     const int* seq_lens, const int* slots, int req_begin, int req_end, int T, int H,
+                                     int Hk, int dk, int dv, int unit, int gate_silu, float eps, float q_mult,
+                                     float k_mult, int zero_rows, void* scratch, int chunk_begin, int slab, int elem,
+                                     cudaStream_t stream) {
+  using namespace b200;
+  const int R = req_end - req_begin;
+  if (R <= 0 || T <= 0) return 0;
+  if (Hk <= 0 || H % Hk || 2 * pairs > dk || R > 65535 || dk <= 0 || dv <= 0) {
+    b200_set_last_error("linear attention: heads must be a multiple of the q / k heads, pairs at most dk / 2", __FILE__,
+                        __LINE__);
+    return -1;
+  }
+  lin::Params p;
+  memset(&p, 0, sizeof(p));
+  p.row = row; p.a = a; p.gate = gate; p.conv_w = conv_w; p.ring = ring; p.y = y; p.state = state;
+  p.inv_freq = inv_freq; p.decay = decay; p.A_log = A_log; p.dt_bias = dt_bias; p.norm_w = norm_w;
+  p.qsl = qsl; p.seq_lens = seq_lens; p.slots = slots;
+  p.ldr = ldr; p.q_off = q_off; p.k_off = k_off; p.v_off = v_off; p.beta_off = beta_off; p.lda = lda; p.ldg = ldg;
+  p.taps = taps; p.pairs = pairs; p.unit = unit; p.gate_silu = gate_silu;
+  p.T = T; p.H = H; p.Hk = Hk; p.dk = dk; p.dv = dv; p.req_begin = req_begin; p.zero_rows = zero_rows;
+  p.eps = eps; p.q_mult = q_mult; p.k_mult = k_mult;
+  p.dkp = lin::padded_dk(dk); p.dvp = (dv + 63) / 64 * 64;
+  p.slab = slab; p.chunk_begin = chunk_begin;
+  if (mode == 0) return elem == 4 ? lin::launch_step<float>(p, R, stream) : lin::launch_step<__nv_bfloat16>(p, R, stream);
+  if (mode == 1) {
+    if (elem != 2 || dk > 256 || taps > 8 || slab <= 0 || scratch == nullptr) {
+      b200_set_last_error("linear attention in chunks: bf16, dk of at most 256, at most 8 taps", __FILE__, __LINE__);
+      return -1;
+    }
+    return decay == nullptr ? lin::launch_chunks<true>(p, R, (float*)scratch, stream)
+                            : lin::launch_chunks<false>(p, R, (float*)scratch, stream);
+  }
+  const dim3 grid((2 * Hk * dk + H * dv + 255) / 256, R);
+  if (elem == 4) B200_CUDA_CHECK(launch_pdl(lin::lin_ring_kernel<float>, grid, dim3(256), (size_t)0, stream, p));
+  else B200_CUDA_CHECK(launch_pdl(lin::lin_ring_kernel<__nv_bfloat16>, grid, dim3(256), (size_t)0, stream, p));
+  return 0;
+}

@@ -17,6 +17,7 @@ from ..layers.linear import ColumnParallelLinear, RowParallelLinear, seeded_norm
 from ..parallel.communicator import get_tp_comm
 from ..parallel.state import get_state
 from ..quantization import QuantConfig
+from ..quantization.unquantized import UnquantizedLinearMethod
 
 
 def pad_q_heads(t: torch.Tensor, dim: int, num_kv_heads: int, g: int, g_padded: int, head_dim: int):
@@ -109,6 +110,9 @@ class LlamaMLP:
 
     def forward(self, x):
         gu = self.gate_up
+        if self.act == "gelu_tanh" and gu.bias is None and not gu.lora_targets \
+                and type(gu.method) is UnquantizedLinearMethod:
+            return self.down(ops.gemm_gated(x, gu.weight, self.act))
         if self.act != "silu":
             # other gated activations (GELU-tanh, clamped and OAI-style SwiGLU, SiTU): GEMM, activation kernel, GEMM
             h = self.gate_up(x)

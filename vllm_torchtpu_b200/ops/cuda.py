@@ -65,7 +65,7 @@ def reload_lib(path: Optional[str] = None) -> str:
     # local scope and own symbols first: the copy must not bind to the functions of the library it replaces
     new = ctypes.CDLL(tmp, mode=os.RTLD_LOCAL | os.RTLD_DEEPBIND)
     new.b200_get_last_error.restype = ctypes.c_char_p
-    new.b200_attn_decode_scratch_bytes.restype = c_size_t
+    new.b200_attn_decode_scratch_bytes.restype = new.b200_linear_attention_chunk_bytes.restype = c_size_t
     _lib = new
     return src
 
@@ -75,8 +75,9 @@ def load_lib(path: str) -> None:
     global _lib, _sms
     _lib = ctypes.CDLL(path, mode=ctypes.RTLD_GLOBAL)
     _lib.b200_get_last_error.restype = ctypes.c_char_p
-    if hasattr(_lib, "b200_attn_decode_scratch_bytes"):
-        _lib.b200_attn_decode_scratch_bytes.restype = c_size_t
+    for name in ("b200_attn_decode_scratch_bytes", "b200_linear_attention_chunk_bytes"):
+        if hasattr(_lib, name):
+            getattr(_lib, name).restype = c_size_t
     if torch.cuda.is_available():
         _sms = torch.cuda.get_device_properties(torch.cuda.current_device()).multi_processor_count
 
@@ -194,16 +195,16 @@ def fused_add_rms_norm(x, residual, weight, eps):
 
 
 def gated_act_and_mul(x, spec: str = "silu"):
-    """x [T, 2I] bf16 (gate columns first) -> act(gate, up) [T, I]; ``spec`` as in
+    """x [T, 2I] (gate columns first) -> act(gate, up) [T, I]; ``spec`` as in
     ``ops.reference.parse_gated_act`` (silu, gelu, gelu_tanh, swigluoai, silu_clamp, situ)."""
     from .reference import parse_gated_act
-    _require_bf16(x)
+    elem = _mixed(x)
     act, a, b = parse_gated_act(spec)
     x = x.contiguous()
     T, I2 = x.shape
     y = torch.empty((T, I2 // 2), dtype=x.dtype, device=x.device)
     _check(lib().b200_gated_act(_p(x), _p(y), c_int(T), c_int(I2 // 2), c_int(act), ctypes.c_float(a),
-                                ctypes.c_float(b), _stream()), "gated_act")
+                                ctypes.c_float(b), c_int(elem), _stream()), "gated_act")
     count_launch()
     return y
 
@@ -253,6 +254,26 @@ def layer_norm_add(y, residual, weight, eps):
     return (r if h is None else h), r
 
 
+def add_rms_norm(y, residual, weight, eps, offset: float = 0.0, update: bool = True):
+    """r = residual (+ y), h = r / rms(r) * (offset + weight).  Returns (h in the weight's dtype, r fp32); an fp32
+    residual is updated in place, a bf16 one (the embedding rows) starts the 32-bit stream.  Without ``update`` the
+    residual is only read."""
+    assert residual.is_contiguous() and (y is None or y.dtype == weight.dtype)
+    y = y.contiguous() if y is not None else None
+    H = residual.shape[-1]
+    r = out = None
+    if update:
+        r = residual if residual.dtype == torch.float32 else torch.empty(residual.shape, dtype=torch.float32,
+                                                                         device=residual.device)
+        out = r if y is not None or r is not residual else None
+    h = torch.empty(residual.shape, dtype=weight.dtype, device=residual.device)
+    _check(lib().b200_add_rms_norm(_p(y), _p(residual), c_int(_mixed(residual)), _p(weight), c_int(_mixed(weight)),
+                                   _p(out), _p(h), c_int(residual.numel() // H), c_int(H), c_float(eps),
+                                   c_float(offset), _stream()), "add_rms_norm")
+    count_launch()
+    return h, r
+
+
 def softcap(x, cap: float):
     """cap * tanh(x / cap) in fp32 (in place when x is fp32)."""
     x = x.contiguous()
@@ -278,6 +299,8 @@ def embedding(ids, table, token_src=None, last_tokens=None):
 def gather_rows(hidden, residual, idx):
     R, H = idx.numel(), hidden.shape[1]
     oh = torch.empty((R, H), dtype=hidden.dtype, device=hidden.device)
+    if residual is not None and residual.dtype != hidden.dtype:
+        return gather_rows(hidden, None, idx)[0], gather_rows(residual, None, idx)[0]
     orr = torch.empty_like(oh) if residual is not None else None
     _check(lib().b200_gather_rows(_p(hidden), _p(residual), _p(idx), _p(oh), _p(orr), c_int(R),
                                   c_int(H * hidden.element_size()), c_int(hidden.shape[0]), _stream()), "gather_rows")
@@ -316,20 +339,39 @@ def rope_and_cache(qkv, positions, inv_freq, kv_cache, slot_mapping, num_q_heads
     return q
 
 
+def norm_and_cache(qkv, positions, kv_cache, slot_mapping, num_q_heads, num_kv_heads, dim, vdim, q_norm_w=None,
+                   k_norm_w=None, eps=1e-6, q_temp=None, q_sumsq=None, k_sumsq=None, norm_sizes=None, offsets=None):
+    """See ``ops.reference.norm_and_cache``; rows of ``qkv`` may be strided."""
+    elem = _mixed(qkv)
+    assert qkv.stride(1) == 1 and kv_cache.dtype == qkv.dtype and kv_cache.is_contiguous()
+    T, (nb, _, _, bs, D) = qkv.shape[0], kv_cache.shape
+    q = torch.empty((T, num_q_heads, D), dtype=qkv.dtype, device=qkv.device)
+    k0, v0 = offsets or (num_q_heads * dim, (num_q_heads + num_kv_heads) * dim)
+    nq, nk = norm_sizes or (num_q_heads * dim, num_kv_heads * dim)
+    coef, every = q_temp or (0.0, 0)
+    _check(lib().b200_norm_cache(
+        _p(qkv), c_int(qkv.stride(0)), c_int(k0), c_int(v0), _p(q_norm_w), _p(k_norm_w), _p(positions),
+        _p(slot_mapping), _p(q_sumsq), _p(k_sumsq), _p(q), _p(kv_cache), c_int(T), c_int(num_q_heads),
+        c_int(num_kv_heads), c_int(dim), c_int(vdim), c_int(D), c_int(bs), c_longlong(nb), c_float(eps), c_float(nq),
+        c_float(nk), c_float(coef), c_int(every), c_int(elem), _stream()), "norm_cache")
+    count_launch()
+    return q
+
+
 # ------------------------------------------------------------------------ GEMM
 def _tma_ready(t, stride: int) -> bool:
     """bf16 operand that a TMA tensor map can describe: 16-byte rows and base."""
     return t.dtype == torch.bfloat16 and stride % 8 == 0 and t.data_ptr() % 16 == 0
 
 
-def gemm_simt(x, w, y, T, N, K, ldx, ldy, *, bias=None, gate=None, ldg=0, batch=1, xs=0, ys=0, act=0, cap=0.0):
+def gemm_simt(x, w, y, T, N, K, ldx, ldy, *, bias=None, gate=None, ldg=0, batch=1, xs=0, ys=0, act=0, cap=0.0, scale=1.0):
     """CUDA-core GEMM (``csrc/gemm_simt.cu``): fp32 operands, or bf16 ones without the TMA's alignment."""
     elem = _mixed(x)
     assert all(t is None or t.dtype == x.dtype for t in (w, bias, gate)), "operands of one dtype"
     assert y.dtype == (torch.float32 if act == 2 else x.dtype)
     _check(lib().b200_gemm_simt(_p(x), _p(w), _p(y), _p(bias), _p(gate), c_int(T), c_int(N), c_int(K), c_int(batch),
                                 c_longlong(ldx), c_longlong(K), c_longlong(ldy), c_longlong(ldg), c_longlong(xs),
-                                c_longlong(ys), c_int(act), c_float(cap), c_int(elem), _stream()), "gemm_simt")
+                                c_longlong(ys), c_int(act), c_float(cap), c_float(scale), c_int(elem), _stream()), "gemm_simt")
     count_launch()
     return y
 
@@ -353,23 +395,32 @@ def gemm_gelu(x, w):
     else:
         _check(lib().b200_gemm_bf16_heads(_p(x2), _p(w), _p(y), c_void_p(0), c_int(T), c_int(N), c_int(K), c_int(1),
                                           c_int(x2.stride(0)), c_int(K), c_int(N), c_int(0), c_int(0), c_int(0),
-                                          c_int(1), c_float(0), _p(ws.status), c_int(_sms), _stream()), "gemm_gelu")
+                                          c_int(1), c_float(0), c_float(1), _p(ws.status), c_int(_sms), _stream()), "gemm_gelu")
     count_launch()
     return y.reshape(*lead, N)
 
 
-def gemm_softcap(x, w, cap: float = 0.0):
-    """fp32 cap * tanh((x @ w.T) / cap) straight from the accumulator (cap 0: x @ w.T): logits."""
+def gemm_gated(x, w, act: str):
+    """act(x @ w[:I].T) * (x @ w[I:].T), w [2I, K]: in the GEMM's epilogue for bf16 silu and gelu_tanh."""
+    if act in ("silu", "gelu_tanh") and x.shape[-1] % 8 == 0 and _tma_ready(x, x.stride(-2)) and _tma_ready(w, w.shape[1]):
+        from .cuda_moe import gemm_swiglu
+        return gemm_swiglu(x, w, gelu_tanh=act == "gelu_tanh")
+    h = gemm(x, w)
+    return gated_act_and_mul(h.reshape(-1, h.shape[-1]), act).reshape(*x.shape[:-1], w.shape[0] // 2)
+
+
+def gemm_softcap(x, w, cap: float = 0.0, scale: float = 1.0):
+    """fp32 cap * tanh(scale * (x @ w.T) / cap) straight from the accumulator (cap 0: scale * (x @ w.T)): logits."""
     (T, K), N = x.shape, w.shape[0]
     y = torch.empty((T, N), dtype=torch.float32, device=x.device)
     if T == 0:
         return y
     if not (_tma_ready(x, x.stride(0)) and _tma_ready(w, K)):
-        return gemm_simt(x, w, y, T, N, K, x.stride(0), N, act=2, cap=cap)
+        return gemm_simt(x, w, y, T, N, K, x.stride(0), N, act=2, cap=cap, scale=scale)
     ws = Workspace.get(x.device)
     _check(lib().b200_gemm_bf16_heads(_p(x), _p(w), _p(y), c_void_p(0), c_int(T), c_int(N), c_int(K), c_int(1),
                                       c_int(x.stride(0)), c_int(K), c_int(N), c_int(0), c_int(0), c_int(0), c_int(2),
-                                      c_float(cap), _p(ws.status), c_int(_sms), _stream()), "gemm_softcap")
+                                      c_float(cap), c_float(scale), _p(ws.status), c_int(_sms), _stream()), "gemm_softcap")
     count_launch()
     return y
 
@@ -394,7 +445,7 @@ def gemm_heads(x, w, gate=None, out=None):
     ws = Workspace.get(x.device)
     _check(lib().b200_gemm_bf16_heads(_p(x), _p(w), _p(y), _p(gate), c_int(T), c_int(N), c_int(K), c_int(H), c_int(ldx),
                                       c_int(K), c_int(ldy), c_int(ldg), c_int(xs), c_int(ys), c_int(0), c_float(0),
-                                      _p(ws.status), c_int(_sms), _stream()), "gemm_heads")
+                                      c_float(1), _p(ws.status), c_int(_sms), _stream()), "gemm_heads")
     count_launch()
     return y
 
@@ -402,7 +453,7 @@ def gemm_heads(x, w, gate=None, out=None):
 def gemm(x, w, bias=None, out=None, force_splits: int = 0):
     """y[T,N] = x[T,K] @ w[N,K]^T (+bias) on the tcgen05 kernel; fp32 operands, and bf16 ones a tensor map
     cannot describe, run on the CUDA cores."""
-    if x.dtype == torch.float32 or x.shape[-1] % 8:
+    if x.dtype == torch.float32 or x.shape[-1] % 8 or x.data_ptr() % 16 or (x.dim() == 2 and x.stride(0) % 8):
         x2 = x.reshape(-1, x.shape[-1])
         x2 = x2 if x2.stride(-1) == 1 else x2.contiguous()
         T, N = x2.shape[0], w.shape[0]
@@ -465,6 +516,10 @@ def decode_splits(num_reqs: int, num_kv_heads: int) -> int:
 def paged_attention(q, kv_cache, meta, scale, *, sliding_window=None, softcap=None, sinks=None,
                     k_scale=1.0, v_scale=1.0, return_lse=False):
     """Ragged paged attention over [decode | prefill/mixed] request ranges of the batch."""
+    if kv_cache.dtype == q.dtype and (q.dtype == torch.float32 or q.shape[2] not in (64, 128)):
+        if return_lse or meta.dcp_size > 1:
+            raise NotImplementedError("log-sum-exp and position-sharded caches: bf16, heads of 64 or 128")
+        return attention_simt(q, kv_cache, meta, scale, sliding_window, softcap, sinks)
     _require_bf16(q)
     # an e4m3 cache is expanded to bf16 in shared memory by the mma.sync kernels; k_scale joins the
     # logit scale and v_scale the output normalisation (reference: layers/adapter/quantization.py:91)
@@ -546,6 +601,22 @@ def paged_attention(q, kv_cache, meta, scale, *, sliding_window=None, softcap=No
         count_launch()
     if return_lse:
         return out, lse
+    return out
+
+
+def attention_simt(q, kv_cache, meta, scale, sliding_window=None, softcap=None, sinks=None):
+    """Paged attention on the CUDA cores (``csrc/attention_simt.cu``): fp32, or head sizes the tensor-core kernels are
+    not built for."""
+    T, Hq, D = q.shape
+    nb, _, Hkv, bs, _ = kv_cache.shape
+    R = meta.padded_num_reqs if meta.padded_num_reqs is not None else meta.num_reqs
+    out = torch.empty_like(q)
+    _check(lib().b200_attn_simt(
+        _p(q), _p(kv_cache), _p(out), _p(meta.block_tables), _p(meta.seq_lens), _p(meta.query_start_loc), c_int(T),
+        c_int(R), c_int(Hq), c_int(Hkv), c_int(D), c_int(meta.block_tables.shape[1]), c_int(bs), c_longlong(nb),
+        c_float(scale), c_int(int(sliding_window or 0)), c_float(float(softcap or 0.0)), _p(sinks), c_int(_mixed(q)),
+        _stream()), "attn_simt")
+    count_launch()
     return out
 
 
@@ -880,6 +951,7 @@ _SUBMODULE_EXPORTS = {
                  "moe_experts_fp8", "quant_act_1x128", "quant_act_int8", "quant_rows_1x128"),
     "cuda_fp4": ("grouped_w4a16_gemm", "moe_experts_w4a16", "w4a16_gemm", "w4a16_int4_gemm", "dequant_w4", "dequant_int4"),
     "cuda_gdn": ("gdn_forward", "kda_forward", "short_conv"),
+    "cuda_linear": ("carried_state_attention",),
     "cuda_mla": ("latent_prep", "mla_absorb", "mla_paged_attention", "mla_unabsorb", "mla_write_cache", "permute_rows", "rope_heads_into",
                  "rope_rows"),
 }

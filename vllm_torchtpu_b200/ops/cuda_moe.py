@@ -10,8 +10,8 @@ from . import count_launch
 from . import cuda as _c
 
 
-def gemm_swiglu(x, w, out=None):
-    """silu(x @ w[:I].T) * (x @ w[I:].T) in one tcgen05 kernel; w is [2I, K]."""
+def gemm_swiglu(x, w, out=None, gelu_tanh: bool = False):
+    """silu(x @ w[:I].T) * (x @ w[I:].T) in one tcgen05 kernel; w is [2I, K].  ``gelu_tanh``: that activation instead."""
     _c._require_bf16(x, w)
     if x.stride(-1) != 1:
         x = x.contiguous()
@@ -25,12 +25,12 @@ def gemm_swiglu(x, w, out=None):
     if 0 < envs.B200_GEMM_2SM_MIN_T <= T:
         _c._check(_c.lib().b200_gemm_bf16_swiglu_2sm(
             _c._p(x2), _c._p(w), _c._p(y), c_int(T), c_int(I), c_int(K), c_int(x2.stride(0)), c_int(w.stride(0)),
-            c_int(y.stride(0)), _c._p(ws.status), c_int(_c._sms), _c._stream()), "gemm_swiglu_2sm")
+            c_int(y.stride(0)), c_int(gelu_tanh), _c._p(ws.status), c_int(_c._sms), _c._stream()), "gemm_swiglu_2sm")
         count_launch()
         return y
     _c._check(_c.lib().b200_gemm_bf16_swiglu(
         _c._p(x2), _c._p(w), _c._p(y), c_int(T), c_int(I), c_int(K), c_int(x2.stride(0)), c_int(w.stride(0)),
-        c_int(y.stride(0)), _c._p(ws.status), c_int(_c._sms), _c._stream()), "gemm_swiglu")
+        c_int(y.stride(0)), c_int(gelu_tanh), _c._p(ws.status), c_int(_c._sms), _c._stream()), "gemm_swiglu")
     count_launch()
     return y
 
