@@ -72,7 +72,7 @@ def parse_args():
     ap.add_argument("--enforce-eager", action="store_true")
     ap.add_argument("--warmup-requests", type=int, default=0,
                     help="requests per warm-up serve (0 = the full workload)")
-    ap.add_argument("--layer-bench", default="", choices=["", "mazivik"],
+    ap.add_argument("--layer-bench", default="", choices=["", "mazivik", "popanex"],
                     help="instead of the serving workload: layer throughput and kernels of this model beside its "
                          "closest neighbour, one JSON line per measurement")
     ap.add_argument("--layer-size", default="2048x16,4096x32,7168x128", help="--layer-bench: width x heads, ...")
@@ -173,7 +173,9 @@ def main():
         print(json.dumps({"impl": "reference", "unavailable": REFERENCE_UNAVAILABLE}))
         return 0
     if args.layer_bench:
-        from vllm_torchtpu_b200.ops.bench_latent import run
+        from importlib import import_module
+        module = {"mazivik": "bench_latent", "popanex": "bench_linear"}[args.layer_bench]
+        run = import_module(f"vllm_torchtpu_b200.ops.{module}").run
         for row in run(args.layer_size, args.layer_parts):
             print(json.dumps(row))
         return 0

@@ -161,6 +161,13 @@ __global__ void __launch_bounds__(HOLD ? 512 : 1024) lin_step_kernel(const Param
   const float decay = DELTA ? 0.f : p.decay[h];
   for (int t = q.qs; t < q.qs + q.len; ++t) {
     const int pos = q.start + t - q.qs;
+    // needed late, loaded early: step size, output gate and norm weight of this thread's first value column
+    const float b_raw = DELTA ? to_f(reinterpret_cast<const E*>(p.row)[(size_t)t * p.ldr + p.beta_off + h]) : 0.f;
+    float g_raw = 0.f, nw = 1.f;
+    if (tid < dv) {
+      g_raw = to_f(reinterpret_cast<const E*>(p.gate)[(size_t)t * p.ldg + h * dv + tid]);
+      if (p.norm_w != nullptr) nw = p.norm_w[tid];
+    }
     for (int x = tid; x < 2 * dk + dv; x += NT) {
       const int c = x < dk ? hk * dk + x : (x < 2 * dk ? n + hk * dk + x - dk : 2 * n + h * dv + x - 2 * dk);
       const int col = column(p, c);
@@ -245,8 +252,7 @@ __global__ void __launch_bounds__(HOLD ? 512 : 1024) lin_step_kernel(const Param
       }
     }
     __syncthreads();
-    const float beta =
-        DELTA ? sigmoid(to_f(reinterpret_cast<const E*>(p.row)[(size_t)t * p.ldr + p.beta_off + h])) : 1.f;
+    const float beta = DELTA ? sigmoid(b_raw) : 1.f;
     float ss = 0.f;
     for (int j = tid; j < dv; j += NT) {
       float m = 0.f, o = 0.f;
@@ -263,9 +269,13 @@ __global__ void __launch_bounds__(HOLD ? 512 : 1024) lin_step_kernel(const Param
     ss = block_sum(ss, red);            // also orders su for the update
     const float inv = 1.f / sqrtf(ss / (float)dv + p.eps);
     for (int j = tid; j < dv; j += NT) {
-      float v = po[j] * inv;
-      if (p.norm_w != nullptr) v *= p.norm_w[j];
-      const float g = to_f(reinterpret_cast<const E*>(p.gate)[(size_t)t * p.ldg + h * dv + j]);
+      float v = po[j] * inv, g = g_raw;
+      if (j == tid) {
+        v *= nw;
+      } else {
+        if (p.norm_w != nullptr) v *= p.norm_w[j];
+        g = to_f(reinterpret_cast<const E*>(p.gate)[(size_t)t * p.ldg + h * dv + j]);
+      }
       v *= p.gate_silu ? silu(g) : sigmoid(g);
       put(reinterpret_cast<E*>(p.y) + (size_t)t * p.H * dv + h * dv + j, v);
     }
@@ -326,27 +336,36 @@ typedef __nv_bfloat16 bf16;
 // window is unrolled for (0: no convolution).
 template <int KM>
 __device__ __forceinline__ void chunk_column(const Params& p, const Req& q, int pos0, int n, int c, float (&v)[C]) {
-  const int col = column(p, c);
+  const int col = column(p, c), t0 = pos0 - q.start;
+  // rows of this step, in one batch of loads; rows outside the chunk's window are clamped and dropped below
+  const bf16* row = reinterpret_cast<const bf16*>(p.row) + (size_t)q.qs * p.ldr + col;
   if constexpr (KM == 0) {
-    const bf16* x = reinterpret_cast<const bf16*>(p.row) + (size_t)(q.qs + pos0 - q.start) * p.ldr + col;
 #pragma unroll
-    for (int i = 0; i < C; ++i) v[i] = i < n ? to_f(x[(size_t)i * p.ldr]) : 0.f;
+    for (int i = 0; i < C; ++i) v[i] = to_f(row[(size_t)(t0 + min(i, n - 1)) * p.ldr]);
+#pragma unroll
+    for (int i = 0; i < C; ++i) v[i] = i < n ? v[i] : 0.f;
   } else {
     float x[C + KM - 1], w[KM];
     const bf16* wp = reinterpret_cast<const bf16*>(p.conv_w) + (size_t)c * p.taps;
 #pragma unroll
-    for (int j = 0; j < KM; ++j) w[j] = j >= KM - p.taps ? to_f(wp[j - (KM - p.taps)]) : 0.f;
+    for (int j = 0; j < KM; ++j) w[j] = to_f(wp[max(0, j - (KM - p.taps))]);
 #pragma unroll
-    for (int m = 0; m < C + KM - 1; ++m) {
-      const int i = m - (KM - 1);
-      x[m] = (i > -p.taps && i < n) ? input_at<bf16>(p, q, pos0 + i, c, col) : 0.f;
+    for (int m = 0; m < C + KM - 1; ++m)
+      x[m] = to_f(row[(size_t)max(0, t0 + min(m - (KM - 1), n - 1)) * p.ldr]);
+#pragma unroll
+    for (int j = 0; j < KM; ++j)
+      if (j < KM - p.taps) w[j] = 0.f;
+    if (t0 == 0) {                       // the portion's first chunk looks back into the ring
+#pragma unroll
+      for (int m = 0; m < KM - 1; ++m)
+        x[m] = m - (KM - 1) > -p.taps ? input_at<bf16>(p, q, pos0 + m - (KM - 1), c, col) : 0.f;
     }
 #pragma unroll
     for (int i = 0; i < C; ++i) {
       float s = 0.f;
 #pragma unroll
       for (int j = 0; j < KM; ++j) s = fmaf(w[j], x[i + j], s);
-      v[i] = i < n ? silu(s) : 0.f;
+      v[i] = i < n ? s / (1.f + __expf(-s)) : 0.f;
     }
   }
 }
@@ -385,12 +404,16 @@ __global__ void __launch_bounds__(256, 2) lin_chunk_kernel(const Params p) {
     const float a_log = expf(p.A_log[h]) * LOG2E;
     for (int c = tid; c < dkp; c += 256) {
       float g = 0.f;
-      const float b = c < dk ? p.dt_bias[h * dk + c] : 0.f;
-      const bf16* a = reinterpret_cast<const bf16*>(p.a) + (size_t)row0 * p.lda + h * dk + c;
+      const int cc = min(c, dk - 1);
+      const float b = p.dt_bias[h * dk + cc];
+      const bf16* a = reinterpret_cast<const bf16*>(p.a) + (size_t)row0 * p.lda + h * dk + cc;
+      float z[C];
+#pragma unroll
+      for (int i = 0; i < C; ++i) z[i] = to_f(a[(size_t)min(i, n - 1) * p.lda]);
 #pragma unroll
       for (int i = 0; i < C; ++i) {
         // a factor below 2^-64 leaves nothing of the state in fp32: the sum keeps its digits
-        if (c < dk && i < n) g -= fminf(a_log * softplus(to_f(a[(size_t)i * p.lda]) + b), 64.f);
+        if (c < dk && i < n) g -= fminf(a_log * softplus(z[i] + b), 64.f);
         sg[i * ds + c] = g;
       }
     }

@@ -26,15 +26,43 @@ struct Params {
   float eps, q_size, k_size, temp_coef;
 };
 
+// V elements at a time: 16 bytes, or one element where sizes and strides are no multiple of that
+template <int V, typename E>
+__device__ __forceinline__ void load(const E* p, float (&v)[V]) {
+  if constexpr (V == 1) {
+    v[0] = to_f(p[0]);
+  } else {
+    const uint4 u = *reinterpret_cast<const uint4*>(p);
+    const E* e = reinterpret_cast<const E*>(&u);
+#pragma unroll
+    for (int j = 0; j < V; ++j) v[j] = to_f(e[j]);
+  }
+}
+template <int V, typename E>
+__device__ __forceinline__ void store(E* p, const float (&v)[V]) {
+  if constexpr (V == 1) {
+    put(p, v[0]);
+  } else {
+    uint4 u;
+    E* e = reinterpret_cast<E*>(&u);
+#pragma unroll
+    for (int j = 0; j < V; ++j) put(e + j, v[j]);
+    *reinterpret_cast<uint4*>(p) = u;
+  }
+}
+
 // One CTA per token.
-template <typename E>
+template <typename E, int V>
 __global__ void __launch_bounds__(256) norm_cache_kernel(const Params p) {
   pdl_launch_dependents();
   pdl_wait();
-  __shared__ float red[32];
-  const int t = blockIdx.x;
+  __shared__ float red[2][8];
+  const int t = blockIdx.x, tid = threadIdx.x;
   const E* row = reinterpret_cast<const E*>(p.row) + (size_t)t * p.ldr;
   const int nq = p.Hq * p.dim, nk = p.Hkv * p.dim;
+  const long long slot = p.slots[t];
+  float temp = 1.f;
+  if (p.temp_every > 0) temp += p.temp_coef * logf((float)((p.positions[t] + 1) / p.temp_every) + 1.f);
   float qs = 1.f, ks = 1.f;
   if (p.q_w != nullptr) {
     float sq = 0.f, sk = 0.f;
@@ -42,52 +70,81 @@ __global__ void __launch_bounds__(256) norm_cache_kernel(const Params p) {
       sq = p.q_sumsq[t];
       sk = p.k_sumsq[t];
     } else {
-      for (int i = threadIdx.x; i < nq; i += blockDim.x) {
-        const float v = to_f(row[i]);
-        sq += v * v;
+      for (int i = tid * V; i < nq + nk; i += blockDim.x * V) {
+        float v[V], s = 0.f;
+        load<V>(row + (i < nq ? i : p.k_off + i - nq), v);
+#pragma unroll
+        for (int j = 0; j < V; ++j) s += v[j] * v[j];
+        if (i < nq) sq += s;
+        else sk += s;
       }
-      for (int i = threadIdx.x; i < nk; i += blockDim.x) {
-        const float v = to_f(row[p.k_off + i]);
-        sk += v * v;
+      sq = warp_sum(sq);
+      sk = warp_sum(sk);
+      if ((tid & 31) == 0) {
+        red[0][tid >> 5] = sq;
+        red[1][tid >> 5] = sk;
       }
-      sq = block_sum(sq, red);
-      sk = block_sum(sk, red);
+      __syncthreads();
+      sq = sk = 0.f;
+      for (int i = 0; i < (int)blockDim.x / 32; ++i) {
+        sq += red[0][i];
+        sk += red[1][i];
+      }
     }
     qs = 1.f / sqrtf(sq / p.q_size + p.eps);
     ks = 1.f / sqrtf(sk / p.k_size + p.eps);
   }
-  float temp = 1.f;
-  if (p.temp_every > 0) temp += p.temp_coef * logf((float)((p.positions[t] + 1) / p.temp_every) + 1.f);
+  qs *= temp;
   E* qo = reinterpret_cast<E*>(p.q_out) + (size_t)t * p.Hq * p.D;
   const E* qw = reinterpret_cast<const E*>(p.q_w);
-  for (int i = threadIdx.x; i < p.Hq * p.D; i += blockDim.x) {
-    const int h = i / p.D, d = i - h * p.D, src = h * p.dim + d;
-    float v = 0.f;
-    if (d < p.dim) {
-      v = to_f(row[src]) * qs;
-      if (qw != nullptr) v *= to_f(qw[src]);
-      v *= temp;
-    }
-    put(qo + i, v);
-  }
-  const long long slot = p.slots[t];
-  if (slot < 0 || slot >= p.num_slots) return;
-  const long long blk = slot / p.block_size;
-  const int off = (int)(slot - blk * p.block_size);
   const E* kw = reinterpret_cast<const E*>(p.k_w);
+  const bool cached = slot >= 0 && slot < p.num_slots;
+  const long long blk = cached ? slot / p.block_size : 0;
+  const int off = (int)(slot - blk * p.block_size);
   const size_t page = (size_t)p.block_size * p.D;
   E* base = reinterpret_cast<E*>(p.cache) + (size_t)blk * 2 * p.Hkv * page + (size_t)off * p.D;
-  for (int i = threadIdx.x; i < p.Hkv * p.D; i += blockDim.x) {
+  // heads: q, then k, then v
+  const int total = (p.Hq + (cached ? 2 * p.Hkv : 0)) * p.D;
+  for (int i = tid * V; i < total; i += blockDim.x * V) {
     const int h = i / p.D, d = i - h * p.D;
-    float k = 0.f, v = 0.f;
-    if (d < p.dim) {
-      k = to_f(row[p.k_off + h * p.dim + d]) * ks;
-      if (kw != nullptr) k *= to_f(kw[h * p.dim + d]);
+    float v[V], w[V];
+#pragma unroll
+    for (int j = 0; j < V; ++j) v[j] = 0.f;
+    if (h < p.Hq) {
+      if (d < p.dim) {
+        load<V>(row + h * p.dim + d, v);
+        if (qw != nullptr) load<V>(qw + h * p.dim + d, w);
+#pragma unroll
+        for (int j = 0; j < V; ++j) v[j] *= qw != nullptr ? qs * w[j] : qs;
+      }
+      store<V>(qo + i, v);
+    } else {
+      const int hk = h - p.Hq;
+      if (hk < p.Hkv) {
+        if (d < p.dim) {
+          load<V>(row + p.k_off + hk * p.dim + d, v);
+          if (kw != nullptr) load<V>(kw + hk * p.dim + d, w);
+#pragma unroll
+          for (int j = 0; j < V; ++j) v[j] *= kw != nullptr ? ks * w[j] : ks;
+        }
+      } else if (d < p.vdim) {
+        load<V>(row + p.v_off + (hk - p.Hkv) * p.vdim + d, v);
+      }
+      store<V>(base + (size_t)hk * page + d, v);
     }
-    if (d < p.vdim) v = to_f(row[p.v_off + h * p.vdim + d]);
-    put(base + (size_t)h * page + d, k);
-    put(base + (size_t)(p.Hkv + h) * page + d, v);
   }
+}
+
+template <typename E>
+static int launch(const Params& p, int T, cudaStream_t stream) {
+  constexpr int V = 16 / sizeof(E);
+  const uintptr_t a = (uintptr_t)p.row | (uintptr_t)p.q_w | (uintptr_t)p.k_w | (uintptr_t)p.q_out | (uintptr_t)p.cache;
+  const bool vec = a % 16 == 0 && (p.ldr | p.k_off | p.v_off | p.dim | p.vdim | p.D) % V == 0;
+  int threads = ((p.Hq + 2 * p.Hkv) * p.D / (vec ? V : 4) + 31) / 32 * 32;
+  threads = threads < 64 ? 64 : (threads > 256 ? 256 : threads);
+  if (vec) B200_CUDA_CHECK(launch_pdl(norm_cache_kernel<E, V>, dim3(T), dim3(threads), (size_t)0, stream, p));
+  else B200_CUDA_CHECK(launch_pdl(norm_cache_kernel<E, 1>, dim3(T), dim3(threads), (size_t)0, stream, p));
+  return 0;
 }
 
 }  // namespace nc
@@ -107,11 +164,5 @@ extern "C" int b200_norm_cache(const void* row, int ldr, int k_off, int v_off, c
   }
   nc::Params p{row, q_w, k_w, q_out, cache, positions, slots, q_sumsq, k_sumsq, ldr, k_off, v_off, Hq, Hkv, dim, vdim,
                D, block_size, temp_every, num_blocks * block_size, eps, q_size, k_size, temp_coef};
-  int threads = ((Hq * dim + 3) / 4 + 31) / 32 * 32;
-  threads = threads < 64 ? 64 : (threads > 256 ? 256 : threads);
-  if (elem == 4)
-    B200_CUDA_CHECK(launch_pdl(nc::norm_cache_kernel<float>, dim3(T), dim3(threads), (size_t)0, stream, p));
-  else
-    B200_CUDA_CHECK(launch_pdl(nc::norm_cache_kernel<__nv_bfloat16>, dim3(T), dim3(threads), (size_t)0, stream, p));
-  return 0;
+  return elem == 4 ? nc::launch<float>(p, T, stream) : nc::launch<__nv_bfloat16>(p, T, stream);
 }

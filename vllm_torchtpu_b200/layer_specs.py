@@ -5,7 +5,7 @@ layer's feed-forward.  ``ModelConfig.from_layer_list`` builds them."""
 from __future__ import annotations
 
 import math
-from dataclasses import dataclass
+from dataclasses import dataclass, replace
 from typing import Optional, Union
 
 
@@ -181,13 +181,17 @@ def layer_specs(layers: list, mixers: tuple, act: str, gated: bool) -> list:
         if mlp and mlp.get("kind") != "dense":
             raise ValueError(f"layer {i}: unknown feed-forward kind {mlp.get('kind')!r}")
         spec = LayerSpec(MIXER_TYPES[layer["type"]].from_dict(layer["mixer"]), int(mlp["ff"]) if mlp else 0, act, gated)
-        src = layer.get("weights_of")
-        if src is not None:
-            if not 0 <= src < i:
-                raise ValueError(f"layer {i}: weights_of {src} must name an earlier layer")
-            src = specs[src].weights_of if specs[src].weights_of is not None else int(src)
-            if (spec.mixer, spec.ff) != (specs[src].mixer, specs[src].ff):
-                raise ValueError(f"layer {i}: its sizes differ from those of layer {src}, whose weights it uses")
-            spec = LayerSpec(spec.mixer, spec.ff, act, gated, src)
         specs.append(spec)
+    for i, layer in enumerate(layers):
+        src, seen = layer.get("weights_of"), {i}
+        if src is None:
+            continue
+        while layers[src].get("weights_of") is not None and src not in seen:
+            seen.add(src)
+            src = layers[src]["weights_of"]
+        if src in seen:
+            raise ValueError(f"layer {i}: weights_of leads back to the layer itself")
+        if (specs[i].mixer, specs[i].ff) != (specs[src].mixer, specs[src].ff):
+            raise ValueError(f"layer {i}: its sizes differ from those of layer {src}, whose weights it uses")
+        specs[i] = replace(specs[i], weights_of=int(src))
     return specs

@@ -52,7 +52,8 @@ def step_meta(q_len: int, ctx: int, reqs: int, device="cuda"):
     to = lambda t: t.to(torch.int32).to(device)
     return AttentionMetadata(to(pos), to(slots), to(bt), to(torch.full((reqs,), n)), to(qsl), reqs, T,
                              num_decode_reqs=dec, max_query_len=q_len, max_seq_len=n, padded_num_reqs=reqs,
-                             padded_num_tokens=T, query_start_loc_cpu=qsl), reqs * nblk + 1
+                             padded_num_tokens=T, query_start_loc_cpu=qsl, state_slots=to(torch.arange(reqs))), \
+        reqs * nblk + 1
 
 
 def build(cfg: ModelConfig):
