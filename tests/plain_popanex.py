@@ -42,26 +42,36 @@ def rotate_halves(x, rot, first=0):
     """x [S, heads, d], row t at position first + t: dimension i turns with dimension i + dims/2 (i < dims/2)."""
     half = rot["dims"] // 2
     out = x.clone()
-    for t in range(x.shape[0]):
-        for i in range(half):
-            a = (first + t) * rot["base"] ** (-2.0 * i / rot["dims"])
-            c, s = math.cos(a), math.sin(a)
-            u, v = x[t, :, i], x[t, :, i + half]
-            out[t, :, i] = u * c - v * s
-            out[t, :, i + half] = v * c + u * s
+    for i in range(half):
+        a = [(first + t) * rot["base"] ** (-2.0 * i / rot["dims"]) for t in range(x.shape[0])]
+        c = torch.tensor([math.cos(v) for v in a], dtype=x.dtype)[:, None]
+        s = torch.tensor([math.sin(v) for v in a], dtype=x.dtype)[:, None]
+        u, v = x[:, :, i], x[:, :, i + half]
+        out[:, :, i] = u * c - v * s
+        out[:, :, i + half] = v * c + u * s
     return out
+
+
+def outer(k, v):
+    """Per head: [H, d], [H, dv] -> [H, d, dv]."""
+    return k[:, :, None] * v[:, None, :]
+
+
+def read(st, q):
+    """Per head: st^T q."""
+    return (st * q[:, :, None]).sum(1)
 
 
 def retention_states(q, k, v, decay, state=None):
     """q, k [S, H, d], v [S, H, dv], decay [H] -> o [S, H, dv] and the state after the last token."""
     S, H, d = q.shape
-    st = torch.zeros(H, d, v.shape[2], dtype=q.dtype) if state is None else state.clone()
-    o = torch.empty(S, H, v.shape[2], dtype=q.dtype)
+    st = torch.zeros(H, d, v.shape[2], dtype=q.dtype) if state is None else state
+    gamma = torch.as_tensor(decay, dtype=q.dtype)[:, None, None]
+    o = []
     for t in range(S):
-        for h in range(H):
-            st[h] = decay[h] * st[h] + torch.outer(k[t, h], v[t, h])
-            o[t, h] = q[t, h] @ st[h]
-    return o, st
+        st = gamma * st + outer(k[t], v[t])
+        o.append(read(st, q[t]))
+    return torch.stack(o), st
 
 
 def retention(h, w, p, m, eps, forget_at=None):
@@ -84,10 +94,11 @@ def query_temperature(p, qt):
 
 
 def sink_softmax(scores, sink):
-    """scores [S keys] of one query and head; one more term exp(sink) in the denominator."""
-    top = torch.maximum(scores.max(), sink)
+    """scores [..., keys], sink [...]: one more term exp(sink) in the denominator."""
+    sink = sink[..., None]
+    top = torch.maximum(scores.max(-1, keepdim=True).values, sink)
     e = torch.exp(scores - top)
-    return e / (e.sum() + torch.exp(sink - top))
+    return e / (e.sum(-1, keepdim=True) + torch.exp(sink - top))
 
 
 def attention(h, w, p, m, eps, lost_key=None, no_sink=False, no_temp=False):
@@ -96,15 +107,17 @@ def attention(h, w, p, m, eps, lost_key=None, no_sink=False, no_temp=False):
     q = (rms(h @ w[p + "q"].t(), eps) * w[p + "q.norm"]).reshape(S, H, d)
     k = (rms(h @ w[p + "k"].t(), eps) * w[p + "k.norm"]).reshape(S, G, d)
     v = (h @ w[p + "v"].t()).reshape(S, G, dv)
+    t = [1.0 if no_temp else query_temperature(i, m["q_temp"]) for i in range(S)]
+    q = q * torch.tensor(t, dtype=h.dtype)[:, None, None]
+    hidden = torch.ones(S, S, dtype=torch.bool).triu(1)
+    if lost_key is not None:
+        hidden[lost_key + 1:, lost_key] = True
     out = torch.zeros(S, H, dv, dtype=h.dtype)
-    for i in range(S):
-        t = 1.0 if no_temp else query_temperature(i, m["q_temp"])
-        keys = [j for j in range(i + 1) if j != lost_key or j == i]
-        for hh in range(H):
-            g = hh // (H // G)
-            s = (k[keys, g] @ (q[i, hh] * t)) * m["scale"]
-            sink = w[p + "sink"][hh] if not no_sink else torch.tensor(-1e9, dtype=h.dtype)
-            out[i, hh] = sink_softmax(s, sink) @ v[keys, g]
+    for hh in range(H):
+        g = hh // (H // G)
+        s = ((q[:, hh] @ k[:, g].t()) * m["scale"]).masked_fill(hidden, float("-inf"))
+        sink = torch.tensor(-1e9, dtype=h.dtype) if no_sink else w[p + "sink"][hh]
+        out[:, hh] = sink_softmax(s, sink.expand(S)) @ v[:, g]
     return out.reshape(S, H * dv) @ w[p + "o"].t()
 
 
@@ -121,15 +134,14 @@ def short_conv(x, taps, before=None):
 def delta_states(q, k, v, g, beta, state=None):
     """Unit q (scaled), unit k, decay factors g [S, H, d], beta [S, H]; q, k [S, H, d] with one entry per head."""
     S, H, d = g.shape
-    st = torch.zeros(H, d, v.shape[2], dtype=q.dtype) if state is None else state.clone()
-    o = torch.empty(S, H, v.shape[2], dtype=q.dtype)
+    st = torch.zeros(H, d, v.shape[2], dtype=q.dtype) if state is None else state
+    o = []
     for t in range(S):
-        for h in range(H):
-            st[h] = g[t, h][:, None] * st[h]
-            u = beta[t, h] * (v[t, h] - k[t, h] @ st[h])
-            st[h] = st[h] + torch.outer(k[t, h], u)
-            o[t, h] = q[t, h] @ st[h]
-    return o, st
+        st = g[t][:, :, None] * st
+        u = beta[t][:, None] * (v[t] - read(st, k[t]))
+        st = st + outer(k[t], u)
+        o.append(read(st, q[t]))
+    return torch.stack(o), st
 
 
 def delta_decay(a, A_log, dt_bias, H):

@@ -424,7 +424,7 @@ def model_preset(name: str) -> ModelConfig:
         return mc
     if n in ("tiny-popanex",):
         # every mixer, unequal sizes, a layer that runs a second time with a state of its own, layers without an MLP
-        ret = {"heads": 3, "dim": 24, "vdim": 40, "rot": {"base": 5000.0, "dims": 16}, "decay": [0.9, 0.97, 0.995]}
+        ret = {"heads": 2, "dim": 24, "vdim": 40, "rot": {"base": 5000.0, "dims": 16}, "decay": [0.9, 0.99]}
         att = {"heads": 6, "kv_heads": 2, "dim": 24, "vdim": 32, "scale": 0.2, "q_temp": {"coef": 0.3, "every": 48}}
         delta = {"heads": 4, "kv_heads": 2, "dim": 16, "vdim": 24, "conv": 3, "gate_rank": 12}
         ff = {"kind": "dense", "ff": 136}

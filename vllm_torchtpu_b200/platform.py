@@ -211,11 +211,21 @@ class B200Platform:
             if p.pipeline_parallel_size > 1:
                 raise ValueError(f"pipeline parallelism is not built for {m.architecture}: its 32-bit residual stream "
                                  "and shared caches do not cross the stage hand-off")
-            bad = [i for i, l in enumerate(m.layer_specs) if l.mixer.heads % tp]
+            bad = [i for i, l in enumerate(m.layer_specs) if l.mixer.heads % tp
+                   or (l.mixer.recurrent and getattr(l.mixer, "kv_heads", tp) % tp)]
             if bad:
-                raise ValueError(f"the query heads of layers {bad[:8]} do not divide over tp={tp}")
+                raise ValueError(f"the heads of layers {bad[:8]} do not divide over tp={tp}")
+            if not m.is_mla and max(p.decode_context_parallel_size, p.prefill_context_parallel_size) > 1:
+                raise ValueError(f"context parallelism is not built for {m.architecture}")
             if cfg.speculative and cfg.speculative.get("method") not in ("ngram", "suffix", "medusa"):
                 raise ValueError(f"drafters that run a layer of the target are not built for {m.architecture}")
+        if m.has_recurrent_state:
+            if cfg.cache.enable_prefix_caching:
+                # a cached prefix has pages but no state to continue from
+                logger.warning("--enable-prefix-caching ignored: %s carries a recurrent state", m.name)
+                cfg.cache.enable_prefix_caching = False
+            if cfg.kv_transfer:
+                raise ValueError(f"KV transfer is not built for {m.architecture}: its recurrent state would stay behind")
         if p.enable_expert_parallel and not m.is_moe:
             logger.warning("--enable-expert-parallel ignored: %s has no experts", m.name)
             p.enable_expert_parallel = False
