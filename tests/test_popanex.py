@@ -356,7 +356,7 @@ def test_carried_state_over_portions_batches_and_reused_slots(dev, dtype, kind, 
         assert err < (3e-6 if dtype == F32 else 6e-3), (k, err)
         if k != "b":
             es = ((state[slot_of[k]].double().cpu() - st).norm() / st.norm()).item()
-            assert es < (3e-6 if dtype == F32 else 4e-3), (k, es)
+            assert es < (3e-6 if dtype == F32 else 2e-5), (k, es)
     assert (state[1] == 5.0).all()                        # a slot that nobody used
 
 
@@ -373,7 +373,7 @@ def test_strong_decays_leave_recent_tokens_exact(dev, dtype):
     want, st = _carried("delta", p, row.double().cpu(), a.double().cpu(), gate.double().cpu())
     assert torch.isfinite(y).all()
     assert ((y.double().cpu() - want).norm() / want.norm()).item() < (2e-5 if dtype == F32 else 6e-3)
-    assert ((cache[1][0].double().cpu() - st).norm() / st.norm()).item() < (2e-5 if dtype == F32 else 4e-3)
+    assert ((cache[1][0].double().cpu() - st).norm() / st.norm()).item() < 2e-5
 
 
 @pytest.mark.gpu

@@ -384,7 +384,7 @@ template <bool GELU_TANH>
 __device__ __forceinline__ float gated_pair(float g, float u) {
   if constexpr (!GELU_TANH) return g / (1.f + __expf(-g)) * u;
   const float z = 0.7978845608028654f * (g + 0.044715f * g * g * g);
-  return g * (1.f - 1.f / (1.f + __expf(2.f * z))) * u;      // 0.5 (1 + tanh z) = 1 - 1 / (1 + e^2z)
+  return g * (1.f - __fdividef(1.f, 1.f + __expf(2.f * z))) * u;      // 0.5 (1 + tanh z) = 1 - 1 / (1 + e^2z)
 }
 
 __device__ __forceinline__ float soft_cap(float v, float cap) { return cap > 0.f ? cap * tanhf(v / cap) : v; }

@@ -14,7 +14,7 @@
 //
 // Kernels:
 //  * lin_step_kernel: one CTA per (head, request), token by token, everything fused (convolution to gate).  The state
-//    is held in registers, so a decoded token reads and writes it once.  Decoding, and prompts in 32-bit.
+//    is held on chip, so a decoded token reads and writes it once.  Decoding, and prompts in 32-bit.
 //  * prompts in bf16, chunks of 16 tokens:
 //      lin_chunk_kernel (parallel over chunks): with G_i the decays accumulated up to token i of the chunk (log2),
 //        A_ij = beta_i sum_c k_ic k_jc 2^(G_ic - G_jc) (i > j),  Q_ij the same with q_i and i >= j;
@@ -24,9 +24,9 @@
 //        U' = U - W S,  O = q' S + Q U',  S <- 2^G_last S + k'^T U'.
 //        The warp keeps S^T as mma accumulators: they are at the same time the A operand of the two products with S
 //        (the contraction index is permuted alike in the B operand), and U'^T comes out in the layout that the update
-//        and Q U' take.  tf32 operands, fp32 accumulation and state.
+//        and Q U' take.  Every operand is a pair of tf32 numbers (three products), fp32 accumulation and state.
 //      lin_finish_kernel: norm and gate.
-//    The scratch of a slab of chunks stays within the L2.
+//    The scratch of a slab of chunks is read back from the L2; the products of the next slab overlap the scan of this one.
 #include <cstring>
 
 #include "common.cuh"
@@ -41,22 +41,51 @@ __device__ __forceinline__ void put(__nv_bfloat16* p, float v) { *p = __float2bf
 __device__ __forceinline__ float silu(float v) { return v / (1.f + expf(-v)); }
 __device__ __forceinline__ float sigmoid(float v) { return 1.f / (1.f + expf(-v)); }
 __device__ __forceinline__ float softplus(float v) { return fmaxf(v, 0.f) + log1pf(expf(-fabsf(v))); }
+// the same from one exponential and one logarithm; ln(1 + e) by its series where 1 + e would drop digits
+__device__ __forceinline__ float softplus_fast(float v) {
+  const float e = __expf(-fabsf(v));
+  const float s = e < 0.0156f ? e * fmaf(e, fmaf(e, 0.33333333f, -0.5f), 1.f) : __logf(1.f + e);
+  return fmaxf(v, 0.f) + s;
+}
 __device__ __forceinline__ float ex2(float x) {
   float y;
   asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
   return y;
 }
-__device__ __forceinline__ uint32_t tf32(float v) {
-  uint32_t r;
-  asm("cvt.rna.tf32.f32 %0, %1;" : "=r"(r) : "f"(v));
-  return r;
+// x = hi + lo, hi a tf32 number and lo what it leaves out: products of such pairs on the tf32 tensor path, lo * lo
+// dropped, keep 21 bits of the operands
+struct Split {
+  uint32_t hi, lo;
+};
+__device__ __forceinline__ Split split(float v) {
+  Split s;
+  s.hi = __float_as_uint(v) & 0xffffe000u;
+  s.lo = __float_as_uint(v - __uint_as_float(s.hi));
+  return s;
 }
-__device__ __forceinline__ float tf32f(float v) { return __uint_as_float(tf32(v)); }
 __device__ __forceinline__ void mma_tf32(float* c, const uint32_t* a, uint32_t b0, uint32_t b1) {
   asm volatile(
       "mma.sync.aligned.m16n8k8.row.col.f32.tf32.tf32.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
       : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
       : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
+}
+struct SplitA {
+  uint32_t hi[4], lo[4];
+};
+// an accumulator tile (C layout) as the A operand of a product over its columns; see lin_scan_kernel
+__device__ __forceinline__ SplitA split_tile(const float* c) {
+  SplitA a;
+  const Split x0 = split(c[0]), x1 = split(c[2]), x2 = split(c[1]), x3 = split(c[3]);
+  a.hi[0] = x0.hi; a.hi[1] = x1.hi; a.hi[2] = x2.hi; a.hi[3] = x3.hi;
+  a.lo[0] = x0.lo; a.lo[1] = x1.lo; a.lo[2] = x2.lo; a.lo[3] = x3.lo;
+  return a;
+}
+// c += a b, the small terms into c2 (may be c)
+__device__ __forceinline__ void mma_split(float* c, float* c2, const SplitA& a, float b0, float b1) {
+  const Split x = split(b0), y = split(b1);
+  mma_tf32(c, a.hi, x.hi, y.hi);
+  mma_tf32(c2, a.lo, x.hi, y.hi);
+  mma_tf32(c2, a.hi, x.lo, y.lo);
 }
 __device__ __forceinline__ void cp_async16(uint32_t dst, const void* src) {
   asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(dst), "l"(src) : "memory");
@@ -97,20 +126,46 @@ __device__ __forceinline__ int column(const Params& p, int c) {
   const int n = p.Hk * p.dk;
   return c < n ? p.q_off + c : (c < 2 * n ? p.k_off + c - n : p.v_off + c - 2 * n);
 }
-// input of channel c at position pos (zero in front of the sequence): from this step's rows or from the ring
+// input of channel c at position pos > start - taps (zero in front of the sequence): from this step's rows or from the
+// ring, without a branch, so that several of these loads are in flight together
 template <typename E>
 __device__ __forceinline__ float input_at(const Params& p, const Req& q, int pos, int c, int col) {
-  if (pos < 0) return 0.f;
-  if (pos >= q.start) return to_f(reinterpret_cast<const E*>(p.row)[(size_t)(q.qs + pos - q.start) * p.ldr + col]);
-  const int ch = 2 * p.Hk * p.dk + p.H * p.dv;
-  return to_f(reinterpret_cast<const E*>(p.ring)[((size_t)q.slot * p.taps + pos % p.taps) * ch + c]);
+  const int ch = 2 * p.Hk * p.dk + p.H * p.dv, m = pos % p.taps;
+  const E* x = reinterpret_cast<const E*>(p.row) + (size_t)(q.qs + max(pos - q.start, 0)) * p.ldr + col;
+  const E* y = reinterpret_cast<const E*>(p.ring) + ((size_t)q.slot * p.taps + (m < 0 ? m + p.taps : m)) * ch + c;
+  const float v = to_f(*(pos >= q.start ? x : y));
+  return pos < 0 ? 0.f : v;
+}
+// convolution and silu of channel c at position pos; KM: taps it is unrolled for (0: any number)
+template <typename E, int KM>
+__device__ __forceinline__ float conv_at(const Params& p, const Req& q, int pos, int c, int col) {
+  const E* w = reinterpret_cast<const E*>(p.conv_w) + (size_t)c * p.taps;
+  float v = 0.f;
+  if constexpr (KM == 0) {
+    for (int j = 0; j < p.taps; ++j) v = fmaf(to_f(w[j]), input_at<E>(p, q, pos - p.taps + 1 + j, c, col), v);
+  } else {
+    float x[KM], k[KM];
+#pragma unroll
+    for (int j = 0; j < KM; ++j) {
+      const int back = min(KM - 1 - j, p.taps - 1);
+      k[j] = to_f(w[p.taps - 1 - back]);
+      x[j] = input_at<E>(p, q, pos - back, c, col);
+    }
+#pragma unroll
+    for (int j = 0; j < KM; ++j)
+      if (KM - 1 - j < p.taps) v = fmaf(k[j], x[j], v);
+  }
+  return silu(v);
 }
 
 // ------------------------------------------------------------------------------------------- token by token
 // Thread (row group rg, column group cg) owns columns VEC * cg .. of rows rg, rg + RG, ... of the state.
-// HOLD: they stay in registers (at most RPT rows); otherwise the pool is read twice and written once per token.
-template <typename E, bool DELTA, int VEC, int RPT, bool HOLD>
-__global__ void __launch_bounds__(HOLD ? 512 : 1024) lin_step_kernel(const Params p) {
+// Between the reads of a token they are in shared memory, where a CTA's whole state arrives by asynchronous copies while
+// q, k, v are prepared (SMEM), in registers, at most RPT rows (REGS), or nowhere: the pool is read twice (POOL).
+enum Hold { POOL, REGS, SMEM };
+template <typename E, bool DELTA, int VEC, int RPT, Hold HOLD>
+__global__ void __launch_bounds__(HOLD == POOL ? 1024 : (HOLD == REGS ? 512 : 256), HOLD == SMEM ? 3 : 1)
+lin_step_kernel(const Params p) {
   pdl_launch_dependents();
   pdl_wait();
   extern __shared__ __align__(16) float sm[];
@@ -148,8 +203,17 @@ __global__ void __launch_bounds__(HOLD ? 512 : 1024) lin_step_kernel(const Param
     if constexpr (VEC == 4) *reinterpret_cast<float4*>(st + (size_t)i * dv) = make_float4(s[0], s[1], s[2], s[3]);
     else st[(size_t)i * dv] = s[0];
   };
-  float S[HOLD ? RPT : 1][VEC];
-  if constexpr (HOLD) {
+  float* held = po + RG * dv + VEC * cg;      // SMEM: [dk][dv]
+  if constexpr (HOLD == SMEM) {
+    for (int x = 0; x < rows; ++x) {
+      float* d = held + (size_t)(rg + x * RG) * dv;
+      if (fresh) *reinterpret_cast<float4*>(d) = make_float4(0.f, 0.f, 0.f, 0.f);
+      else cp_async16(smem_u32(d), st + (size_t)(rg + x * RG) * dv);
+    }
+    asm volatile("cp.async.commit_group;" ::: "memory");
+  }
+  float S[HOLD == REGS ? RPT : 1][VEC];
+  if constexpr (HOLD == REGS) {
 #pragma unroll
     for (int x = 0; x < RPT; ++x) {
 #pragma unroll
@@ -173,10 +237,7 @@ __global__ void __launch_bounds__(HOLD ? 512 : 1024) lin_step_kernel(const Param
       const int col = column(p, c);
       float v;
       if (p.taps > 0) {
-        const E* w = reinterpret_cast<const E*>(p.conv_w) + (size_t)c * p.taps;
-        v = 0.f;
-        for (int j = 0; j < p.taps; ++j) v += to_f(w[j]) * input_at<E>(p, q, pos - p.taps + 1 + j, c, col);
-        v = silu(v);
+        v = p.taps <= 4 ? conv_at<E, 4>(p, q, pos, c, col) : conv_at<E, 0>(p, q, pos, c, col);
         // a single token enters the ring here; longer portions once all of their readers are done
         if (q.len == 1 && (x >= 2 * dk || h % group == 0))
           reinterpret_cast<E*>(p.ring)[((size_t)q.slot * p.taps + pos % p.taps) * (2 * n + p.H * dv) + c] =
@@ -223,7 +284,7 @@ __global__ void __launch_bounds__(HOLD ? 512 : 1024) lin_step_kernel(const Param
     float mem[VEC], os[VEC];
 #pragma unroll
     for (int e = 0; e < VEC; ++e) mem[e] = os[e] = 0.f;
-    const bool zero = !HOLD && fresh && t == q.qs;
+    const bool zero = HOLD == POOL && fresh && t == q.qs;
     auto pass = [&](int i, float (&s)[VEC]) {
       const float g = DELTA ? sg[i] : decay, kk = sk[i] * ik, qq = sq[i] * iq;
 #pragma unroll
@@ -233,10 +294,18 @@ __global__ void __launch_bounds__(HOLD ? 512 : 1024) lin_step_kernel(const Param
         os[e] = fmaf(qq, s[e], os[e]);
       }
     };
-    if constexpr (HOLD) {
+    if constexpr (HOLD == REGS) {
 #pragma unroll
       for (int x = 0; x < RPT; ++x)
         if (x < rows) pass(rg + x * RG, S[x]);
+    } else if constexpr (HOLD == SMEM) {
+      asm volatile("cp.async.wait_all;" ::: "memory");      // a thread copies and reads its own elements only
+#pragma unroll 4
+      for (int x = 0; x < rows; ++x) {
+        const float4 f = *reinterpret_cast<const float4*>(held + (size_t)(rg + x * RG) * dv);
+        float s[4] = {f.x, f.y, f.z, f.w};
+        pass(rg + x * RG, reinterpret_cast<float(&)[VEC]>(s));
+      }
     } else if (!zero) {
       for (int x = 0; x < rows; ++x) {
         float s[VEC];
@@ -282,7 +351,20 @@ __global__ void __launch_bounds__(HOLD ? 512 : 1024) lin_step_kernel(const Param
     float u[VEC];
 #pragma unroll
     for (int e = 0; e < VEC; ++e) u[e] = act ? su[VEC * cg + e] : 0.f;
-    if constexpr (HOLD) {
+    if constexpr (HOLD == SMEM) {
+      const bool last = t + 1 == q.qs + q.len;
+#pragma unroll 4
+      for (int x = 0; x < rows; ++x) {
+        const int i = rg + x * RG;
+        const float g = DELTA ? sg[i] : decay, kk = sk[i] * ik;
+        float4* d = reinterpret_cast<float4*>(held + (size_t)i * dv);
+        const float4 f = *d;
+        const float4 n4 = make_float4(fmaf(kk, u[0], f.x * g), fmaf(kk, u[1 % VEC], f.y * g),
+                                      fmaf(kk, u[2 % VEC], f.z * g), fmaf(kk, u[3 % VEC], f.w * g));
+        if (last) *reinterpret_cast<float4*>(st + (size_t)i * dv) = n4;
+        else *d = n4;
+      }
+    } else if constexpr (HOLD == REGS) {
 #pragma unroll
       for (int x = 0; x < RPT; ++x)
         if (x < rows) {
@@ -308,7 +390,7 @@ __global__ void __launch_bounds__(HOLD ? 512 : 1024) lin_step_kernel(const Param
     }
     __syncthreads();                    // before the next token's q, k, v
   }
-  if constexpr (HOLD) {
+  if constexpr (HOLD == REGS) {
 #pragma unroll
     for (int x = 0; x < RPT; ++x)
       if (x < rows) store_row(rg + x * RG, S[x]);
@@ -340,18 +422,30 @@ __device__ __forceinline__ void chunk_column(const Params& p, const Req& q, int 
   // rows of this step, in one batch of loads; rows outside the chunk's window are clamped and dropped below
   const bf16* row = reinterpret_cast<const bf16*>(p.row) + (size_t)q.qs * p.ldr + col;
   if constexpr (KM == 0) {
+    if (n == C) {
+      const bf16* x = row + (size_t)t0 * p.ldr;
 #pragma unroll
-    for (int i = 0; i < C; ++i) v[i] = to_f(row[(size_t)(t0 + min(i, n - 1)) * p.ldr]);
+      for (int i = 0; i < C; ++i, x += p.ldr) v[i] = to_f(*x);
+    } else {
 #pragma unroll
-    for (int i = 0; i < C; ++i) v[i] = i < n ? v[i] : 0.f;
+      for (int i = 0; i < C; ++i) v[i] = to_f(row[(size_t)(t0 + min(i, n - 1)) * p.ldr]);
+#pragma unroll
+      for (int i = 0; i < C; ++i) v[i] = i < n ? v[i] : 0.f;
+    }
   } else {
     float x[C + KM - 1], w[KM];
     const bf16* wp = reinterpret_cast<const bf16*>(p.conv_w) + (size_t)c * p.taps;
 #pragma unroll
     for (int j = 0; j < KM; ++j) w[j] = to_f(wp[max(0, j - (KM - p.taps))]);
+    if (n == C && t0 > 0) {
+      const bf16* y = row + (size_t)(t0 - (KM - 1)) * p.ldr;
 #pragma unroll
-    for (int m = 0; m < C + KM - 1; ++m)
-      x[m] = to_f(row[(size_t)max(0, t0 + min(m - (KM - 1), n - 1)) * p.ldr]);
+      for (int m = 0; m < C + KM - 1; ++m, y += p.ldr) x[m] = to_f(*y);
+    } else {
+#pragma unroll
+      for (int m = 0; m < C + KM - 1; ++m)
+        x[m] = to_f(row[(size_t)max(0, t0 + min(m - (KM - 1), n - 1)) * p.ldr]);
+    }
 #pragma unroll
     for (int j = 0; j < KM; ++j)
       if (j < KM - p.taps) w[j] = 0.f;
@@ -365,28 +459,31 @@ __device__ __forceinline__ void chunk_column(const Params& p, const Req& q, int 
       float s = 0.f;
 #pragma unroll
       for (int j = 0; j < KM; ++j) s = fmaf(w[j], x[i + j], s);
-      v[i] = i < n ? s / (1.f + __expf(-s)) : 0.f;
+      v[i] = i < n ? __fdividef(s, 1.f + __expf(-s)) : 0.f;
     }
   }
 }
 
 // grid (requests * slab, H), 256 threads
-template <bool DELTA, int KM>
-__global__ void __launch_bounds__(256, 2) lin_chunk_kernel(const Params p) {
+template <bool DELTA, int KM, int DKP>
+__global__ void __launch_bounds__(256, 3) lin_chunk_kernel(const Params p) {
+  constexpr int dkp = DKP, ds = DKP + 4;
   pdl_launch_dependents();
   pdl_wait();
   extern __shared__ __align__(16) float sm[];
-  __shared__ float beta[C], sa[C][C + 4], norm[2][C];
+  __shared__ float beta[C], power[C + 1];
+  __shared__ __align__(16) float sa[C][C + 4];
   const int slot = blockIdx.x, h = blockIdx.y, tid = threadIdx.x;
   const Req q = request(p, p.req_begin + slot / p.slab);
   const int t0 = (p.chunk_begin + slot % p.slab) * C, n = min(C, q.len - t0);
   if (n <= 0 || q.slot < 0) return;
   const int pos0 = q.start + t0, row0 = q.qs + t0;
-  const int dk = p.dk, dv = p.dv, dkp = p.dkp, ds = dkp + 4, nk = p.Hk * dk, hk = h / (p.H / p.Hk);
+  const int dk = p.dk, dv = p.dv, nk = p.Hk * dk, hk = h / (p.H / p.Hk);
   float* sq = sm;                       // [C][ds]
   float* sk = sq + C * ds;
   float* sg = sk + C * ds;              // decays accumulated from the chunk's first token on, log2 (delta rule)
   // ---- q, k and the accumulated decays
+#pragma unroll 1
   for (int x = tid; x < 2 * dkp; x += 256) {
     const int i0 = x < dkp ? x : x - dkp;
     float v[C];
@@ -402,6 +499,7 @@ __global__ void __launch_bounds__(256, 2) lin_chunk_kernel(const Params p) {
   }
   if constexpr (DELTA) {
     const float a_log = expf(p.A_log[h]) * LOG2E;
+#pragma unroll 1
     for (int c = tid; c < dkp; c += 256) {
       float g = 0.f;
       const int cc = min(c, dk - 1);
@@ -413,7 +511,7 @@ __global__ void __launch_bounds__(256, 2) lin_chunk_kernel(const Params p) {
 #pragma unroll
       for (int i = 0; i < C; ++i) {
         // a factor below 2^-64 leaves nothing of the state in fp32: the sum keeps its digits
-        if (c < dk && i < n) g -= fminf(a_log * softplus(z[i] + b), 64.f);
+        if (c < dk && i < n) g -= fminf(a_log * softplus_fast(z[i] + b), 64.f);
         sg[i * ds + c] = g;
       }
     }
@@ -423,6 +521,7 @@ __global__ void __launch_bounds__(256, 2) lin_chunk_kernel(const Params p) {
   }
   __syncthreads();
   if (p.pairs > 0) {
+#pragma unroll 1
     for (int x = tid; x < C * p.pairs; x += 256) {
       const int i = x / p.pairs, f = x - i * p.pairs;
       float sn, cs;
@@ -447,17 +546,27 @@ __global__ void __launch_bounds__(256, 2) lin_chunk_kernel(const Params p) {
         for (int i = lane; i < dk; i += 32) s += d[i] * d[i];
         m /= sqrtf(warp_sum(s) + UNIT_EPS);
       }
-      if (lane == 0) norm[x >= C][x & (C - 1)] = m;
+      for (int i = lane; i < dk; i += 32) d[i] *= m;
     }
+    if (!DELTA && tid <= C) power[tid] = exp2f(fmaxf(log2f(p.decay[h]), -64.f) * (float)tid);
   }
   __syncthreads();
   const size_t unit = (size_t)slot * p.H + h;
-  const float ld = DELTA ? 0.f : fmaxf(log2f(p.decay[h]), -64.f);
   // ---- products of the tokens of the chunk
   {
-    const int i = tid >> 4, j = tid & 15;
-    float qk = 0.f, kk = 0.f;
-    if (j <= i) {
+    // thread -> pair (i, j <= i): rows r and 15 - r of the triangle are 17 pairs together
+    int i = 0, j = C;
+    if (tid < 8 * 17) {
+      const int r = tid / 17, x = tid - 17 * r;
+      i = x <= r ? r : 15 - r;
+      j = x <= r ? x : x - r - 1;
+    } else if (tid - 8 * 17 < 120) {     // pairs above the diagonal: zeros
+      const int y = tid - 8 * 17, r = y / 15, x = y - 15 * r;
+      i = x < 15 - r ? r : 15 - r;
+      j = x < 15 - r ? r + 1 + x : x + 1;
+    }
+    if (tid < 8 * 17) {
+      float qk = 0.f, kk = 0.f;
       const float *qi = sq + i * ds, *ki = sk + i * ds, *kj = sk + j * ds, *gi = sg + i * ds, *gj = sg + j * ds;
       for (int c = 0; c < dkp; c += 4) {
         const float4 a = *reinterpret_cast<const float4*>(qi + c), b = *reinterpret_cast<const float4*>(kj + c);
@@ -472,36 +581,38 @@ __global__ void __launch_bounds__(256, 2) lin_chunk_kernel(const Params p) {
           qk = fmaf(a.x, b.x, qk); qk = fmaf(a.y, b.y, qk); qk = fmaf(a.z, b.z, qk); qk = fmaf(a.w, b.w, qk);
         }
       }
-      qk *= norm[0][i] * norm[1][j];
-      if constexpr (!DELTA) qk *= exp2f(ld * (float)(i - j));
-      kk *= norm[1][i] * norm[1][j];
+      if constexpr (!DELTA) qk *= power[i - j];
+      p.aq[(unit * C + i) * AQ_LD + j] = qk;
+      if constexpr (DELTA) sa[i][j] = j < i ? beta[i] * kk : 0.f;
+    } else if (j < C) {
+      p.aq[(unit * C + i) * AQ_LD + j] = 0.f;
     }
-    p.aq[(unit * C + i) * AQ_LD + j] = tf32f(qk);
-    if constexpr (DELTA) sa[i][j] = j < i ? beta[i] * kk : 0.f;
   }
   if constexpr (DELTA) __syncthreads();
   // ---- columns of W and U (forward substitution), q', k', last decay
+#pragma unroll 1
   for (int x = tid; x < dkp + p.dvp; x += 256) {
     float v[C];
+    asm volatile("" ::: "memory");       // values that do not depend on the column stay in shared memory
     if (x < dkp) {
       float *qd = p.qd + unit * C * (dkp + 8) + x, *kd = p.kd + unit * C * (dkp + 4) + x;
       if constexpr (DELTA) {
         const float last = sg[(C - 1) * ds + x];
 #pragma unroll
         for (int i = 0; i < C; ++i) {
-          const float g = sg[i * ds + x], e = ex2(g), k = sk[i * ds + x] * norm[1][i];
-          qd[i * (dkp + 8)] = tf32f(sq[i * ds + x] * norm[0][i] * e);
-          kd[i * (dkp + 4)] = tf32f(k * ex2(last - g));
+          const float g = sg[i * ds + x], e = ex2(g), k = sk[i * ds + x];
+          qd[i * (dkp + 8)] = sq[i * ds + x] * e;
+          kd[i * (dkp + 4)] = k * ex2(last - g);
           v[i] = beta[i] * k * e;
         }
         p.gl[unit * dkp + x] = ex2(last);
       } else {
 #pragma unroll
         for (int i = 0; i < C; ++i) {
-          qd[i * (dkp + 8)] = tf32f(sq[i * ds + x] * norm[0][i] * exp2f(ld * (float)(i + 1)));
-          kd[i * (dkp + 4)] = i < n ? tf32f(sk[i * ds + x] * norm[1][i] * exp2f(ld * (float)(n - 1 - i))) : 0.f;
+          qd[i * (dkp + 8)] = sq[i * ds + x] * power[i + 1];
+          kd[i * (dkp + 4)] = sk[i * ds + x] * power[max(n - 1 - i, 0)];      // k is zero from token n on
         }
-        p.gl[unit * dkp + x] = exp2f(ld * (float)n);
+        p.gl[unit * dkp + x] = power[n];
       }
     } else {
       const int j = x - dkp;
@@ -519,19 +630,27 @@ __global__ void __launch_bounds__(256, 2) lin_chunk_kernel(const Params p) {
     if constexpr (DELTA) {
 #pragma unroll
       for (int i = 1; i < C; ++i) {
+        asm volatile("" ::: "memory");   // one row of A in registers at a time
 #pragma unroll
-        for (int j = 0; j < i; ++j) v[i] = fmaf(-sa[i][j], v[j], v[i]);
+        for (int j = 0; j < i; j += 4) {
+          const float4 a = *reinterpret_cast<const float4*>(&sa[i][j]);      // zeros from column i on
+          v[i] = fmaf(-a.x, v[j], v[i]);
+          if (j + 1 < i) v[i] = fmaf(-a.y, v[j + 1], v[i]);
+          if (j + 2 < i) v[i] = fmaf(-a.z, v[j + 2], v[i]);
+          if (j + 3 < i) v[i] = fmaf(-a.w, v[j + 3], v[i]);
+        }
       }
       if (x < dkp) {
         float* w = p.w + unit * C * (dkp + 8) + x;
 #pragma unroll
-        for (int i = 0; i < C; ++i) w[i * (dkp + 8)] = tf32f(-v[i]);
+        for (int i = 0; i < C; ++i) w[i * (dkp + 8)] = -v[i];
       }
     }
     if (x >= dkp) {
-      float* u = p.u + unit * C * p.dvp + x - dkp;
+      const int j = x - dkp;             // [dvp / 64][C][64]: a CTA of the scan reads one block
+      float* u = p.u + (unit * (p.dvp / 64) + j / 64) * C * 64 + j % 64;
 #pragma unroll
-      for (int i = 0; i < C; ++i) u[i * p.dvp] = v[i];
+      for (int i = 0; i < C; ++i) u[i * 64] = v[i];
     }
   }
 }
@@ -574,7 +693,7 @@ __global__ void __launch_bounds__(128) lin_scan_kernel(const Params p) {
 #pragma unroll
     for (int i = tid; i < C * 16; i += 128) {
       const int r = i >> 4, s = (i & 15) * 4;
-      cp_async16(d + (L::U + r * L::U_LD + s) * 4, p.u + (unit * C + r) * p.dvp + col0 + s);
+      cp_async16(d + (L::U + r * L::U_LD + s) * 4, p.u + ((unit * splits + col0 / 64) * C + r) * 64 + s);
     }
   };
   float* st = p.state + ((size_t)q.slot * p.H + h) * dk * dv;
@@ -601,40 +720,46 @@ __global__ void __launch_bounds__(128) lin_scan_kernel(const Params p) {
     asm volatile("cp.async.commit_group;" ::: "memory");
     const float* b = sm + (c % L::STAGES) * L::WORDS;
     float U[2][4], O[2][4];              // transposed: rows value columns, columns tokens 8 x + 2 t, + 1
+    float U2[2][4], O2[2][4];            // small terms
 #pragma unroll
     for (int x = 0; x < 2; ++x) {
       const float* u = b + L::U + (8 * x + 2 * t) * L::U_LD + warp * 16 + g;
       U[x][0] = u[0]; U[x][1] = u[L::U_LD]; U[x][2] = u[8]; U[x][3] = u[L::U_LD + 8];
-      O[x][0] = O[x][1] = O[x][2] = O[x][3] = 0.f;
+#pragma unroll
+      for (int e = 0; e < 4; ++e) O[x][e] = O2[x][e] = U2[x][e] = 0.f;
     }
     const float* qd = b + L::QD + g * (DKP + 8) + 2 * t;
     const float* w = b + L::W + g * (DKP + 8) + 2 * t;
 #pragma unroll
     for (int x = 0; x < NT; ++x) {
-      const uint32_t a[4] = {tf32(S[x][0]), tf32(S[x][2]), tf32(S[x][1]), tf32(S[x][3])};
+      const SplitA a = split_tile(S[x]);
 #pragma unroll
       for (int y = 0; y < 2; ++y) {
-        const uint2 bq = *reinterpret_cast<const uint2*>(qd + 8 * y * (DKP + 8) + 8 * x);
-        mma_tf32(O[y], a, bq.x, bq.y);
         if constexpr (DELTA) {
-          const uint2 bw = *reinterpret_cast<const uint2*>(w + 8 * y * (DKP + 8) + 8 * x);
-          mma_tf32(U[y], a, bw.x, bw.y);
+          const float2 bw = *reinterpret_cast<const float2*>(w + 8 * y * (DKP + 8) + 8 * x);
+          mma_split(U[y], U2[y], a, bw.x, bw.y);
         }
+        const float2 bq = *reinterpret_cast<const float2*>(qd + 8 * y * (DKP + 8) + 8 * x);
+        mma_split(O[y], O2[y], a, bq.x, bq.y);
       }
     }
-    uint32_t ua[2][4];
+    SplitA ua[2];
 #pragma unroll
     for (int x = 0; x < 2; ++x) {
-      ua[x][0] = tf32(U[x][0]); ua[x][1] = tf32(U[x][2]); ua[x][2] = tf32(U[x][1]); ua[x][3] = tf32(U[x][3]);
+#pragma unroll
+      for (int e = 0; e < 4; ++e) U[x][e] += U2[x][e];
+      ua[x] = split_tile(U[x]);
     }
 #pragma unroll
     for (int y = 0; y < 2; ++y) {
 #pragma unroll
       for (int x = 0; x < 2; ++x) {
         if (x > y) continue;             // Q is lower triangular
-        const uint2 bq = *reinterpret_cast<const uint2*>(b + L::AQ + (8 * y + g) * AQ_LD + 8 * x + 2 * t);
-        mma_tf32(O[y], ua[x], bq.x, bq.y);
+        const float2 bq = *reinterpret_cast<const float2*>(b + L::AQ + (8 * y + g) * AQ_LD + 8 * x + 2 * t);
+        mma_split(O[y], O2[y], ua[x], bq.x, bq.y);
       }
+#pragma unroll
+      for (int e = 0; e < 4; ++e) O[y][e] += O2[y][e];
     }
     const float* kd = b + L::KD + 2 * t * (DKP + 4) + g;
     const float* gl = b + L::GL + 2 * t;
@@ -645,7 +770,7 @@ __global__ void __launch_bounds__(128) lin_scan_kernel(const Params p) {
 #pragma unroll
       for (int y = 0; y < 2; ++y) {
         const float* k = kd + 8 * y * (DKP + 4) + 8 * x;
-        mma_tf32(S[x], ua[y], __float_as_uint(k[0]), __float_as_uint(k[DKP + 4]));
+        mma_split(S[x], S[x], ua[y], k[0], k[DKP + 4]);
       }
     }
     const int rows = min(C, q.len - (p.chunk_begin + c) * C);
@@ -695,13 +820,13 @@ __global__ void __launch_bounds__(256) lin_finish_kernel(const Params p) {
 }
 
 // ------------------------------------------------------------------------------------------- host
-template <typename E, bool DELTA, int VEC, int RPT, bool HOLD>
+template <typename E, bool DELTA, int VEC, int RPT, Hold HOLD>
 static int launch_step_as(const Params& p, int R, int threads, cudaStream_t stream) {
   const int RG = threads / (p.dv / VEC);
-  const int smem = (3 * p.dk + 2 * p.dv + 2 * RG * p.dv) * (int)sizeof(float);
+  const int smem = (3 * p.dk + 2 * p.dv + 2 * RG * p.dv + (HOLD == SMEM ? p.dk * p.dv : 0)) * (int)sizeof(float);
   static unsigned long long seen = 0;
-  if (smem > 48 * 1024)
-    B200_CUDA_CHECK(ensure_dynamic_smem(lin_step_kernel<E, DELTA, VEC, RPT, HOLD>, 200 * 1024, &seen));
+  if (smem > 46 * 1024)
+    B200_CUDA_CHECK(ensure_dynamic_smem(lin_step_kernel<E, DELTA, VEC, RPT, HOLD>, 220 * 1024, &seen));
   B200_CUDA_CHECK(launch_pdl(lin_step_kernel<E, DELTA, VEC, RPT, HOLD>, dim3(p.H, R), dim3(threads), (size_t)smem,
                              stream, p));
   return 0;
@@ -710,11 +835,16 @@ static int launch_step_as(const Params& p, int R, int threads, cudaStream_t stre
 template <typename E, bool DELTA, int VEC>
 static int launch_step_v(const Params& p, int R, cudaStream_t stream) {
   const int ncg = p.dv / VEC;
+  if constexpr (VEC == 4) {
+    // q, k and the decays are read as floats: the state behind them starts on 16 bytes when 3 dk is a multiple of 4
+    if (p.dk % 4 == 0 && ncg <= 256 && p.dk * p.dv <= 48 * 1024)
+      return launch_step_as<E, DELTA, VEC, 1, SMEM>(p, R, p.dk * p.dv <= 2048 && ncg <= 128 ? 128 : 256, stream);
+  }
   for (int threads = 128; threads <= 512; threads *= 2) {
     if (threads < ncg) continue;
     const int RG = threads / ncg, rows = (p.dk + RG - 1) / RG;
-    if (rows <= 4) return launch_step_as<E, DELTA, VEC, 4, true>(p, R, threads, stream);
-    if (rows <= 16) return launch_step_as<E, DELTA, VEC, 16, true>(p, R, threads, stream);
+    if (rows <= 4) return launch_step_as<E, DELTA, VEC, 4, REGS>(p, R, threads, stream);
+    if (rows <= 16) return launch_step_as<E, DELTA, VEC, 16, REGS>(p, R, threads, stream);
   }
   int threads = 512;
   while (threads < ncg) threads *= 2;
@@ -722,7 +852,7 @@ static int launch_step_v(const Params& p, int R, cudaStream_t stream) {
     b200_set_last_error("linear attention: at most 1024 value columns per thread group", __FILE__, __LINE__);
     return -1;
   }
-  return launch_step_as<E, DELTA, VEC, 1, false>(p, R, threads, stream);
+  return launch_step_as<E, DELTA, VEC, 1, POOL>(p, R, threads, stream);
 }
 
 template <typename E>
@@ -743,13 +873,22 @@ static int launch_scan(const Params& p, int R, cudaStream_t stream) {
   return 0;
 }
 
+template <bool DELTA, int KM, int DKP>
+static int launch_chunk_as(const Params& p, int R, cudaStream_t stream) {
+  constexpr int smem = (DELTA ? 3 : 2) * C * (DKP + 4) * (int)sizeof(float);
+  static unsigned long long seen = 0;
+  if (smem > 44 * 1024) B200_CUDA_CHECK(ensure_dynamic_smem(lin_chunk_kernel<DELTA, KM, DKP>, smem, &seen));
+  B200_CUDA_CHECK(launch_pdl(lin_chunk_kernel<DELTA, KM, DKP>, dim3(R * p.slab, p.H), dim3(256), (size_t)smem, stream, p));
+  return 0;
+}
 template <bool DELTA, int KM>
 static int launch_chunk(const Params& p, int R, cudaStream_t stream) {
-  const int smem = (DELTA ? 3 : 2) * C * (p.dkp + 4) * (int)sizeof(float);
-  static unsigned long long seen = 0;
-  if (smem > 44 * 1024) B200_CUDA_CHECK(ensure_dynamic_smem(lin_chunk_kernel<DELTA, KM>, 100 * 1024, &seen));
-  B200_CUDA_CHECK(launch_pdl(lin_chunk_kernel<DELTA, KM>, dim3(R * p.slab, p.H), dim3(256), (size_t)smem, stream, p));
-  return 0;
+  switch (p.dkp) {
+    case 32: return launch_chunk_as<DELTA, KM, 32>(p, R, stream);
+    case 64: return launch_chunk_as<DELTA, KM, 64>(p, R, stream);
+    case 128: return launch_chunk_as<DELTA, KM, 128>(p, R, stream);
+    default: return launch_chunk_as<DELTA, KM, 256>(p, R, stream);
+  }
 }
 
 static int padded_dk(int dk) { return dk <= 32 ? 32 : (dk <= 64 ? 64 : (dk <= 128 ? 128 : 256)); }
@@ -760,8 +899,9 @@ static size_t chunk_words(int dk, int dv, bool delta) {
   return (size_t)C * ((delta ? 2 : 1) * (dkp + 8) + dkp + 4 + dvp + AQ_LD + dv) + dkp;
 }
 
+// one of the three kernels of a slab of chunks
 template <bool DELTA>
-static int launch_chunks(Params& p, int R, float* scratch, cudaStream_t stream) {
+static int launch_chunks(Params& p, int R, float* scratch, int mode, cudaStream_t stream) {
   const size_t units = (size_t)R * p.slab * p.H;
   p.qd = scratch;
   p.w = p.qd + units * C * (p.dkp + 8);
@@ -770,16 +910,17 @@ static int launch_chunks(Params& p, int R, float* scratch, cudaStream_t stream) 
   p.aq = p.u + units * C * p.dvp;
   p.gl = p.aq + units * C * AQ_LD;
   p.o = p.gl + units * p.dkp;
-  int rc = p.taps == 0 ? launch_chunk<DELTA, 0>(p, R, stream)
+  if (mode == 1)
+    return p.taps == 0 ? launch_chunk<DELTA, 0>(p, R, stream)
                        : (p.taps <= 4 ? launch_chunk<DELTA, 4>(p, R, stream) : launch_chunk<DELTA, 8>(p, R, stream));
-  if (rc) return rc;
-  switch (p.dkp) {
-    case 32: rc = launch_scan<DELTA, 4>(p, R, stream); break;
-    case 64: rc = launch_scan<DELTA, 8>(p, R, stream); break;
-    case 128: rc = launch_scan<DELTA, 16>(p, R, stream); break;
-    default: rc = launch_scan<DELTA, 32>(p, R, stream); break;
+  if (mode == 3) {
+    switch (p.dkp) {
+      case 32: return launch_scan<DELTA, 4>(p, R, stream);
+      case 64: return launch_scan<DELTA, 8>(p, R, stream);
+      case 128: return launch_scan<DELTA, 16>(p, R, stream);
+      default: return launch_scan<DELTA, 32>(p, R, stream);
+    }
   }
-  if (rc) return rc;
   B200_CUDA_CHECK(launch_pdl(lin_finish_kernel, dim3(R * p.slab * C, (p.H + 7) / 8), dim3(256), (size_t)0, stream, p));
   return 0;
 }
@@ -793,9 +934,9 @@ extern "C" size_t b200_linear_attention_chunk_bytes(int dk, int dv, int delta) {
 }
 
 // Requests [req_begin, req_end) of the batch.  mode 0: token by token (any sizes; the ring takes portions of more than
-// one token when ring_update is set); mode 1: chunks [chunk_begin, chunk_begin + slab) of every request (bf16,
-// dk <= 256, taps <= 8; scratch for (req_end - req_begin) * slab * H chunks); mode 2: the ring of a prompt that ran in
-// mode 1.  decay != null: fixed decay per head, otherwise the delta rule with a, A_log, dt_bias and the step sizes in
+// one token through mode 2); mode 1: products of chunks [chunk_begin, chunk_begin + slab) of every request (bf16, dk <=
+// 256, taps <= 8; into scratch for (req_end - req_begin) * slab * H chunks), mode 3: their recurrence, mode 4: their
+// norm and gate; mode 2: the ring of a prompt.  decay != null: fixed decay per head, otherwise the delta rule with a, A_log, dt_bias and the step sizes in
 // column beta_off of the row.  elem: 2 = bf16, 4 = fp32.
 extern "C" int b200_linear_attention(int mode, const void* row, int ldr, int q_off, int k_off, int v_off, int beta_off,
                                      const void* a, int lda, const void* gate, int ldg, const void* conv_w, void* ring,
@@ -825,13 +966,13 @@ extern "C" int b200_linear_attention(int mode, const void* row, int ldr, int q_o
   p.dkp = lin::padded_dk(dk); p.dvp = (dv + 63) / 64 * 64;
   p.slab = slab; p.chunk_begin = chunk_begin;
   if (mode == 0) return elem == 4 ? lin::launch_step<float>(p, R, stream) : lin::launch_step<__nv_bfloat16>(p, R, stream);
-  if (mode == 1) {
+  if (mode == 1 || mode == 3 || mode == 4) {
     if (elem != 2 || dk > 256 || taps > 8 || slab <= 0 || scratch == nullptr) {
       b200_set_last_error("linear attention in chunks: bf16, dk of at most 256, at most 8 taps", __FILE__, __LINE__);
       return -1;
     }
-    return decay == nullptr ? lin::launch_chunks<true>(p, R, (float*)scratch, stream)
-                            : lin::launch_chunks<false>(p, R, (float*)scratch, stream);
+    return decay == nullptr ? lin::launch_chunks<true>(p, R, (float*)scratch, mode, stream)
+                            : lin::launch_chunks<false>(p, R, (float*)scratch, mode, stream);
   }
   const dim3 grid((2 * Hk * dk + H * dv + 255) / 256, R);
   if (elem == 4) B200_CUDA_CHECK(launch_pdl(lin::lin_ring_kernel<float>, grid, dim3(256), (size_t)0, stream, p));

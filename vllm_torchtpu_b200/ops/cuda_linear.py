@@ -1,16 +1,17 @@
 """Bindings of the carried-state linear-attention kernels (``csrc/linear_attention.cu``)."""
 from __future__ import annotations
 
-from ctypes import c_float, c_int
+from ctypes import c_float, c_int, c_void_p
 
 import torch
 
 from . import count_launch
 from . import cuda as _c
 
-STEP, CHUNKS, RING = 0, 1, 2
+STEP, CHUNKS, RING, SCAN, FINISH = 0, 1, 2, 3, 4
 CHUNK = 16
-SCRATCH_BYTES = 48 << 20                 # of one slab of chunks: stays within the L2
+SCRATCH_BYTES = 64 << 20                 # of one slab of chunks: two of them about fill the L2
+_side: dict = {}                         # device index -> stream of the scans
 
 
 def slabs(lens, heads: int, chunk_bytes: int, budget: int = SCRATCH_BYTES) -> list:
@@ -28,6 +29,13 @@ def slabs(lens, heads: int, chunk_bytes: int, budget: int = SCRATCH_BYTES) -> li
         out += [(i, j, c, min(n, most - c)) for c in range(0, most, n)]
         i = j
     return out
+
+
+def _side_stream(device):
+    i = torch.device(device).index or 0
+    if i not in _side:
+        _side[i] = torch.cuda.Stream(device)
+    return _side[i]
 
 
 def carried_state_attention(plan, row, decay_in, gate, meta, cache):
@@ -49,7 +57,7 @@ def carried_state_attention(plan, row, decay_in, gate, meta, cache):
     y = (torch.empty if whole else torch.zeros)((T, p.heads * p.vdim), dtype=row.dtype, device=row.device)
     L = _c.lib()
 
-    def call(mode, lo, hi, scratch=None, chunk=0, slab=0):
+    def call(mode, lo, hi, scratch=None, chunk=0, slab=0, stream=None):
         _c._check(L.b200_linear_attention(
             c_int(mode), _c._p(row), c_int(row.stride(0)), *(c_int(o) for o in p.offsets), c_int(p.beta_offset),
             _c._p(decay_in), c_int(decay_in.stride(0) if decay_in is not None else 0), _c._p(gate),
@@ -59,19 +67,34 @@ def carried_state_attention(plan, row, decay_in, gate, meta, cache):
             _c._p(meta.seq_lens), _c._p(meta.state_slots), c_int(lo), c_int(hi), c_int(T), c_int(p.heads),
             c_int(p.k_heads), c_int(p.dim), c_int(p.vdim), c_int(int(p.unit_norm)), c_int(int(p.gate_act == "silu")),
             c_float(p.eps), c_float(p.q_mult), c_float(p.k_mult), c_int(int(decode_only)), _c._p(scratch),
-            c_int(chunk), c_int(slab), c_int(elem), _c._stream()), "linear_attention")
-        count_launch(3 if mode == CHUNKS else 1)
+            c_int(chunk), c_int(slab), c_int(elem),
+            _c._stream() if stream is None else c_void_p(stream.cuda_stream)), "linear_attention")
+        count_launch()
 
     if n_dec:
         call(STEP, 0, n_dec)
     if lens:
         if elem == 2 and p.dim <= 256 and p.taps <= 8:
             per = int(L.b200_linear_attention_chunk_bytes(c_int(p.dim), c_int(p.vdim), c_int(int(p.delta))))
-            plan_ = slabs(lens, p.heads, per)
-            scratch = torch.empty(max((j - i) * n for i, j, _, n in plan_) * p.heads * per, dtype=torch.uint8,
-                                  device=row.device)
-            for i, j, c, n in plan_:
-                call(CHUNKS, nd + i, nd + j, scratch, c, n)
+            parts = slabs(lens, p.heads, per)
+            room = max((j - i) * n for i, j, _, n in parts) * p.heads * per
+            scratch = torch.empty((min(2, len(parts)), room), dtype=torch.uint8, device=row.device)
+            main = torch.cuda.current_stream()
+            side = main if len(parts) == 1 else _side_stream(row.device)
+            last = None                   # slab whose scan is on its way: (arguments, event)
+            for x, (i, j, c, n) in enumerate(parts):
+                args = (nd + i, nd + j, scratch[x & 1], c, n)
+                call(CHUNKS, *args)
+                if side is not main:
+                    side.wait_event(main.record_event())
+                call(SCAN, *args, side)   # a chain over the chunks with few CTAs: beside the next slab's products
+                if last is not None:
+                    main.wait_event(last[1])
+                    call(FINISH, *last[0])
+                last = (args, side.record_event() if side is not main else None)
+            if last[1] is not None:
+                main.wait_event(last[1])
+            call(FINISH, *last[0])
         else:
             call(STEP, nd, R)
         if p.taps:
