@@ -14,7 +14,7 @@ import torch
 from test_mazivik import BF16, DEV_DTYPE, DEVS, F32, ROOT, _close, _rand, logit_error, portions, replay_logits, tokens_of
 
 from vllm_torchtpu_b200 import SamplingParams, ops
-from vllm_torchtpu_b200.config import EngineConfig, ModelConfig, ParallelConfig, model_preset
+from vllm_torchtpu_b200.config import CacheConfig, EngineConfig, ModelConfig, ParallelConfig, model_preset
 from vllm_torchtpu_b200.entrypoints.trace_replay import make_replay
 from vllm_torchtpu_b200.ops import linear_attention as la
 from vllm_torchtpu_b200.runner.attn_metadata import AttentionMetadata
@@ -609,6 +609,7 @@ def test_configuration_reads_every_size_and_refuses_what_is_not_built():
                     (MIXED, dict(parallel=ParallelConfig(pipeline_parallel_size=2))),
                     (MIXED, dict(speculative={"method": "mtp"})),
                     (MIXED, dict(kv_transfer={"kv_connector": "B200HostConnector"})),
+                    (MIXED, dict(cache=CacheConfig(kv_cache_dtype="fp8"))),
                     (MODELS["attention_only"], dict(parallel=ParallelConfig(prefill_context_parallel_size=2)))):
         with pytest.raises(ValueError):
             EngineConfig(model=ModelConfig.from_hf_dict(cfg), device="cpu", **kw).finalize()

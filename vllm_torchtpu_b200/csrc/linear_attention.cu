@@ -839,12 +839,13 @@ static int launch_step_v(const Params& p, int R, cudaStream_t stream) {
     // q, k and the decays are read as floats: the state behind them starts on 16 bytes when 3 dk is a multiple of 4
     if (p.dk % 4 == 0 && ncg <= 256 && p.dk * p.dv <= 48 * 1024)
       return launch_step_as<E, DELTA, VEC, 1, SMEM>(p, R, p.dk * p.dv <= 2048 && ncg <= 128 ? 128 : 256, stream);
-  }
-  for (int threads = 128; threads <= 512; threads *= 2) {
-    if (threads < ncg) continue;
-    const int RG = threads / ncg, rows = (p.dk + RG - 1) / RG;
-    if (rows <= 4) return launch_step_as<E, DELTA, VEC, 4, REGS>(p, R, threads, stream);
-    if (rows <= 16) return launch_step_as<E, DELTA, VEC, 16, REGS>(p, R, threads, stream);
+  } else {
+    for (int threads = 128; threads <= 512; threads *= 2) {
+      if (threads < ncg) continue;
+      const int RG = threads / ncg, rows = (p.dk + RG - 1) / RG;
+      if (rows <= 4) return launch_step_as<E, DELTA, VEC, 4, REGS>(p, R, threads, stream);
+      if (rows <= 16) return launch_step_as<E, DELTA, VEC, 16, REGS>(p, R, threads, stream);
+    }
   }
   int threads = 512;
   while (threads < ncg) threads *= 2;

@@ -217,6 +217,8 @@ class B200Platform:
                 raise ValueError(f"the heads of layers {bad[:8]} do not divide over tp={tp}")
             if not m.is_mla and max(p.decode_context_parallel_size, p.prefill_context_parallel_size) > 1:
                 raise ValueError(f"context parallelism is not built for {m.architecture}")
+            if not m.is_mla and cfg.cache.kv_cache_dtype.startswith("fp8"):
+                raise ValueError(f"an fp8 KV cache is not built for {m.architecture}")
             if cfg.speculative and cfg.speculative.get("method") not in ("ngram", "suffix", "medusa"):
                 raise ValueError(f"drafters that run a layer of the target are not built for {m.architecture}")
         if m.has_recurrent_state:
