@@ -389,6 +389,43 @@ def test_decode_rows_of_padded_requests_come_back_as_zeros():
     assert (y[2:] == 0).all() and (y[:2] != 0).any() and (cache[1][1] == 0).all()
 
 
+@pytest.mark.gpu
+@pytest.mark.parametrize("kind,taps", [("retention", 0), ("delta", 4)])
+@pytest.mark.parametrize("chunks", [1, 5])
+def test_prompts_in_several_slabs_on_two_streams(monkeypatch, kind, taps, chunks):
+    """A scratch of few chunks: states cross slabs in the pool, requests of unequal lengths end in different slabs."""
+    from vllm_torchtpu_b200.ops import cuda, cuda_linear
+    H, d, dv = 2, 64, 96
+    per = cuda.lib().b200_linear_attention_chunk_bytes(d, dv, int(kind == "delta"))
+    monkeypatch.setattr(cuda_linear.slabs, "__defaults__", (chunks * H * per,))
+    p, n = _plan(kind, BF16, "cuda", H, H, d, dv, taps)
+    lens, slots = [1, 150, 33, 2, 97], [4, 2, 0, 3, 1]
+    assert len(cuda_linear.slabs(lens[1:], H, per)) > 3
+    state = torch.full(p.state_shape(5), 5.0, device="cuda")
+    cache = (torch.full(p.ring_shape(5), 5.0, dtype=BF16, device="cuda"), state) if taps else (state,)
+    seqs = []
+    for i, t in enumerate(lens):
+        t += i == 0
+        seqs.append((_rand("cuda", BF16, t, n, seed=i), _rand("cuda", BF16, t, H * d, seed=i + 20) if taps else None,
+                     _rand("cuda", BF16, t, H * dv, seed=i + 40)))
+    first = tuple(t[:1] if t is not None else None for t in seqs[0])
+    ops.carried_state_attention(p, *first, _state_meta("cuda", [1], [0], [4]), cache)
+    parts = [tuple(t[1:] if t is not None else None for t in seqs[0])] + seqs[1:]
+    row, a, gate = (torch.cat(t) if t[0] is not None else None for t in zip(*parts))
+    for _ in range(2):                                    # the second time over states that the first one left
+        y = ops.carried_state_attention(p, row, a, gate, _state_meta("cuda", lens, [1, 0, 0, 0, 0], slots), cache)
+        if _ == 0:
+            y0 = y.clone()
+    at = 1
+    for (r, a_, g), x, slot in list(zip(seqs, lens, slots))[1:]:
+        want, st = _carried(kind, p, r.double().cpu(), a_.double().cpu() if taps else None, g.double().cpu())
+        for got in (y0, y):
+            e = got[at:at + x].double().cpu() - want
+            assert (e.norm() / want.norm()).item() < 6e-3
+        assert ((state[slot].double().cpu() - st).norm() / st.norm()).item() < 2e-5
+        at += x
+
+
 def test_slabs_cover_every_chunk_once():
     from vllm_torchtpu_b200.ops.cuda_linear import CHUNK, slabs
     for lens in ([1], [16, 17, 1, 400], [5000], [3] * 300 + [2000]):
