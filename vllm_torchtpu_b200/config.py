@@ -16,7 +16,8 @@ from typing import Any, Optional
 
 import torch
 
-from .layer_specs import LatentMixerSpec, LayerSpec, RotarySpec, layer_specs  # noqa: F401
+from .layer_specs import (DeltaMixerSpec, GroupedMixerSpec, LatentMixerSpec, LayerSpec, RetentionMixerSpec,  # noqa: F401
+                          RotarySpec, layer_specs)
 
 _DTYPES = {
     "float32": torch.float32, "fp32": torch.float32, "float": torch.float32,
@@ -33,7 +34,7 @@ def parse_dtype(d) -> torch.dtype:
 
 @dataclass
 class ModelConfig:
-    architecture: str = "llama"          # llama | qwen3_moe | gpt_oss | deepseek_v3 | qwen3_next | kimi_linear | mazivik | popanex
+    architecture: str = "llama"          # llama | qwen3_moe | gpt_oss | deepseek_v3 | qwen3_next | kimi_linear | mazivik | popanex | zeganex
     name: str = "tiny-llama"
     num_layers: int = 2
     hidden_size: int = 256
@@ -73,6 +74,7 @@ class ModelConfig:
     moe_n_group: int = 1
     moe_topk_group: int = 1
     moe_score_bias: bool = False
+    moe_router_fp32: bool = False        # router logits in 32-bit, not rounded to the model dtype
     # MLA
     q_lora_rank: int = 0
     kv_lora_rank: int = 0
@@ -83,6 +85,8 @@ class ModelConfig:
     layer_specs: tuple = ()              # models configured layer by layer (LayerSpec); the scalars above are maxima
     final_logit_softcap: Optional[float] = None    # logits = cap * tanh(logits / cap)
     logit_scale: float = 1.0             # logits = scale * (head x)
+    bigram: Optional[tuple] = None       # (buckets, mul_prev, mul_cur) of an embedding of (previous token, token)
+    residual_mult: float = 1.0           # factor on the normalised sublayer outputs
     # sparse MLA (DSA indexer)
     index_topk: int = 0
     index_n_heads: int = 0
@@ -115,7 +119,7 @@ class ModelConfig:
     @property
     def has_recurrent_state(self) -> bool:
         """Some layers carry a state per request instead of a KV cache."""
-        return self.full_attention_interval > 0 or any(s.mixer.recurrent for s in self.layer_specs)
+        return self.full_attention_interval > 0 or any(s.mixer.carries_state for s in self.layer_specs)
 
     def layer_is_moe(self, i: int) -> bool:
         return self.is_moe and i >= self.first_dense_layers
@@ -159,7 +163,7 @@ class ModelConfig:
     @staticmethod
     def from_hf_dict(cfg: dict, name: str = "") -> "ModelConfig":
         """Map a Hugging Face ``config.json`` dictionary to ModelConfig."""
-        if "architectures" not in cfg and cfg.get("architecture") in ("Mazivik", "Popanex"):
+        if "architectures" not in cfg and cfg.get("architecture") in ("Mazivik", "Popanex", "Zeganex"):
             return ModelConfig.from_layer_list(cfg, name)
         arch = (cfg.get("architectures") or ["LlamaForCausalLM"])[0]
         mc = ModelConfig(name=name or cfg.get("_name_or_path", arch))
@@ -314,10 +318,10 @@ class ModelConfig:
 
     @staticmethod
     def from_layer_list(cfg: dict, name: str = "") -> "ModelConfig":
-        """Map a ``config.json`` that lists its layers one by one (``{"architecture": "Mazivik" | "Popanex",
-        "layers": [...], "norm": {"eps"}, "vocab", "width", ...}``) to ModelConfig."""
+        """Map a ``config.json`` that lists its layers one by one (``{"architecture": "Mazivik" | "Popanex" |
+        "Zeganex", "layers": [...], "norm": {"eps"}, "vocab", "width", ...}``) to ModelConfig."""
         arch = cfg["architecture"].lower()
-        build = {"mazivik": _mazivik_layers, "popanex": _popanex_layers}[arch]
+        build = {"mazivik": _mazivik_layers, "popanex": _popanex_layers, "zeganex": _zeganex_layers}[arch]
         mc = ModelConfig(architecture=arch, name=name or arch, num_layers=len(cfg["layers"]),
                          hidden_size=int(cfg["width"]), vocab_size=int(cfg["vocab"]))
         mc.rms_norm_eps = float(cfg["norm"]["eps"])
@@ -334,7 +338,7 @@ class ModelConfig:
 
 
 def _mazivik_layers(mc: ModelConfig, cfg: dict) -> None:
-    specs = layer_specs(cfg["layers"], ("latent_attention",), act="gelu", gated=False)
+    specs = layer_specs(cfg["layers"], {"latent_attention": LatentMixerSpec.from_dict}, act="gelu", gated=False)
     for i, s in enumerate(specs):
         m = s.mixer
         if m.kv_from is not None:
@@ -362,7 +366,8 @@ def _mazivik_layers(mc: ModelConfig, cfg: dict) -> None:
 
 
 def _popanex_layers(mc: ModelConfig, cfg: dict) -> None:
-    specs = layer_specs(cfg["layers"], ("attention", "retention", "channel_delta"), act="gelu_tanh", gated=True)
+    specs = layer_specs(cfg["layers"], {"attention": GroupedMixerSpec.from_dict, "retention": RetentionMixerSpec.from_dict,
+                                        "channel_delta": DeltaMixerSpec.from_dict}, act="gelu_tanh", gated=True)
     mc.layer_specs = tuple(specs)
     mc.hidden_act = "gelu_tanh"
     mc.logit_scale = float(cfg.get("logit_scale", 1.0))
@@ -372,6 +377,35 @@ def _popanex_layers(mc: ModelConfig, cfg: dict) -> None:
     mc.num_kv_heads = max((m.kv_heads for m in att), default=1)
     mc.head_dim = max(max(m.dim, m.vdim) for m in att or mixers)
     mc.attn_sinks = bool(att)
+
+
+def _zeganex_layers(mc: ModelConfig, cfg: dict) -> None:
+    specs = layer_specs(cfg["layers"], {"attention": GroupedMixerSpec.differential, "attention_2": GroupedMixerSpec.gated},
+                        act="silu", gated=True, expert_act="relu2")
+    for i, s in enumerate(specs):
+        m = s.mixer
+        if m.kv_from is not None:
+            src = specs[m.kv_from].mixer if 0 <= m.kv_from < i else None
+            if src is None or src.kv_from is not None:
+                raise ValueError(f"layer {i}: kv_from {m.kv_from} must name an earlier layer with keys of its own")
+            if (src.heads, src.kv_heads, src.dim, src.vdim, src.maps, src.rot) != (m.heads, m.kv_heads, m.dim, m.vdim,
+                                                                                  m.maps, m.rot):
+                raise ValueError(f"layer {i}: head counts, sizes and rotation differ from layer {m.kv_from}'s")
+    mc.layer_specs = tuple(specs)
+    mixers = [s.mixer for s in specs]
+    mc.num_q_heads, mc.num_kv_heads = max(m.heads for m in mixers), max(m.kv_heads for m in mixers)
+    mc.head_dim = max(max(m.maps * m.dim, m.vdim) for m in mixers)
+    mc.residual_mult = float(cfg.get("residual_mult", 1.0))
+    b = (cfg.get("embedding") or {}).get("bigram")
+    mc.bigram = (int(b["buckets"]), int(b["mul_prev"]), int(b["mul_cur"])) if b else None
+    mc.tie_word_embeddings = True
+    moe = [s.experts for s in specs if s.experts]
+    if moe:
+        mc.num_experts, mc.num_experts_per_tok = max(e.experts for e in moe), max(e.top for e in moe)
+        mc.moe_intermediate_size = max(e.ff for e in moe)
+        mc.moe_renormalize, mc.moe_router_fp32 = False, True
+    spans = [m.rot.scaling["original"] * m.rot.scaling["factor"] for m in mixers if m.rot and m.rot.scaling]
+    mc.max_model_len = int(max([mc.max_model_len] + spans))
 
 
 def _preset(**kw) -> ModelConfig:
@@ -436,6 +470,21 @@ def model_preset(name: str) -> ModelConfig:
                 {"type": "retention", "mixer": ret, "mlp": None, "weights_of": 2},
                 {"type": "attention", "mixer": dict(att, heads=4, kv_heads=1, vdim=24), "mlp": None}]},
             name="tiny-popanex")
+        mc.max_model_len, mc.init_std = 256, 0.1
+        return mc
+    if n in ("tiny-zeganex",):
+        # both mixers, shared keys and values, dense and expert feed-forwards and a layer without one
+        conv = {"heads": 4, "kv_heads": 2, "dim": 24, "vdim": 40, "scale": 0.2, "mask": {"size": 21}}
+        diff = {"type": "attention", "mixer": dict(conv, conv=3, diff=0.4)}
+        rot = {"base": 5000.0, "dims": 12, "scaling": {"factor": 2.0, "original": 64, "fast": 16.0, "slow": 1.0}}
+        gated = {"type": "attention_2", "mixer": dict(conv, conv=4, vdim=24, rot=rot)}
+        moe = {"kind": "moe", "router": {"experts": 6, "top": 2}, "expert": {"ff": 40}}
+        mc = ModelConfig.from_layer_list({
+            "architecture": "Zeganex", "width": 96, "vocab": 320, "norm": {"eps": 1e-5}, "residual_mult": 0.7,
+            "embedding": {"bigram": {"buckets": 211, "mul_prev": 23, "mul_cur": 7}}, "torch_dtype": "float32", "layers": [
+                dict(gated, mlp={"kind": "dense", "ff": 136}), dict(diff, mlp=moe),
+                {"type": "attention", "mixer": dict(diff["mixer"], kv_from=1), "mlp": None}]},
+            name="tiny-zeganex")
         mc.max_model_len, mc.init_std = 256, 0.1
         return mc
     if n in ("tiny-odd-heads",):

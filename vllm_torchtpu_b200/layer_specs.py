@@ -42,7 +42,7 @@ class LatentMixerSpec:
     kv_from: Optional[int] = None        # layer whose cached latent and rotated key this layer reads
     output_gate: bool = True             # heads times sigmoid(W_g x) in front of the output projection
 
-    recurrent = False
+    recurrent = carries_state = False
 
     @staticmethod
     def from_dict(d: dict) -> "LatentMixerSpec":
@@ -69,30 +69,73 @@ class QueryTemperature:
 
 @dataclass(frozen=True)
 class GroupedMixerSpec:
-    """Grouped-query softmax attention: own key and value sizes, norms over the whole q and k projections, no
-    rotation, query temperature, one sink logit per head."""
+    """Grouped-query softmax attention with own key and value sizes.  Norms over the whole q and k projections, a query
+    temperature and sinks; or short convolutions, with a rotation, a window, an output gate or two softmax maps per head
+    (differential attention)."""
     heads: int
     kv_heads: int
-    dim: int
+    dim: int                             # of one map
     vdim: int
     scale: float
     q_temp: Optional[QueryTemperature] = None
     projection_norm: bool = True
-    sinks: bool = True
+    sinks: bool = True                   # one sink logit per head
+    conv: int = 0                        # taps of the short convolutions on q, k and v (0: none)
+    rot: Optional[RotarySpec] = None     # rotation of interleaved pairs
+    window: Optional[int] = None         # keys a query sees, itself included (None: all)
+    maps: int = 1                        # softmax maps per head over the same values; 2: map 1 - lambda * map 2
+    diff: float = 0.0                    # constant part of lambda
+    bias: bool = False                   # of the q, k and v projections
+    out_bias: bool = False
+    output_gate: bool = False            # heads times sigmoid(W_g x) in front of the output projection
+    kv_from: Optional[int] = None        # layer whose cached keys and values this layer reads
 
     recurrent = False
+
+    @property
+    def carries_state(self) -> bool:
+        return self.conv > 0
+
+    def __post_init__(self):
+        if self.heads % self.kv_heads:
+            raise ValueError(f"{self.heads} query heads do not divide over {self.kv_heads} key/value heads")
+        if self.rot is not None and (self.rot.dims % 2 or self.rot.dims > self.dim):
+            raise ValueError(f"rot.dims {self.rot.dims} must be even and at most dim {self.dim}")
+        if self.window is not None and self.window < 1:
+            raise ValueError("a window holds at least the token itself")
+
+    @staticmethod
+    def sizes_of(d: dict) -> tuple:
+        return int(d["heads"]), int(d["kv_heads"]), int(d["dim"]), int(d["vdim"]), float(d["scale"])
 
     @staticmethod
     def from_dict(d: dict) -> "GroupedMixerSpec":
         t = d.get("q_temp")
-        s = GroupedMixerSpec(int(d["heads"]), int(d["kv_heads"]), int(d["dim"]), int(d["vdim"]), float(d["scale"]),
-                             QueryTemperature(float(t["coef"]), int(t["every"])) if t else None)
-        if s.heads % s.kv_heads:
-            raise ValueError(f"{s.heads} query heads do not divide over {s.kv_heads} key/value heads")
-        return s
+        return GroupedMixerSpec(*GroupedMixerSpec.sizes_of(d),
+                                QueryTemperature(float(t["coef"]), int(t["every"])) if t else None)
+
+    @staticmethod
+    def convolved(d: dict, **kw) -> "GroupedMixerSpec":
+        """Biased projections behind short convolutions; ``mask.size`` is the window, ``rot`` the rotation."""
+        if int(d["conv"]) < 1:
+            raise ValueError("a short convolution has at least one tap")
+        r, mask, src = d.get("rot"), d.get("mask"), d.get("kv_from")
+        rot = RotarySpec(int(r["dims"]), float(r["base"]), r.get("scaling") or None) if r else None
+        return GroupedMixerSpec(*GroupedMixerSpec.sizes_of(d), projection_norm=False, sinks=False, conv=int(d["conv"]),
+                                rot=rot, window=int(mask["size"]) if mask else None, bias=True,
+                                kv_from=None if src is None else int(src), **kw)
+
+    @staticmethod
+    def differential(d: dict) -> "GroupedMixerSpec":
+        return GroupedMixerSpec.convolved(d, maps=2, diff=float(d["diff"]))
+
+    @staticmethod
+    def gated(d: dict) -> "GroupedMixerSpec":
+        return GroupedMixerSpec.convolved(d, out_bias=True, output_gate=True)
 
     def num_params(self, h: int) -> int:
-        return h * (self.heads * self.dim + self.kv_heads * (self.dim + self.vdim)) + self.heads * self.vdim * h
+        n = h * self.heads * (self.maps * self.dim + self.vdim * (2 if self.output_gate else 1))
+        return n + (h * self.kv_heads * (self.maps * self.dim + self.vdim) if self.kv_from is None else 0)
 
 
 @dataclass(frozen=True)
@@ -104,7 +147,7 @@ class RetentionMixerSpec:
     rot: RotarySpec
     decay: tuple
 
-    recurrent = True
+    recurrent = carries_state = True
 
     @staticmethod
     def from_dict(d: dict) -> "RetentionMixerSpec":
@@ -130,7 +173,7 @@ class DeltaMixerSpec:
     conv: int                            # taps of the short convolutions
     gate_rank: int = 0                   # rank of the decay and output gate projections until a checkpoint sets it
 
-    recurrent = True
+    recurrent = carries_state = True
 
     @staticmethod
     def from_dict(d: dict) -> "DeltaMixerSpec":
@@ -152,36 +195,58 @@ class DeltaMixerSpec:
 
 
 MixerSpec = Union[LatentMixerSpec, GroupedMixerSpec, RetentionMixerSpec, DeltaMixerSpec]
-MIXER_TYPES = {"latent_attention": LatentMixerSpec, "attention": GroupedMixerSpec, "retention": RetentionMixerSpec,
-               "channel_delta": DeltaMixerSpec}
+
+
+@dataclass(frozen=True)
+class ExpertsSpec:
+    """Mixture of ungated experts: down(act(up(x))) of the ``top`` experts with the largest softmax scores, weighted with
+    these scores."""
+    experts: int
+    top: int
+    ff: int
+    act: str
+
+    @staticmethod
+    def from_dict(d: dict, act: str) -> "ExpertsSpec":
+        s = ExpertsSpec(int(d["router"]["experts"]), int(d["router"]["top"]), int(d["expert"]["ff"]), act)
+        if not 1 <= s.top <= s.experts:
+            raise ValueError(f"top {s.top} of {s.experts} experts")
+        return s
+
+    def num_params(self, h: int) -> int:
+        return self.experts * h * (2 * self.ff + 1)
 
 
 @dataclass(frozen=True)
 class LayerSpec:
     """One entry of a checkpoint configuration that lists its layers one by one."""
     mixer: MixerSpec
-    ff: int = 0                          # width of the dense feed-forward, 0 = the layer has none
+    ff: int = 0                          # width of the dense feed-forward, 0 = the layer has none (or experts)
     act: str = "gelu"
     gated: bool = False                  # down(act(gate) * up) instead of down(act(up))
     weights_of: Optional[int] = None     # layer whose weights this one runs with (its cache and state are its own)
+    experts: Optional[ExpertsSpec] = None
 
     def num_params(self, h: int) -> int:
         if self.weights_of is not None:
             return 0
-        return self.mixer.num_params(h) + (3 if self.gated else 2) * h * self.ff
+        n = self.mixer.num_params(h) + (3 if self.gated else 2) * h * self.ff
+        return n + (self.experts.num_params(h) if self.experts else 0)
 
 
-def layer_specs(layers: list, mixers: tuple, act: str, gated: bool) -> list:
-    """``LayerSpec`` of every entry of a configuration's layer list; ``mixers``: the types the design has."""
+def layer_specs(layers: list, mixers: dict, act: str, gated: bool, expert_act: Optional[str] = None) -> list:
+    """``LayerSpec`` of every entry of a configuration's layer list.  ``mixers``: the types the design has and the
+    functions that read them; ``expert_act``: activation of its experts (None: it has none)."""
     specs: list = []
     for i, layer in enumerate(layers):
         if layer["type"] not in mixers:
             raise ValueError(f"layer {i}: unknown mixer type {layer['type']!r}")
         mlp = layer.get("mlp")
-        if mlp and mlp.get("kind") != "dense":
-            raise ValueError(f"layer {i}: unknown feed-forward kind {mlp.get('kind')!r}")
-        spec = LayerSpec(MIXER_TYPES[layer["type"]].from_dict(layer["mixer"]), int(mlp["ff"]) if mlp else 0, act, gated)
-        specs.append(spec)
+        kind = mlp.get("kind") if mlp else None
+        if mlp and kind not in ("dense", "moe" if expert_act else "dense"):
+            raise ValueError(f"layer {i}: unknown feed-forward kind {kind!r}")
+        specs.append(LayerSpec(mixers[layer["type"]](layer["mixer"]), int(mlp["ff"]) if kind == "dense" else 0, act, gated,
+                               experts=ExpertsSpec.from_dict(mlp, expert_act) if kind == "moe" else None))
     for i, layer in enumerate(layers):
         src, seen = layer.get("weights_of"), {i}
         if src is None:

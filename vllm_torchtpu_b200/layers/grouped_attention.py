@@ -54,13 +54,12 @@ class GroupedAttention:
             raise ValueError(f"{name}: {spec.heads} heads do not divide over tp={tp}")
         self.name, self.spec, self.cfg, self.device = name, spec, cfg, device
         self.Hq, self.Hkv = spec.heads // tp, max(1, spec.kv_heads // tp)
-        self.D = cache_head_dim(spec.dim, spec.vdim, cfg.dtype)
+        self.D = cache_head_dim(spec.maps * spec.dim, spec.vdim, cfg.dtype)
         self.eps = cfg.rms_norm_eps
         kw = dict(dtype=cfg.dtype, device=device, quant_config=quant)
-        self.inp = PackedLinear(f"{name}.qkv_proj", cfg.hidden_size, [
-            Part("q", spec.heads * spec.dim, spec.heads), Part("k", spec.kv_heads * spec.dim, spec.kv_heads),
-            Part("v", spec.kv_heads * spec.vdim, spec.kv_heads)], **kw)
-        self.o = HeadPaddedRowLinear(f"{name}.o_proj", spec.heads, spec.vdim, self.D, cfg.hidden_size, **kw)
+        self.inp = PackedLinear(f"{name}.qkv_proj", cfg.hidden_size, self.parts(spec), bias=spec.bias, **kw)
+        self.o = HeadPaddedRowLinear(f"{name}.o_proj", spec.heads, spec.vdim, self.D, cfg.hidden_size,
+                                     bias=spec.out_bias, **kw)
         ones = lambda n: torch.ones(n, dtype=cfg.dtype, device=device)                  # noqa: E731
         self.q_norm = ones(self.Hq * spec.dim) if spec.projection_norm else None
         self.k_norm = ones(self.Hkv * spec.dim) if spec.projection_norm else None
@@ -68,6 +67,14 @@ class GroupedAttention:
         self.kv_replicas = max(1, tp // spec.kv_heads)
         # sharded norms: the squared sums of all ranks, each replicated key head counted once
         self.norm_sizes = (spec.heads * spec.dim, spec.kv_heads * spec.dim)
+
+    @staticmethod
+    def parts(spec: GroupedMixerSpec) -> list:
+        """Projections of the layer's input, packed into one GEMM."""
+        qk, parts = spec.maps * spec.dim, [Part("q", spec.heads * spec.maps * spec.dim, spec.heads)]
+        if spec.kv_from is None:
+            parts += [Part("k", spec.kv_heads * qk, spec.kv_heads), Part("v", spec.kv_heads * spec.vdim, spec.kv_heads)]
+        return parts + ([Part("g", spec.heads * spec.vdim, spec.heads)] if spec.output_gate else [])
 
     def linears(self):
         return [self.inp, self.o]

@@ -63,6 +63,7 @@ class FusedMoE:
         self.hidden_size = cfg.hidden_size
         self.num_experts = cfg.num_experts
         self.activation = getattr(cfg, "hidden_act", "silu")
+        self.gated = self.activation not in ops.ref.UNGATED_ACTS
         self.top_k = cfg.num_experts_per_tok
         self.use_ep = st.expert_parallel and st.ep.size > 1
         self.ep_size = st.ep.size if self.use_ep else 1
@@ -100,6 +101,12 @@ class FusedMoE:
         self.b13[local_e, I:] = up_b[r * I:(r + 1) * I].to(self.b13.dtype)
         self.b2[local_e, :self.hidden_size] = (down_b.float() / self.tp_size).to(self.b2.dtype)
 
+    def load_ungated(self, local_e: int, up, down) -> None:
+        """Unsharded matrices of one expert without a gate projection."""
+        if self.w13 is None:
+            self.method.alloc(self)
+        self.method.load_expert(self, local_e, None, up, down)
+
     def init_dummy(self, std: float, seed: int) -> None:
         # router logits come from N(0,1) gate weights so that routing is well spread
         self.gate.init_dummy(1.0, seed)
@@ -125,8 +132,8 @@ class FusedMoE:
         return self.method.weight_bytes(self) + self.gate.weight_bytes()
 
     def route(self, x: torch.Tensor):
-        logits = self.gate(x)
         c = self.cfg
+        logits = ops.gemm_softcap(x, self.gate.weight) if c.moe_router_fp32 else self.gate(x)
         ids, w = ops.moe_route(logits, self.top_k, scoring=c.moe_scoring, renormalize=c.moe_renormalize,
                                routed_scaling=c.moe_routed_scaling, score_bias=self.score_bias,
                                n_group=c.moe_n_group, topk_group=c.moe_topk_group)

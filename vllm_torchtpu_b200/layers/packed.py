@@ -48,6 +48,16 @@ class PackedLinear(ColumnParallelLinear):
             p.rows = rows.get(p.name, p.rows)
         self.layout()
 
+    def load_bias(self, **full: torch.Tensor) -> None:
+        """Bias vectors of some parts; the others get none."""
+        if self.bias is None:
+            self.bias = torch.zeros(self.out_features, dtype=self.dtype, device=self.device)
+        for p, n in zip(self.parts, self.shard_sizes):
+            if p.name in full:
+                i = self.tp_rank // max(1, self.tp_size // p.units) if p.units else 0
+                at = self.offset[p.name]
+                self.bias[at:at + n] = full[p.name][i * n:(i + 1) * n].to(self.bias.device, self.dtype)
+
     def shard_of(self, full_weight):
         out, at = [], 0
         for p, n in zip(self.parts, self.shard_sizes):

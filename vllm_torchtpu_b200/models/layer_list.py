@@ -50,24 +50,27 @@ class LayerListForCausalLM(LlamaForCausalLM):
         std, seed = cfg.init_std, cfg.seed
         self.embed = seeded_normal("model.embed_tokens", (cfg.vocab_size, cfg.hidden_size), std, cfg.dtype, self.device,
                                    seed)
-        self.lm_head = self._shard_vocab(seeded_normal("lm_head", (cfg.vocab_size, cfg.hidden_size), std, cfg.dtype,
-                                                       self.device, seed))
+        self.lm_head = self._shard_vocab(self.embed if cfg.tie_word_embeddings else seeded_normal(
+            "lm_head", (cfg.vocab_size, cfg.hidden_size), std, cfg.dtype, self.device, seed))
         for l in self.weight_owners():
             l.self_attn.init_dummy(std, seed)
             l.mlp.init_dummy(std, seed)
 
     def weight_bytes(self) -> int:
-        n = sum(t.numel() * t.element_size() for t in (self.embed, self.lm_head) if t is not None)
+        n = sum(t.numel() * t.element_size() for t in {id(t): t for t in (self.embed, self.lm_head)}.values() if t is not None)
         return n + sum(l.self_attn.weight_bytes() + l.mlp.weight_bytes() for l in self.weight_owners())
 
     def embedding_groups(self) -> list:
         """[(checkpoint tensors that make up one parameter, loader of these tensors)] of what is outside the layers."""
         def embed(t):
             self.embed = t.to(device=self.device, dtype=self.cfg.dtype).contiguous()
+            if self.cfg.tie_word_embeddings:
+                self.lm_head = self._shard_vocab(self.embed)
 
         def head(t):
             self.lm_head = self._shard_vocab(t.to(device=self.device, dtype=self.cfg.dtype).contiguous())
-        return [(("embed",), embed), (("head",), head), (("final.norm",), vector_loader(self.norm))]
+        groups = [(("embed",), embed), (("final.norm",), vector_loader(self.norm))]
+        return groups if self.cfg.tie_word_embeddings else groups + [(("head",), head)]
 
     def setup_decode_fusion(self, kv_caches) -> None:
         self.decode_mega, self.decode_mega_reason = None, self.fusion_reason

@@ -121,7 +121,7 @@ class LlamaMLP:
         if (x.is_cuda and gu.bias is None and getattr(gu.method, "supports_fused_reduce", False)
                 and not gu.lora_targets):
             # gate and up tiles share the activation tile; SiLU*mul happens in the GEMM epilogue
-            return self.down(ops.cuda_ops().gemm_swiglu(x, gu.weight))
+            return self.down(ops.gemm_gated(x, gu.weight, "silu"))
         if (x.is_cuda and x.dtype == torch.bfloat16 and hasattr(self.down.method, "apply_quantised")
                 and not self.down.lora_targets and type(self.down.method) is type(gu.method)):
             # block-scaled fp8: SiLU*mul runs inside the quantisation kernel of the down projection's input

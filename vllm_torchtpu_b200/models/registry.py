@@ -30,8 +30,11 @@ def get_model_class(cfg: ModelConfig):
     if a == "popanex":
         from .popanex import PopanexForCausalLM
         return PopanexForCausalLM
+    if a == "zeganex":
+        from .zeganex import ZeganexForCausalLM
+        return ZeganexForCausalLM
     raise ValueError(f"no model class for architecture {a!r}")
 
 
 def supported_architectures() -> list[str]:
-    return ["llama", "qwen3_moe", "gpt_oss", "deepseek_v3", "qwen3_next", "kimi_linear", "mazivik", "popanex"]
+    return ["llama", "qwen3_moe", "gpt_oss", "deepseek_v3", "qwen3_next", "kimi_linear", "mazivik", "popanex", "zeganex"]

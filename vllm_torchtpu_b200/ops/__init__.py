@@ -40,12 +40,13 @@ def layer_norm_add(y, residual, weight, eps):
         ref.layer_norm_add(y, residual, weight, eps)
 
 
-def add_rms_norm(y, residual, weight, eps, offset=0.0, update=True):
+def add_rms_norm(y, residual, weight, eps, offset=0.0, update=True, post=None, mult=1.0):
     """(h, fp32 r) of r = residual (+ y), h = RMS norm of r times (offset + weight); an fp32 residual is updated in
-    place on a GPU.  ``y`` None: r = residual.  Without ``update`` the stream is only read and r is None."""
+    place on a GPU.  ``y`` None: r = residual.  ``post``: the RMS norm of y with this weight, times ``mult``, is added
+    instead of y.  Without ``update`` the stream is only read and r is None."""
     y = materialize(y)
-    return cuda_ops().add_rms_norm(y, residual, weight, eps, offset, update) if _on_gpu(residual) else \
-        ref.add_rms_norm(y, residual, weight, eps, offset, update)
+    return cuda_ops().add_rms_norm(y, residual, weight, eps, offset, update, post, mult) if _on_gpu(residual) else \
+        ref.add_rms_norm(y, residual, weight, eps, offset, update, post, mult)
 
 
 def softcap(x, cap):
@@ -114,6 +115,35 @@ def latent_prep(*a, **kw):
 
 def rope_heads_into(q, out, *a, **kw):
     return cuda_ops().rope_heads_into(q, out, *a, **kw) if _on_gpu(q) else ref.rope_heads_into(q, out, *a, **kw)
+
+
+def embedding_pairs(ids, prev, table, pairs, bigram, token_src, last_tokens, last_inputs):
+    """fp32 sum of token and bigram embeddings; see ``ops.reference.embedding_pairs``."""
+    f = cuda_ops().embedding_pairs if _on_gpu(table) else ref.embedding_pairs
+    return f(ids, prev, table, pairs, bigram, token_src, last_tokens, last_inputs)
+
+
+def conv_and_cache(plan, row, kv_cache, ring, meta):
+    """Short convolutions, rotation and cache write of an attention layer; see ``ops.short_conv``."""
+    if _on_gpu(row):
+        return cuda_ops().conv_and_cache(plan, row, kv_cache, ring, meta)
+    from .short_conv import conv_and_cache as f
+    return f(plan, row, kv_cache, ring, meta)
+
+
+def conv_ring_update(plan, row, ring, meta):
+    if _on_gpu(row):
+        return cuda_ops().conv_ring_update(plan, row, ring, meta)
+    from .short_conv import ring_update as f
+    return f(plan, row, ring, meta)
+
+
+def combine_heads(a, vdim, gate=None, lam=None, diff=0.0, eps=0.0):
+    """Difference of two softmax maps with its norm, output gate; see ``ops.short_conv``."""
+    if _on_gpu(a):
+        return cuda_ops().combine_heads(a, vdim, gate, lam, diff, eps)
+    from .short_conv import combine_heads as f
+    return f(a, vdim, gate, lam, diff, eps)
 
 
 def embedding(ids, table):

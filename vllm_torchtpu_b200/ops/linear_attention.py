@@ -25,6 +25,8 @@ from typing import Optional
 import torch
 import torch.nn.functional as F
 
+from .short_conv import conv_with_ring
+
 UNIT_EPS = 1e-6
 
 
@@ -80,17 +82,6 @@ def rotate_half_split(x: torch.Tensor, positions: torch.Tensor, inv_freq: torch.
     return torch.cat([u * c - v * s, v * c + u * s, x[..., 2 * P:]], -1)
 
 
-def _conv_with_ring(plan, x, ring, start: int):
-    """x [L, C] of one request from position ``start`` on; ring [taps, C] is read and updated."""
-    K = plan.taps
-    hist = [ring[p % K] if p >= 0 else torch.zeros_like(x[0]) for p in range(start - K + 1, start)]
-    full = torch.cat([torch.stack(hist), x], 0) if hist else x
-    out = sum(full[j:j + x.shape[0]].float() * plan.conv_w[:, j].float() for j in range(K))
-    for p in range(max(start, start + x.shape[0] - K), start + x.shape[0]):
-        ring[p % K] = x[p - start]
-    return F.silu(out)
-
-
 def linear_attention_reference(plan: LinearAttentionPlan, row, decay_in, gate, meta, cache):
     T, H, G, d, dv = row.shape[0], plan.heads, plan.k_heads, plan.dim, plan.vdim
     y = torch.zeros(T, H * dv, dtype=row.dtype, device=row.device)
@@ -102,7 +93,7 @@ def linear_attention_reference(plan: LinearAttentionPlan, row, decay_in, gate, m
             continue
         start, S = sl[r] - (b - a), state[slots[r]]
         x = split_qkv(plan, row[a:b])
-        x = _conv_with_ring(plan, x, ring[slots[r]], start) if plan.taps else x.float()
+        x = F.silu(conv_with_ring(x, plan.conv_w, ring[slots[r]], start)) if plan.taps else x.float()
         q, k, v = x.split([G * d, G * d, H * dv], -1)
         q, k, v = q.reshape(-1, G, d), k.reshape(-1, G, d), v.reshape(-1, H, dv)
         if plan.inv_freq is not None:

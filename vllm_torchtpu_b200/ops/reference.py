@@ -54,10 +54,16 @@ def layer_norm_add(y: torch.Tensor, residual: torch.Tensor, weight: torch.Tensor
 
 
 def add_rms_norm(y: Optional[torch.Tensor], residual: torch.Tensor, weight: torch.Tensor, eps: float,
-                 offset: float = 0.0, update: bool = True):
-    """32-bit residual stream in front of a sublayer: r = residual (+ y); h = r / rms(r) * (offset + w).
+                 offset: float = 0.0, update: bool = True, post: Optional[torch.Tensor] = None, mult: float = 1.0):
+    """32-bit residual stream in front of a sublayer: r = residual (+ y); h = r / rms(r) * (offset + w).  With ``post``
+    the output y is normalised first: r = residual + mult * y / rms(y) * post.
     Returns (h in the weight's dtype, r fp32 or None without ``update``)."""
-    r = residual.float() if y is None else residual.float() + y.float()
+    r = residual.float()
+    if y is not None:
+        a = y.float()
+        if post is not None:
+            a = mult * (a * torch.rsqrt(a.pow(2).mean(-1, keepdim=True) + eps) * post.float())
+        r = r + a
     h = r * torch.rsqrt(r.pow(2).mean(-1, keepdim=True) + eps) * (offset + weight.float())
     return h.to(weight.dtype), (r if update else None)
 
@@ -370,6 +376,21 @@ def merge_attn_states(outs: list, lses: list):
     return o.to(outs[0].dtype), m + torch.log(denom.clamp_min(1e-38))
 
 
+def embedding_pairs(ids, prev, table, pairs, bigram, token_src, last_tokens, last_inputs):
+    """fp32 table[token] + pairs[(prev * mul_prev + token * mul_cur) % buckets] with ``bigram`` = (buckets, mul_prev,
+    mul_cur); row number ``buckets`` in front of a sequence's first token.  ``token_src`` >= 0: the token is
+    last_tokens[token_src]; it is kept in last_inputs[token_src], where the next step's row finds it.  ``prev``: the
+    previous token, -1 none, -2 last_inputs[token_src]."""
+    src = token_src.clamp_min(0).long()
+    late = token_src >= 0
+    cur = torch.where(late, last_tokens[src], ids)
+    before = torch.where((prev == -2) & late, last_inputs[src], prev).long()
+    last_inputs[src[late]] = cur[late]
+    buckets, mul_prev, mul_cur = bigram
+    row = torch.where(before < 0, torch.full_like(before, buckets), (before * mul_prev + cur.long() * mul_cur) % buckets)
+    return table[cur.long()].float() + pairs[row].float()
+
+
 def embedding(ids: torch.Tensor, table: torch.Tensor) -> torch.Tensor:
     return table[ids.long()]
 
@@ -470,10 +491,14 @@ def moe_route_post(ids, w, num_experts: int, num_valid=None, sim: str = ""):
     return ids, w
 
 
+UNGATED_ACTS = ("relu2",)                # of experts without a gate projection: the square of relu
+
+
 def moe_experts(x, w13, w2, topk_ids, topk_w, expert_offset: int = 0, act: str = "silu", b13=None, b2=None):
     """Σ_k w_k · FFN_e(x) over the experts this rank owns.  w13: [E_local, 2I, H] (gate rows first),
     w2: [E_local, H, I] (rows beyond H, padding for the kernels' tile width, are ignored); ``act``: gated
-    activation (``parse_gated_act``); optional expert biases b13 [E_local, 2I], b2 [E_local, H]."""
+    activation (``parse_gated_act``), or one of ``UNGATED_ACTS`` with w13 [E_local, I, H]; optional expert biases b13
+    [E_local, 2I], b2 [E_local, H]."""
     T, H = x.shape
     E_local = w13.shape[0]
     out = torch.zeros(T, H, dtype=torch.float32, device=x.device)
@@ -487,7 +512,7 @@ def moe_experts(x, w13, w2, topk_ids, topk_w, expert_offset: int = 0, act: str =
         h = xf[rows] @ w13[e].float().t()
         if b13 is not None:
             h = (h.to(x.dtype).float() + b13[e].float())
-        a = gated_act_and_mul(h, act).to(x.dtype).float()
+        a = (h.clamp_min(0).square() if act == "relu2" else gated_act_and_mul(h, act)).to(x.dtype).float()
         y = (a @ w2[e, :H].float().t()).to(x.dtype).float()
         if b2 is not None:
             y = (y + b2[e, :H].float()).to(x.dtype).float()

@@ -212,9 +212,11 @@ class B200Platform:
                 raise ValueError(f"pipeline parallelism is not built for {m.architecture}: its 32-bit residual stream "
                                  "and shared caches do not cross the stage hand-off")
             bad = [i for i, l in enumerate(m.layer_specs) if l.mixer.heads % tp
-                   or (l.mixer.recurrent and getattr(l.mixer, "kv_heads", tp) % tp)]
+                   or (l.mixer.recurrent and getattr(l.mixer, "kv_heads", tp) % tp)
+                   or (l.mixer.carries_state and not l.mixer.recurrent and l.mixer.kv_heads % tp and tp % l.mixer.kv_heads)
+                   or (l.experts and not p.enable_expert_parallel and l.experts.ff % tp)]
             if bad:
-                raise ValueError(f"the heads of layers {bad[:8]} do not divide over tp={tp}")
+                raise ValueError(f"the heads or experts of layers {bad[:8]} do not divide over tp={tp}")
             if not m.is_mla and max(p.decode_context_parallel_size, p.prefill_context_parallel_size) > 1:
                 raise ValueError(f"context parallelism is not built for {m.architecture}")
             if not m.is_mla and cfg.cache.kv_cache_dtype.startswith("fp8"):
@@ -233,7 +235,7 @@ class B200Platform:
             p.enable_expert_parallel = False
         if p.enable_expert_parallel:
             ep = tp * p.data_parallel_size
-            if m.num_experts % ep:
+            if m.num_experts % ep or any(l.experts and l.experts.experts % ep for l in m.layer_specs):
                 raise ValueError(f"{m.num_experts} experts do not divide over ep={ep}")
         if p.pipeline_parallel_size > 1:
             from .parallel.pp import validate_pipeline_parallel_config

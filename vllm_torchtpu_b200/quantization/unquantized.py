@@ -81,11 +81,16 @@ def padded_hidden(moe) -> int:
     return (moe.hidden_size + 127) // 128 * 128
 
 
+def padded_inter(moe) -> int:
+    """Rows of the up projection of ungated experts, rounded up alike: zero rows stay zero through the activation."""
+    return moe.intermediate_size if moe.gated else (moe.intermediate_size + 127) // 128 * 128
+
+
 class UnquantizedMoEMethod:
     name = "unquantized"
 
     def create_weights(self, moe) -> None:
-        moe.w13 = None      # [E_local, 2I, H]
+        moe.w13 = None      # [E_local, 2I, H]; ungated experts [E_local, I padded, H]
         moe.w2 = None       # [E_local, H, I]
 
     def init_dummy(self, moe, std, seed) -> None:
@@ -95,16 +100,26 @@ class UnquantizedMoEMethod:
         w13 = []
         w2 = []
         for e in range(lo, hi):
-            w13.append(seeded_normal(f"{moe.name}.experts.{e}.w13", (2 * I, H), std, moe.dtype, moe.device, seed))
+            w13.append(seeded_normal(f"{moe.name}.experts.{e}.w13", (2 * I if moe.gated else I, H), std, moe.dtype,
+                                     moe.device, seed))
             w2.append(seeded_normal(f"{moe.name}.experts.{e}.w2", (H, I), std, moe.dtype, moe.device, seed))
         moe.w13 = torch.stack(w13).contiguous()
         moe.w2 = torch.stack(w2).contiguous()
         if padded_hidden(moe) != H:
             moe.w2 = torch.nn.functional.pad(moe.w2, (0, 0, 0, padded_hidden(moe) - H)).contiguous()
+        if padded_inter(moe) != I:
+            more = padded_inter(moe) - I
+            moe.w13 = torch.nn.functional.pad(moe.w13, (0, 0, 0, more)).contiguous()
+            moe.w2 = torch.nn.functional.pad(moe.w2, (0, more)).contiguous()
 
     def load_expert(self, moe, local_e, gate, up, down, scales=(None, None, None)) -> None:
-        """Unsharded checkpoint matrices of one expert; the intermediate dimension is sliced for this
-        TP rank here.  Block-scaled fp8 pieces (``scales`` given) are expanded first."""
+        """Unsharded checkpoint matrices of one expert (``gate`` None: ungated); the intermediate dimension is sliced
+        for this TP rank here.  Block-scaled fp8 pieces (``scales`` given) are expanded first."""
+        if gate is None:
+            I, r = moe.intermediate_size, moe.tp_rank
+            moe.w13[local_e, :I] = up[r * I:(r + 1) * I].to(moe.w13.dtype)
+            moe.w2[local_e, :moe.hidden_size, :I] = down[:, r * I:(r + 1) * I].to(moe.w2.dtype)
+            return
         gate, up, down = expert_tp_shard(moe, *dequant_expert_pieces(moe, (gate, up, down), scales))
         I = moe.intermediate_size
         moe.w13[local_e, :I] = gate.to(moe.w13.dtype)
@@ -113,8 +128,9 @@ class UnquantizedMoEMethod:
 
     def alloc(self, moe) -> None:
         E, I, H = moe.num_local_experts, moe.intermediate_size, moe.hidden_size
-        moe.w13 = torch.zeros(E, 2 * I, H, dtype=moe.dtype, device=moe.device)
-        moe.w2 = torch.zeros(E, padded_hidden(moe), I, dtype=moe.dtype, device=moe.device)
+        up = 2 * I if moe.gated else padded_inter(moe)
+        moe.w13 = torch.zeros(E, up, H, dtype=moe.dtype, device=moe.device)
+        moe.w2 = torch.zeros(E, padded_hidden(moe), padded_inter(moe), dtype=moe.dtype, device=moe.device)
 
     def apply(self, moe, x, topk_ids, topk_w):
         kw = dict(act=moe.activation, b13=getattr(moe, "b13", None), b2=getattr(moe, "b2", None))

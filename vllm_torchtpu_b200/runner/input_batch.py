@@ -81,6 +81,7 @@ class StepBuffers:
 
     int32 region:  input_ids[T] positions[T] slot_mapping[T] token_src[T]
                    query_start_loc[R+1] seq_lens[R] logits_indices[R] top_k[R] batch_slots[R]
+                   prev_ids[T] (token in front of each row's; filled for models that read pairs of tokens)
     fp32 region:   temperature[R] top_p[R]
     block tables:  [R, max_blocks] int32 (separate copy)
     """
@@ -92,7 +93,7 @@ class StepBuffers:
         sizes = [("input_ids", T), ("positions", T), ("slot_mapping", T), ("token_src", T),
                  ("query_start_loc", R + 1), ("seq_lens", R), ("logits_indices", T), ("top_k", T),
                  ("batch_slots", R), ("temperature", T), ("top_p", T), ("rng_step", 2), ("global_seq_lens", R),
-                 ("num_valid", 1)]
+                 ("num_valid", 1), ("prev_ids", T)]
         self.offsets, off = {}, 0
         for name, n in sizes:
             self.offsets[name] = (off, n)

@@ -219,6 +219,8 @@ class ModelRunner:
                              "(they step in lockstep, which the exchanges rely on)")
         if st.tp.size > 1 or st.pp.size > 1 or self.dcp_size > 1:
             raise ValueError("dp_vocab_parallel is built for replicas of one GPU (no TP / PP / DCP inside a replica)")
+        if self.mcfg.bigram:
+            raise ValueError("dp_vocab_parallel is not built for models with a bigram embedding")
         if self.cfg.speculative:
             raise ValueError("dp_vocab_parallel and speculative decoding are exclusive (drafters call the lm_head a "
                              "data-dependent number of times)")
@@ -231,6 +233,8 @@ class ModelRunner:
         self.bufs_prefill = StepBuffers(self.max_tokens, self.max_reqs, mb, self.device)
         self.bufs_decode = StepBuffers(self.max_reqs, self.max_reqs, mb, self.device)
         self.last_tokens = torch.zeros(self.max_reqs, dtype=torch.int32, device=self.device)
+        # the token that a request's last step read from last_tokens (models whose embedding reads pairs of tokens)
+        self.last_inputs = torch.zeros(self.max_reqs, dtype=torch.int32, device=self.device)
         self._spec_k_dev = torch.zeros(self.max_reqs, dtype=torch.int32, device=self.device)
         self.tokens_host = [torch.zeros(self.max_reqs * 9, dtype=torch.int32, pin_memory=self.is_cuda)
                             for _ in range(4)]
@@ -381,6 +385,11 @@ class ModelRunner:
         v = hv("positions", T_pad); v[:T] = pos; v[T:] = 0
         v = hv("slot_mapping", T_pad); v[:T] = slot_map; v[T:] = -1
         v = hv("token_src", T_pad); v[:T] = np.where(known, -1, tslots); v[T:] = -1
+        if self.mcfg.bigram:
+            # the token in front: known to the host, none (-1), or still on the device where the last step read it (-2)
+            before = np.maximum(pos - 1, 0)
+            prev = np.where(before < b.num_known[tslots] + spec_k[req_idx], b.token_ids[tslots, before], -2)
+            v = hv("prev_ids", T_pad); v[:T] = np.where(pos == 0, -1, prev); v[T:] = -1
         v = hv("query_start_loc", R_pad + 1); v[:n + 1] = qsl; v[n + 1:] = T
         v = hv("seq_lens", R_pad); v[:n] = local_lens; v[n:] = 0
         v = hv("global_seq_lens", R_pad); v[:n] = seq_lens_np; v[n:] = 0
@@ -440,7 +449,7 @@ class ModelRunner:
         st = get_state()
         if st.pp.size > 1:
             return self._forward_and_sample_pp(bufs, meta, T, R, n_req_pad, all_greedy, verify)
-        hidden0 = self._embed(ids, dv("token_src", T))
+        hidden0 = self._embed(ids, dv("token_src", T), dv("prev_ids", T) if self.mcfg.bigram else None)
         if self._mm_plan and hidden0 is not None:
             # image / video embeddings replace the placeholder-token rows of the prompt
             for rid, start, row0, nrows in self._mm_plan:
@@ -678,9 +687,12 @@ class ModelRunner:
             return None
         return (acc[0] / max(1, acc[1])).cpu().tolist()
 
-    def _embed(self, ids, token_src):
+    def _embed(self, ids, token_src, prev=None):
         if self.model.embed is None:
             return None
+        if prev is not None:
+            return ops.embedding_pairs(ids, prev, self.model.embed, self.model.bigram, self.mcfg.bigram, token_src,
+                                       self.last_tokens, self.last_inputs)
         dpv = getattr(self.model, "dp_vocab", None)
         if dpv is not None:
             # the table is sharded over the replicas: resolve the on-device token feedback first, then exchange
@@ -740,6 +752,7 @@ class ModelRunner:
         v = hv("positions", T); v[:] = 0; v[:per] = np.arange(per)
         hv("slot_mapping", T)[:] = -1
         hv("token_src", T)[:] = -1
+        hv("prev_ids", T)[:] = -1
         hv("query_start_loc", 2)[:] = [0, per]
         hv("seq_lens", 1)[:] = per
         hv("logits_indices", 1)[:] = per - 1
@@ -969,6 +982,7 @@ class ModelRunner:
         hv("positions", R)[:] = 0
         hv("slot_mapping", R)[:] = -1
         hv("token_src", R)[:] = -1
+        hv("prev_ids", R)[:] = -1
         hv("query_start_loc", R + 1)[:] = np.arange(R + 1)
         hv("seq_lens", R)[:] = 1
         hv("logits_indices", R)[:] = np.arange(R)
@@ -1001,6 +1015,7 @@ class ModelRunner:
         hv("positions", T)[:] = np.tile(np.arange(per), R)
         hv("slot_mapping", T)[:] = -1
         hv("token_src", T)[:] = -1
+        hv("prev_ids", T)[:] = -1
         qsl = np.arange(R + 1, dtype=np.int64) * per
         hv("query_start_loc", R + 1)[:] = qsl
         hv("seq_lens", R)[:] = per
