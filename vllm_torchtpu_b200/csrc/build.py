@@ -78,6 +78,9 @@ FAMILY_SOURCES = {
     "popanex": ("attention.cu", "attention_simt.cu", "attention_tc.cu", "elementwise.cu", "gemm_2sm_tcgen05.cu",
                 "gemm_simt.cu", "gemm_tcgen05.cu", "layer_norm.cu", "linear_attention.cu", "norm_cache.cu", "runtime.cu",
                 "sample.cu"),
+    "zeganex": ("attention.cu", "attention_simt.cu", "attention_tc.cu", "conv_cache.cu", "elementwise.cu",
+                "gemm_2sm_tcgen05.cu", "gemm_simt.cu", "gemm_tcgen05.cu", "layer_norm.cu", "moe.cu", "runtime.cu",
+                "sample.cu"),
 }
 
 

@@ -387,6 +387,7 @@ __device__ __forceinline__ float gated_pair(float g, float u) {
   return g * (1.f - __fdividef(1.f, 1.f + __expf(2.f * z))) * u;      // 0.5 (1 + tanh z) = 1 - 1 / (1 + e^2z)
 }
 
+__device__ __forceinline__ float relu_squared(float v) { return v > 0.f ? v * v : 0.f; }
 __device__ __forceinline__ float soft_cap(float v, float cap) { return cap > 0.f ? cap * tanhf(v / cap) : v; }
 
 struct alignas(16) bf16x8 {

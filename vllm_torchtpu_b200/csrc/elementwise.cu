@@ -167,6 +167,65 @@ __global__ void embedding_kernel(const int* __restrict__ ids, const int* __restr
   for (int i = threadIdx.x; i < n; i += blockDim.x) dst[i] = srcp[i];
 }
 
+__device__ __forceinline__ float emb_f(float v) { return v; }
+__device__ __forceinline__ float emb_f(__nv_bfloat16 v) { return __bfloat162float(v); }
+
+// out[t] = table[token] + pairs[(prev * mul_prev + token * mul_cur) % buckets], fp32; row `buckets` without a previous
+// token.  A token that is still on the device (token_src >= 0) is kept in last_inputs for the next step, whose previous
+// token it is (prev -2).  V elements per thread and pass.
+template <typename E, int V>
+__global__ void embedding_pairs_kernel(const int* __restrict__ ids, const int* __restrict__ prev,
+                                       const int* __restrict__ token_src, const int* __restrict__ last_tokens,
+                                       int* __restrict__ last_inputs, const E* __restrict__ table,
+                                       const E* __restrict__ pairs, float* __restrict__ out, int H, int vocab,
+                                       long long buckets, long long mul_prev, long long mul_cur) {
+  __shared__ long long s_row;
+  __shared__ int s_id;
+  const int t = blockIdx.x;
+  if (threadIdx.x == 0) {
+    const int src = token_src[t];
+    int id = src >= 0 ? last_tokens[src] : ids[t], before = prev[t];
+    if (before == -2) before = src >= 0 ? last_inputs[src] : -1;
+    if (src >= 0) last_inputs[src] = id;
+    id = min(max(id, 0), vocab - 1);
+    s_row = before < 0 ? buckets : ((long long)before * mul_prev + (long long)id * mul_cur) % buckets;
+    s_id = id;
+  }
+  __syncthreads();
+  const E* a = table + (size_t)s_id * H;
+  const E* b = pairs + (size_t)s_row * H;
+  float* o = out + (size_t)t * H;
+  for (int i = threadIdx.x * V; i < H; i += blockDim.x * V) {
+    if constexpr (V == 1) {
+      o[i] = emb_f(a[i]) + emb_f(b[i]);
+    } else {
+      const uint4 x = *reinterpret_cast<const uint4*>(a + i), y = *reinterpret_cast<const uint4*>(b + i);
+      const E *xe = reinterpret_cast<const E*>(&x), *ye = reinterpret_cast<const E*>(&y);
+      float v[V];
+#pragma unroll
+      for (int j = 0; j < V; ++j) v[j] = emb_f(xe[j]) + emb_f(ye[j]);
+#pragma unroll
+      for (int j = 0; j < V; j += 4) *reinterpret_cast<float4*>(o + i + j) = make_float4(v[j], v[j + 1], v[j + 2], v[j + 3]);
+    }
+  }
+}
+
+template <typename E>
+static int embedding_pairs(const int* ids, const int* prev, const int* token_src, const int* last_tokens, int* last_inputs,
+                           const void* table, const void* pairs, float* out, int T, int H, int vocab, long long buckets,
+                           long long mul_prev, long long mul_cur, cudaStream_t stream) {
+  constexpr int V = 16 / sizeof(E);
+  const bool vec = H % V == 0 && ((uintptr_t)table | (uintptr_t)pairs | (uintptr_t)out) % 16 == 0;
+  if (vec)
+    embedding_pairs_kernel<E, V><<<T, 128, 0, stream>>>(ids, prev, token_src, last_tokens, last_inputs, (const E*)table,
+                                                        (const E*)pairs, out, H, vocab, buckets, mul_prev, mul_cur);
+  else
+    embedding_pairs_kernel<E, 1><<<T, 128, 0, stream>>>(ids, prev, token_src, last_tokens, last_inputs, (const E*)table,
+                                                        (const E*)pairs, out, H, vocab, buckets, mul_prev, mul_cur);
+  B200_CUDA_CHECK(cudaGetLastError());
+  return 0;
+}
+
 // out_h[r] = hidden[idx[r]], out_r[r] = residual[idx[r]]
 template <typename V>
 __global__ void gather_rows_kernel(const V* __restrict__ hidden, const V* __restrict__ residual,
@@ -374,6 +433,22 @@ extern "C" int b200_embedding(const int* ids, const int* token_src, const int* l
                                                       (uint16_t*)out, row_bytes / 2, vocab);
   B200_CUDA_CHECK(cudaGetLastError());
   return 0;
+}
+
+// table, pairs: elem bytes (2 = bf16, 4 = fp32); pairs has buckets + 1 rows
+extern "C" int b200_embedding_pairs(const int* ids, const int* prev, const int* token_src, const int* last_tokens,
+                                    int* last_inputs, const void* table, const void* pairs, float* out, int T, int H,
+                                    int vocab, long long buckets, long long mul_prev, long long mul_cur, int elem,
+                                    cudaStream_t stream) {
+  if (T == 0) return 0;
+  if (buckets < 1) {
+    b200_set_last_error("embedding_pairs: at least one bucket", __FILE__, __LINE__);
+    return -1;
+  }
+  return elem == 4 ? embedding_pairs<float>(ids, prev, token_src, last_tokens, last_inputs, table, pairs, out, T, H, vocab,
+                                            buckets, mul_prev, mul_cur, stream)
+                   : embedding_pairs<__nv_bfloat16>(ids, prev, token_src, last_tokens, last_inputs, table, pairs, out, T, H,
+                                                    vocab, buckets, mul_prev, mul_cur, stream);
 }
 
 extern "C" int b200_gather_rows(const void* hidden, const void* residual, const int* idx, void* out_h,

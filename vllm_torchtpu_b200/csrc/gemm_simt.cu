@@ -85,8 +85,69 @@ __global__ void __launch_bounds__(256) gemm_kernel(const Params p) {
   }
 }
 
+// Rows [off[e], off[e + 1]) of x times w[e] [N, K]: experts on the CUDA cores.  grid (column tiles, experts); a CTA walks
+// over the row tiles of its expert.
+template <typename E>
+__global__ void __launch_bounds__(256) grouped_kernel(const E* __restrict__ x, const E* __restrict__ w, E* __restrict__ y,
+                                                      const int* __restrict__ off, int N, int K, int act) {
+  __shared__ float sx[TK][TM + 4];
+  __shared__ float sw[TK][TN + 4];
+  pdl_launch_dependents();
+  pdl_wait();
+  const int e = blockIdx.y, n0 = blockIdx.x * TN, r0 = off[e], r1 = off[e + 1];
+  const int tx = threadIdx.x & 15, ty = threadIdx.x >> 4;
+  const E* we = w + (size_t)e * N * K;
+  for (int t0 = r0; t0 < r1; t0 += TM) {
+    float acc[4][4] = {};
+    for (int k0 = 0; k0 < K; k0 += TK) {
+#pragma unroll
+      for (int i = 0; i < TM * TK / 256; ++i) {
+        const int idx = threadIdx.x + i * 256, k = idx & (TK - 1), r = idx / TK;
+        const bool kin = k0 + k < K;
+        sx[k][r] = (kin && t0 + r < r1) ? to_f(x[(size_t)(t0 + r) * K + k0 + k]) : 0.f;
+        sw[k][r] = (kin && n0 + r < N) ? to_f(we[(size_t)(n0 + r) * K + k0 + k]) : 0.f;
+      }
+      __syncthreads();
+#pragma unroll
+      for (int k = 0; k < TK; ++k) {
+        const float4 a = *reinterpret_cast<const float4*>(&sx[k][ty * 4]);
+        const float4 c = *reinterpret_cast<const float4*>(&sw[k][tx * 4]);
+        const float av[4] = {a.x, a.y, a.z, a.w}, cv[4] = {c.x, c.y, c.z, c.w};
+#pragma unroll
+        for (int i = 0; i < 4; ++i)
+#pragma unroll
+          for (int j = 0; j < 4; ++j) acc[i][j] = fmaf(av[i], cv[j], acc[i][j]);
+      }
+      __syncthreads();
+    }
+#pragma unroll
+    for (int i = 0; i < 4; ++i)
+#pragma unroll
+      for (int j = 0; j < 4; ++j) {
+        const int t = t0 + ty * 4 + i, n = n0 + tx * 4 + j;
+        if (t < r1 && n < N) y[(size_t)t * N + n] = from_f<E>(act == 4 ? relu_squared(acc[i][j]) : acc[i][j]);
+      }
+  }
+}
+
 }  // namespace simt
 }  // namespace b200
+
+// x [R, K], y [R, N], w [groups, N, K], off int[groups + 1] on the device; act 0 none, 4 the square of relu; elem: 2 = bf16,
+// 4 = fp32 (all operands alike).
+extern "C" int b200_grouped_gemm_simt(const void* x, const void* w, void* y, const int* off, int groups, int N, int K,
+                                      int act, int elem, cudaStream_t stream) {
+  using namespace b200;
+  if (groups <= 0 || N <= 0) return 0;
+  const dim3 grid((N + simt::TN - 1) / simt::TN, groups);
+  if (elem == 4)
+    B200_CUDA_CHECK(launch_pdl(simt::grouped_kernel<float>, grid, dim3(256), (size_t)0, stream, (const float*)x,
+                               (const float*)w, (float*)y, off, N, K, act));
+  else
+    B200_CUDA_CHECK(launch_pdl(simt::grouped_kernel<__nv_bfloat16>, grid, dim3(256), (size_t)0, stream,
+                               (const __nv_bfloat16*)x, (const __nv_bfloat16*)w, (__nv_bfloat16*)y, off, N, K, act));
+  return 0;
+}
 
 // elem: 2 = bf16, 4 = fp32 (all operands alike); strides in elements.
 extern "C" int b200_gemm_simt(const void* x, const void* w, void* y, const void* bias, const void* gate, int T, int N,

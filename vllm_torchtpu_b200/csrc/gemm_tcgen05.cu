@@ -99,7 +99,7 @@ struct GemmParams {
   unsigned long long ag_done_off;
   int ag_flip;
   unsigned long long* dbg;               // optional: per-CTA phase timestamps (ns), 16 slots per CTA
-  // ---- gate / up pairs: act 0 silu, 3 gelu (tanh form)
+  // ---- gate / up pairs: act 0 silu, 3 gelu (tanh form); grouped products without a gate: act 4 the square of relu
   // ---- MODE 3: epilogue (act 0 none / 1 gelu / 2 fp32 output Yf: out_scale * y, then the soft cap (cap 0: none);
   // optional gate: y *= sigmoid(gate[t, b * N + n])) and batch over heads: head b reads activation columns from
   // b * x_head_cols, weight rows from b * N and writes output columns from b * y_head_cols
@@ -776,7 +776,11 @@ gemm_bf16_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant_
               }
 #pragma unroll
               for (int j = 0; j < 32; ++j) {
-                if (c0 + j < t_valid) yp[(size_t)j * td.cs] = __float2bfloat16(__uint_as_float(r[j]) + bias);
+                if (c0 + j < t_valid) {
+                  float v = __uint_as_float(r[j]) + bias;
+                  if (FULL && p.act == 4) v = relu_squared(v);
+                  yp[(size_t)j * td.cs] = __float2bfloat16(v);
+                }
               }
             }
           }
@@ -1675,8 +1679,9 @@ extern "C" int b200_gemm_bf16_swiglu(const void* X, const void* W, void* Y, int 
 //   rows [group_off[e], group_off[e+1]) of X use weight W[e] ([N, K], or [2N, K] gate/up when swiglu).
 // X: [R, K]; Y: [R, N].  group_off lives in device memory, so the launch is CUDA-graph safe; the
 // grid is one persistent CTA per SM and CTAs without work exit.  avg_rows_hint picks the token tile.
+// act (without swiglu): 0 none, 4 the square of relu.
 extern "C" int b200_grouped_gemm_bf16(const void* X, const void* W, void* Y, const int* group_off,
-                                      int num_groups, int R, int N, int K, int swiglu, int avg_rows_hint,
+                                      int num_groups, int R, int N, int K, int swiglu, int act, int avg_rows_hint,
                                       int* status, int num_sms, cudaStream_t stream) {
   using namespace b200;
   if (R <= 0 || N <= 0 || K <= 0 || num_groups <= 0) return 0;
@@ -1690,6 +1695,7 @@ extern "C" int b200_grouped_gemm_bf16(const void* X, const void* W, void* Y, con
   init_params(p, Y, R, N, K, N, bn, status);
   p.group_off = group_off;
   p.num_groups = num_groups;
+  if (!swiglu) p.act = act;
   p.w_rows_per_group = swiglu ? 2 * N : N;
   p.up_row_off = N;
   p.w_evict_first = avg_rows_hint <= bn ? 1 : 0;

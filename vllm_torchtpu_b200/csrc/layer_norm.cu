@@ -8,6 +8,8 @@
 //
 //   add_rms: r' = r (+ y),  o = r' / rms(r') * (offset + w)     (r' fp32)
 //
+// and of blocks that do both: the output y is normalised and scaled first, r' = r + mult * y / rms(y) * post.
+//
 // mean and variance (mean of the squared deviations) in fp32 over the row, which stays in shared memory between
 // the passes.  Also the tanh soft cap of the logits.
 #include "common.cuh"
@@ -119,20 +121,39 @@ static int launch_v(const void* x, const void* res, const void* w, void* res_out
 }
 
 // One CTA per row.  TY: type of the sublayer output y (null: nothing is added), TR: of the stream that comes in, TO: of
-// w and of the normalised output; res_out (fp32, may be res itself) is written when given.
-template <int V, typename TY, typename TR, typename TO>
-__global__ void add_rms_norm_kernel(const TY* __restrict__ y, const TR* res, const TO* __restrict__ w, float* res_out,
-                                    TO* __restrict__ out, int H, float eps, float offset) {
+// w and of the normalised output; res_out (fp32, may be res itself) is written when given.  POST: y passes a norm with the
+// weight post and the factor mult first.
+template <int V, typename TY, typename TR, typename TO, bool POST>
+__global__ void add_rms_norm_kernel(const TY* __restrict__ y, const TR* res, const TO* __restrict__ w,
+                                    const TO* __restrict__ post, float* res_out, TO* __restrict__ out, int H, float eps,
+                                    float offset, float mult) {
   pdl_launch_dependents();
   pdl_wait();
   extern __shared__ __align__(16) float row[];
   __shared__ float red[32];
   const size_t base = (size_t)blockIdx.x * H;
-  float ss = 0.f;
+  float ss = 0.f, scale = 1.f;
+  if constexpr (POST) {
+    float sy = 0.f;
+    for (int i = threadIdx.x * V; i < H; i += blockDim.x * V) {
+      float a[V];
+      load<V>(y + base + i, a);
+#pragma unroll
+      for (int j = 0; j < V; ++j) sy += a[j] * a[j];
+      store<V>(row + i, a);
+    }
+    scale = mult / sqrtf(block_sum(sy, red) / (float)H + eps);
+  }
   for (int i = threadIdx.x * V; i < H; i += blockDim.x * V) {
     float v[V];
     load<V>(res + base + i, v);
-    if (y != nullptr) {
+    if constexpr (POST) {
+      float a[V], g[V];
+      load<V>(row + i, a);
+      load<V>(post + i, g);
+#pragma unroll
+      for (int j = 0; j < V; ++j) v[j] += a[j] * scale * g[j];
+    } else if (y != nullptr) {
       float a[V];
       load<V>(y + base + i, a);
 #pragma unroll
@@ -154,10 +175,10 @@ __global__ void add_rms_norm_kernel(const TY* __restrict__ y, const TR* res, con
   }
 }
 
-template <typename TY, typename TR, typename TO>
-static int launch_add_rms(const void* y, const void* res, const void* w, void* res_out, void* out, int T, int H,
-                          float eps, float offset, cudaStream_t stream) {
-  const uintptr_t a = (uintptr_t)y | (uintptr_t)res | (uintptr_t)w | (uintptr_t)res_out | (uintptr_t)out;
+template <typename TY, typename TR, typename TO, bool POST>
+static int launch_add_rms(const void* y, const void* res, const void* w, const void* post, void* res_out, void* out, int T,
+                          int H, float eps, float offset, float mult, cudaStream_t stream) {
+  const uintptr_t a = (uintptr_t)y | (uintptr_t)res | (uintptr_t)w | (uintptr_t)post | (uintptr_t)res_out | (uintptr_t)out;
   const bool vec = H % 8 == 0 && a % 16 == 0;
   int threads = (H / (vec ? 8 : 1) + 31) / 32 * 32;
   threads = threads < 32 ? 32 : (threads > 512 ? 512 : threads);
@@ -165,14 +186,16 @@ static int launch_add_rms(const void* y, const void* res, const void* w, void* r
   static unsigned long long seen8 = 0, seen1 = 0;
   if (vec) {
     if (smem > 48 * 1024)
-      B200_CUDA_CHECK(ensure_dynamic_smem(add_rms_norm_kernel<8, TY, TR, TO>, 200 * 1024, &seen8));
-    B200_CUDA_CHECK(launch_pdl(add_rms_norm_kernel<8, TY, TR, TO>, dim3(T), dim3(threads), (size_t)smem, stream,
-                               (const TY*)y, (const TR*)res, (const TO*)w, (float*)res_out, (TO*)out, H, eps, offset));
+      B200_CUDA_CHECK(ensure_dynamic_smem(add_rms_norm_kernel<8, TY, TR, TO, POST>, 200 * 1024, &seen8));
+    B200_CUDA_CHECK(launch_pdl(add_rms_norm_kernel<8, TY, TR, TO, POST>, dim3(T), dim3(threads), (size_t)smem, stream,
+                               (const TY*)y, (const TR*)res, (const TO*)w, (const TO*)post, (float*)res_out, (TO*)out, H,
+                               eps, offset, mult));
   } else {
     if (smem > 48 * 1024)
-      B200_CUDA_CHECK(ensure_dynamic_smem(add_rms_norm_kernel<1, TY, TR, TO>, 200 * 1024, &seen1));
-    B200_CUDA_CHECK(launch_pdl(add_rms_norm_kernel<1, TY, TR, TO>, dim3(T), dim3(threads), (size_t)smem, stream,
-                               (const TY*)y, (const TR*)res, (const TO*)w, (float*)res_out, (TO*)out, H, eps, offset));
+      B200_CUDA_CHECK(ensure_dynamic_smem(add_rms_norm_kernel<1, TY, TR, TO, POST>, 200 * 1024, &seen1));
+    B200_CUDA_CHECK(launch_pdl(add_rms_norm_kernel<1, TY, TR, TO, POST>, dim3(T), dim3(threads), (size_t)smem, stream,
+                               (const TY*)y, (const TR*)res, (const TO*)w, (const TO*)post, (float*)res_out, (TO*)out, H,
+                               eps, offset, mult));
   }
   return 0;
 }
@@ -227,20 +250,24 @@ extern "C" int b200_layer_norm(const void* x, int x_elem, const void* w, int w_e
   return -1;
 }
 
-// y (or null): type of w; res: element bytes res_elem; w and out: w_elem (2 = bf16, 4 = fp32); res_out fp32 or null.
-extern "C" int b200_add_rms_norm(const void* y, const void* res, int res_elem, const void* w, int w_elem, void* res_out,
-                                 void* out, int T, int H, float eps, float offset, cudaStream_t stream) {
+// y (or null): type of w; res: element bytes res_elem; w, post and out: w_elem (2 = bf16, 4 = fp32); res_out fp32 or null;
+// post (or null): weight of the norm y passes first, times mult.
+extern "C" int b200_add_rms_norm(const void* y, const void* res, int res_elem, const void* w, const void* post, int w_elem,
+                                 void* res_out, void* out, int T, int H, float eps, float offset, float mult,
+                                 cudaStream_t stream) {
   if (T <= 0 || H <= 0) return 0;
   if (H > 50000) {
     b200_set_last_error("add_rms_norm: rows of at most 50000 elements", __FILE__, __LINE__);
     return -1;
   }
-  if (res_elem == 2 && w_elem == 2)
-    return ln::launch_add_rms<bf16, bf16, bf16>(y, res, w, res_out, out, T, H, eps, offset, stream);
-  if (res_elem == 4 && w_elem == 2)
-    return ln::launch_add_rms<bf16, float, bf16>(y, res, w, res_out, out, T, H, eps, offset, stream);
-  if (res_elem == 4 && w_elem == 4)
-    return ln::launch_add_rms<float, float, float>(y, res, w, res_out, out, T, H, eps, offset, stream);
+  const bool pn = post != nullptr && y != nullptr;
+#define ADD_RMS(TY, TR, TO)                                                                                             \
+  return pn ? ln::launch_add_rms<TY, TR, TO, true>(y, res, w, post, res_out, out, T, H, eps, offset, mult, stream)      \
+            : ln::launch_add_rms<TY, TR, TO, false>(y, res, w, nullptr, res_out, out, T, H, eps, offset, mult, stream)
+  if (res_elem == 2 && w_elem == 2) ADD_RMS(bf16, bf16, bf16);
+  if (res_elem == 4 && w_elem == 2) ADD_RMS(bf16, float, bf16);
+  if (res_elem == 4 && w_elem == 4) ADD_RMS(float, float, float);
+#undef ADD_RMS
   b200_set_last_error("add_rms_norm: unsupported combination of types", __FILE__, __LINE__);
   return -1;
 }

@@ -151,21 +151,21 @@ moe_permute_plan_kernel(const int* __restrict__ ids, int entries, int top_k, int
   }
 }
 
-// x_perm[pos] = x[row_src[pos]] for pos < group_off[E_local]
-__global__ void moe_gather_kernel(const __nv_bfloat16* __restrict__ x, const int* __restrict__ row_src,
-                                  const int* __restrict__ group_off, int E_local,
-                                  __nv_bfloat16* __restrict__ x_perm, int H, int T) {
+// x_perm[pos] = x[row_src[pos]] for pos < group_off[E_local]; rows of n pieces of type P (16 bytes, or 2)
+template <typename P>
+__global__ void moe_gather_kernel(const P* __restrict__ x, const int* __restrict__ row_src,
+                                  const int* __restrict__ group_off, int E_local, P* __restrict__ x_perm, int n, int T) {
   const int total = group_off[E_local];
   for (int pos = blockIdx.x; pos < total; pos += gridDim.x) {
     const int t = min(max(row_src[pos], 0), T - 1);
-    const uint4* src = reinterpret_cast<const uint4*>(x + (size_t)t * H);
-    uint4* dst = reinterpret_cast<uint4*>(x_perm + (size_t)pos * H);
-    for (int i = threadIdx.x; i < (H >> 3); i += blockDim.x) dst[i] = src[i];
+    const P* src = x + (size_t)t * n;
+    P* dst = x_perm + (size_t)pos * n;
+    for (int i = threadIdx.x; i < n; i += blockDim.x) dst[i] = src[i];
   }
 }
 
 // out[t] = sum_j w[t,j] * y[inv_pos[t,j]]   (rows with inv_pos < 0 belong to other ranks)
-__global__ void moe_unpermute_kernel(const __nv_bfloat16* __restrict__ y, const int* __restrict__ inv_pos,
+__global__ void moe_unpermute_kernel(const __nv_bfloat16* __restrict__ y, int ldy, const int* __restrict__ inv_pos,
                                      const float* __restrict__ w, __nv_bfloat16* __restrict__ out, int H,
                                      int top_k, int rows_cap) {
   const int t = blockIdx.x;
@@ -175,7 +175,7 @@ __global__ void moe_unpermute_kernel(const __nv_bfloat16* __restrict__ y, const 
       const int pos = inv_pos[(size_t)t * top_k + j];
       if (pos < 0 || pos >= rows_cap) continue;
       const float wt = w[(size_t)t * top_k + j];
-      const uint4 raw = *(reinterpret_cast<const uint4*>(y + (size_t)pos * H) + i);
+      const uint4 raw = *(reinterpret_cast<const uint4*>(y + (size_t)pos * ldy) + i);
       const __nv_bfloat162* h = reinterpret_cast<const __nv_bfloat162*>(&raw);
 #pragma unroll
       for (int q = 0; q < 4; ++q) {
@@ -189,6 +189,22 @@ __global__ void moe_unpermute_kernel(const __nv_bfloat16* __restrict__ y, const 
 #pragma unroll
     for (int q = 0; q < 4; ++q) oh[q] = __floats2bfloat162_rn(acc[2 * q], acc[2 * q + 1]);
     *(reinterpret_cast<uint4*>(out + (size_t)t * H) + i) = o;
+  }
+}
+
+// the same for 32-bit rows and widths that are no multiple of 16 bytes; y rows are ldy elements apart
+template <typename E>
+__global__ void moe_unpermute_any_kernel(const E* __restrict__ y, int ldy, const int* __restrict__ inv_pos,
+                                         const float* __restrict__ w, E* __restrict__ out, int H, int top_k, int rows_cap) {
+  const int t = blockIdx.x;
+  for (int i = threadIdx.x; i < H; i += blockDim.x) {
+    float acc = 0.f;
+    for (int j = 0; j < top_k; ++j) {
+      const int pos = inv_pos[(size_t)t * top_k + j];
+      if (pos >= 0 && pos < rows_cap) acc = fmaf(w[(size_t)t * top_k + j], to_f(y[(size_t)pos * ldy + i]), acc);
+    }
+    if constexpr (sizeof(E) == 2) out[(size_t)t * H + i] = __float2bfloat16(acc);
+    else out[(size_t)t * H + i] = acc;
   }
 }
 
@@ -294,29 +310,40 @@ extern "C" int b200_moe_route(const void* logits, int dtype, int ld, int T, int 
   return 0;
 }
 
-extern "C" int b200_moe_permute(const void* x, const int* ids, int T, int top_k, int H, int e_lo, int E_local,
+extern "C" int b200_moe_permute(const void* x, const int* ids, int T, int top_k, int row_bytes, int e_lo, int E_local,
                                 int* group_off, int* row_src, int* inv_pos, void* x_perm,
                                 cudaStream_t stream) {
   if (T == 0) return 0;
-  if (H % 8 || E_local > 8191) {
-    b200_set_last_error("moe_permute: H % 8 == 0 required", __FILE__, __LINE__);
+  if (row_bytes % 2 || E_local > 8191) {
+    b200_set_last_error("moe_permute: at most 8191 experts, rows of an even number of bytes", __FILE__, __LINE__);
     return -1;
   }
   moe_permute_plan_kernel<<<1, 1024, (E_local + 1) * sizeof(int), stream>>>(ids, T * top_k, top_k, e_lo,
                                                                            E_local, group_off, row_src, inv_pos);
   int blocks = T * top_k;
   if (blocks > 148 * 16) blocks = 148 * 16;
-  moe_gather_kernel<<<blocks, 128, 0, stream>>>((const __nv_bfloat16*)x, row_src, group_off, E_local,
-                                                (__nv_bfloat16*)x_perm, H, T);
+  if (row_bytes % 16 == 0 && ((uintptr_t)x | (uintptr_t)x_perm) % 16 == 0)
+    moe_gather_kernel<uint4><<<blocks, 128, 0, stream>>>((const uint4*)x, row_src, group_off, E_local, (uint4*)x_perm,
+                                                         row_bytes / 16, T);
+  else
+    moe_gather_kernel<uint16_t><<<blocks, 128, 0, stream>>>((const uint16_t*)x, row_src, group_off, E_local,
+                                                            (uint16_t*)x_perm, row_bytes / 2, T);
   B200_CUDA_CHECK(cudaGetLastError());
   return 0;
 }
 
-extern "C" int b200_moe_unpermute(const void* y, const int* inv_pos, const float* w, void* out, int T, int H,
-                                  int top_k, int rows_cap, cudaStream_t stream) {
+// y rows are ldy elements apart, out rows H; elem: 2 = bf16, 4 = fp32
+extern "C" int b200_moe_unpermute(const void* y, int ldy, const int* inv_pos, const float* w, void* out, int T, int H,
+                                  int top_k, int rows_cap, int elem, cudaStream_t stream) {
   if (T == 0) return 0;
-  moe_unpermute_kernel<<<T, 128, 0, stream>>>((const __nv_bfloat16*)y, inv_pos, w, (__nv_bfloat16*)out, H,
-                                              top_k, rows_cap);
+  if (elem == 4)
+    moe_unpermute_any_kernel<float><<<T, 128, 0, stream>>>((const float*)y, ldy, inv_pos, w, (float*)out, H, top_k, rows_cap);
+  else if (H % 8 || ldy % 8)
+    moe_unpermute_any_kernel<__nv_bfloat16><<<T, 128, 0, stream>>>((const __nv_bfloat16*)y, ldy, inv_pos, w,
+                                                                   (__nv_bfloat16*)out, H, top_k, rows_cap);
+  else
+    moe_unpermute_kernel<<<T, 128, 0, stream>>>((const __nv_bfloat16*)y, ldy, inv_pos, w, (__nv_bfloat16*)out, H,
+                                                top_k, rows_cap);
   B200_CUDA_CHECK(cudaGetLastError());
   return 0;
 }

@@ -50,7 +50,7 @@ class ConvAttention(GroupedAttention):
     def load_conv(self, q, k=None, v=None) -> None:
         s = self.spec
         parts = [self._own(q, s.heads)] + [self._own(t, s.kv_heads) for t in (k, v) if t is not None]
-        self.plan.conv_w = torch.cat(parts, 0).to(device=self.device, dtype=self.cfg.dtype).contiguous()
+        self.plan.conv_w = torch.cat(parts, 0).t().to(device=self.device, dtype=self.cfg.dtype).contiguous()
 
     def load_bias(self, q, k=None, v=None) -> None:
         self.inp.load_bias(**{n: t for n, t in (("q", q), ("k", k), ("v", v)) if t is not None})

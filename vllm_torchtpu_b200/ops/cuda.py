@@ -254,10 +254,10 @@ def layer_norm_add(y, residual, weight, eps):
     return (r if h is None else h), r
 
 
-def add_rms_norm(y, residual, weight, eps, offset: float = 0.0, update: bool = True):
-    """r = residual (+ y), h = r / rms(r) * (offset + weight).  Returns (h in the weight's dtype, r fp32); an fp32
-    residual is updated in place, a bf16 one (the embedding rows) starts the 32-bit stream.  Without ``update`` the
-    residual is only read."""
+def add_rms_norm(y, residual, weight, eps, offset: float = 0.0, update: bool = True, post=None, mult: float = 1.0):
+    """r = residual (+ y, or + mult * RMS norm of y with the weight ``post``), h = r / rms(r) * (offset + weight).
+    Returns (h in the weight's dtype, r fp32); an fp32 residual is updated in place, a bf16 one (the embedding rows)
+    starts the 32-bit stream.  Without ``update`` the residual is only read."""
     assert residual.is_contiguous() and (y is None or y.dtype == weight.dtype)
     y = y.contiguous() if y is not None else None
     H = residual.shape[-1]
@@ -267,9 +267,10 @@ def add_rms_norm(y, residual, weight, eps, offset: float = 0.0, update: bool = T
                                                                          device=residual.device)
         out = r if y is not None or r is not residual else None
     h = torch.empty(residual.shape, dtype=weight.dtype, device=residual.device)
-    _check(lib().b200_add_rms_norm(_p(y), _p(residual), c_int(_mixed(residual)), _p(weight), c_int(_mixed(weight)),
-                                   _p(out), _p(h), c_int(residual.numel() // H), c_int(H), c_float(eps),
-                                   c_float(offset), _stream()), "add_rms_norm")
+    assert post is None or post.dtype == weight.dtype
+    _check(lib().b200_add_rms_norm(_p(y), _p(residual), c_int(_mixed(residual)), _p(weight), _p(post),
+                                   c_int(_mixed(weight)), _p(out), _p(h), c_int(residual.numel() // H), c_int(H),
+                                   c_float(eps), c_float(offset), c_float(mult), _stream()), "add_rms_norm")
     count_launch()
     return h, r
 
@@ -292,6 +293,20 @@ def embedding(ids, table, token_src=None, last_tokens=None):
     _check(lib().b200_embedding(_p(ids), _p(token_src), _p(last_tokens), _p(table), _p(out), c_int(T),
                                 c_int(table.shape[1] * table.element_size()), c_int(table.shape[0]), _stream()),
            "embedding")
+    count_launch()
+    return out
+
+
+def embedding_pairs(ids, prev, table, pairs, bigram, token_src, last_tokens, last_inputs):
+    """See ``ops.reference.embedding_pairs``."""
+    T, H = ids.numel(), table.shape[1]
+    buckets, mul_prev, mul_cur = bigram
+    assert pairs.dtype == table.dtype and pairs.shape == (buckets + 1, H) and ids.dtype == prev.dtype == torch.int32
+    out = torch.empty((T, H), dtype=torch.float32, device=table.device)
+    _check(lib().b200_embedding_pairs(
+        _p(ids), _p(prev), _p(token_src), _p(last_tokens), _p(last_inputs), _p(table), _p(pairs), _p(out), c_int(T),
+        c_int(H), c_int(table.shape[0]), c_longlong(buckets), c_longlong(mul_prev), c_longlong(mul_cur),
+        c_int(_mixed(table)), _stream()), "embedding_pairs")
     count_launch()
     return out
 
@@ -951,6 +966,7 @@ _SUBMODULE_EXPORTS = {
                  "moe_experts_fp8", "quant_act_1x128", "quant_act_int8", "quant_rows_1x128"),
     "cuda_fp4": ("grouped_w4a16_gemm", "moe_experts_w4a16", "w4a16_gemm", "w4a16_int4_gemm", "dequant_w4", "dequant_int4"),
     "cuda_gdn": ("gdn_forward", "kda_forward", "short_conv"),
+    "cuda_conv": ("combine_heads", "conv_and_cache", "conv_ring_update"),
     "cuda_linear": ("carried_state_attention",),
     "cuda_mla": ("latent_prep", "mla_absorb", "mla_paged_attention", "mla_unabsorb", "mla_write_cache", "permute_rows", "rope_heads_into",
                  "rope_rows"),

@@ -8,6 +8,7 @@ import torch
 from .. import envs
 from . import count_launch
 from . import cuda as _c
+from .reference import UNGATED_ACTS
 
 
 def gemm_swiglu(x, w, out=None, gelu_tanh: bool = False):
@@ -35,8 +36,19 @@ def gemm_swiglu(x, w, out=None, gelu_tanh: bool = False):
     return y
 
 
-def grouped_gemm(x_perm, w, group_off, swiglu: bool, avg_rows: int, out=None):
-    """Rows [group_off[e], group_off[e+1]) of x_perm times w[e] ([N,K] or [2N,K] when swiglu)."""
+def grouped_gemm(x_perm, w, group_off, swiglu: bool, avg_rows: int, out=None, act: str = ""):
+    """Rows [group_off[e], group_off[e+1]) of x_perm times w[e] ([N,K] or [2N,K] when swiglu); ``act`` (without swiglu)
+    "relu2": the square of relu in the epilogue.  32-bit operands, and sizes a tensor map cannot describe, run on the
+    CUDA cores."""
+    code = {"": 0, "relu2": 4}[act]
+    if not swiglu and (x_perm.dtype == torch.float32 or x_perm.shape[1] % 8 or w.shape[1] % 128):
+        assert x_perm.is_contiguous() and w.is_contiguous() and x_perm.dtype == w.dtype and out is None
+        y = torch.empty((x_perm.shape[0], w.shape[1]), dtype=x_perm.dtype, device=x_perm.device)
+        _c._check(_c.lib().b200_grouped_gemm_simt(
+            _c._p(x_perm), _c._p(w), _c._p(y), _c._p(group_off), c_int(w.shape[0]), c_int(w.shape[1]), c_int(w.shape[2]),
+            c_int(code), c_int(_c._mixed(x_perm)), _c._stream()), "grouped_gemm_simt")
+        count_launch()
+        return y
     _c._require_bf16(x_perm, w)
     R, K = x_perm.shape
     E = w.shape[0]
@@ -47,7 +59,7 @@ def grouped_gemm(x_perm, w, group_off, swiglu: bool, avg_rows: int, out=None):
     ws = _c.Workspace.get(x_perm.device)
     _c._check(_c.lib().b200_grouped_gemm_bf16(
         _c._p(x_perm), _c._p(w), _c._p(y), _c._p(group_off), c_int(E), c_int(R), c_int(N), c_int(K),
-        c_int(1 if swiglu else 0), c_int(max(1, avg_rows)), _c._p(ws.status), c_int(_c._sms), _c._stream()),
+        c_int(1 if swiglu else 0), c_int(code), c_int(max(1, avg_rows)), _c._p(ws.status), c_int(_c._sms), _c._stream()),
         "grouped_gemm")
     count_launch()
     return y
@@ -89,18 +101,19 @@ def moe_permute(x, topk_ids, e_lo: int, e_local: int):
     inv_pos = torch.empty(T * k, dtype=torch.int32, device=dev)
     x_perm = torch.empty((T * k, H), dtype=x.dtype, device=dev)
     _c._check(_c.lib().b200_moe_permute(
-        _c._p(x), _c._p(topk_ids), c_int(T), c_int(k), c_int(H), c_int(e_lo), c_int(e_local), _c._p(group_off),
+        _c._p(x), _c._p(topk_ids), c_int(T), c_int(k), c_int(H * x.element_size()), c_int(e_lo), c_int(e_local), _c._p(group_off),
         _c._p(row_src), _c._p(inv_pos), _c._p(x_perm), _c._stream()), "moe_permute")
     count_launch(2)
     return x_perm, group_off, row_src, inv_pos
 
 
-def moe_unpermute(y, inv_pos, topk_w, T: int):
-    H = y.shape[1]
+def moe_unpermute(y, inv_pos, topk_w, T: int, H: int = 0):
+    """[T, H] weighted sums of the rows of y, whose first H columns count (0: all)."""
+    H = H or y.shape[1]
     k = topk_w.shape[1]
     out = torch.empty((T, H), dtype=y.dtype, device=y.device)
-    _c._check(_c.lib().b200_moe_unpermute(_c._p(y), _c._p(inv_pos), _c._p(topk_w), _c._p(out), c_int(T),
-                                          c_int(H), c_int(k), c_int(y.shape[0]), _c._stream()),
+    _c._check(_c.lib().b200_moe_unpermute(_c._p(y), c_int(y.stride(0)), _c._p(inv_pos), _c._p(topk_w), _c._p(out), c_int(T),
+                                          c_int(H), c_int(k), c_int(y.shape[0]), c_int(_c._mixed(y)), _c._stream()),
               "moe_unpermute")
     count_launch()
     return out
@@ -126,6 +139,8 @@ def moe_experts(x, w13, w2, topk_ids, topk_w, expert_offset: int = 0, act: str =
     avg = (T * k + E_local - 1) // E_local
     if act == "silu" and b13 is None:
         h = grouped_gemm(x_perm, w13, group_off, True, avg)          # SiLU * mul in the GEMM epilogue
+    elif act in UNGATED_ACTS:
+        h = grouped_gemm(x_perm, w13, group_off, False, avg, act=act)
     else:
         # other gated activations / expert biases: one grouped GEMM over the stacked [gate; up] rows, bias,
         # then the activation kernel
@@ -136,8 +151,7 @@ def moe_experts(x, w13, w2, topk_ids, topk_w, expert_offset: int = 0, act: str =
     y = grouped_gemm(h, w2, group_off, False, avg)
     if b2 is not None:
         group_bias_add(y, b2, group_off)
-    out = moe_unpermute(y, inv_pos, topk_w.contiguous(), T)
-    return out if out.shape[1] == H else out[:, :H].contiguous()      # down projection padded to the tile width
+    return moe_unpermute(y, inv_pos, topk_w.contiguous(), T, H)      # (y: down projection padded to the tile width)
 
 
 # ----------------------------------------------------------------- expert parallel, fused plane

@@ -48,7 +48,7 @@ class ConvAttentionPlan:
     width: int                           # columns of a stored head
     offsets: tuple                       # first columns of q, k, v in the row
     taps: int
-    conv_w: Optional[torch.Tensor] = None       # [channels, taps] in the model dtype, channels = q | k | v
+    conv_w: Optional[torch.Tensor] = None       # [taps, channels] in the model dtype, channels = q | k | v
     inv_freq: Optional[torch.Tensor] = None     # [pairs] fp32, None: no rotation
     rot_mult: float = 1.0
 
@@ -86,7 +86,7 @@ def conv_and_cache(plan: ConvAttentionPlan, row, kv_cache, ring, meta):
     x, y = plan.split(row), torch.zeros(T, plan.channels, device=row.device)
     for a, b, start, slot in portions_of(meta):
         mine = ring[slot] if slot >= 0 else torch.zeros_like(ring[0])
-        y[a:b] = conv_with_ring(x[a:b], p.conv_w, mine, start)
+        y[a:b] = conv_with_ring(x[a:b], p.conv_w.t(), mine, start)
     q, k, v = y.split(p.sizes, -1)
     q, k = q.reshape(T, p.heads * p.maps, p.dim), k.reshape(T, p.kv_heads * p.maps, p.dim)
     if p.inv_freq is not None:
