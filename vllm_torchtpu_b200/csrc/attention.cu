@@ -48,6 +48,7 @@ struct AttnParams {
   // ones; a query at global position g sees the first dcp_local_len(g + 1) local keys
   const int* global_seq_lens;
   int dcp_size, dcp_rank, dcp_interleave;
+  HeadFinish fin;                // decode kernel with FIN
 };
 
 // number of positions < n that live on `rank` when positions are dealt round-robin in runs of `il`
@@ -189,7 +190,8 @@ struct DecodeSmem {
   static constexpr int TOTAL = 4 * WARP_BYTES;
 };
 
-template <int D, bool FP8 = false>
+// FIN: the epilogue goes on to what p.fin describes.
+template <int D, bool FP8 = false, bool FIN = false>
 __global__ void __launch_bounds__(128, 2) attn_decode_kernel(const AttnParams p) {
   using SM = DecodeSmem<D, FP8>;
   constexpr int STAGES = SM::STAGES;
@@ -402,6 +404,43 @@ __global__ void __launch_bounds__(128, 2) attn_decode_kernel(const AttnParams p)
   const int tok_row = qs + row / G, head = h * G + row % G;
 
   auto finish = [&](float mfin, float Lfin, const float* a) {
+    if constexpr (FIN) {
+      const float inv = row_ok && Lfin > 0.f ? 1.f / Lfin : 0.f;
+      float v[SEG];
+#pragma unroll
+      for (int d = 0; d < SEG; ++d) v[d] = a[d] * inv;
+      int h_out = head, heads = p.Hq;
+      bool write = row_ok;
+      if (p.fin.lam != nullptr) {                   // rows 2i, 2i + 1 (lanes 8 apart) are the maps of one head
+        const float lam = *p.fin.lam;
+        float ss = 0.f;
+#pragma unroll
+        for (int d = 0; d < SEG; ++d) {
+          v[d] -= lam * __shfl_xor_sync(0xffffffffu, v[d], 8);
+          ss += v[d] * v[d];
+        }
+        ss += __shfl_xor_sync(0xffffffffu, ss, 1);
+        ss += __shfl_xor_sync(0xffffffffu, ss, 2);
+        ss += __shfl_xor_sync(0xffffffffu, ss, 4);
+        const float sc = p.fin.keep / sqrtf(ss / (float)p.fin.vdim + p.fin.eps);
+#pragma unroll
+        for (int d = 0; d < SEG; ++d) v[d] *= sc;
+        write = row_ok && !(row & 1);
+        h_out = head >> 1;
+        heads = p.Hq >> 1;
+      }
+      if (!write) return;
+      if (p.fin.gate != nullptr) gate_columns<SEG>(p.fin, tok_row, h_out, seg * SEG, v);
+      __nv_bfloat16* dst = p.out + ((size_t)tok_row * heads + h_out) * D + seg * SEG;
+#pragma unroll
+      for (int d = 0; d < SEG; d += 8) {
+        bf16x8 o8;
+#pragma unroll
+        for (int u = 0; u < 4; ++u) o8.v[u] = __floats2bfloat162_rn(v[d + 2 * u], v[d + 2 * u + 1]);
+        *reinterpret_cast<bf16x8*>(dst + d) = o8;
+      }
+      return;
+    }
     if (!row_ok) return;
     if (p.sinks != nullptr) {
       // attention sink: one extra logit per head that only joins the normaliser
@@ -730,13 +769,13 @@ static void set_fp8_scales(AttnParams& p, float k_scale, float v_scale) {
   p.v_scale = v_scale * (kHwV ? 1.f : 256.f);
 }
 
-template <int D, bool FP8>
+template <int D, bool FP8, bool FIN = false>
 static cudaError_t launch_decode(dim3 grid, cudaStream_t stream, const AttnParams& p) {
   constexpr int smem = DecodeSmem<D, FP8>::TOTAL;
   static unsigned long long seen = 0;
-  cudaError_t e = ensure_dynamic_smem(attn_decode_kernel<D, FP8>, smem, &seen);
+  cudaError_t e = ensure_dynamic_smem(attn_decode_kernel<D, FP8, FIN>, smem, &seen);
   if (e != cudaSuccess) return e;
-  return launch_pdl(attn_decode_kernel<D, FP8>, grid, dim3(128), smem, stream, p);
+  return launch_pdl(attn_decode_kernel<D, FP8, FIN>, grid, dim3(128), smem, stream, p);
 }
 
 template <int D, bool FP8>
@@ -762,7 +801,7 @@ static int attn_decode_impl(const void* q, const void* kv, void* out, float* lse
                             int max_blocks, int block_size, long long num_blocks, int Hq, int Hkv, int D,
                             float scale, int window, float softcap, const float* sinks, int num_splits,
                             void* scratch, int* counters, int kv_fp8, float k_scale, float v_scale,
-                            cudaStream_t stream) {
+                            cudaStream_t stream, const HeadFinish* fin = nullptr) {
   const int R = req_end - req_begin;
   if (R <= 0) return 0;
   if (block_size % 16 || (Hq % Hkv) || Hq / Hkv > 16) {
@@ -783,6 +822,16 @@ static int attn_decode_impl(const void* q, const void* kv, void* out, float* lse
   p.counters = counters;
   dim3 grid(Hkv, R, num_splits);
   if (kv_fp8) set_fp8_scales(p, k_scale, v_scale);
+  if (fin != nullptr) {
+    if ((D != 128 && D != 64) || (fin->lam != nullptr && (Hq / Hkv) % 2) || fin->vdim < 1 || fin->vdim > D) {
+      b200_set_last_error("attn_decode_heads: heads of 64 or 128, pairs of maps within a kv head", __FILE__, __LINE__);
+      return -1;
+    }
+    p.fin = *fin;
+    if (D == 128) B200_CUDA_CHECK((launch_decode<128, false, true>(grid, stream, p)));
+    else B200_CUDA_CHECK((launch_decode<64, false, true>(grid, stream, p)));
+    return 0;
+  }
   if (D == 128 && kv_fp8) B200_CUDA_CHECK((launch_decode<128, true>(grid, stream, p)));
   else if (D == 128) B200_CUDA_CHECK((launch_decode<128, false>(grid, stream, p)));
   else if (D == 64 && kv_fp8) B200_CUDA_CHECK((launch_decode<64, true>(grid, stream, p)));
@@ -804,6 +853,18 @@ extern "C" int b200_attn_decode(const void* q, const void* kv, void* out, float*
                           block_size, num_blocks, Hq, Hkv, D, scale, window, softcap, sinks, num_splits, scratch,
                           counters, 0, 1.f, 1.f, stream);
 }
+// The same with the epilogue of HeadFinish: out [T, lam ? Hq / 2 : Hq, D].
+extern "C" int b200_attn_decode_heads(const void* q, const void* kv, void* out, const int* block_tables,
+                                      const int* seq_lens, const int* qsl, int req_begin, int req_end, int max_blocks,
+                                      int block_size, long long num_blocks, int Hq, int Hkv, int D, float scale,
+                                      int window, int num_splits, void* scratch, int* counters, const float* lam,
+                                      const void* gate, int ldg, int vdim, float keep, float eps, cudaStream_t stream) {
+  const HeadFinish fin{lam, (const __nv_bfloat16*)gate, ldg, vdim, keep, eps};
+  return attn_decode_impl(q, kv, out, nullptr, block_tables, seq_lens, qsl, req_begin, req_end, max_blocks,
+                          block_size, num_blocks, Hq, Hkv, D, scale, window, 0.f, nullptr, num_splits, scratch,
+                          counters, 0, 1.f, 1.f, stream, &fin);
+}
+
 // The cache holds e4m3 bytes: stored value * k_scale (v_scale) is the key (value).
 extern "C" int b200_attn_decode_fp8kv(const void* q, const void* kv, void* out, float* lse,
                                       const int* block_tables, const int* seq_lens, const int* qsl,

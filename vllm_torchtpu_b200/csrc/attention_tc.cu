@@ -54,6 +54,7 @@ struct Params {
   int non_causal;                 // 1: every query row sees the whole sequence (encoders, diffusion)
   long long num_blocks;
   float scale_log2, softcap;
+  HeadFinish fin;                 // with FIN
 };
 
 // MN-major operand whose rows (K index) are 128 bytes = 64 elements of the MN dimension, written by
@@ -77,6 +78,8 @@ __device__ __forceinline__ float ex2f(float x) {
   return y;
 }
 
+// FIN: the epilogue goes on to what p.fin describes.
+template <bool FIN>
 __global__ void __launch_bounds__(NUM_THREADS, 1)
 attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmKV,
                        const Params p) {
@@ -410,7 +413,57 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
       if (ok && !mbar_wait(l_bar, 0, abort_flag, p.status, ST_TIMEOUT_FLAG)) ok = false;
       if (ok) l += l_sh[(half ^ 1) * 128 + row];
     }
-    if (ok && row_ok) {
+    if constexpr (FIN) {
+      const float inv = ok && l > 0.f ? 1.f / l : 0.f;
+#pragma unroll
+      for (int i = 0; i < HD; ++i) acc[i] *= inv;
+      const long long t = qs + q0 + pos_local;
+      if (p.fin.lam != nullptr) {
+        // the maps of a head are neighbouring rows (lanes): each of the two takes half of this thread's columns
+        const bool odd = lane & 1;
+        const float lam = *p.fin.lam;
+        constexpr int HQ = HD / 2;
+        float o[HQ], ss = 0.f;
+#pragma unroll
+        for (int i = 0; i < HQ; ++i) {
+          const float got = __shfl_xor_sync(0xffffffffu, odd ? acc[i] : acc[HQ + i], 1);
+          o[i] = odd ? got - lam * acc[HQ + i] : acc[i] - lam * got;
+          ss += o[i] * o[i];
+        }
+        ss += __shfl_xor_sync(0xffffffffu, ss, 1);
+        if (nchunks > 0) {
+          mx_sh[half * 128 + row] = ss;             // (the row maxima have been read: every thread passed l_bar)
+          mbar_arrive(l_bar);
+          if (ok && !mbar_wait(l_bar, 1, abort_flag, p.status, ST_TIMEOUT_FLAG)) ok = false;
+          if (ok) ss += mx_sh[(half ^ 1) * 128 + row];
+        }
+        const float sc = p.fin.keep / sqrtf(ss / (float)p.fin.vdim + p.fin.eps);
+        if (ok && row_ok) {
+#pragma unroll
+          for (int i = 0; i < HQ; ++i) o[i] *= sc;
+          const int col = half * HD + (odd ? HQ : 0);
+          if (p.fin.gate != nullptr) gate_columns<HQ>(p.fin, t, head >> 1, col, o);
+          __nv_bfloat16* dst = p.out + ((size_t)t * (p.Hq >> 1) + (head >> 1)) * D + col;
+#pragma unroll
+          for (int i = 0; i < HQ; i += 8) {
+            bf16x8 o8;
+#pragma unroll
+            for (int u = 0; u < 4; ++u) o8.v[u] = __floats2bfloat162_rn(o[i + 2 * u], o[i + 2 * u + 1]);
+            *reinterpret_cast<bf16x8*>(dst + i) = o8;
+          }
+        }
+      } else if (ok && row_ok) {
+        if (p.fin.gate != nullptr) gate_columns<HD>(p.fin, t, head, half * HD, acc);
+        __nv_bfloat16* dst = p.out + ((size_t)t * p.Hq + head) * D + half * HD;
+#pragma unroll
+        for (int i = 0; i < HD; i += 8) {
+          bf16x8 o8;
+#pragma unroll
+          for (int u = 0; u < 4; ++u) o8.v[u] = __floats2bfloat162_rn(acc[i + 2 * u], acc[i + 2 * u + 1]);
+          *reinterpret_cast<bf16x8*>(dst + i) = o8;
+        }
+      }
+    } else if (ok && row_ok) {
       float sc = 1.f;
       if (p.sinks != nullptr) {
         const float sk = p.sinks[head] * 1.4426950408889634f;
@@ -455,7 +508,7 @@ static int attn_prefill_tc_impl(const void* q, const void* kv, void* out, float*
                                 const int* seq_lens, const int* qsl, int req_begin, int req_end, int num_tiles_64,
                                 int total_tokens, int max_blocks, int block_size, long long num_blocks, int Hq,
                                 int Hkv, int D, float scale, int window, float softcap, const float* sinks,
-                                int* status, int non_causal, cudaStream_t stream) {
+                                int* status, int non_causal, cudaStream_t stream, const HeadFinish* fin = nullptr) {
   if (req_end <= req_begin || num_tiles_64 <= 0) return 0;
   const int G = Hkv > 0 ? Hq / Hkv : 0;
   if (D != 128 || Hq % Hkv || (G != 1 && G != 2 && G != 4 && G != 8) || block_size % 16) {
@@ -481,13 +534,22 @@ static int attn_prefill_tc_impl(const void* q, const void* kv, void* out, float*
   rc = b200_make_tmap_2d(&tmKV, kv, 2, (uint64_t)num_blocks * 2 * Hkv * block_size, (uint64_t)D, (uint64_t)D * 2,
                          16, 64);
   if (rc) return rc;
-  static unsigned long long attr_seen = 0;
-  B200_CUDA_CHECK(ensure_dynamic_smem(fa::attn_prefill_tc_kernel, fa::SMEM_TOTAL, &attr_seen));
+  static unsigned long long attr_seen = 0, attr_seen_fin = 0;
+  if (fin != nullptr) {
+    if ((fin->lam != nullptr && G % 2) || fin->vdim < 1 || fin->vdim > D) {
+      b200_set_last_error("attn_prefill_tc_heads: pairs of maps within a kv head", __FILE__, __LINE__);
+      return -1;
+    }
+    p.fin = *fin;
+    B200_CUDA_CHECK(ensure_dynamic_smem(fa::attn_prefill_tc_kernel<true>, fa::SMEM_TOTAL, &attr_seen_fin));
+  } else {
+    B200_CUDA_CHECK(ensure_dynamic_smem(fa::attn_prefill_tc_kernel<false>, fa::SMEM_TOTAL, &attr_seen));
+  }
   // ceil(q_len / BQ) <= ceil(q_len / 64) * (64 / BQ) for BQ <= 64; BQ = 128 needs at most as many tiles
   const int tiles = p.BQ >= 64 ? num_tiles_64 : num_tiles_64 * (64 / p.BQ);
   dim3 grid(Hkv, tiles);
-  B200_CUDA_CHECK(launch_pdl(fa::attn_prefill_tc_kernel, grid, dim3(fa::NUM_THREADS), (size_t)fa::SMEM_TOTAL, stream,
-                             tmQ, tmKV, p));
+  B200_CUDA_CHECK(launch_pdl(fin != nullptr ? fa::attn_prefill_tc_kernel<true> : fa::attn_prefill_tc_kernel<false>, grid,
+                             dim3(fa::NUM_THREADS), (size_t)fa::SMEM_TOTAL, stream, tmQ, tmKV, p));
   return 0;
 }
 
@@ -499,6 +561,19 @@ extern "C" int b200_attn_prefill_tc(const void* q, const void* kv, void* out, fl
   return attn_prefill_tc_impl(q, kv, out, lse, block_tables, seq_lens, qsl, req_begin, req_end, num_tiles_64,
                               total_tokens, max_blocks, block_size, num_blocks, Hq, Hkv, D, scale, window, softcap,
                               sinks, status, 0, stream);
+}
+
+// The same with the epilogue of HeadFinish: out [T, lam ? Hq / 2 : Hq, D].
+extern "C" int b200_attn_prefill_tc_heads(const void* q, const void* kv, void* out, const int* block_tables,
+                                          const int* seq_lens, const int* qsl, int req_begin, int req_end,
+                                          int num_tiles_64, int total_tokens, int max_blocks, int block_size,
+                                          long long num_blocks, int Hq, int Hkv, int D, float scale, int window,
+                                          const float* lam, const void* gate, int ldg, int vdim, float keep, float eps,
+                                          int* status, cudaStream_t stream) {
+  const HeadFinish fin{lam, (const __nv_bfloat16*)gate, ldg, vdim, keep, eps};
+  return attn_prefill_tc_impl(q, kv, out, nullptr, block_tables, seq_lens, qsl, req_begin, req_end, num_tiles_64,
+                              total_tokens, max_blocks, block_size, num_blocks, Hq, Hkv, D, scale, window, 0.f, nullptr,
+                              status, 0, stream, &fin);
 }
 
 // Bidirectional form (vision encoders, diffusion transformers): each request's q_len equals its seq_len and

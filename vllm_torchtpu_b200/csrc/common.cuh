@@ -390,6 +390,25 @@ __device__ __forceinline__ float gated_pair(float g, float u) {
 __device__ __forceinline__ float relu_squared(float v) { return v > 0.f ? v * v : 0.f; }
 __device__ __forceinline__ float soft_cap(float v, float cap) { return cap > 0.f ? cap * tanhf(v / cap) : v; }
 
+// What follows the softmax of a head before the output projection, in the epilogue of the attention kernels:
+//   lam:  query heads 2h and 2h + 1 are two maps of head h over the same values; o = o1 - lam * o2, then
+//         o / rms(o over vdim) * keep.  The output has half as many heads.
+//   gate: o times sigmoid(gate[t, h * vdim + d])
+struct HeadFinish {
+  const float* lam;
+  const __nv_bfloat16* gate;
+  int ldg, vdim;
+  float keep, eps;
+};
+// v[i] *= sigmoid of the gate of columns col + i (those below vdim)
+template <int N>
+__device__ __forceinline__ void gate_columns(const HeadFinish& f, long long t, int head, int col, float* v) {
+  const __nv_bfloat16* g = f.gate + (size_t)t * f.ldg + (size_t)head * f.vdim + col;
+#pragma unroll
+  for (int i = 0; i < N; ++i)
+    if (col + i < f.vdim) v[i] = __fdividef(v[i], 1.f + __expf(-__bfloat162float(g[i])));
+}
+
 struct alignas(16) bf16x8 {
   __nv_bfloat162 v[4];
 };

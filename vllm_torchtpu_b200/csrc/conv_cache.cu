@@ -84,147 +84,196 @@ __device__ __forceinline__ void store(E* p, const float (&v)[V], int e0 = 0, int
   }
 }
 
-// grid (token runs of TT, vectors / blockDim).  KM: taps the window is held in registers for (0: any number, re-read).
+// The channels that vector `vec` of the stored heads takes: row column and ring channel of its element 0 (elements e0 ..
+// e1 - 1 exist, the others are zeros), head index (q rows, then k, then v heads) and first column in the head.
+struct Where {
+  int hh, d0, ch, col, e0, e1;
+  bool rotated;
+};
+template <int V>
+__device__ __forceinline__ Where where_is(const Params& p, int vec) {
+  const int nv = p.D / V, nq = p.H * p.maps, cq = nq * p.dim, ck = p.G * p.maps * p.dim;
+  Where w;
+  w.hh = vec / nv;
+  w.d0 = (vec - w.hh * nv) * V;
+  int lo = 0, hi;
+  w.rotated = p.pairs > 0;
+  if (w.hh < nq) {
+    const int h = w.hh / p.maps, m = w.hh - h * p.maps;
+    w.ch = h * p.maps * p.dim + w.d0;
+    w.col = p.q_off + w.ch;
+    lo = m * p.dim;
+    hi = lo + p.dim;
+  } else if (w.hh < nq + p.G) {
+    w.ch = (w.hh - nq) * p.maps * p.dim + w.d0;
+    w.col = p.k_off + w.ch;
+    w.ch += cq;
+    hi = p.maps * p.dim;
+  } else {
+    w.ch = (w.hh - nq - p.G) * p.vdim + w.d0;
+    w.col = p.v_off + w.ch;
+    w.ch += cq + ck;
+    hi = p.vdim;
+    w.rotated = false;
+  }
+  w.e0 = max(lo - w.d0, 0);
+  w.e1 = min(hi - w.d0, V);
+  return w;
+}
+
+// grid (token runs of TT, parts of the vectors).  KM: taps the window is held in registers for (0: any number, re-read).
+// A run is walked in groups of up to four tokens whose inputs are requested together; the inputs in front of the run are
+// requested before the tokens' requests are known, and what turns out to belong to another portion is replaced.
 template <typename E, int V, bool VEC, int KM, int TT>
-__global__ void __launch_bounds__(256) conv_cache_kernel(const Params p) {
-  pdl_launch_dependents();
-  pdl_wait();
+__global__ void __launch_bounds__(256, 2) conv_cache_kernel(const Params p) {
   extern __shared__ __align__(16) float2 turn[];          // [TT][pairs]
   __shared__ Token tok[TT];
   const int tid = threadIdx.x, t0 = blockIdx.x * TT;
-  if (tid < TT) tok[tid] = token_of(p, t0 + tid);
-  __syncthreads();
-  for (int i = tid; i < TT * p.pairs; i += blockDim.x) {
-    const int k = i / p.pairs;
-    float sn, cs;
-    sincosf((float)tok[k].pos * p.inv_freq[i - k * p.pairs], &sn, &cs);
-    turn[i] = make_float2(cs * p.rot_mult, sn * p.rot_mult);
-  }
-  __syncthreads();
-  const int nv = p.D / V, vec = blockIdx.y * blockDim.x + tid, hh = vec / nv, d0 = (vec - hh * nv) * V;
-  const int nq = p.H * p.maps;
-  if (hh >= nq + 2 * p.G) return;
-  // channels of this thread: elements e0 .. e1 - 1 exist; turn0: index within the map of element 0
-  const int cq = nq * p.dim, ck = p.G * p.maps * p.dim, C = cq + ck + p.G * p.vdim;
-  int ch, col, lo, hi;
-  bool rotated = p.pairs > 0;
-  if (hh < nq) {
-    const int h = hh / p.maps, m = hh - h * p.maps;
-    ch = h * p.maps * p.dim + d0;
-    col = p.q_off + ch;
-    lo = m * p.dim;
-    hi = lo + p.dim;
-  } else if (hh < nq + p.G) {
-    ch = (hh - nq) * p.maps * p.dim + d0;
-    col = p.k_off + ch;
-    ch += cq;
-    lo = 0;
-    hi = p.maps * p.dim;
-  } else {
-    ch = (hh - nq - p.G) * p.vdim + d0;
-    col = p.v_off + ch;
-    ch += cq + ck;
-    lo = 0;
-    hi = p.vdim;
-    rotated = false;
-  }
-  const int e0 = max(lo - d0, 0), e1 = min(hi - d0, V);
-  const bool any = e0 < e1;
+  const int nq = p.H * p.maps, C = (nq + p.G * p.maps) * p.dim + p.G * p.vdim, vecs = (nq + 2 * p.G) * (p.D / V);
   const E* row = reinterpret_cast<const E*>(p.row);
-  const E* w = reinterpret_cast<const E*>(p.w) + ch;
   E* ring = reinterpret_cast<E*>(p.ring);
-  // input of position pos - back for the token with info k in row t
-  auto input = [&](const Token& k, int t, int back, float (&u)[V]) {
-    const int pos = k.pos - back;
-    if (pos >= 0 && t - back >= k.qs) {
-      load<E, V, VEC>(row + (size_t)(t - back) * p.ldr + col, e0, e1, u);
-    } else if (pos >= 0 && k.state >= 0) {
-      load<E, V, VEC>(ring + ((size_t)k.state * p.taps + pos % p.taps) * C + ch, e0, e1, u);
-    } else {
-#pragma unroll
-      for (int e = 0; e < V; ++e) u[e] = 0.f;
-    }
-  };
   constexpr int HB = KM > 1 ? KM - 1 : 1;
-  float wt[KM > 0 ? KM : 1][V], hist[HB][V];               // hist[j]: input of j + 1 positions before
+  bool ready = false;
+  for (int v0 = blockIdx.y * blockDim.x; v0 < vecs; v0 += gridDim.y * blockDim.x) {
+    const int vec = v0 + tid;
+    const Where x = where_is<V>(p, min(vec, vecs - 1));
+    const bool any = x.e0 < x.e1 && vec < vecs;
+    const E* w = reinterpret_cast<const E*>(p.w) + x.ch;
+    constexpr int GR = TT < 4 ? TT : 4;
+    uint4 raw[GR], before[HB];                             // inputs of a group and of the rows in front of the run
+    uint4 wt[VEC && KM > 0 ? KM : 1];                      // wt[j]: weights of the inputs j positions before
+    auto request = [&](int t) {
+      return any && t >= 0 && t < p.T ? *reinterpret_cast<const uint4*>(row + (size_t)t * p.ldr + x.col)
+                                      : make_uint4(0u, 0u, 0u, 0u);
+    };
+    if constexpr (VEC) {
 #pragma unroll
-  for (int j = 0; j < HB; ++j)
-#pragma unroll
-    for (int e = 0; e < V; ++e) hist[j][e] = 0.f;
-  if constexpr (KM > 0) {
-#pragma unroll
-    for (int j = 0; j < KM; ++j) {                         // wt[j]: weight of the input j positions before
-#pragma unroll
-      for (int e = 0; e < V; ++e) wt[j][e] = 0.f;
-      if (any && j < p.taps) load<E, V, VEC>(w + (size_t)(p.taps - 1 - j) * C, e0, e1, wt[j]);
-    }
-  }
-  float u[TT][V];
-#pragma unroll
-  for (int i = 0; i < TT; ++i) {
-#pragma unroll
-    for (int e = 0; e < V; ++e) u[i][e] = 0.f;
-    if (any && tok[i].len > 0) load<E, V, VEC>(row + (size_t)(t0 + i) * p.ldr + col, e0, e1, u[i]);
-  }
-#pragma unroll
-  for (int i = 0; i < TT; ++i) {
-    const int t = t0 + i;
-    if (t >= p.T) break;
-    const Token k = tok[i];
-    float y[V];
-#pragma unroll
-    for (int e = 0; e < V; ++e) y[e] = 0.f;
-    if (any && k.len > 0) {
+      for (int i = 0; i < GR; ++i) raw[i] = request(t0 + i);
       if constexpr (KM > 0) {
-        if (i == 0 || tok[i > 0 ? i - 1 : 0].qs != k.qs) {
 #pragma unroll
-          for (int j = 0; j < KM - 1; ++j)
-            if (j + 1 < p.taps) input(k, t, j + 1, hist[j]);
-        }
+        for (int i = 0; i < HB; ++i) before[i] = request(t0 - 1 - i);
+      }
+    }
+    if constexpr (VEC && KM > 0) {
 #pragma unroll
-        for (int j = KM - 2; j >= 0; --j)
-#pragma unroll
-          for (int e = 0; e < V; ++e) y[e] = fmaf(wt[j + 1][e], hist[j][e], y[e]);
-#pragma unroll
-        for (int e = 0; e < V; ++e) y[e] = fmaf(wt[0][e], u[i][e], y[e]);
-#pragma unroll
-        for (int j = KM - 2; j > 0; --j)
-#pragma unroll
-          for (int e = 0; e < V; ++e) hist[j][e] = hist[j - 1][e];
-#pragma unroll
-        for (int e = 0; e < V; ++e) hist[0][e] = u[i][e];
+      for (int j = 0; j < KM; ++j) {
+        wt[j] = make_uint4(0u, 0u, 0u, 0u);
+        if (any && j < p.taps) wt[j] = *reinterpret_cast<const uint4*>(w + (size_t)(p.taps - 1 - j) * C);
+      }
+    }
+    if (!ready) {                                          // uniform over the CTA
+      if (tid < TT) tok[tid] = token_of(p, t0 + tid);
+      __syncthreads();
+      for (int i = tid; i < TT * p.pairs; i += blockDim.x) {
+        const int k = i / p.pairs;
+        float sn, cs;
+        sincosf((float)tok[k].pos * p.inv_freq[i - k * p.pairs], &sn, &cs);
+        turn[i] = make_float2(cs * p.rot_mult, sn * p.rot_mult);
+      }
+      __syncthreads();
+      ready = true;
+    }
+    if (vec >= vecs) continue;
+    // input of position pos - back for the token with info k in row t
+    auto input = [&](const Token& k, int t, int back, float (&u)[V]) {
+      const int pos = k.pos - back;
+      if (pos >= 0 && t - back >= k.qs) {
+        load<E, V, VEC>(row + (size_t)(t - back) * p.ldr + x.col, x.e0, x.e1, u);
+      } else if (pos >= 0 && k.state >= 0) {
+        load<E, V, VEC>(ring + ((size_t)k.state * p.taps + pos % p.taps) * C + x.ch, x.e0, x.e1, u);
       } else {
-        for (int j = p.taps - 1; j >= 0; --j) {
-          float x[V], g[V];
-          input(k, t, j, x);
-          load<E, V, VEC>(w + (size_t)(p.taps - 1 - j) * C, e0, e1, g);
 #pragma unroll
-          for (int e = 0; e < V; ++e) y[e] = fmaf(g[e], x[e], y[e]);
+        for (int e = 0; e < V; ++e) u[e] = 0.f;
+      }
+    };
+    auto unpack = [&](const uint4& r, float (&u)[V]) {
+      const E* e = reinterpret_cast<const E*>(&r);
+#pragma unroll
+      for (int j = 0; j < V; ++j) u[j] = to_f(e[j]);
+    };
+    float hist[HB][V];                                     // hist[j]: input of j + 1 positions before
+    if constexpr (VEC && KM > 0) {
+#pragma unroll
+      for (int j = 0; j < HB; ++j) unpack(before[j], hist[j]);
+    }
+#pragma unroll 1
+    for (int g0 = 0; g0 < TT && t0 + g0 < p.T; g0 += GR) {
+      if constexpr (VEC) {
+        if (g0 > 0) {
+#pragma unroll
+          for (int i = 0; i < GR; ++i) raw[i] = request(t0 + g0 + i);
         }
       }
-      if (k.len == 1 && k.state >= 0)
-        store<E, V, VEC>(ring + ((size_t)k.state * p.taps + k.pos % p.taps) * C + ch, u[i], e0, e1);
-      if (rotated) {
 #pragma unroll
-        for (int e = 0; e < V; e += 2) {
-          // a pair never straddles two maps or the end of the rotated part, both are even
-          const int x = (d0 + e) % p.dim;
-          if (e + 1 < e1 && e >= e0 && x < 2 * p.pairs && x + 1 < p.dim) {
-            const float2 cs = turn[i * p.pairs + (x >> 1)];
-            const float a = y[e], b = y[e + 1];
-            y[e] = a * cs.x - b * cs.y;
-            y[e + 1] = b * cs.x + a * cs.y;
+    for (int gi = 0; gi < GR; ++gi) {
+      const int i = g0 + gi, t = t0 + i;
+      if (t >= p.T) break;
+      const Token k = tok[i];
+      float y[V], u[V];
+#pragma unroll
+      for (int e = 0; e < V; ++e) y[e] = u[e] = 0.f;
+      if (any && k.len > 0) {
+        if constexpr (VEC) unpack(raw[gi], u);
+        else load<E, V, VEC>(row + (size_t)t * p.ldr + x.col, x.e0, x.e1, u);
+        if constexpr (VEC && KM > 0) {
+          if (t - k.qs < KM - 1 && (i == 0 || t == k.qs)) {       // the window reaches back in front of the portion
+#pragma unroll
+            for (int j = 0; j < KM - 1; ++j)
+              if (j + 1 < p.taps && t - j - 1 < k.qs) input(k, t, j + 1, hist[j]);
+          }
+#pragma unroll
+          for (int j = KM - 2; j >= 0; --j) {
+            float g[V];
+            unpack(wt[j + 1], g);
+#pragma unroll
+            for (int e = 0; e < V; ++e) y[e] = fmaf(g[e], hist[j][e], y[e]);
+          }
+          float g[V];
+          unpack(wt[0], g);
+#pragma unroll
+          for (int e = 0; e < V; ++e) y[e] = fmaf(g[e], u[e], y[e]);
+#pragma unroll
+          for (int j = KM - 2; j > 0; --j)
+#pragma unroll
+            for (int e = 0; e < V; ++e) hist[j][e] = hist[j - 1][e];
+#pragma unroll
+          for (int e = 0; e < V; ++e) hist[0][e] = u[e];
+        } else {
+          for (int j = p.taps - 1; j >= 0; --j) {
+            float z[V], g[V];
+            input(k, t, j, z);
+            load<E, V, VEC>(w + (size_t)(p.taps - 1 - j) * C, x.e0, x.e1, g);
+#pragma unroll
+            for (int e = 0; e < V; ++e) y[e] = fmaf(g[e], z[e], y[e]);
+          }
+        }
+        if (k.len == 1 && k.state >= 0)
+          store<E, V, VEC>(ring + ((size_t)k.state * p.taps + k.pos % p.taps) * C + x.ch, u, x.e0, x.e1);
+        if (x.rotated) {
+          const int first = x.d0 % p.dim;                  // (of one map: heads with two are rotated in even maps only)
+#pragma unroll
+          for (int e = 0; e < V; e += 2) {
+            // a pair never straddles two maps or the end of the rotated part, both are even
+            int f = first + e;
+            if (f >= p.dim) f = (x.d0 + e) % p.dim;
+            if (e + 1 < x.e1 && e >= x.e0 && f < 2 * p.pairs && f + 1 < p.dim) {
+              const float2 cs = turn[i * p.pairs + (f >> 1)];
+              const float a = y[e], b = y[e + 1];
+              y[e] = a * cs.x - b * cs.y;
+              y[e + 1] = b * cs.x + a * cs.y;
+            }
           }
         }
       }
+      if (x.hh < nq) {
+        store<E, V, VEC>(reinterpret_cast<E*>(p.q_out) + ((size_t)t * nq + x.hh) * p.D + x.d0, y);
+      } else if (k.slot >= 0 && k.slot < p.num_slots) {
+        const long long blk = k.slot / p.block_size;
+        const int off = (int)(k.slot - blk * p.block_size);
+        store<E, V, VEC>(reinterpret_cast<E*>(p.cache) +
+                             ((size_t)(blk * 2 * p.G + x.hh - nq) * p.block_size + off) * p.D + x.d0, y);
+      }
     }
-    if (hh < nq) {
-      store<E, V, VEC>(reinterpret_cast<E*>(p.q_out) + ((size_t)t * nq + hh) * p.D + d0, y);
-    } else if (k.slot >= 0 && k.slot < p.num_slots) {
-      const long long blk = k.slot / p.block_size;
-      const int off = (int)(k.slot - blk * p.block_size);
-      store<E, V, VEC>(reinterpret_cast<E*>(p.cache) + ((size_t)(blk * 2 * p.G + hh - nq) * p.block_size + off) * p.D + d0,
-                       y);
     }
   }
 }
@@ -232,8 +281,6 @@ __global__ void __launch_bounds__(256) conv_cache_kernel(const Params p) {
 // The last inputs of every portion from request `first` on.  grid (channels / 256, requests)
 template <typename E>
 __global__ void ring_kernel(const Params p, int first) {
-  pdl_launch_dependents();
-  pdl_wait();
   const int r = first + blockIdx.y, qs = p.qsl[r], len = p.qsl[r + 1] - qs, slot = p.state_slots[r];
   const int cq = p.H * p.maps * p.dim, ck = p.G * p.maps * p.dim, C = cq + ck + p.G * p.vdim;
   const int c = blockIdx.x * blockDim.x + threadIdx.x;
@@ -245,12 +292,15 @@ __global__ void ring_kernel(const Params p, int first) {
         reinterpret_cast<const E*>(p.row)[(size_t)(qs + pos - start) * p.ldr + col];
 }
 
+// Launched in stream order, without programmatic overlap with the kernels around them.
 template <typename E, int V, bool VEC, int KM, int TT>
 static int launch_conv(const Params& p, cudaStream_t stream) {
   const int vecs = (p.H * p.maps + 2 * p.G) * (p.D / V), threads = vecs < 256 ? (vecs + 31) / 32 * 32 : 256;
-  const dim3 grid((p.T + TT - 1) / TT, (vecs + threads - 1) / threads);
-  B200_CUDA_CHECK(launch_pdl(conv_cache_kernel<E, V, VEC, KM, TT>, grid, dim3(threads),
-                             (size_t)TT * p.pairs * sizeof(float2), stream, p));
+  const int runs = (p.T + TT - 1) / TT, most = (vecs + threads - 1) / threads;
+  int parts = (4 * 148 + runs - 1) / runs;                 // enough CTAs for every SM, else one over all vectors
+  parts = parts > most ? most : parts;
+  conv_cache_kernel<E, V, VEC, KM, TT><<<dim3(runs, parts), threads, (size_t)TT * p.pairs * sizeof(float2), stream>>>(p);
+  B200_CUDA_CHECK(cudaGetLastError());
   return 0;
 }
 
@@ -265,13 +315,13 @@ static int launch(const Params& p, int ring_from, int only_ring, int single, cud
     if (!vec) rc = launch_conv<E, 2, false, 0, 4>(p, stream);
     else if (p.taps > 4) rc = launch_conv<E, V, true, 0, 4>(p, stream);
     else if (single) rc = launch_conv<E, V, true, 4, 1>(p, stream);
-    else rc = launch_conv<E, V, true, 4, 8>(p, stream);
+    else rc = launch_conv<E, V, true, 4, 16>(p, stream);
     if (rc) return rc;
   }
   if (ring_from < p.R && p.taps > 1) {
     const int C = p.H * p.maps * p.dim + p.G * (p.maps * p.dim + p.vdim);
-    B200_CUDA_CHECK(launch_pdl(ring_kernel<E>, dim3((C + 255) / 256, p.R - ring_from), dim3(256), (size_t)0, stream, p,
-                               ring_from));
+    ring_kernel<E><<<dim3((C + 255) / 256, p.R - ring_from), 256, 0, stream>>>(p, ring_from);
+    B200_CUDA_CHECK(cudaGetLastError());
   }
   return 0;
 }
@@ -289,8 +339,6 @@ struct CombineParams {
 // One warp per token and head, at most NV vectors per lane.
 template <typename E, int V, bool VEC, int NV>
 __global__ void __launch_bounds__(256) combine_kernel(const CombineParams p) {
-  pdl_launch_dependents();
-  pdl_wait();
   const long long n = (long long)blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
   const int lane = threadIdx.x & 31;
   if (n >= p.rows) return;
@@ -338,9 +386,10 @@ static int launch_combine(const CombineParams& p, cudaStream_t stream) {
   constexpr int V = 16 / sizeof(E);
   const dim3 grid((unsigned)((p.rows + 7) / 8)), block(256);
   const bool vec = ((uintptr_t)p.a | (uintptr_t)p.out) % 16 == 0 && p.D % V == 0;
-  if (vec && p.D <= 32 * V) B200_CUDA_CHECK(launch_pdl(combine_kernel<E, V, true, 1>, grid, block, (size_t)0, stream, p));
-  else if (vec && p.D <= 128 * V) B200_CUDA_CHECK(launch_pdl(combine_kernel<E, V, true, 4>, grid, block, (size_t)0, stream, p));
-  else B200_CUDA_CHECK(launch_pdl(combine_kernel<E, 2, false, 8>, grid, block, (size_t)0, stream, p));
+  if (vec && p.D <= 32 * V) combine_kernel<E, V, true, 1><<<grid, block, 0, stream>>>(p);
+  else if (vec && p.D <= 128 * V) combine_kernel<E, V, true, 4><<<grid, block, 0, stream>>>(p);
+  else combine_kernel<E, 2, false, 8><<<grid, block, 0, stream>>>(p);
+  B200_CUDA_CHECK(cudaGetLastError());
   return 0;
 }
 

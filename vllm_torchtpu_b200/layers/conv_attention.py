@@ -94,18 +94,21 @@ class ConvAttention(GroupedAttention):
         ops.conv_ring_update(self.plan, inputs[0], cache[0], meta)
 
     def forward(self, x, cache, meta):
-        s, T = self.spec, x.shape[0]
+        T = x.shape[0]
         ring, pages = cache
         row = self.inp(x)
         rb = getattr(meta, "state_rollback", None)
         if rb is not None:
             rb.capture(self, (ring,), (row,))      # verification step: rejected drafts are rolled back later
         q = ops.conv_and_cache(self.plan, row, pages, ring, meta)
-        o = ops.paged_attention(q, pages, meta, s.scale, sliding_window=s.window)
-        gate = None
+        return self.o(self.attend(q, row, pages, meta).reshape(T, self.Hq * self.D))
+
+    def attend(self, q, row, pages, meta):
+        """Softmax over the window and what follows it: [T, heads, D]."""
+        s, gate = self.spec, None
         if s.output_gate:
             at = self.inp.offset["g"]
             gate = row[:, at:at + self.Hq * s.vdim]
-        if gate is not None or s.maps == 2:
-            o = ops.combine_heads(o, s.vdim, gate, self.lam, s.diff, self.eps)
-        return self.o(o.reshape(T, self.Hq * self.D))
+        if gate is None and s.maps == 1:
+            return ops.paged_attention(q, pages, meta, s.scale, sliding_window=s.window)
+        return ops.paged_attention_heads(q, pages, meta, s.scale, s.window, s.vdim, gate, self.lam, s.diff, self.eps)

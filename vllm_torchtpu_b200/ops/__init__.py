@@ -138,6 +138,14 @@ def conv_ring_update(plan, row, ring, meta):
     return f(plan, row, ring, meta)
 
 
+def paged_attention_heads(q, kv_cache, meta, scale, window, vdim, gate=None, lam=None, diff=0.0, eps=0.0):
+    """Paged attention over a window and ``combine_heads`` behind it, in the attention kernels' epilogue where they have
+    it: [T, heads, width]."""
+    if _on_gpu(q):
+        return cuda_ops().paged_attention_heads(q, kv_cache, meta, scale, window, vdim, gate, lam, diff, eps)
+    return combine_heads(paged_attention(q, kv_cache, meta, scale, sliding_window=window), vdim, gate, lam, diff, eps)
+
+
 def combine_heads(a, vdim, gate=None, lam=None, diff=0.0, eps=0.0):
     """Difference of two softmax maps with its norm, output gate; see ``ops.short_conv``."""
     if _on_gpu(a):

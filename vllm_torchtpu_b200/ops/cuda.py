@@ -966,7 +966,7 @@ _SUBMODULE_EXPORTS = {
                  "moe_experts_fp8", "quant_act_1x128", "quant_act_int8", "quant_rows_1x128"),
     "cuda_fp4": ("grouped_w4a16_gemm", "moe_experts_w4a16", "w4a16_gemm", "w4a16_int4_gemm", "dequant_w4", "dequant_int4"),
     "cuda_gdn": ("gdn_forward", "kda_forward", "short_conv"),
-    "cuda_conv": ("combine_heads", "conv_and_cache", "conv_ring_update"),
+    "cuda_conv": ("combine_heads", "conv_and_cache", "conv_ring_update", "paged_attention_heads"),
     "cuda_linear": ("carried_state_attention",),
     "cuda_mla": ("latent_prep", "mla_absorb", "mla_paged_attention", "mla_unabsorb", "mla_write_cache", "permute_rows", "rope_heads_into",
                  "rope_rows"),

@@ -97,20 +97,23 @@ class UnquantizedMoEMethod:
         from ..layers.linear import seeded_normal
         E, I, H = moe.num_experts, moe.intermediate_size, moe.hidden_size
         lo, hi = moe.expert_range
+        if not moe.gated:
+            self.alloc(moe)
+            for e in range(lo, hi):
+                pre, full = f"{moe.name}.experts.{e}", I * moe.tp_size
+                self.load_expert(moe, e - lo, None,
+                                 seeded_normal(f"{pre}.up", (full, H), std, moe.dtype, moe.device, seed),
+                                 seeded_normal(f"{pre}.down", (H, full), std, moe.dtype, moe.device, seed))
+            return
         w13 = []
         w2 = []
         for e in range(lo, hi):
-            w13.append(seeded_normal(f"{moe.name}.experts.{e}.w13", (2 * I if moe.gated else I, H), std, moe.dtype,
-                                     moe.device, seed))
+            w13.append(seeded_normal(f"{moe.name}.experts.{e}.w13", (2 * I, H), std, moe.dtype, moe.device, seed))
             w2.append(seeded_normal(f"{moe.name}.experts.{e}.w2", (H, I), std, moe.dtype, moe.device, seed))
         moe.w13 = torch.stack(w13).contiguous()
         moe.w2 = torch.stack(w2).contiguous()
         if padded_hidden(moe) != H:
             moe.w2 = torch.nn.functional.pad(moe.w2, (0, 0, 0, padded_hidden(moe) - H)).contiguous()
-        if padded_inter(moe) != I:
-            more = padded_inter(moe) - I
-            moe.w13 = torch.nn.functional.pad(moe.w13, (0, 0, 0, more)).contiguous()
-            moe.w2 = torch.nn.functional.pad(moe.w2, (0, more)).contiguous()
 
     def load_expert(self, moe, local_e, gate, up, down, scales=(None, None, None)) -> None:
         """Unsharded checkpoint matrices of one expert (``gate`` None: ungated); the intermediate dimension is sliced
