@@ -404,6 +404,15 @@ struct HeadFinish {
 template <int N>
 __device__ __forceinline__ void gate_columns(const HeadFinish& f, long long t, int head, int col, float* v) {
   const __nv_bfloat16* g = f.gate + (size_t)t * f.ldg + (size_t)head * f.vdim + col;
+  if ((reinterpret_cast<uintptr_t>(g) & 15) == 0 && col + N <= f.vdim) {
+    uint4 raw[N / 8];
+#pragma unroll
+    for (int i = 0; i < N / 8; ++i) raw[i] = reinterpret_cast<const uint4*>(g)[i];
+#pragma unroll
+    for (int i = 0; i < N; ++i)
+      v[i] = __fdividef(v[i], 1.f + __expf(-__bfloat162float(reinterpret_cast<const __nv_bfloat16*>(raw)[i])));
+    return;
+  }
 #pragma unroll
   for (int i = 0; i < N; ++i)
     if (col + i < f.vdim) v[i] = __fdividef(v[i], 1.f + __expf(-__bfloat162float(g[i])));

@@ -36,31 +36,40 @@ struct Params {
 
 struct Token {
   int qs, len, pos, state;             // first row and length of its portion, position, state slot (-1: none)
-  long long slot;
+  long long cell;                      // element of the cache where its first key head begins (-1: not cached)
 };
 
-// request of row t: qsl is monotone and repeats its last value behind the last request
-__device__ __forceinline__ Token token_of(const Params& p, int t) {
+// request of row t, by a whole warp: as many requests as end at t or before (qsl is monotone and repeats its last value
+// behind the last request)
+__device__ __forceinline__ Token token_of(const Params& p, int t, int lane) {
+  int r = 0;
+  for (int i = lane; i < p.R + lane; i += 32)
+    r += __popc(__ballot_sync(0xffffffffu, i < p.R && p.qsl[min(i, p.R - 1) + 1] <= t));
   Token k{t, 0, 0, -1, -1};
-  if (t >= p.T || t >= p.qsl[p.R]) return k;
-  int lo = 0, hi = p.R;                // qsl[lo] <= t < qsl[hi]
-  while (hi - lo > 1) {
-    const int mid = (lo + hi) >> 1;
-    if (p.qsl[mid] <= t) lo = mid;
-    else hi = mid;
+  if (t >= p.T || r >= p.R) return k;
+  k.qs = p.qsl[r];
+  k.len = p.qsl[r + 1] - k.qs;
+  k.pos = p.seq_lens[r] - k.len + t - k.qs;
+  k.state = p.state_slots[r];
+  const long long slot = p.slots[t];
+  if (p.G > 0 && slot >= 0 && slot < p.num_slots) {
+    const long long blk = slot / p.block_size;
+    k.cell = (blk * 2 * p.G * p.block_size + slot - blk * p.block_size) * p.D;
   }
-  k.qs = p.qsl[lo];
-  k.len = p.qsl[lo + 1] - k.qs;
-  k.pos = p.seq_lens[lo] - k.len + t - k.qs;
-  k.state = p.state_slots[lo];
-  k.slot = p.slots[t];
   return k;
 }
+
+// V elements as they lie in memory
+template <int BYTES> struct Pack;
+template <> struct Pack<16> { typedef uint4 type; };
+template <> struct Pack<8> { typedef uint2 type; };
+template <> struct Pack<4> { typedef uint32_t type; };
+template <typename E, int V> using PackOf = typename Pack<V * sizeof(E)>::type;
 
 template <typename E, int V, bool VEC>
 __device__ __forceinline__ void load(const E* p, int e0, int e1, float (&v)[V]) {
   if constexpr (VEC) {
-    const uint4 u = *reinterpret_cast<const uint4*>(p);
+    const PackOf<E, V> u = *reinterpret_cast<const PackOf<E, V>*>(p);
     const E* e = reinterpret_cast<const E*>(&u);
 #pragma unroll
     for (int j = 0; j < V; ++j) v[j] = to_f(e[j]);
@@ -72,17 +81,19 @@ __device__ __forceinline__ void load(const E* p, int e0, int e1, float (&v)[V]) 
 template <typename E, int V, bool VEC>
 __device__ __forceinline__ void store(E* p, const float (&v)[V], int e0 = 0, int e1 = V) {
   if constexpr (VEC) {
-    uint4 u;
+    PackOf<E, V> u;
     E* e = reinterpret_cast<E*>(&u);
 #pragma unroll
     for (int j = 0; j < V; ++j) put(e + j, v[j]);
-    *reinterpret_cast<uint4*>(p) = u;
+    *reinterpret_cast<PackOf<E, V>*>(p) = u;
   } else {
 #pragma unroll
     for (int j = 0; j < V; ++j)
       if (j >= e0 && j < e1) put(p + j, v[j]);
   }
 }
+
+constexpr int THREADS = 128;
 
 // The channels that vector `vec` of the stored heads takes: row column and ring channel of its element 0 (elements e0 ..
 // e1 - 1 exist, the others are zeros), head index (q rows, then k, then v heads) and first column in the head.
@@ -121,50 +132,48 @@ __device__ __forceinline__ Where where_is(const Params& p, int vec) {
   return w;
 }
 
-// grid (token runs of TT, parts of the vectors).  KM: taps the window is held in registers for (0: any number, re-read).
-// A run is walked in groups of up to four tokens whose inputs are requested together; the inputs in front of the run are
-// requested before the tokens' requests are known, and what turns out to belong to another portion is replaced.
+// grid (token runs of TT, parts of the vectors).  A run within one portion, as most are, takes the way with the window in
+// registers (at most KM taps, 0: none do): the inputs of the next four tokens are on their way at any time, and the first
+// ones are requested before the tokens' portion is known.  Other runs read every input where it lies.
 template <typename E, int V, bool VEC, int KM, int TT>
-__global__ void __launch_bounds__(256, 2) conv_cache_kernel(const Params p) {
+__global__ void __launch_bounds__(THREADS, 4) conv_cache_kernel(const Params p) {
   extern __shared__ __align__(16) float2 turn[];          // [TT][pairs]
   __shared__ Token tok[TT];
   const int tid = threadIdx.x, t0 = blockIdx.x * TT;
   const int nq = p.H * p.maps, C = (nq + p.G * p.maps) * p.dim + p.G * p.vdim, vecs = (nq + 2 * p.G) * (p.D / V);
   const E* row = reinterpret_cast<const E*>(p.row);
   E* ring = reinterpret_cast<E*>(p.ring);
-  constexpr int HB = KM > 1 ? KM - 1 : 1;
-  bool ready = false;
-  for (int v0 = blockIdx.y * blockDim.x; v0 < vecs; v0 += gridDim.y * blockDim.x) {
+  constexpr int HB = KM > 1 ? KM - 1 : 1, GR = TT < 4 ? TT : 4;
+  typedef PackOf<E, V> Raw;
+  bool ready = false, whole = false;
+  for (int v0 = blockIdx.y * THREADS; v0 < vecs; v0 += gridDim.y * THREADS) {
     const int vec = v0 + tid;
     const Where x = where_is<V>(p, min(vec, vecs - 1));
     const bool any = x.e0 < x.e1 && vec < vecs;
     const E* w = reinterpret_cast<const E*>(p.w) + x.ch;
-    constexpr int GR = TT < 4 ? TT : 4;
-    uint4 raw[GR], before[HB];                             // inputs of a group and of the rows in front of the run
-    uint4 wt[VEC && KM > 0 ? KM : 1];                      // wt[j]: weights of the inputs j positions before
-    auto request = [&](int t) {
-      return any && t >= 0 && t < p.T ? *reinterpret_cast<const uint4*>(row + (size_t)t * p.ldr + x.col)
-                                      : make_uint4(0u, 0u, 0u, 0u);
+    const E* col = row + x.col;
+    Raw raw[GR];                                           // inputs of the next tokens
+    float wt[KM > 0 ? KM : 1][V], hist[HB][V];             // weight of, and the input itself, j (+ 1) positions before
+    auto request = [&](int t) { return any && t < p.T ? *reinterpret_cast<const Raw*>(col + (size_t)t * p.ldr) : Raw(); };
+    auto unpack = [&](const Raw& r, float (&u)[V]) {
+      const E* e = reinterpret_cast<const E*>(&r);
+#pragma unroll
+      for (int j = 0; j < V; ++j) u[j] = to_f(e[j]);
     };
-    if constexpr (VEC) {
-#pragma unroll
-      for (int i = 0; i < GR; ++i) raw[i] = request(t0 + i);
-      if constexpr (KM > 0) {
-#pragma unroll
-        for (int i = 0; i < HB; ++i) before[i] = request(t0 - 1 - i);
-      }
-    }
     if constexpr (VEC && KM > 0) {
 #pragma unroll
-      for (int j = 0; j < KM; ++j) {
-        wt[j] = make_uint4(0u, 0u, 0u, 0u);
-        if (any && j < p.taps) wt[j] = *reinterpret_cast<const uint4*>(w + (size_t)(p.taps - 1 - j) * C);
-      }
+      for (int i = 0; i < GR; ++i) raw[i] = request(t0 + i);
+#pragma unroll
+      for (int j = 0; j < KM; ++j)
+        unpack(any && j < p.taps ? *reinterpret_cast<const Raw*>(w + (size_t)(p.taps - 1 - j) * C) : Raw(), wt[j]);
     }
     if (!ready) {                                          // uniform over the CTA
-      if (tid < TT) tok[tid] = token_of(p, t0 + tid);
+      for (int i = tid >> 5; i < TT; i += THREADS / 32) {
+        const Token k = token_of(p, t0 + i, tid & 31);
+        if ((tid & 31) == 0) tok[i] = k;
+      }
       __syncthreads();
-      for (int i = tid; i < TT * p.pairs; i += blockDim.x) {
+      for (int i = tid; i < TT * p.pairs; i += THREADS) {
         const int k = i / p.pairs;
         float sn, cs;
         sincosf((float)tok[k].pos * p.inv_freq[i - k * p.pairs], &sn, &cs);
@@ -172,13 +181,15 @@ __global__ void __launch_bounds__(256, 2) conv_cache_kernel(const Params p) {
       }
       __syncthreads();
       ready = true;
+      whole = tok[0].len > 0 && tok[TT - 1].len > 0 && tok[TT - 1].qs == tok[0].qs;
     }
     if (vec >= vecs) continue;
+    const int first = x.d0 % p.dim;                        // index of element 0 within its map
     // input of position pos - back for the token with info k in row t
     auto input = [&](const Token& k, int t, int back, float (&u)[V]) {
       const int pos = k.pos - back;
       if (pos >= 0 && t - back >= k.qs) {
-        load<E, V, VEC>(row + (size_t)(t - back) * p.ldr + x.col, x.e0, x.e1, u);
+        load<E, V, VEC>(col + (size_t)(t - back) * p.ldr, x.e0, x.e1, u);
       } else if (pos >= 0 && k.state >= 0) {
         load<E, V, VEC>(ring + ((size_t)k.state * p.taps + pos % p.taps) * C + x.ch, x.e0, x.e1, u);
       } else {
@@ -186,71 +197,88 @@ __global__ void __launch_bounds__(256, 2) conv_cache_kernel(const Params p) {
         for (int e = 0; e < V; ++e) u[e] = 0.f;
       }
     };
-    auto unpack = [&](const uint4& r, float (&u)[V]) {
-      const E* e = reinterpret_cast<const E*>(&r);
-#pragma unroll
-      for (int j = 0; j < V; ++j) u[j] = to_f(e[j]);
-    };
-    float hist[HB][V];                                     // hist[j]: input of j + 1 positions before
-    if constexpr (VEC && KM > 0) {
-#pragma unroll
-      for (int j = 0; j < HB; ++j) unpack(before[j], hist[j]);
-    }
-#pragma unroll 1
-    for (int g0 = 0; g0 < TT && t0 + g0 < p.T; g0 += GR) {
-      if constexpr (VEC) {
-        if (g0 > 0) {
-#pragma unroll
-          for (int i = 0; i < GR; ++i) raw[i] = request(t0 + g0 + i);
-        }
+    E* q_out = reinterpret_cast<E*>(p.q_out) + ((size_t)t0 * nq + x.hh) * p.D + x.d0;
+    E* cache = reinterpret_cast<E*>(p.cache) + (size_t)(x.hh - nq) * p.block_size * p.D + x.d0;
+    const size_t q_step = (size_t)nq * p.D;
+    const bool is_q = x.hh < nq;
+    auto save = [&](int i, const float (&y)[V]) {          // (a thread's rows of q are written in order)
+      if (is_q) {
+        store<E, V, VEC>(q_out, y);
+        q_out += q_step;
+      } else if (tok[i].cell >= 0) {
+        store<E, V, VEC>(cache + tok[i].cell, y);
       }
+    };
+    if constexpr (VEC && KM > 0) {
+      if (whole) {
+        const int turns = x.rotated && any ? min(max(p.pairs - (first >> 1), 0), V / 2) : 0;   // pairs that rotate
+        const Token k = tok[0];
 #pragma unroll
-    for (int gi = 0; gi < GR; ++gi) {
-      const int i = g0 + gi, t = t0 + i;
-      if (t >= p.T) break;
-      const Token k = tok[i];
-      float y[V], u[V];
+        for (int j = 0; j < HB; ++j) {
+          if (any && KM > 1 && j + 1 < p.taps) {
+            input(k, t0, j + 1, hist[j]);
+          } else {
 #pragma unroll
-      for (int e = 0; e < V; ++e) y[e] = u[e] = 0.f;
-      if (any && k.len > 0) {
-        if constexpr (VEC) unpack(raw[gi], u);
-        else load<E, V, VEC>(row + (size_t)t * p.ldr + x.col, x.e0, x.e1, u);
-        if constexpr (VEC && KM > 0) {
-          if (t - k.qs < KM - 1 && (i == 0 || t == k.qs)) {       // the window reaches back in front of the portion
+            for (int e = 0; e < V; ++e) hist[j][e] = 0.f;
+          }
+        }
+#pragma unroll 1
+        for (int g0 = 0; g0 < TT; g0 += GR) {
+          const E* ahead = col + (size_t)(t0 + g0 + GR) * p.ldr;
+#pragma unroll
+          for (int gi = 0; gi < GR; ++gi) {
+            float u[V], y[V];
+            unpack(raw[gi], u);
+            if (TT > GR && any && g0 + GR < TT) raw[gi] = *reinterpret_cast<const Raw*>(ahead + (size_t)gi * p.ldr);
+#pragma unroll
+            for (int e = 0; e < V; ++e) y[e] = wt[0][e] * u[e];
 #pragma unroll
             for (int j = 0; j < KM - 1; ++j)
-              if (j + 1 < p.taps && t - j - 1 < k.qs) input(k, t, j + 1, hist[j]);
-          }
 #pragma unroll
-          for (int j = KM - 2; j >= 0; --j) {
-            float g[V];
-            unpack(wt[j + 1], g);
+              for (int e = 0; e < V; ++e) y[e] = fmaf(wt[j + 1][e], hist[j][e], y[e]);
 #pragma unroll
-            for (int e = 0; e < V; ++e) y[e] = fmaf(g[e], hist[j][e], y[e]);
-          }
-          float g[V];
-          unpack(wt[0], g);
+            for (int j = KM - 2; j > 0; --j)
 #pragma unroll
-          for (int e = 0; e < V; ++e) y[e] = fmaf(g[e], u[e], y[e]);
+              for (int e = 0; e < V; ++e) hist[j][e] = hist[j - 1][e];
 #pragma unroll
-          for (int j = KM - 2; j > 0; --j)
+            for (int e = 0; e < V; ++e) hist[0][e] = u[e];
+            if (TT == 1 && any && k.len == 1 && k.state >= 0)
+              store<E, V, VEC>(ring + ((size_t)k.state * p.taps + k.pos % p.taps) * C + x.ch, u);
+            if (turns > 0) {
+              const float2* cs = turn + (g0 + gi) * p.pairs + (first >> 1);
 #pragma unroll
-            for (int e = 0; e < V; ++e) hist[j][e] = hist[j - 1][e];
-#pragma unroll
-          for (int e = 0; e < V; ++e) hist[0][e] = u[e];
-        } else {
-          for (int j = p.taps - 1; j >= 0; --j) {
-            float z[V], g[V];
-            input(k, t, j, z);
-            load<E, V, VEC>(w + (size_t)(p.taps - 1 - j) * C, x.e0, x.e1, g);
-#pragma unroll
-            for (int e = 0; e < V; ++e) y[e] = fmaf(g[e], z[e], y[e]);
+              for (int e = 0; e < V; e += 2)
+                if ((e >> 1) < turns) {
+                  const float2 c = cs[e >> 1];
+                  const float a = y[e], b = y[e + 1];
+                  y[e] = a * c.x - b * c.y;
+                  y[e + 1] = b * c.x + a * c.y;
+                }
+            }
+            save(g0 + gi, y);
           }
         }
-        if (k.len == 1 && k.state >= 0)
-          store<E, V, VEC>(ring + ((size_t)k.state * p.taps + k.pos % p.taps) * C + x.ch, u, x.e0, x.e1);
+        continue;
+      }
+    }
+#pragma unroll 1
+    for (int i = 0; i < TT && t0 + i < p.T; ++i) {
+      const Token k = tok[i];
+      float y[V];
+#pragma unroll
+      for (int e = 0; e < V; ++e) y[e] = 0.f;
+      if (any && k.len > 0) {
+#pragma unroll 1
+        for (int j = p.taps - 1; j >= 0; --j) {
+          float z[V], g[V];
+          input(k, t0 + i, j, z);
+          load<E, V, VEC>(w + (size_t)(p.taps - 1 - j) * C, x.e0, x.e1, g);
+#pragma unroll
+          for (int e = 0; e < V; ++e) y[e] = fmaf(g[e], z[e], y[e]);
+          if (j == 0 && k.len == 1 && k.state >= 0)
+            store<E, V, VEC>(ring + ((size_t)k.state * p.taps + k.pos % p.taps) * C + x.ch, z, x.e0, x.e1);
+        }
         if (x.rotated) {
-          const int first = x.d0 % p.dim;                  // (of one map: heads with two are rotated in even maps only)
 #pragma unroll
           for (int e = 0; e < V; e += 2) {
             // a pair never straddles two maps or the end of the rotated part, both are even
@@ -265,15 +293,7 @@ __global__ void __launch_bounds__(256, 2) conv_cache_kernel(const Params p) {
           }
         }
       }
-      if (x.hh < nq) {
-        store<E, V, VEC>(reinterpret_cast<E*>(p.q_out) + ((size_t)t * nq + x.hh) * p.D + x.d0, y);
-      } else if (k.slot >= 0 && k.slot < p.num_slots) {
-        const long long blk = k.slot / p.block_size;
-        const int off = (int)(k.slot - blk * p.block_size);
-        store<E, V, VEC>(reinterpret_cast<E*>(p.cache) +
-                             ((size_t)(blk * 2 * p.G + x.hh - nq) * p.block_size + off) * p.D + x.d0, y);
-      }
-    }
+      save(i, y);
     }
   }
 }
@@ -295,11 +315,11 @@ __global__ void ring_kernel(const Params p, int first) {
 // Launched in stream order, without programmatic overlap with the kernels around them.
 template <typename E, int V, bool VEC, int KM, int TT>
 static int launch_conv(const Params& p, cudaStream_t stream) {
-  const int vecs = (p.H * p.maps + 2 * p.G) * (p.D / V), threads = vecs < 256 ? (vecs + 31) / 32 * 32 : 256;
-  const int runs = (p.T + TT - 1) / TT, most = (vecs + threads - 1) / threads;
-  int parts = (4 * 148 + runs - 1) / runs;                 // enough CTAs for every SM, else one over all vectors
-  parts = parts > most ? most : parts;
-  conv_cache_kernel<E, V, VEC, KM, TT><<<dim3(runs, parts), threads, (size_t)TT * p.pairs * sizeof(float2), stream>>>(p);
+  const int vecs = (p.H * p.maps + 2 * p.G) * (p.D / V), most = (vecs + THREADS - 1) / THREADS;
+  const int runs = (p.T + TT - 1) / TT;
+  int parts = 1;                                           // even shares of the vectors, enough CTAs for every SM
+  while (parts < most && (most % parts || (long long)parts * runs < 12 * 148)) ++parts;
+  conv_cache_kernel<E, V, VEC, KM, TT><<<dim3(runs, parts), THREADS, (size_t)TT * p.pairs * sizeof(float2), stream>>>(p);
   B200_CUDA_CHECK(cudaGetLastError());
   return 0;
 }
