@@ -26,12 +26,12 @@ EXPERTS, TOP, FF, GATED_FF = 32, 4, 1152, 768
 def zeganex_config(width: int, heads: int, kind: str, layers: int = 4) -> ModelConfig:
     mix = {"heads": heads, "kv_heads": heads // 4, "vdim": D, "conv": TAPS, "mask": {"size": WINDOW}}
     mixer = {"attention": dict(mix, dim=D // 2, scale=(D // 2) ** -0.5, diff=0.4),
-             "attention_2": dict(mix, dim=D, scale=D ** -0.5, rot={"base": 50000.0, "dims": D // 2, "scaling": {
+             "attention_2": dict(mix, dim=D, scale=D ** -0.5, rot={"base": 10000.0, "dims": D // 2, "scaling": {
                  "factor": 4.0, "original": 4096, "fast": 32.0, "slow": 1.0}})}[kind]
     mlp = {"kind": "moe", "router": {"experts": EXPERTS, "top": TOP}, "expert": {"ff": FF}}
     return ModelConfig.from_layer_list({
         "architecture": "Zeganex", "width": width, "vocab": 1024, "norm": {"eps": 1e-6}, "residual_mult": 0.5,
-        "embedding": {"bigram": {"buckets": 4099, "mul_prev": 31, "mul_cur": 17}},
+        "embedding": {"bigram": {"buckets": 4099, "mul_prev": 29, "mul_cur": 13}},
         "layers": [{"type": kind, "mixer": mixer, "mlp": mlp}] * layers}, "zeganex-bench")
 
 
@@ -128,7 +128,7 @@ def _pairs(width: int, heads: int, step: str):
     table, pairs = rnd(8192, width), rnd(4100, width)
     tok = torch.randint(0, 8192, (T,), device="cuda", dtype=torch.int32)
     src, last = torch.full((T,), -1, dtype=torch.int32, device="cuda"), torch.zeros(reqs, dtype=torch.int32, device="cuda")
-    yield "embedding", lambda: cuda.embedding_pairs(tok, tok, table, pairs, (4099, 31, 17), src, last, last.clone()), 0.0, \
+    yield "embedding", lambda: cuda.embedding_pairs(tok, tok, table, pairs, (4099, 29, 13), src, last, last.clone()), 0.0, \
         T * width * 8.0, lambda: cuda.embedding(tok, table), 0.0, T * width * 4.0
     if step == "decode":
         V = 128256
