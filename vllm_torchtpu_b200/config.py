@@ -11,13 +11,13 @@ from __future__ import annotations
 
 import json
 import os
-from dataclasses import dataclass, field, asdict
+from dataclasses import dataclass, field, asdict, replace
 from typing import Any, Optional
 
 import torch
 
-from .layer_specs import (DeltaMixerSpec, GroupedMixerSpec, LatentMixerSpec, LayerSpec, RetentionMixerSpec,  # noqa: F401
-                          RotarySpec, layer_specs)
+from .layer_specs import (DeltaMixerSpec, ExpertsSpec, GlaMixerSpec, GroupedMixerSpec, LatentMixerSpec,  # noqa: F401
+                          LayerSpec, ParallelMixerSpec, RetentionMixerSpec, RotarySpec, layer_specs)
 
 _DTYPES = {
     "float32": torch.float32, "fp32": torch.float32, "float": torch.float32,
@@ -34,7 +34,7 @@ def parse_dtype(d) -> torch.dtype:
 
 @dataclass
 class ModelConfig:
-    architecture: str = "llama"          # llama | qwen3_moe | gpt_oss | deepseek_v3 | qwen3_next | kimi_linear | mazivik | popanex | zeganex
+    architecture: str = "llama"          # llama | qwen3_moe | gpt_oss | deepseek_v3 | qwen3_next | kimi_linear | mazivik | popanex | zeganex | vipolix
     name: str = "tiny-llama"
     num_layers: int = 2
     hidden_size: int = 256
@@ -67,6 +67,7 @@ class ModelConfig:
     num_shared_experts: int = 0
     shared_expert_intermediate_size: int = 0   # 0: moe_intermediate_size x num_shared_experts
     shared_expert_gate: bool = False           # shared expert output scaled by sigmoid(x . w) (Qwen2-MoE, Qwen3-Next)
+    shared_expert_act: str = ""                # activation of the shared expert; "": hidden_act
     first_dense_layers: int = 0          # leading layers with a dense FFN
     moe_scoring: str = "softmax"         # softmax | sigmoid
     moe_renormalize: bool = True
@@ -87,6 +88,7 @@ class ModelConfig:
     logit_scale: float = 1.0             # logits = scale * (head x)
     bigram: Optional[tuple] = None       # (buckets, mul_prev, mul_cur) of an embedding of (previous token, token)
     residual_mult: float = 1.0           # factor on the normalised sublayer outputs
+    token_side_dim: int = 0              # width of one layer's part of the per-layer token embedding (0: none)
     # sparse MLA (DSA indexer)
     index_topk: int = 0
     index_n_heads: int = 0
@@ -119,7 +121,7 @@ class ModelConfig:
     @property
     def has_recurrent_state(self) -> bool:
         """Some layers carry a state per request instead of a KV cache."""
-        return self.full_attention_interval > 0 or any(s.mixer.carries_state for s in self.layer_specs)
+        return self.full_attention_interval > 0 or any(s.carries_state for s in self.layer_specs)
 
     def layer_is_moe(self, i: int) -> bool:
         return self.is_moe and i >= self.first_dense_layers
@@ -163,7 +165,7 @@ class ModelConfig:
     @staticmethod
     def from_hf_dict(cfg: dict, name: str = "") -> "ModelConfig":
         """Map a Hugging Face ``config.json`` dictionary to ModelConfig."""
-        if "architectures" not in cfg and cfg.get("architecture") in ("Mazivik", "Popanex", "Zeganex"):
+        if "architectures" not in cfg and cfg.get("architecture") in LAYER_LIST_DESIGNS:
             return ModelConfig.from_layer_list(cfg, name)
         arch = (cfg.get("architectures") or ["LlamaForCausalLM"])[0]
         mc = ModelConfig(name=name or cfg.get("_name_or_path", arch))
@@ -318,10 +320,10 @@ class ModelConfig:
 
     @staticmethod
     def from_layer_list(cfg: dict, name: str = "") -> "ModelConfig":
-        """Map a ``config.json`` that lists its layers one by one (``{"architecture": "Mazivik" | "Popanex" |
-        "Zeganex", "layers": [...], "norm": {"eps"}, "vocab", "width", ...}``) to ModelConfig."""
+        """Map a ``config.json`` that lists its layers one by one (``{"architecture": a key of
+        LAYER_LIST_DESIGNS, "layers": [...], "norm": {"eps"}, "vocab", "width", ...}``) to ModelConfig."""
         arch = cfg["architecture"].lower()
-        build = {"mazivik": _mazivik_layers, "popanex": _popanex_layers, "zeganex": _zeganex_layers}[arch]
+        build = LAYER_LIST_DESIGNS[cfg["architecture"]]
         mc = ModelConfig(architecture=arch, name=name or arch, num_layers=len(cfg["layers"]),
                          hidden_size=int(cfg["width"]), vocab_size=int(cfg["vocab"]))
         mc.rms_norm_eps = float(cfg["norm"]["eps"])
@@ -408,6 +410,31 @@ def _zeganex_layers(mc: ModelConfig, cfg: dict) -> None:
     mc.max_model_len = int(max([mc.max_model_len] + spans))
 
 
+def _vipolix_layers(mc: ModelConfig, cfg: dict) -> None:
+    side = cfg.get("token_side")
+    mc.token_side_dim = int(side["dim"]) if side else 0
+    specs = layer_specs(cfg["layers"], {"gla": GlaMixerSpec.from_dict, "parallel": ParallelMixerSpec.from_dict}, act="silu",
+                        gated=True, expert_act="swigluoai:1.702", experts=ExpertsSpec.clamped, dense=False)
+    specs = [replace(s, token_shift=True, side_dim=mc.token_side_dim) for s in specs]
+    mc.layer_specs = tuple(specs)
+    mixers = [s.mixer for s in specs]
+    att = [m.left for m in mixers if not m.recurrent]
+    mc.num_q_heads = max(m.heads for m in att or mixers)
+    mc.num_kv_heads = max((m.kv_heads for m in att), default=1)
+    mc.head_dim = max(max(m.dim, m.vdim) for m in att or mixers)
+    mc.attn_sinks = bool(att)
+    moe = [s.experts for s in specs if s.experts]
+    if moe:
+        mc.num_experts, mc.num_experts_per_tok = max(e.experts for e in moe), max(e.top for e in moe)
+        mc.moe_intermediate_size = max(e.ff for e in moe)
+        mc.moe_scoring, mc.moe_router_fp32, mc.moe_score_bias = "sigmoid", True, True
+
+
+# "architecture" of a config.json that lists its layers -> the function that reads it
+LAYER_LIST_DESIGNS = {"Mazivik": _mazivik_layers, "Popanex": _popanex_layers, "Zeganex": _zeganex_layers,
+                      "Vipolix": _vipolix_layers}
+
+
 def _preset(**kw) -> ModelConfig:
     return ModelConfig(**kw)
 
@@ -485,6 +512,23 @@ def model_preset(name: str) -> ModelConfig:
                 dict(gated, mlp={"kind": "dense", "ff": 136}), dict(diff, mlp=moe),
                 {"type": "attention", "mixer": dict(diff["mixer"], kv_from=1), "mlp": None}]},
             name="tiny-zeganex")
+        mc.max_model_len, mc.init_std = 256, 0.1
+        return mc
+    if n in ("tiny-vipolix",):
+        # both mixers, unequal sizes, one layer without a feed-forward
+        left = {"heads": 4, "kv_heads": 2, "dim": 24, "vdim": 40, "scale": 0.2, "conv": 3, "mask": {"size": 21},
+                "rot": {"base": 5000.0, "dims": 12}}
+        par = {"type": "parallel", "mixer": {"left": left, "right": {"heads": 2, "dim": 24, "decay_rank": 12},
+                                             "left_scale": 0.8, "right_scale": 0.6}}
+        gla = {"type": "gla", "mixer": {"heads": 2, "dim": 16, "vdim": 40, "tau": 12.0, "decay_rank": 8}}
+        moe = {"kind": "moe", "expert": {"ff": 40, "limit": 3.0}, "shared": {"ff": 56, "limit": 2.5},
+               "router": {"experts": 8, "top": 2, "scale": 1.3, "groups": {"count": 4, "keep": 2}}}
+        mc = ModelConfig.from_layer_list({
+            "architecture": "Vipolix", "width": 96, "vocab": 320, "norm": {"eps": 1e-5}, "token_side": {"dim": 20},
+            "torch_dtype": "float32", "layers": [
+                dict(gla, mlp=moe), dict(par, mlp=moe), dict(gla, mlp=None),
+                dict(par, mlp=dict(moe, router={"experts": 6, "top": 3, "scale": 0.9, "groups": {"count": 3, "keep": 2}}))]},
+            name="tiny-vipolix")
         mc.max_model_len, mc.init_std = 256, 0.1
         return mc
     if n in ("tiny-odd-heads",):

@@ -89,6 +89,9 @@ class GroupedMixerSpec:
     out_bias: bool = False
     output_gate: bool = False            # heads times sigmoid(W_g x) in front of the output projection
     kv_from: Optional[int] = None        # layer whose cached keys and values this layer reads
+    chunk: Optional[int] = None          # a query sees the keys of its own chunk of that many positions (None: no chunks)
+    head_temp: bool = False              # scores times one number per query head
+    zero_sink: bool = False              # one is added to the denominator of the softmax (a sink logit of 0)
 
     recurrent = False
 
@@ -96,13 +99,20 @@ class GroupedMixerSpec:
     def carries_state(self) -> bool:
         return self.conv > 0
 
+    @property
+    def mask(self) -> Optional[int]:
+        """The window, or minus the size of the chunks, as the attention ops take it."""
+        return -self.chunk if self.chunk is not None else self.window
+
     def __post_init__(self):
         if self.heads % self.kv_heads:
             raise ValueError(f"{self.heads} query heads do not divide over {self.kv_heads} key/value heads")
         if self.rot is not None and (self.rot.dims % 2 or self.rot.dims > self.dim):
             raise ValueError(f"rot.dims {self.rot.dims} must be even and at most dim {self.dim}")
-        if self.window is not None and self.window < 1:
-            raise ValueError("a window holds at least the token itself")
+        if any(n is not None and n < 1 for n in (self.window, self.chunk)):
+            raise ValueError("a window or a chunk holds at least the token itself")
+        if self.window is not None and self.chunk is not None:
+            raise ValueError("a window and chunks at the same time are not built")
 
     @staticmethod
     def sizes_of(d: dict) -> tuple:
@@ -132,6 +142,12 @@ class GroupedMixerSpec:
     @staticmethod
     def gated(d: dict) -> "GroupedMixerSpec":
         return GroupedMixerSpec.convolved(d, out_bias=True, output_gate=True)
+
+    @staticmethod
+    def chunked(d: dict) -> "GroupedMixerSpec":
+        """``mask.size`` is the size of the chunks; a temperature per head and a sink of 0."""
+        s = GroupedMixerSpec.convolved(d, head_temp=True, zero_sink=True)
+        return replace(s, chunk=s.window, window=None)
 
     def num_params(self, h: int) -> int:
         n = h * self.heads * (self.maps * self.dim + self.vdim * (2 if self.output_gate else 1))
@@ -194,27 +210,131 @@ class DeltaMixerSpec:
         return n + self.rank * self.heads * (self.dim + self.vdim)
 
 
-MixerSpec = Union[LatentMixerSpec, GroupedMixerSpec, RetentionMixerSpec, DeltaMixerSpec]
+@dataclass(frozen=True)
+class GlaMixerSpec:
+    """Gated linear attention: one decay sigmoid(z)^(1 / tau) per head and key channel, z from a low-rank projection."""
+    heads: int
+    dim: int
+    vdim: int
+    tau: float
+    decay_rank: int = 0                  # rank of the decay projection until a checkpoint sets it
+
+    recurrent = carries_state = True
+
+    @staticmethod
+    def from_dict(d: dict) -> "GlaMixerSpec":
+        s = GlaMixerSpec(int(d["heads"]), int(d["dim"]), int(d["vdim"]), float(d["tau"]), int(d.get("decay_rank", 0)))
+        if s.tau <= 0:
+            raise ValueError(f"tau {s.tau} must be positive")
+        return s
+
+    @property
+    def rank(self) -> int:
+        return self.decay_rank or 16
+
+    def num_params(self, h: int) -> int:
+        return h * (self.heads * (2 * self.dim + 3 * self.vdim) + self.rank) + self.rank * self.heads * self.dim
+
+
+@dataclass(frozen=True)
+class RemovalMixerSpec:
+    """Generalised delta rule: one decay and one removal rate per head and key channel, both acting on the old state."""
+    heads: int
+    dim: int                             # of keys and values alike
+    decay_rank: int = 0                  # rank of the decay projection until a checkpoint sets it
+
+    recurrent = carries_state = True
+
+    @property
+    def vdim(self) -> int:
+        return self.dim
+
+    @staticmethod
+    def from_dict(d: dict) -> "RemovalMixerSpec":
+        return RemovalMixerSpec(int(d["heads"]), int(d["dim"]), int(d.get("decay_rank", 0)))
+
+    @property
+    def rank(self) -> int:
+        return self.decay_rank or 16
+
+    def num_params(self, h: int) -> int:
+        return h * (6 * self.heads * self.dim + self.rank) + self.rank * self.heads * self.dim
+
+
+@dataclass(frozen=True)
+class ParallelMixerSpec:
+    """Two mixers over the same input, y = left_scale * left + right_scale * right; the left one has pages."""
+    left: GroupedMixerSpec
+    right: RemovalMixerSpec
+    left_scale: float
+    right_scale: float
+
+    recurrent = False
+    carries_state = True
+
+    @staticmethod
+    def from_dict(d: dict) -> "ParallelMixerSpec":
+        return ParallelMixerSpec(GroupedMixerSpec.chunked(d["left"]), RemovalMixerSpec.from_dict(d["right"]),
+                                 float(d["left_scale"]), float(d["right_scale"]))
+
+    @property
+    def heads(self) -> int:
+        return math.gcd(self.left.heads, self.right.heads)      # what tensor parallelism has to divide
+
+    @property
+    def kv_heads(self) -> int:
+        return self.left.kv_heads
+
+    def num_params(self, h: int) -> int:
+        return self.left.num_params(h) + self.right.num_params(h)
+
+
+MixerSpec = Union[LatentMixerSpec, GroupedMixerSpec, RetentionMixerSpec, DeltaMixerSpec, GlaMixerSpec, RemovalMixerSpec,
+                  ParallelMixerSpec]
 
 
 @dataclass(frozen=True)
 class ExpertsSpec:
-    """Mixture of ungated experts: down(act(up(x))) of the ``top`` experts with the largest softmax scores, weighted with
-    these scores."""
+    """Mixture of experts: down(act(up(x))), or down(act(gate(x), up(x))), of the ``top`` chosen experts.  Softmax scores
+    that are the weights themselves; or sigmoid scores (``sigmoid``), chosen after a correction within the best groups and
+    renormalised.  ``shared_ff``: an expert that every token uses, times the sigmoid of one number per token."""
     experts: int
     top: int
     ff: int
     act: str
+    gated: bool = False
+    sigmoid: bool = False
+    groups: int = 1
+    keep: int = 1                        # groups whose experts can be chosen
+    scale: float = 1.0
+    shared_ff: int = 0
+    shared_act: str = ""
+
+    def __post_init__(self):
+        if not 1 <= self.top <= self.experts:
+            raise ValueError(f"top {self.top} of {self.experts} experts")
+        if self.groups < 1 or self.experts % self.groups or not 1 <= self.keep <= self.groups:
+            raise ValueError(f"{self.keep} of {self.groups} groups of {self.experts} experts")
+        if self.top > self.keep * (self.experts // self.groups):
+            raise ValueError(f"top {self.top} experts out of {self.keep} groups of {self.experts // self.groups}")
 
     @staticmethod
     def from_dict(d: dict, act: str) -> "ExpertsSpec":
-        s = ExpertsSpec(int(d["router"]["experts"]), int(d["router"]["top"]), int(d["expert"]["ff"]), act)
-        if not 1 <= s.top <= s.experts:
-            raise ValueError(f"top {s.top} of {s.experts} experts")
-        return s
+        return ExpertsSpec(int(d["router"]["experts"]), int(d["router"]["top"]), int(d["expert"]["ff"]), act)
+
+    @staticmethod
+    def clamped(d: dict, act: str) -> "ExpertsSpec":
+        """Gated experts whose gate and up projections are clamped at ``limit``, behind sigmoid scores in groups."""
+        r, g, sh = d["router"], d["router"].get("groups") or {}, d.get("shared")
+        groups = int(g.get("count", 1))
+        return ExpertsSpec(int(r["experts"]), int(r["top"]), int(d["expert"]["ff"]), f"{act}:{float(d['expert']['limit'])}",
+                           gated=True, sigmoid=True, groups=groups, keep=int(g.get("keep", groups)),
+                           scale=float(r.get("scale", 1.0)), shared_ff=int(sh["ff"]) if sh else 0,
+                           shared_act=f"{act}:{float(sh['limit'])}" if sh else "")
 
     def num_params(self, h: int) -> int:
-        return self.experts * h * (2 * self.ff + 1)
+        n = 3 if self.gated else 2
+        return self.experts * h * (n * self.ff + 1) + (h * (3 * self.shared_ff + 1) if self.shared_ff else 0)
 
 
 @dataclass(frozen=True)
@@ -226,27 +346,36 @@ class LayerSpec:
     gated: bool = False                  # down(act(gate) * up) instead of down(act(up))
     weights_of: Optional[int] = None     # layer whose weights this one runs with (its cache and state are its own)
     experts: Optional[ExpertsSpec] = None
+    token_shift: bool = False            # the mixer's input is mixed with the one of the token before
+    side_dim: int = 0                    # width of the layer's own token input behind the feed-forward (0: none)
+
+    @property
+    def carries_state(self) -> bool:
+        return self.token_shift or self.mixer.carries_state
 
     def num_params(self, h: int) -> int:
         if self.weights_of is not None:
             return 0
-        n = self.mixer.num_params(h) + (3 if self.gated else 2) * h * self.ff
+        n = self.mixer.num_params(h) + (3 if self.gated else 2) * h * self.ff + 2 * h * self.side_dim
         return n + (self.experts.num_params(h) if self.experts else 0)
 
 
-def layer_specs(layers: list, mixers: dict, act: str, gated: bool, expert_act: Optional[str] = None) -> list:
+def layer_specs(layers: list, mixers: dict, act: str, gated: bool, expert_act: Optional[str] = None,
+                experts=ExpertsSpec.from_dict, dense: bool = True) -> list:
     """``LayerSpec`` of every entry of a configuration's layer list.  ``mixers``: the types the design has and the
-    functions that read them; ``expert_act``: activation of its experts (None: it has none)."""
+    functions that read them; ``expert_act``: activation of its experts (None: it has none), ``experts``: the function that
+    reads them; ``dense``: it has dense feed-forwards."""
+    kinds = (["dense"] if dense else []) + (["moe"] if expert_act else [])
     specs: list = []
     for i, layer in enumerate(layers):
         if layer["type"] not in mixers:
             raise ValueError(f"layer {i}: unknown mixer type {layer['type']!r}")
         mlp = layer.get("mlp")
         kind = mlp.get("kind") if mlp else None
-        if mlp and kind not in ("dense", "moe" if expert_act else "dense"):
+        if mlp and kind not in kinds:
             raise ValueError(f"layer {i}: unknown feed-forward kind {kind!r}")
         specs.append(LayerSpec(mixers[layer["type"]](layer["mixer"]), int(mlp["ff"]) if kind == "dense" else 0, act, gated,
-                               experts=ExpertsSpec.from_dict(mlp, expert_act) if kind == "moe" else None))
+                               experts=experts(mlp, expert_act) if kind == "moe" else None))
     for i, layer in enumerate(layers):
         src, seen = layer.get("weights_of"), {i}
         if src is None:

@@ -1,5 +1,6 @@
 """Grouped-query attention behind short convolutions (``layer_specs.GroupedMixerSpec`` with ``conv``): a sliding window,
-optionally rotated q and k with an output gate, or two softmax maps per head (differential attention).
+optionally rotated q and k with an output gate, or two softmax maps per head (differential attention); or chunks of the
+sequence instead of the window, a factor on the scores of every head and a sink of 0.
 
     row  = [W_q ‖ W_k ‖ W_v ‖ W_g] x + b                              one packed GEMM
     q, cache <- conv(row_q), conv(row_k), conv(row_v), rotated        one launch (``conv_and_cache``)
@@ -30,13 +31,15 @@ from .linear import seeded_normal
 
 
 class ConvAttention(GroupedAttention):
-    def __init__(self, name: str, spec: GroupedMixerSpec, cfg: ModelConfig, device, quant=None):
-        super().__init__(name, spec, cfg, device, quant)
+    def __init__(self, name: str, spec: GroupedMixerSpec, cfg: ModelConfig, device, quant=None, more=(), output=True):
+        super().__init__(name, spec, cfg, device, quant, more, output)
         s, at = spec, self.inp.offset
         inv = ops.ref.rope_inv_freq(s.rot.dims, s.rot.base, s.rot.rope_scaling).to(device) if s.rot else None
         mult = ops.ref.rope_attention_factor(s.rot.rope_scaling) if s.rot else 1.0
         self.plan = ConvAttentionPlan(self.Hq, self.Hkv if s.kv_from is None else 0, s.dim, s.vdim, s.maps, self.D,
                                       (at["q"], at.get("k", 0), at.get("v", 0)), s.conv, inv_freq=inv, rot_mult=mult)
+        if s.head_temp:
+            self.plan.q_scale = torch.ones(self.Hq, dtype=torch.float32, device=device)
         self.lam = torch.zeros(1, dtype=torch.float32, device=device) if s.maps == 2 else None
 
     # ---- weights ---------------------------------------------------------------
@@ -55,6 +58,10 @@ class ConvAttention(GroupedAttention):
     def load_bias(self, q, k=None, v=None) -> None:
         self.inp.load_bias(**{n: t for n, t in (("q", q), ("k", k), ("v", v)) if t is not None})
 
+    def load_temp(self, full) -> None:
+        """Factors on the scores of the heads; they go onto the queries, in 32-bit."""
+        self.plan.q_scale.copy_(self._own(full, self.spec.heads))
+
     def load_out_bias(self, b) -> None:
         self.o.bias = b.to(device=self.device, dtype=self.cfg.dtype).contiguous()
 
@@ -72,6 +79,8 @@ class ConvAttention(GroupedAttention):
                                  ("v", s.kv_heads * s.vdim)) if n == "q" or s.kv_from is None}
         self.load_conv(**{n: vec(f"{n}_conv", r, s.conv) for n, r in own.items()})
         self.load_bias(**{n: vec(f"{n}_bias", r, scale=0.1) for n, r in own.items()})
+        if s.head_temp:
+            self.load_temp(1.0 + vec("temp", s.heads, scale=0.2))
         if s.out_bias:
             self.load_out_bias(vec("o_bias", self.cfg.hidden_size, scale=0.1))
         if s.maps == 2:
@@ -94,21 +103,24 @@ class ConvAttention(GroupedAttention):
         ops.conv_ring_update(self.plan, inputs[0], cache[0], meta)
 
     def forward(self, x, cache, meta):
-        T = x.shape[0]
+        T, row = x.shape[0], self.inp(x)
+        q = self.queries(row, cache, meta)
+        return self.o(self.attend(q, row, cache[1], meta).reshape(T, self.Hq * self.D))
+
+    def queries(self, row, cache, meta):
+        """Convolved and rotated queries of the projected rows; keys and values go to their pages."""
         ring, pages = cache
-        row = self.inp(x)
         rb = getattr(meta, "state_rollback", None)
         if rb is not None:
             rb.capture(self, (ring,), (row,))      # verification step: rejected drafts are rolled back later
-        q = ops.conv_and_cache(self.plan, row, pages, ring, meta)
-        return self.o(self.attend(q, row, pages, meta).reshape(T, self.Hq * self.D))
+        return ops.conv_and_cache(self.plan, row, pages, ring, meta)
 
-    def attend(self, q, row, pages, meta):
-        """Softmax over the window and what follows it: [T, heads, D]."""
+    def attend(self, q, row, pages, meta, out=None):
+        """Softmax over the visible keys and what follows it: [T, heads, D], or the rows ``out``."""
         s, gate = self.spec, None
         if s.output_gate:
             at = self.inp.offset["g"]
             gate = row[:, at:at + self.Hq * s.vdim]
         if gate is None and s.maps == 1:
-            return ops.paged_attention(q, pages, meta, s.scale, sliding_window=s.window)
-        return ops.paged_attention_heads(q, pages, meta, s.scale, s.window, s.vdim, gate, self.lam, s.diff, self.eps)
+            return ops.paged_attention(q, pages, meta, s.scale, sliding_window=s.mask, sinks=self.sinks, out=out)
+        return ops.paged_attention_heads(q, pages, meta, s.scale, s.mask, s.vdim, gate, self.lam, s.diff, self.eps)

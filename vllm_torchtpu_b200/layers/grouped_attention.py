@@ -47,7 +47,9 @@ class HeadPaddedRowLinear(RowParallelLinear):
 
 
 class GroupedAttention:
-    def __init__(self, name: str, spec: GroupedMixerSpec, cfg: ModelConfig, device, quant=None):
+    def __init__(self, name: str, spec: GroupedMixerSpec, cfg: ModelConfig, device, quant=None, more=(), output=True):
+        """``more``: parts of other mixers that the packed projection of the input computes too; without ``output`` the
+        owner applies the output projection."""
         st = get_state()
         tp = st.tp.size
         if spec.heads % tp:
@@ -57,13 +59,15 @@ class GroupedAttention:
         self.D = cache_head_dim(spec.maps * spec.dim, spec.vdim, cfg.dtype)
         self.eps = cfg.rms_norm_eps
         kw = dict(dtype=cfg.dtype, device=device, quant_config=quant)
-        self.inp = PackedLinear(f"{name}.qkv_proj", cfg.hidden_size, self.parts(spec), bias=spec.bias, **kw)
+        self.inp = PackedLinear(f"{name}.qkv_proj", cfg.hidden_size, self.parts(spec) + list(more), bias=spec.bias,
+                                **kw)
         self.o = HeadPaddedRowLinear(f"{name}.o_proj", spec.heads, spec.vdim, self.D, cfg.hidden_size,
-                                     bias=spec.out_bias, **kw)
+                                     bias=spec.out_bias, **kw) if output else None
         ones = lambda n: torch.ones(n, dtype=cfg.dtype, device=device)                  # noqa: E731
         self.q_norm = ones(self.Hq * spec.dim) if spec.projection_norm else None
         self.k_norm = ones(self.Hkv * spec.dim) if spec.projection_norm else None
-        self.sinks = torch.zeros(self.Hq, dtype=torch.float32, device=device) if spec.sinks else None
+        self.sinks = torch.zeros(self.Hq, dtype=torch.float32, device=device) if spec.sinks or spec.zero_sink \
+            else None
         self.kv_replicas = max(1, tp // spec.kv_heads)
         # sharded norms: the squared sums of all ranks, each replicated key head counted once
         self.norm_sizes = (spec.heads * spec.dim, spec.kv_heads * spec.dim)
@@ -77,12 +81,12 @@ class GroupedAttention:
         return parts + ([Part("g", spec.heads * spec.vdim, spec.heads)] if spec.output_gate else [])
 
     def linears(self):
-        return [self.inp, self.o]
+        return [self.inp] + ([self.o] if self.o is not None else [])
 
     def init_dummy(self, std: float, seed: int) -> None:
         for lin in self.linears():
             lin.init_dummy(std, seed)
-        if self.sinks is not None:
+        if self.spec.sinks:
             self.load_sinks(seeded_normal(f"{self.name}.sinks", (self.spec.heads,), 1.0, torch.float32, self.device, seed))
 
     def load_sinks(self, full) -> None:

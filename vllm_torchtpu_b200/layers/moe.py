@@ -75,7 +75,9 @@ class FusedMoE:
         lo = self.ep_rank * self.num_local_experts
         self.expert_range = (lo, lo + self.num_local_experts)
         self.has_bias = bool(getattr(cfg, "moe_bias", False))      # router and expert biases (GPT-OSS)
-        self.gate = ReplicatedLinear(f"{name}.gate", cfg.hidden_size, cfg.num_experts, dtype=cfg.dtype,
+        # with router logits in 32-bit, the gate of a shared expert is one more row of the router
+        self.gate_rows = cfg.num_experts + int(cfg.shared_expert_gate and cfg.moe_router_fp32)
+        self.gate = ReplicatedLinear(f"{name}.gate", cfg.hidden_size, self.gate_rows, dtype=cfg.dtype,
                                      device=device, quant_config=None, bias=self.has_bias)
         self.b13 = self.b2 = None
         self.score_bias = None
@@ -107,6 +109,12 @@ class FusedMoE:
             self.method.alloc(self)
         self.method.load_expert(self, local_e, None, up, down)
 
+    def load_gated(self, local_e: int, gate, up, down) -> None:
+        """Unsharded matrices of one expert with a gate projection."""
+        if self.w13 is None:
+            self.method.alloc(self)
+        self.method.load_expert(self, local_e, gate, up, down)
+
     def init_dummy(self, std: float, seed: int) -> None:
         # router logits come from N(0,1) gate weights so that routing is well spread
         self.gate.init_dummy(1.0, seed)
@@ -131,9 +139,13 @@ class FusedMoE:
     def weight_bytes(self) -> int:
         return self.method.weight_bytes(self) + self.gate.weight_bytes()
 
-    def route(self, x: torch.Tensor):
+    def router_logits(self, x: torch.Tensor) -> torch.Tensor:
+        """[T, gate_rows]; the columns behind the experts are not theirs."""
+        return ops.gemm_softcap(x, self.gate.weight) if self.cfg.moe_router_fp32 else self.gate(x)
+
+    def route(self, x: torch.Tensor, logits: Optional[torch.Tensor] = None):
         c = self.cfg
-        logits = ops.gemm_softcap(x, self.gate.weight) if c.moe_router_fp32 else self.gate(x)
+        logits = (self.router_logits(x) if logits is None else logits)[:, :self.num_experts]
         ids, w = ops.moe_route(logits, self.top_k, scoring=c.moe_scoring, renormalize=c.moe_renormalize,
                                routed_scaling=c.moe_routed_scaling, score_bias=self.score_bias,
                                n_group=c.moe_n_group, topk_group=c.moe_topk_group)
@@ -148,8 +160,8 @@ class FusedMoE:
             ids, w = post(ids, w, self.num_experts, nv, sim)
         return ids, w
 
-    def forward(self, x: torch.Tensor) -> torch.Tensor:
-        topk_ids, topk_w = self.route(x)
+    def forward(self, x: torch.Tensor, logits: Optional[torch.Tensor] = None) -> torch.Tensor:
+        topk_ids, topk_w = self.route(x, logits)
         if not self.use_ep:
             y = self.method.apply(self, x, topk_ids, topk_w)
             if self.tp_size > 1:

@@ -33,8 +33,12 @@ def get_model_class(cfg: ModelConfig):
     if a == "zeganex":
         from .zeganex import ZeganexForCausalLM
         return ZeganexForCausalLM
+    if a == "vipolix":
+        from .vipolix import VipolixForCausalLM
+        return VipolixForCausalLM
     raise ValueError(f"no model class for architecture {a!r}")
 
 
 def supported_architectures() -> list[str]:
-    return ["llama", "qwen3_moe", "gpt_oss", "deepseek_v3", "qwen3_next", "kimi_linear", "mazivik", "popanex", "zeganex"]
+    return ["llama", "qwen3_moe", "gpt_oss", "deepseek_v3", "qwen3_next", "kimi_linear", "mazivik", "popanex", "zeganex",
+            "vipolix"]

@@ -41,12 +41,47 @@ def layer_norm_add(y, residual, weight, eps):
 
 
 def add_rms_norm(y, residual, weight, eps, offset=0.0, update=True, post=None, mult=1.0):
-    """(h, fp32 r) of r = residual (+ y), h = RMS norm of r times (offset + weight); an fp32 residual is updated in
+    """(h, fp32 r) of r = residual (+ mult * y), h = RMS norm of r times (offset + weight); an fp32 residual is updated in
     place on a GPU.  ``y`` None: r = residual.  ``post``: the RMS norm of y with this weight, times ``mult``, is added
     instead of y.  Without ``update`` the stream is only read and r is None."""
     y = materialize(y)
     return cuda_ops().add_rms_norm(y, residual, weight, eps, offset, update, post, mult) if _on_gpu(residual) else \
         ref.add_rms_norm(y, residual, weight, eps, offset, update, post, mult)
+
+
+def add_rms_norm_shift(y, residual, weight, eps, offset, shift, state, meta, post=None, mult=1.0, keep=False):
+    """Residual sum and norm of ``add_rms_norm`` with a token shift behind them; see ``ops.token_shift``."""
+    if _on_gpu(residual):
+        return cuda_ops().add_rms_norm_shift(materialize(y), residual, weight, eps, offset, shift, state, meta, post, mult,
+                                             keep)
+    from .token_shift import add_rms_norm_shift as f
+    return f(materialize(y), residual, weight, eps, offset, shift, state, meta, post, mult, keep)
+
+
+def add_gated(y, z, gate):
+    """y + sigmoid(gate)[:, None] * z, gate fp32 [T] (rows may be strided)."""
+    if _on_gpu(y):
+        return cuda_ops().add_gated(y, z, gate)
+    return (y.float() + torch.sigmoid(gate.float())[:, None] * z.float()).to(y.dtype)
+
+
+def residual_add(y, residual, mult=1.0, dtype=None):
+    """(r rounded to ``dtype``, fp32 r) of r = residual + mult * y; r may be the residual's storage."""
+    y = materialize(y)
+    return cuda_ops().residual_add(y, residual, mult, dtype) if _on_gpu(y) else ref.residual_add(y, residual, mult, dtype)
+
+
+def gemm_token_gate(x, w, table, first, ids):
+    """gelu_tanh(x @ w.T) * table[ids, first : first + N], in the GEMM's epilogue on a GPU."""
+    f = cuda_ops().gemm_token_gate if _on_gpu(x) else ref.gemm_token_gate
+    return f(x, w, table, first, ids)
+
+
+def resolve_tokens(ids, token_src, last_tokens):
+    """Token ids of a step's rows: those still on the device (token_src >= 0) are last_tokens[token_src]."""
+    if _on_gpu(ids):
+        return cuda_ops().resolve_tokens(ids, token_src, last_tokens)
+    return torch.where(token_src >= 0, last_tokens[token_src.clamp_min(0).long()], ids)
 
 
 def softcap(x, cap):
@@ -96,12 +131,25 @@ def gemm_gated(x, w, act):
     return cuda_ops().gemm_gated(x, w, act) if _on_gpu(x) else ref.gated_act_and_mul(ref.gemm(x, w), act)
 
 
-def carried_state_attention(plan, row, decay_in, gate, meta, cache):
-    """Linear attention with a carried state; see ``ops.linear_attention``."""
+def carried_state_attention(plan, row, decay_in, gate, meta, cache, out=None):
+    """Linear attention with a carried state; see ``ops.linear_attention``.  ``out``: [T, heads * vdim], rows may be
+    strided."""
     if _on_gpu(row):
-        return cuda_ops().carried_state_attention(plan, row, decay_in, gate, meta, cache)
+        return cuda_ops().carried_state_attention(plan, row, decay_in, gate, meta, cache, out)
     from .linear_attention import linear_attention_reference
-    return linear_attention_reference(plan, row, decay_in, gate, meta, cache)
+    return linear_attention_reference(plan, row, decay_in, gate, meta, cache, out)
+
+
+def mixer_rows(x, width: int):
+    """[T, width] rows that mixers write into; rows of padding stay finite."""
+    if _on_gpu(x) and x.dtype == torch.bfloat16:
+        return cuda_ops().Workspace.get(x.device).attn_out(x.shape[0], 1, width)[:, 0]
+    return torch.zeros(x.shape[0], width, dtype=x.dtype, device=x.device)
+
+
+def tanh_(x):
+    """In place, fp32 inside; rows may be strided."""
+    return cuda_ops().tanh_(x) if _on_gpu(x) else x.copy_(torch.tanh(x.float()))
 
 
 def gemm_heads(x, w, gate=None, out=None):
@@ -172,11 +220,16 @@ def norm_and_cache(qkv, positions, kv_cache, slot_mapping, *a, **kw):
 
 
 def paged_attention(q, kv_cache, meta, scale, *, sliding_window=None, softcap=None, sinks=None,
-                    k_scale=1.0, v_scale=1.0, return_lse=False):
+                    k_scale=1.0, v_scale=1.0, return_lse=False, out=None):
+    """``sliding_window`` n > 0: a query sees the last n keys; n < 0: the keys of its own chunk of -n positions.  ``out``:
+    [T, >= heads * dim] rows, which may be strided, for the heads side by side."""
     if _on_gpu(q):
         return cuda_ops().paged_attention(q, kv_cache, meta, scale, sliding_window=sliding_window,
                                           softcap=softcap, sinks=sinks, k_scale=k_scale,
-                                          v_scale=v_scale, return_lse=return_lse)
+                                          v_scale=v_scale, return_lse=return_lse, out=out)
+    if out is not None:
+        o = paged_attention(q, kv_cache, meta, scale, sliding_window=sliding_window, softcap=softcap, sinks=sinks)
+        return out[:, :o.shape[1] * o.shape[2]].copy_(o.reshape(o.shape[0], -1))
     return ref.paged_attention(q, kv_cache, meta.block_tables, meta.seq_lens, meta.query_start_loc,
                                scale, num_reqs=meta.num_reqs, sliding_window=sliding_window,
                                softcap=softcap, sinks=sinks, k_scale=k_scale, v_scale=v_scale,

@@ -55,17 +55,29 @@ def layer_norm_add(y: torch.Tensor, residual: torch.Tensor, weight: torch.Tensor
 
 def add_rms_norm(y: Optional[torch.Tensor], residual: torch.Tensor, weight: torch.Tensor, eps: float,
                  offset: float = 0.0, update: bool = True, post: Optional[torch.Tensor] = None, mult: float = 1.0):
-    """32-bit residual stream in front of a sublayer: r = residual (+ y); h = r / rms(r) * (offset + w).  With ``post``
-    the output y is normalised first: r = residual + mult * y / rms(y) * post.
+    """32-bit residual stream in front of a sublayer: r = residual (+ mult * y); h = r / rms(r) * (offset + w).  With
+    ``post`` the output y is normalised first: r = residual + mult * y / rms(y) * post.
     Returns (h in the weight's dtype, r fp32 or None without ``update``)."""
     r = residual.float()
     if y is not None:
         a = y.float()
         if post is not None:
-            a = mult * (a * torch.rsqrt(a.pow(2).mean(-1, keepdim=True) + eps) * post.float())
-        r = r + a
+            a = a * torch.rsqrt(a.pow(2).mean(-1, keepdim=True) + eps) * post.float()
+        r = r + mult * a
     h = r * torch.rsqrt(r.pow(2).mean(-1, keepdim=True) + eps) * (offset + weight.float())
     return h.to(weight.dtype), (r if update else None)
+
+
+def residual_add(y: torch.Tensor, residual: torch.Tensor, mult: float = 1.0, dtype=None):
+    """(r rounded to ``dtype``, fp32 r) of r = residual + mult * y."""
+    r = residual.float() + mult * y.float()
+    return r.to(dtype or y.dtype), r
+
+
+def gemm_token_gate(x, w, table, first: int, ids):
+    """gelu_tanh(x @ w.T) times the columns from ``first`` on of the rows ``ids`` of ``table``."""
+    e = table[ids.long(), first:first + w.shape[0]].float()
+    return (F.gelu(x.float() @ w.float().t(), approximate="tanh") * e).to(x.dtype)
 
 
 def softcap(x: torch.Tensor, cap: float) -> torch.Tensor:
@@ -343,7 +355,7 @@ def paged_attention(q, kv_cache, block_tables, seq_lens, query_start_loc, scale,
             qpos = torch.arange(kv_len - q_len, kv_len, device=q.device)[:, None]
         mask = kpos <= qpos
         if sliding_window:
-            mask &= kpos > qpos - sliding_window
+            mask &= kpos > qpos - sliding_window if sliding_window > 0 else kpos >= qpos - qpos % -sliding_window
         s = s.masked_fill(~mask, float("-inf"))
         if sinks is not None:
             sink = sinks.float().reshape(Hkv, G, 1, 1).expand(Hkv, G, q_len, 1)
@@ -454,7 +466,7 @@ def moe_route(router_logits, top_k: int, scoring: str = "softmax", renormalize: 
     if n_group > 1:
         g = choice.view(T, n_group, E // n_group)
         if score_bias is not None:
-            gs = g.topk(2, dim=-1).values.sum(-1)
+            gs = g.topk(min(2, g.shape[-1]), dim=-1).values.sum(-1)
         else:
             gs = g.max(-1).values
         gidx = gs.topk(topk_group, dim=-1).indices

@@ -8,7 +8,8 @@ stands behind them in attention layers (``ConvAttentionPlan``): plain-PyTorch st
 none of those it reads; a portion that starts at position 0 reads none of it, so nothing has to be cleared.
 
 Attention layers: q, k and v channels of one packed projection ``row`` pass the convolution, then q and k turn (the first
-``2 * pairs`` dimensions of a head, interleaved pairs, cos and sin times ``rot_mult``), k and v go to the token's page.
+``2 * pairs`` dimensions of a head, interleaved pairs, cos and sin times ``rot_mult``), q is multiplied by one number per
+head where the plan has them, k and v go to the token's page.
 Heads are stored in ``width`` columns, zeros behind them.  With two maps per head, a key row is both maps side by side,
 and the query of a head becomes two rows, each with its map's columns and zeros in the other's place: scores against the
 whole key row are then the scores of that map, and the values are shared.
@@ -51,6 +52,7 @@ class ConvAttentionPlan:
     conv_w: Optional[torch.Tensor] = None       # [taps, channels] in the model dtype, channels = q | k | v
     inv_freq: Optional[torch.Tensor] = None     # [pairs] fp32, None: no rotation
     rot_mult: float = 1.0
+    q_scale: Optional[torch.Tensor] = None      # [heads] fp32, None: 1
 
     @property
     def sizes(self) -> tuple:
@@ -91,6 +93,8 @@ def conv_and_cache(plan: ConvAttentionPlan, row, kv_cache, ring, meta):
     q, k = q.reshape(T, p.heads * p.maps, p.dim), k.reshape(T, p.kv_heads * p.maps, p.dim)
     if p.inv_freq is not None:
         q, k = (rope_scaled(t, meta.positions, p.inv_freq, p.rot_mult, True) for t in (q, k))
+    if p.q_scale is not None:
+        q = q.reshape(T, p.heads, -1) * p.q_scale[:, None]
     wide = torch.zeros(T, p.heads, p.maps, p.width, device=row.device)
     for m in range(p.maps):
         wide[:, :, m, m * p.dim:(m + 1) * p.dim] = q.reshape(T, p.heads, p.maps, p.dim)[:, :, m]

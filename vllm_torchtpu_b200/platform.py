@@ -214,7 +214,8 @@ class B200Platform:
             bad = [i for i, l in enumerate(m.layer_specs) if l.mixer.heads % tp
                    or (l.mixer.recurrent and getattr(l.mixer, "kv_heads", tp) % tp)
                    or (l.mixer.carries_state and not l.mixer.recurrent and l.mixer.kv_heads % tp and tp % l.mixer.kv_heads)
-                   or (l.experts and not p.enable_expert_parallel and l.experts.ff % tp)]
+                   or (l.experts and not p.enable_expert_parallel and l.experts.ff % tp)
+                   or (l.experts and l.experts.shared_ff % tp)]
             if bad:
                 raise ValueError(f"the heads or experts of layers {bad[:8]} do not divide over tp={tp}")
             if not m.is_mla and max(p.decode_context_parallel_size, p.prefill_context_parallel_size) > 1:

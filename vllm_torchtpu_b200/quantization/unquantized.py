@@ -141,6 +141,12 @@ class UnquantizedMoEMethod:
             return ops.cuda_ops().moe_experts(x, moe.w13, moe.w2, topk_ids, topk_w, moe.expert_range[0], **kw)
         return ops.ref.moe_experts(x, moe.w13, moe.w2, topk_ids, topk_w, moe.expert_range[0], **kw)
 
+    def apply_add(self, moe, x, topk_ids, topk_w, shared, residual):
+        """``apply`` with the shared expert ((output, gate column) or None) and the residual stream in the last kernel:
+        (sum rounded, fp32 sum)."""
+        return ops.cuda_ops().moe_experts(x, moe.w13, moe.w2, topk_ids, topk_w, moe.expert_range[0], act=moe.activation,
+                                          shared=shared, residual=residual)
+
     def apply_fused_ep(self, moe, x, topk_ids, topk_w, comm):
         return ops.cuda_ops().moe_experts_ep(x, moe.w13, moe.w2, topk_ids, topk_w, comm.heap, moe.num_experts)
 

@@ -454,6 +454,9 @@ class ModelRunner:
             # image / video embeddings replace the placeholder-token rows of the prompt
             for rid, start, row0, nrows in self._mm_plan:
                 self.mm_manager.merge_into(hidden0, rid, start, row0, nrows)
+        if self.mcfg.token_side_dim:
+            # every layer reads the token once more: ids that are still on the device are filled in
+            ids = ops.resolve_tokens(ids, dv("token_src", T), self.last_tokens)
         hidden, residual = self.model.forward(ids, meta, self.kv_caches, hidden=hidden0)
         if self._pool_plan:
             self._pool(hidden, residual)

@@ -41,9 +41,13 @@ class StateRollback:
         self.saved: list = []           # (layer, cache, snapshots, input rows)
         self.stats = {"snapshots": 0, "rolled_back": 0, "replayed_rows": 0}
 
-    def capture(self, layer, cache, inputs) -> None:
-        """Called by a recurrent layer in front of its stateful part."""
-        snap = tuple(pool.index_select(0, self._slots_t) for pool in cache)
+    def snapshot(self, cache) -> tuple:
+        """The verifying requests' part of the pools."""
+        return tuple(pool.index_select(0, self._slots_t) for pool in cache)
+
+    def capture(self, layer, cache, inputs, snap=None) -> None:
+        """Called by a recurrent layer in front of its stateful part; behind it with the ``snapshot`` taken in front."""
+        snap = self.snapshot(cache) if snap is None else snap
         rows = tuple(t.index_select(0, self._rows_t) for t in inputs)
         self.saved.append((layer, cache, snap, rows))
         self.stats["snapshots"] += 1
