@@ -59,7 +59,7 @@ def _existing(L, q, cache, bt, sl, qsl, maxb, nb, Hq, Hkv, D, splits):
     rc = L.b200_attn_decode(_p(q), _p(cache), _p(out), _p(lse), _p(bt), _p(sl), _p(qsl), c_int(0), c_int(R),
                             c_int(maxb), c_int(cache.shape[3]), c_longlong(nb), c_int(Hq), c_int(Hkv), c_int(D),
                             c_float(D ** -0.5), c_int(0), c_float(0.0), c_void_p(0), c_int(splits), _p(scratch),
-                            _p(counters), stream)
+                            _p(counters), c_int(0), stream)
     assert rc == 0, L.b200_get_last_error().decode()
     torch.cuda.synchronize()
     return out, lse

@@ -39,6 +39,7 @@ struct AttnParams {
   int* counters;                 // decode scratch [R * Hkv]
   const float* sinks;            // optional [Hq]
   int max_blocks, block_size, Hq, Hkv, req_begin, req_end, num_splits, window;
+  int ldo;                             // elements between the output rows of neighbouring tokens (without an epilogue)
   int non_causal;                // prefill kernel: every query sees all seq_len keys (encoder attention)
   long long num_blocks;
   float scale_log2, softcap;
@@ -235,8 +236,7 @@ __global__ void __launch_bounds__(128, 2) attn_decode_kernel(const AttnParams p)
   }
 
   // this (split, warp) unit's range of 16-token chunks
-  int first_tok = 0;
-  if (p.window > 0) first_tok = max(0, ctx - p.window + 1);
+  const int first_tok = first_key(p.window, ctx);
   const int c_lo = first_tok >> 4;
   const int C = ((seq_len + 15) >> 4) - c_lo;
   const int units = p.num_splits * 4;
@@ -284,7 +284,8 @@ __global__ void __launch_bounds__(128, 2) attn_decode_kernel(const AttnParams p)
   for (int i = 0; i < D / 8; ++i) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f;
   float m[2] = {-INFINITY, -INFINITY}, l[2] = {0.f, 0.f};
   const int row0 = lane >> 2, row1 = row0 + 8;
-  const int lim0 = ctx + row0 / G, lim1 = ctx + row1 / G;       // last visible key per row
+  const int lim0 = ctx + row0 / G, lim1 = ctx + row1 / G;       // last and first visible key per row
+  const int lo0 = first_key(p.window, lim0), lo1 = first_key(p.window, lim1);
 
 #pragma unroll
   for (int s = 0; s < STAGES - 1; ++s) {
@@ -312,7 +313,7 @@ __global__ void __launch_bounds__(128, 2) attn_decode_kernel(const AttnParams p)
         const int lim = (e < 2) ? lim0 : lim1;
         float v = s[nb][e] * p.scale_log2;
         if (p.softcap > 0.f) v = p.softcap * tanhf(v / p.softcap);
-        const bool ok = tok <= lim && (p.window <= 0 || tok > lim - p.window);
+        const bool ok = tok <= lim && tok >= (e < 2 ? lo0 : lo1);
         v = ok ? v : -INFINITY;
         s[nb][e] = v;
         if (e < 2) mx0 = fmaxf(mx0, v); else mx1 = fmaxf(mx1, v);
@@ -450,12 +451,12 @@ __global__ void __launch_bounds__(128, 2) attn_decode_kernel(const AttnParams p)
       Lfin = Lfin * sc + ex2(sk - mnew);
       mfin = mnew;
       const float inv = (FP8 ? p.v_scale : 1.f) / Lfin;
-      __nv_bfloat16* dst = p.out + ((size_t)tok_row * p.Hq + head) * D + seg * SEG;
+      __nv_bfloat16* dst = p.out + (size_t)tok_row * p.ldo + head * D + seg * SEG;
 #pragma unroll
       for (int d = 0; d < SEG; ++d) dst[d] = __float2bfloat16(a[d] * sc * inv);
     } else {
       const float inv = Lfin > 0.f ? (FP8 ? p.v_scale : 1.f) / Lfin : 0.f;
-      __nv_bfloat16* dst = p.out + ((size_t)tok_row * p.Hq + head) * D + seg * SEG;
+      __nv_bfloat16* dst = p.out + (size_t)tok_row * p.ldo + head * D + seg * SEG;
 #pragma unroll
       for (int d = 0; d < SEG; ++d) dst[d] = __float2bfloat16(a[d] * inv);
     }
@@ -562,8 +563,7 @@ __global__ void __launch_bounds__(128, 3) attn_prefill_kernel(const AttnParams p
     }
   }
   const int kv_end = p.non_causal ? seq_len : min(seq_len, last_key(q0 + BQ - 1) + 1);   // causal bound of the tile
-  int kv_begin = 0;
-  if (p.window > 0) kv_begin = max(0, ctx + q0 - p.window + 1) / BKV * BKV;
+  const int kv_begin = first_key(p.window, ctx + q0) / BKV * BKV;
   const int nchunks = (kv_end - kv_begin + BKV - 1) / BKV;
 
   const int* bt = p.block_tables + (size_t)r * p.max_blocks;
@@ -601,6 +601,7 @@ __global__ void __launch_bounds__(128, 3) attn_prefill_kernel(const AttnParams p
   for (int i = 0; i < D / 8; ++i) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f;
   float m[2] = {-INFINITY, -INFINITY}, l[2] = {0.f, 0.f};
   const int lim0 = p.non_causal ? 0x3fffffff : last_key(row0), lim1 = p.non_causal ? 0x3fffffff : last_key(row1);
+  const int lo0 = first_key(p.window, max(lim0, 0)), lo1 = first_key(p.window, max(lim1, 0));
 
   if (nchunks > 0) issue(0, 0);
   cp_async_commit();
@@ -633,7 +634,7 @@ __global__ void __launch_bounds__(128, 3) attn_prefill_kernel(const AttnParams p
         const int lim = (e < 2) ? lim0 : lim1;
         float v = s[nb][e] * p.scale_log2;
         if (p.softcap > 0.f) v = p.softcap * tanhf(v / p.softcap);
-        const bool ok = tok <= lim && tok < kv_end && (p.window <= 0 || tok > lim - p.window);
+        const bool ok = tok <= lim && tok < kv_end && tok >= (e < 2 ? lo0 : lo1);
         v = ok ? v : -INFINITY;
         s[nb][e] = v;
         if (e < 2) mx0 = fmaxf(mx0, v); else mx1 = fmaxf(mx1, v);
@@ -696,7 +697,7 @@ __global__ void __launch_bounds__(128, 3) attn_prefill_kernel(const AttnParams p
   if constexpr (FP8) { sc0 *= p.v_scale; sc1 *= p.v_scale; }
   const float inv0 = l[0] > 0.f ? sc0 / l[0] : 0.f, inv1 = l[1] > 0.f ? sc1 / l[1] : 0.f;
   if (row0 < q_len) {
-    __nv_bfloat16* dst = p.out + ((size_t)(qs + row0) * p.Hq + hq) * D + (FP8 ? 4 : 2) * (lane & 3);
+    __nv_bfloat16* dst = p.out + (size_t)(qs + row0) * p.ldo + hq * D + (FP8 ? 4 : 2) * (lane & 3);
     if constexpr (FP8) {
 #pragma unroll
       for (int dc = 0; dc < D / 16; ++dc)
@@ -713,7 +714,7 @@ __global__ void __launch_bounds__(128, 3) attn_prefill_kernel(const AttnParams p
           l[0] > 0.f ? (m[0] + log2f(l[0])) * 0.6931471805599453f : -INFINITY;
   }
   if (row1 < q_len) {
-    __nv_bfloat16* dst = p.out + ((size_t)(qs + row1) * p.Hq + hq) * D + (FP8 ? 4 : 2) * (lane & 3);
+    __nv_bfloat16* dst = p.out + (size_t)(qs + row1) * p.ldo + hq * D + (FP8 ? 4 : 2) * (lane & 3);
     if constexpr (FP8) {
 #pragma unroll
       for (int dc = 0; dc < D / 16; ++dc)
@@ -759,7 +760,7 @@ static void fill_params(AttnParams& p, const void* q, const void* kv, void* out,
   p.non_causal = 0;
   p.global_seq_lens = nullptr;
   p.dcp_size = 1; p.dcp_rank = 0; p.dcp_interleave = 1;
-  (void)D;
+  p.ldo = Hq * D;
 }
 
 // fp8 (e4m3) cache: K's dequantisation factor joins the logit scale, V's the output normalisation.
@@ -801,10 +802,10 @@ static int attn_decode_impl(const void* q, const void* kv, void* out, float* lse
                             int max_blocks, int block_size, long long num_blocks, int Hq, int Hkv, int D,
                             float scale, int window, float softcap, const float* sinks, int num_splits,
                             void* scratch, int* counters, int kv_fp8, float k_scale, float v_scale,
-                            cudaStream_t stream, const HeadFinish* fin = nullptr) {
+                            cudaStream_t stream, const HeadFinish* fin = nullptr, int ldo = 0) {
   const int R = req_end - req_begin;
   if (R <= 0) return 0;
-  if (block_size % 16 || (Hq % Hkv) || Hq / Hkv > 16) {
+  if (block_size % 16 || (Hq % Hkv) || Hq / Hkv > 16 || ldo % 8) {
     b200_set_last_error("attn_decode: block_size % 16 == 0 and q heads per kv head <= 16 required", __FILE__,
                         __LINE__);
     return -1;
@@ -820,6 +821,7 @@ static int attn_decode_impl(const void* q, const void* kv, void* out, float* lse
   p.part_o = (float*)scratch;
   p.part_ml = p.part_o + (size_t)R * Hkv * num_splits * 16 * D;
   p.counters = counters;
+  if (ldo > 0) p.ldo = ldo;
   dim3 grid(Hkv, R, num_splits);
   if (kv_fp8) set_fp8_scales(p, k_scale, v_scale);
   if (fin != nullptr) {
@@ -844,14 +846,15 @@ static int attn_decode_impl(const void* q, const void* kv, void* out, float* lse
   return 0;
 }
 
+// window: first_key in common.cuh; ldo: elements between output rows (0: Hq * D).
 extern "C" int b200_attn_decode(const void* q, const void* kv, void* out, float* lse, const int* block_tables,
                                 const int* seq_lens, const int* qsl, int req_begin, int req_end,
                                 int max_blocks, int block_size, long long num_blocks, int Hq, int Hkv, int D,
                                 float scale, int window, float softcap, const float* sinks, int num_splits,
-                                void* scratch, int* counters, cudaStream_t stream) {
+                                void* scratch, int* counters, int ldo, cudaStream_t stream) {
   return attn_decode_impl(q, kv, out, lse, block_tables, seq_lens, qsl, req_begin, req_end, max_blocks,
                           block_size, num_blocks, Hq, Hkv, D, scale, window, softcap, sinks, num_splits, scratch,
-                          counters, 0, 1.f, 1.f, stream);
+                          counters, 0, 1.f, 1.f, stream, nullptr, ldo);
 }
 // The same with the epilogue of HeadFinish: out [T, lam ? Hq / 2 : Hq, D].
 extern "C" int b200_attn_decode_heads(const void* q, const void* kv, void* out, const int* block_tables,
@@ -888,9 +891,9 @@ static int attn_prefill_impl(const void* q, const void* kv, void* out, float* ls
                              int num_tiles, int max_blocks, int block_size, long long num_blocks, int Hq,
                              int Hkv, int D, float scale, int window, float softcap, const float* sinks,
                              int kv_fp8, float k_scale, float v_scale, cudaStream_t stream,
-                             const DcpArgs& dcp = DcpArgs()) {
+                             const DcpArgs& dcp = DcpArgs(), int ldo = 0) {
   if (req_end <= req_begin || num_tiles <= 0) return 0;
-  if (block_size % 16 || (Hq % Hkv)) {
+  if (block_size % 16 || (Hq % Hkv) || ldo % 8) {
     b200_set_last_error("attn_prefill: block_size % 16 == 0 required", __FILE__, __LINE__);
     return -1;
   }
@@ -902,7 +905,7 @@ static int attn_prefill_impl(const void* q, const void* kv, void* out, float* ls
   p.num_splits = 1;
   p.part_o = nullptr; p.part_ml = nullptr; p.counters = nullptr;
   if (dcp.size > 1) {
-    if (dcp.global_seq_lens == nullptr || dcp.interleave <= 0 || window > 0) {
+    if (dcp.global_seq_lens == nullptr || dcp.interleave <= 0 || window != 0) {
       b200_set_last_error("attn_prefill: decode context parallelism needs the global lengths and no sliding window",
                           __FILE__, __LINE__);
       return -1;
@@ -910,6 +913,7 @@ static int attn_prefill_impl(const void* q, const void* kv, void* out, float* ls
     p.global_seq_lens = dcp.global_seq_lens;
     p.dcp_size = dcp.size; p.dcp_rank = dcp.rank; p.dcp_interleave = dcp.interleave;
   }
+  if (ldo > 0) p.ldo = ldo;
   dim3 grid(Hq, num_tiles);
   if (kv_fp8) set_fp8_scales(p, k_scale, v_scale);
   if (D == 128 && kv_fp8) B200_CUDA_CHECK((launch_prefill<128, true>(grid, stream, p)));
@@ -943,10 +947,10 @@ extern "C" int b200_attn_prefill(const void* q, const void* kv, void* out, float
                                  const int* seq_lens, const int* qsl, int req_begin, int req_end,
                                  int num_tiles, int max_blocks, int block_size, long long num_blocks, int Hq,
                                  int Hkv, int D, float scale, int window, float softcap, const float* sinks,
-                                 cudaStream_t stream) {
+                                 int ldo, cudaStream_t stream) {
   return attn_prefill_impl(q, kv, out, lse, block_tables, seq_lens, qsl, req_begin, req_end, num_tiles,
                            max_blocks, block_size, num_blocks, Hq, Hkv, D, scale, window, softcap, sinks, 0, 1.f,
-                           1.f, stream);
+                           1.f, stream, DcpArgs(), ldo);
 }
 // Bidirectional attention over a ragged batch whose keys and values sit in the paged layout (vision
 // encoders: each request's q_len equals its seq_len).  Same arguments as b200_attn_prefill.

@@ -26,7 +26,7 @@ struct Params {
   void* out;
   const int *block_tables, *seq_lens, *qsl;
   const float* sinks;
-  int T, R, Hq, Hkv, D, max_blocks, block_size, window;
+  int T, R, Hq, Hkv, D, max_blocks, block_size, window, ldo;
   long long num_blocks;
   float scale, softcap;
 };
@@ -45,7 +45,7 @@ __global__ void __launch_bounds__(32 * WARPS) attn_simt_kernel(const Params p) {
   int r = -1;
   for (int i = 0; i < p.R; ++i)
     if (t >= p.qsl[i] && t < p.qsl[i + 1]) { r = i; break; }
-  E* out = reinterpret_cast<E*>(p.out) + ((size_t)t * p.Hq + h) * p.D;
+  E* out = reinterpret_cast<E*>(p.out) + (size_t)t * p.ldo + h * p.D;
   if (r < 0) {                                    // a row of padding
     for (int d = lane; d < p.D; d += 32) put(out + d, 0.f);
     return;
@@ -55,7 +55,7 @@ __global__ void __launch_bounds__(32 * WARPS) attn_simt_kernel(const Params p) {
   for (int d = lane; d < p.D; d += 32) q[d] = to_f(qp[d]);
   __syncwarp();
   const int pos = p.seq_lens[r] - (p.qsl[r + 1] - t);
-  const int first = p.window > 0 ? max(0, pos - p.window + 1) : 0;
+  const int first = first_key(p.window, pos);
   const int hk = h / (p.Hq / p.Hkv);
   const int* bt = p.block_tables + (size_t)r * p.max_blocks;
   const size_t page = (size_t)p.block_size * p.D;
@@ -131,11 +131,11 @@ static int launch(const Params& p, cudaStream_t stream) {
 }  // namespace as
 }  // namespace b200
 
-// q, out [T, Hq, D], kv [blocks, 2, Hkv, block_size, D]; D % 4 == 0, D <= 512; elem: 2 = bf16, 4 = fp32.
+// q, out [T, Hq, D] (out: rows ldo elements apart, 0: Hq * D), kv [blocks, 2, Hkv, block_size, D]; D % 4 == 0, D <= 512; elem: 2 = bf16, 4 = fp32.
 extern "C" int b200_attn_simt(const void* q, const void* kv, void* out, const int* block_tables, const int* seq_lens,
                               const int* qsl, int T, int R, int Hq, int Hkv, int D, int max_blocks, int block_size,
-                              long long num_blocks, float scale, int window, float softcap, const float* sinks, int elem,
-                              cudaStream_t stream) {
+                              long long num_blocks, float scale, int window, float softcap, const float* sinks, int ldo,
+                              int elem, cudaStream_t stream) {
   using namespace b200;
   if (T <= 0 || R <= 0) return 0;
   if (D % 4 || D > 512 || Hkv <= 0 || Hq % Hkv || (T + as::WARPS - 1) / as::WARPS > 65535) {
@@ -144,6 +144,6 @@ extern "C" int b200_attn_simt(const void* q, const void* kv, void* out, const in
     return -1;
   }
   as::Params p{q, kv, out, block_tables, seq_lens, qsl, sinks, T, R, Hq, Hkv, D, max_blocks, block_size, window,
-               num_blocks, scale, softcap};
+               ldo > 0 ? ldo : Hq * D, num_blocks, scale, softcap};
   return elem == 4 ? as::launch<float>(p, stream) : as::launch<__nv_bfloat16>(p, stream);
 }

@@ -51,6 +51,7 @@ struct Params {
   const float* sinks;
   int* status;
   int max_blocks, block_size, Hq, Hkv, G, BQ, req_begin, req_end, window;
+  int ldo;                             // elements between the output rows of neighbouring tokens (without an epilogue)
   int non_causal;                 // 1: every query row sees the whole sequence (encoders, diffusion)
   long long num_blocks;
   float scale_log2, softcap;
@@ -149,8 +150,7 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
   const int ctx = seq_len - q_len;
   // causal bound of the tile; the whole sequence without the mask
   const int kv_end = active ? (p.non_causal ? seq_len : min(seq_len, ctx + q0 + p.BQ)) : 0;
-  int kv_begin = 0;
-  if (active && p.window > 0) kv_begin = max(0, ctx + q0 - p.window + 1) / BKV * BKV;
+  const int kv_begin = active ? first_key(p.window, ctx + q0) / BKV * BKV : 0;
   const int nchunks = active ? (kv_end - kv_begin + BKV - 1) / BKV : 0;
 
   tc_fence_before();
@@ -270,6 +270,7 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
     const int pos_local = row / p.G, head = h * p.G + row % p.G;
     const bool row_ok = active && (q0 + pos_local) < q_len;
     const int lim = p.non_causal ? seq_len - 1 : ctx + q0 + pos_local;    // last visible key of this row
+    const int first = first_key(p.window, max(lim, 0));
     constexpr int HC = BKV / 2, HD = D / 2;
     float acc[HD];
 #pragma unroll
@@ -290,7 +291,7 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
       // columns [c_lo, c_hi) of this thread's 64 are visible to the row (causal limit, end of the
       // sequence, sliding window); most chunks are fully visible
       const int c_hi = min(HC, min(lim, kv_end - 1) - tok0 + 1);
-      const int c_lo = p.window > 0 ? max(0, lim - p.window + 1 - tok0) : 0;
+      const int c_lo = max(0, first - tok0);
       const bool full = c_lo <= 0 && c_hi >= HC;
       const bool capped = p.softcap > 0.f;
       // pass 1: row maximum (raw scores; the scale is positive, the soft-cap monotonic)
@@ -473,7 +474,7 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
         m = n;
       }
       const float inv = l > 0.f ? sc / l : 0.f;
-      __nv_bfloat16* dst = p.out + ((size_t)(qs + q0 + pos_local) * p.Hq + head) * D + half * HD;
+      __nv_bfloat16* dst = p.out + (size_t)(qs + q0 + pos_local) * p.ldo + head * D + half * HD;
 #pragma unroll
       for (int i = 0; i < HD; i += 8) {
         uint4 o;
@@ -508,11 +509,12 @@ static int attn_prefill_tc_impl(const void* q, const void* kv, void* out, float*
                                 const int* seq_lens, const int* qsl, int req_begin, int req_end, int num_tiles_64,
                                 int total_tokens, int max_blocks, int block_size, long long num_blocks, int Hq,
                                 int Hkv, int D, float scale, int window, float softcap, const float* sinks,
-                                int* status, int non_causal, cudaStream_t stream, const HeadFinish* fin = nullptr) {
+                                int* status, int non_causal, cudaStream_t stream, const HeadFinish* fin = nullptr,
+                                int ldo = 0) {
   if (req_end <= req_begin || num_tiles_64 <= 0) return 0;
   const int G = Hkv > 0 ? Hq / Hkv : 0;
-  if (D != 128 || Hq % Hkv || (G != 1 && G != 2 && G != 4 && G != 8) || block_size % 16) {
-    b200_set_last_error("attn_prefill_tc: head_dim 128, q heads per kv head in {1,2,4,8}, block_size % 16 == 0",
+  if (D != 128 || Hq % Hkv || (G != 1 && G != 2 && G != 4 && G != 8) || block_size % 16 || ldo % 8) {
+    b200_set_last_error("attn_prefill_tc: head_dim 128, q heads per kv head in {1,2,4,8}, block_size % 16 == 0, rows of 16 bytes",
                         __FILE__, __LINE__);
     return -1;
   }
@@ -523,6 +525,7 @@ static int attn_prefill_tc_impl(const void* q, const void* kv, void* out, float*
   p.max_blocks = max_blocks; p.block_size = block_size; p.Hq = Hq; p.Hkv = Hkv; p.G = G; p.BQ = fa::BM / G;
   p.req_begin = req_begin; p.req_end = req_end; p.window = window; p.num_blocks = num_blocks;
   p.non_causal = non_causal;
+  p.ldo = ldo > 0 ? ldo : Hq * D;
   p.scale_log2 = scale * 1.4426950408889634f;
   p.softcap = softcap > 0.f ? softcap * 1.4426950408889634f : 0.f;
   CUtensorMap tmQ, tmKV;
@@ -557,10 +560,11 @@ extern "C" int b200_attn_prefill_tc(const void* q, const void* kv, void* out, fl
                                     const int* seq_lens, const int* qsl, int req_begin, int req_end,
                                     int num_tiles_64, int total_tokens, int max_blocks, int block_size,
                                     long long num_blocks, int Hq, int Hkv, int D, float scale, int window,
-                                    float softcap, const float* sinks, int* status, cudaStream_t stream) {
+                                    float softcap, const float* sinks, int ldo, int* status,
+                                    cudaStream_t stream) {
   return attn_prefill_tc_impl(q, kv, out, lse, block_tables, seq_lens, qsl, req_begin, req_end, num_tiles_64,
                               total_tokens, max_blocks, block_size, num_blocks, Hq, Hkv, D, scale, window, softcap,
-                              sinks, status, 0, stream);
+                              sinks, status, 0, stream, nullptr, ldo);
 }
 
 // The same with the epilogue of HeadFinish: out [T, lam ? Hq / 2 : Hq, D].

@@ -81,6 +81,9 @@ FAMILY_SOURCES = {
     "zeganex": ("attention.cu", "attention_simt.cu", "attention_tc.cu", "conv_cache.cu", "elementwise.cu",
                 "gemm_2sm_tcgen05.cu", "gemm_simt.cu", "gemm_tcgen05.cu", "layer_norm.cu", "moe.cu", "runtime.cu",
                 "sample.cu"),
+    "vipolix": ("attention.cu", "attention_simt.cu", "attention_tc.cu", "conv_cache.cu", "elementwise.cu",
+                "gemm_2sm_tcgen05.cu", "gemm_simt.cu", "gemm_tcgen05.cu", "layer_norm.cu", "linear_attention.cu", "moe.cu",
+                "runtime.cu", "sample.cu", "token_shift.cu"),
 }
 
 

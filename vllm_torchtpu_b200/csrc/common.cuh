@@ -379,12 +379,28 @@ __device__ __forceinline__ T warp_max(T v) {
 
 __device__ __forceinline__ float gelu_erf(float v) { return 0.5f * v * (1.f + erff(v * 0.70710678118654752f)); }
 
-// act(gate) * up: silu, or gelu in its tanh form (tanh from one exponential)
-template <bool GELU_TANH>
-__device__ __forceinline__ float gated_pair(float g, float u) {
-  if constexpr (!GELU_TANH) return g / (1.f + __expf(-g)) * u;
-  const float z = 0.7978845608028654f * (g + 0.044715f * g * g * g);
-  return g * (1.f - __fdividef(1.f, 1.f + __expf(2.f * z))) * u;      // 0.5 (1 + tanh z) = 1 - 1 / (1 + e^2z)
+// gelu in its tanh form, tanh from one exponential: 0.5 (1 + tanh z) = 1 - 1 / (1 + e^2z)
+__device__ __forceinline__ float gelu_tanh(float v) {
+  const float z = 0.7978845608028654f * (v + 0.044715f * v * v * v);
+  return v * (1.f - __fdividef(1.f, 1.f + __expf(2.f * z)));
+}
+// gate and up projection of a feed-forward -> its activation.  ACT as the GEMMs number them: 0 silu(g) u,
+// 3 gelu(g) u in the tanh form, 5 g' sigmoid(alpha g') (u' + 1) with g' = min(g, limit), u' = clamp(u, -limit, limit)
+template <int ACT>
+__device__ __forceinline__ float gated_pair(float g, float u, float alpha, float limit) {
+  if constexpr (ACT == 3) return gelu_tanh(g) * u;
+  if constexpr (ACT == 5) {
+    g = fminf(g, limit);
+    u = fminf(fmaxf(u, -limit), limit);
+    return __fdividef(g, 1.f + __expf(-alpha * g)) * (u + 1.f);
+  }
+  return g / (1.f + __expf(-g)) * u;
+}
+
+// First key that the query at position pos sees: of the last `window` ones (> 0), of its own chunk of -window positions (< 0,
+// chunks are counted from position 0), of all (0).
+__device__ __forceinline__ int first_key(int window, int pos) {
+  return window > 0 ? max(0, pos - window + 1) : (window < 0 ? pos - pos % -window : 0);
 }
 
 __device__ __forceinline__ float relu_squared(float v) { return v > 0.f ? v * v : 0.f; }

@@ -3,7 +3,7 @@
 //
 //   y_t = sum_j w[j] u_(t - taps + 1 + j)     per channel of q, k and v (zeros in front of the sequence)
 //   q, k: dimensions 2i, 2i + 1 of a head (of one map) turn by position * inv_freq[i], cos and sin times rot_mult
-//   q -> q_out [T, heads * maps, D];   k, v -> page of the token's slot
+//   q times one number per head (q_scale, optional) -> q_out [T, heads * maps, D];   k, v -> page of the token's slot
 //
 // Heads are stored in D columns with zeros behind them.  With two maps per head a key row holds both maps side by side and
 // query row 2h + m has its map's columns only, so that plain attention over D columns gives the scores of one map.
@@ -27,7 +27,7 @@ __device__ __forceinline__ void put(__nv_bfloat16* p, float v) { *p = __float2bf
 struct Params {
   const void *row, *w;                 // w [taps, channels]
   void *q_out, *cache, *ring;
-  const float* inv_freq;
+  const float *inv_freq, *q_scale;
   const int *slots, *qsl, *seq_lens, *state_slots;
   int ldr, q_off, k_off, v_off, H, G, dim, vdim, maps, D, taps, pairs, block_size, T, R;
   long long num_slots;
@@ -201,8 +201,11 @@ __global__ void __launch_bounds__(THREADS, 4) conv_cache_kernel(const Params p) 
     E* cache = reinterpret_cast<E*>(p.cache) + (size_t)(x.hh - nq) * p.block_size * p.D + x.d0;
     const size_t q_step = (size_t)nq * p.D;
     const bool is_q = x.hh < nq;
-    auto save = [&](int i, const float (&y)[V]) {          // (a thread's rows of q are written in order)
+    const float scale = is_q && p.q_scale != nullptr ? p.q_scale[x.hh / p.maps] : 1.f;
+    auto save = [&](int i, float (&y)[V]) {                // (a thread's rows of q are written in order)
       if (is_q) {
+#pragma unroll
+        for (int e = 0; e < V; ++e) y[e] *= scale;
         store<E, V, VEC>(q_out, y);
         q_out += q_step;
       } else if (tok[i].cell >= 0) {
@@ -420,7 +423,8 @@ static int launch_combine(const CombineParams& p, cudaStream_t stream) {
 // [blocks, 2, G, block_size, D] (G 0: none); elem: 2 = bf16, 4 = fp32 (all alike).  Requests from ring_from on may have
 // portions of several tokens; single: every request has one token; only_ring: nothing but the rings advances.
 extern "C" int b200_conv_cache(const void* row, int ldr, int q_off, int k_off, int v_off, const void* w, int taps,
-                               void* ring, const float* inv_freq, int pairs, float rot_mult, void* q_out, void* cache,
+                               void* ring, const float* inv_freq, int pairs, float rot_mult, const float* q_scale,
+                               void* q_out, void* cache,
                                const int* slots, const int* qsl, const int* seq_lens, const int* state_slots, int T, int R,
                                int H, int G, int dim, int vdim, int maps, int D, int block_size, long long num_blocks,
                                int ring_from, int single, int only_ring, int elem, cudaStream_t stream) {
@@ -432,7 +436,7 @@ extern "C" int b200_conv_cache(const void* row, int ldr, int q_off, int k_off, i
                         __FILE__, __LINE__);
     return -1;
   }
-  cc::Params p{row, w, q_out, cache, ring, inv_freq, slots, qsl, seq_lens, state_slots, ldr, q_off, k_off, v_off, H, G, dim,
+  cc::Params p{row, w, q_out, cache, ring, inv_freq, q_scale, slots, qsl, seq_lens, state_slots, ldr, q_off, k_off, v_off, H, G, dim,
                vdim, maps, D, taps, pairs, block_size, T, R, num_blocks * block_size, rot_mult};
   return elem == 4 ? cc::launch<float>(p, ring_from, only_ring, single, stream)
                    : cc::launch<__nv_bfloat16>(p, ring_from, only_ring, single, stream);

@@ -61,6 +61,7 @@ struct Params {
   int T, N, K, ldy;
   int n_pairs, t_tiles, kb_total;
   int up_row_off;                  // SwiGLU: first up row of W (= I)
+  float alpha, limit;              // of the clamped activation
 };
 
 __device__ __forceinline__ void tmem_alloc_2sm(uint32_t* smem_dst, uint32_t ncols) {
@@ -120,12 +121,12 @@ __device__ __forceinline__ void decode_work(int w, const Params& p, int& n_pair,
   n_pair = first + rem - t_tile * gsize;
 }
 
-// EPI 0: bias, 1: SwiGLU, 2: gelu (erf), 3: gate and up as in 1 with gelu in its tanh form
+// EPI 0: bias, 1: SwiGLU, 2: gelu (erf); gate and up as in 1 with another activation: 3 gelu in its tanh form, 5 clamped
 template <int EPI>
 __global__ void __cluster_dims__(2, 1, 1) __launch_bounds__(THREADS, 1)
 gemm_bf16_2sm_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant__ CUtensorMap tmX,
                      const Params p) {
-  constexpr bool SWIGLU = EPI == 1 || EPI == 3;
+  constexpr bool SWIGLU = EPI == 1 || EPI == 3 || EPI == 5;
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
   uint64_t* bars = reinterpret_cast<uint64_t*>(smem + STAGES * STAGE_BYTES);
@@ -278,7 +279,8 @@ gemm_bf16_2sm_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_const
               for (int j = 0; j < 16; ++j) {
                 if (c0 + 16 + j < t_valid) {
                   const float gv = buf[(16 + j) * 32 + lane], uv = __uint_as_float(r[16 + j]);
-                  yp[(size_t)j * p.ldy] = __float2bfloat16(EPI == 3 ? gated_pair<true>(gv, uv) : __fdividef(gv, 1.f + __expf(-gv)) * uv);
+                  yp[(size_t)j * p.ldy] = __float2bfloat16(EPI == 1 ? __fdividef(gv, 1.f + __expf(-gv)) * uv
+                                                                     : gated_pair<EPI>(gv, uv, p.alpha, p.limit));
                 }
               }
             } else {             // gate warp: columns 0-15, up values from the partner
@@ -287,7 +289,8 @@ gemm_bf16_2sm_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_const
               for (int j = 0; j < 16; ++j) {
                 if (c0 + j < t_valid) {
                   const float gv = __uint_as_float(r[j]), uv = buf[j * 32 + lane];
-                  yp[(size_t)j * p.ldy] = __float2bfloat16(EPI == 3 ? gated_pair<true>(gv, uv) : __fdividef(gv, 1.f + __expf(-gv)) * uv);
+                  yp[(size_t)j * p.ldy] = __float2bfloat16(EPI == 1 ? __fdividef(gv, 1.f + __expf(-gv)) * uv
+                                                                     : gated_pair<EPI>(gv, uv, p.alpha, p.limit));
                 }
               }
             }
@@ -450,10 +453,10 @@ extern "C" int b200_gemm_bf16_gelu_2sm(const void* X, const void* W, void* Y, in
   return gemm_bf16_2sm(X, W, Y, nullptr, T, N, K, ldx, ldw, ldy, status, num_sms, 1, stream);
 }
 
-// Y[T, I] = act(X * W[0:I]^T) * (X * W[I:2I]^T), act silu or gelu (tanh form); W [2I, K] row stride ldw.
+// Y[T, I] = gated_pair<act>(X * W[0:I]^T, X * W[I:2I]^T); W [2I, K] row stride ldw.
 extern "C" int b200_gemm_bf16_swiglu_2sm(const void* X, const void* W, void* Y, int T, int I, int K, int ldx,
-                                         int ldw, int ldy, int gelu_tanh, int* status, int num_sms,
-                                         cudaStream_t stream) {
+                                         int ldw, int ldy, int act, float alpha, float limit, int* status,
+                                         int num_sms, cudaStream_t stream) {
   using namespace b200;
   using namespace b200::g2;
   if (T <= 0 || I <= 0 || K <= 0) return 0;
@@ -475,5 +478,7 @@ extern "C" int b200_gemm_bf16_swiglu_2sm(const void* X, const void* W, void* Y, 
   if (rc) return rc;
   rc = operand_map(&tmX, X, (uint64_t)T, (uint64_t)K, (uint64_t)ldx * 2);
   if (rc) return rc;
-  return gelu_tanh ? launch_pairs<3>(tmW, tmX, p, num_sms, stream) : launch_pairs<1>(tmW, tmX, p, num_sms, stream);
+  p.alpha = alpha; p.limit = limit;
+  if (act == 5) return launch_pairs<5>(tmW, tmX, p, num_sms, stream);
+  return act == 3 ? launch_pairs<3>(tmW, tmX, p, num_sms, stream) : launch_pairs<1>(tmW, tmX, p, num_sms, stream);
 }

@@ -3,6 +3,7 @@
 // the TMA granule.  Batched over heads, with the epilogues the tcgen05 kernels have:
 //
 //   Y[t, b * ys + n] = act( sum_k X[t, b * xs + k] * W[b * N + n, k] + bias[n] ) [ * sigmoid(G[t, b * N + n]) ]
+//   with gate_rows:  Y[t, n] = gelu( . ) * G[gate_rows[t], n], gelu in its tanh form
 //
 // act: 0 none, 1 gelu (erf), 2 out_scale and soft cap (cap * tanh(. / cap), cap 0: none) with fp32 output.  64 x 64 output tile per CTA, 4 x 4 per thread, 16-wide K slices in shared memory.
 #include "common.cuh"
@@ -18,6 +19,8 @@ template <> __device__ __forceinline__ __nv_bfloat16 from_f<__nv_bfloat16>(float
 
 struct Params {
   const void *x, *w, *bias, *gate;
+  const int* gate_rows;
+  int gate_count;
   void* y;
   int T, N, K, batch, act, y_f32;
   float cap, out_scale;
@@ -72,7 +75,11 @@ __global__ void __launch_bounds__(256) gemm_kernel(const Params p) {
         if (p.bias) v += to_f(reinterpret_cast<const E*>(p.bias)[n]);
         if (p.act == 1) v = gelu_erf(v);
         if (p.act == 2) v = soft_cap(v * p.out_scale, p.cap);
-        if (p.gate) {
+        if (p.gate_rows) {
+          const int row = min(max(p.gate_rows[t], 0), p.gate_count - 1);
+          const float z = 0.7978845608028654f * (v + 0.044715f * v * v * v);
+          v = 0.5f * v * (1.f + tanhf(z)) * to_f(reinterpret_cast<const E*>(p.gate)[(size_t)row * p.ldg + n]);
+        } else if (p.gate) {
           const float g = to_f(reinterpret_cast<const E*>(p.gate)[(size_t)t * p.ldg + (size_t)b * p.N + n]);
           v *= 1.f / (1.f + expf(-g));
         }
@@ -149,13 +156,14 @@ extern "C" int b200_grouped_gemm_simt(const void* x, const void* w, void* y, con
   return 0;
 }
 
-// elem: 2 = bf16, 4 = fp32 (all operands alike); strides in elements.
-extern "C" int b200_gemm_simt(const void* x, const void* w, void* y, const void* bias, const void* gate, int T, int N,
-                              int K, int batch, long long ldx, long long ldw, long long ldy, long long ldg,
+// elem: 2 = bf16, 4 = fp32 (all operands alike); strides in elements.  gate_rows (or null): token t's gate is row
+// gate_rows[t] of a table of gate_count rows.
+extern "C" int b200_gemm_simt(const void* x, const void* w, void* y, const void* bias, const void* gate,
+                              const int* gate_rows, int gate_count, int T, int N, int K, int batch, long long ldx, long long ldw, long long ldy, long long ldg,
                               long long xs, long long ys, int act, float cap, float out_scale, int elem, cudaStream_t stream) {
   using namespace b200;
   if (T <= 0 || N <= 0 || batch <= 0) return 0;
-  simt::Params p{x, w, bias, gate, y, T, N, K, batch, act, act == 2 ? 1 : 0, cap, out_scale, ldx, ldw, ldy, ldg, xs, ys};
+  simt::Params p{x, w, bias, gate, gate_rows, gate_count, y, T, N, K, batch, act, act == 2 ? 1 : 0, cap, out_scale, ldx, ldw, ldy, ldg, xs, ys};
   const long long gx = (long long)batch * ((N + simt::TN - 1) / simt::TN);
   int gy = (T + simt::TM - 1) / simt::TM;
   if (gy > 65535) gy = 65535;

@@ -21,6 +21,7 @@
 // Pallas quantized_matmul kernels (reference: src/vllm_torchtpu/kernels/quantized_matmul/).
 #include <cstring>
 #include <mutex>
+#include <type_traits>
 #include <unordered_map>
 
 #include "common.cuh"
@@ -99,10 +100,14 @@ struct GemmParams {
   unsigned long long ag_done_off;
   int ag_flip;
   unsigned long long* dbg;               // optional: per-CTA phase timestamps (ns), 16 slots per CTA
-  // ---- gate / up pairs: act 0 silu, 3 gelu (tanh form); grouped products without a gate: act 4 the square of relu
+  // ---- gate / up pairs: act as in gated_pair (0 silu, 3 gelu in its tanh form, 5 clamped with alpha = out_scale and
+  // limit = cap); grouped products without a gate: act 4 the square of relu
   // ---- MODE 3: epilogue (act 0 none / 1 gelu / 2 fp32 output Yf: out_scale * y, then the soft cap (cap 0: none);
   // optional gate: y *= sigmoid(gate[t, b * N + n])) and batch over heads: head b reads activation columns from
-  // b * x_head_cols, weight rows from b * N and writes output columns from b * y_head_cols
+  // b * x_head_cols, weight rows from b * N and writes output columns from b * y_head_cols.  gate_rows: token t's gate is
+  // row gate_rows[t] (below gate_count) of the table, and y = gelu(y) * gate in the tanh form (one head)
+  const int* gate_rows;
+  int gate_count;
   int act, batch, x_head_cols, y_head_cols, ldg;
   float cap, out_scale;
   const __nv_bfloat16* gate;
@@ -111,6 +116,17 @@ struct GemmParams {
   int* cta_done;                         // local: CTA exit counter
   unsigned int spin_limit;
 };
+
+// gate and up sums -> activation
+__device__ __forceinline__ float gated_by(const GemmParams& p, float g, float u) {
+  if (p.act == 3) return gated_pair<3>(g, u, 0.f, 0.f);
+  if (p.act == 5) return gated_pair<5>(g, u, p.out_scale, p.cap);
+  return gated_pair<0>(g, u, 0.f, 0.f);
+}
+// row of the gate table that belongs to token t
+__device__ __forceinline__ const __nv_bfloat16* token_gate(const GemmParams& p, int t) {
+  return p.gate + (size_t)min(max(p.gate_rows[t], 0), p.gate_count - 1) * p.ldg;
+}
 
 constexpr int NUM_THREADS_FUSED = NUM_THREADS + 128;   // + 4 reducer warps
 
@@ -342,13 +358,15 @@ __device__ __forceinline__ void cluster_reduce_cols(const GemmParams& p, const W
 #pragma unroll
           for (int r2 = 0; r2 < SMAX; ++r2)
             if (r2 < S) { u.x += vu[ci][r2].x; u.y += vu[ci][r2].y; u.z += vu[ci][r2].z; u.w += vu[ci][r2].w; }
-          if (p.act == 3) {
-            a.x = gated_pair<true>(a.x, u.x); a.y = gated_pair<true>(a.y, u.y);
-            a.z = gated_pair<true>(a.z, u.z); a.w = gated_pair<true>(a.w, u.w);
-          } else {
-            a.x = gated_pair<false>(a.x, u.x); a.y = gated_pair<false>(a.y, u.y);
-            a.z = gated_pair<false>(a.z, u.z); a.w = gated_pair<false>(a.w, u.w);
-          }
+          a.x = gated_by(p, a.x, u.x); a.y = gated_by(p, a.y, u.y);
+          a.z = gated_by(p, a.z, u.z); a.w = gated_by(p, a.w, u.w);
+        }
+        if (MODE == 3 && p.gate_rows != nullptr) {
+          const __nv_bfloat16* gp = token_gate(p, wk.t_row + c) + n4;
+          float vals[4] = {a.x, a.y, a.z, a.w};
+#pragma unroll
+          for (int j = 0; j < 4; ++j) vals[j] = n4 + j < p.N ? gelu_tanh(vals[j]) * __bfloat162float(gp[j]) : 0.f;
+          a = make_float4(vals[0], vals[1], vals[2], vals[3]);
         }
         if (MODE == 3 && p.act == 1) {           // (no bias in this mode)
           a.x = gelu_erf(a.x); a.y = gelu_erf(a.y); a.z = gelu_erf(a.z); a.w = gelu_erf(a.w);
@@ -622,19 +640,16 @@ gemm_bf16_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant_
           tmem_ld_wait();
           if (n < p.N) {
             __nv_bfloat16* yp = dst_base + (size_t)(t0 + c0) * p.ldy + n;
-            if (p.act == 3) {
+            auto put = [&](auto act) {
 #pragma unroll
               for (int j = 0; j < 32; ++j)
                 if (c0 + j < t_valid)
-                  yp[(size_t)j * p.ldy] =
-                      __float2bfloat16(gated_pair<true>(__uint_as_float(g[j]), __uint_as_float(u[j])));
-            } else {
-#pragma unroll
-              for (int j = 0; j < 32; ++j)
-                if (c0 + j < t_valid)
-                  yp[(size_t)j * p.ldy] =
-                      __float2bfloat16(gated_pair<false>(__uint_as_float(g[j]), __uint_as_float(u[j])));
-            }
+                  yp[(size_t)j * p.ldy] = __float2bfloat16(gated_pair<decltype(act)::value>(
+                      __uint_as_float(g[j]), __uint_as_float(u[j]), p.out_scale, p.cap));
+            };
+            if (p.act == 3) put(std::integral_constant<int, 3>());
+            else if (p.act == 5) put(std::integral_constant<int, 5>());
+            else put(std::integral_constant<int, 0>());
           }
         }
         tc_fence_before();
@@ -747,6 +762,14 @@ gemm_bf16_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant_
               const TileDst td = tile_dst<BN, MODE>(p, wk, d);
               __nv_bfloat16* yp = td.base + (size_t)c0 * td.cs + row;
               if constexpr (MODE == 3) {
+                if (p.gate_rows != nullptr) {
+#pragma unroll 4
+                  for (int j = 0; j < 32; ++j)
+                    if (c0 + j < t_valid)
+                      yp[(size_t)j * td.cs] = __float2bfloat16(gelu_tanh(__uint_as_float(r[j])) *
+                                                               __bfloat162float(token_gate(p, t0 + c0 + j)[n]));
+                  continue;
+                }
                 if (p.gate != nullptr) {
                   const __nv_bfloat16* gp = p.gate + (size_t)(t0 + c0) * p.ldg + (size_t)wk.head * p.N + n;
                   float gv[32];
@@ -1459,9 +1482,10 @@ extern "C" int b200_gemm_bf16(const void* X, const void* W, void* Y, const void*
 // whose K is no multiple of the 64-wide K block reads into its neighbour's columns; those meet the zero fill
 // behind the weight's K columns.
 // act 2: Y is fp32 and holds cap * tanh(out_scale * . / cap) (cap 0: out_scale * the products).
-extern "C" int b200_gemm_bf16_heads(const void* X, const void* W, void* Y, const void* gate, int T, int N, int K,
-                                    int batch, int ldx, int ldw, int ldy, int ldg, int xs, int ys, int act, float cap,
-                                    float out_scale, int* status, int num_sms, cudaStream_t stream) {
+// gate_rows: Y[t, n] = gelu(.) * gate[gate_rows[t], n], gelu in its tanh form.
+static int gemm_bf16_heads(const void* X, const void* W, void* Y, const void* gate, const int* gate_rows, int gate_count,
+                           int T, int N, int K, int batch, int ldx, int ldw, int ldy, int ldg, int xs, int ys, int act,
+                           float cap, float out_scale, int* status, int num_sms, cudaStream_t stream) {
   using namespace b200;
   if (T <= 0 || N <= 0 || K <= 0 || batch <= 0) return 0;
   if (ldx % 8 || ldw % 8 || xs % 8) {
@@ -1480,6 +1504,8 @@ extern "C" int b200_gemm_bf16_heads(const void* X, const void* W, void* Y, const
     return -3;
   }
   p.gate = reinterpret_cast<const __nv_bfloat16*>(gate);
+  p.gate_rows = gate_rows;
+  p.gate_count = gate_count;
   p.status = status;
   p.T = T; p.N = N; p.K = K; p.ldy = ldy; p.ldg = ldg;
   p.batch = batch; p.x_head_cols = xs; p.y_head_cols = ys; p.act = act;
@@ -1490,7 +1516,7 @@ extern "C" int b200_gemm_bf16_heads(const void* X, const void* W, void* Y, const
   p.t_tiles = (T + bn - 1) / bn;
   p.kb_total = (K + BK - 1) / BK;
   const int tiles = p.n_tiles * p.t_tiles;
-  if (batch > 1 || gate != nullptr) splits = 1;
+  if (batch > 1 || (gate != nullptr && gate_rows == nullptr)) splits = 1;
   if (splits > p.kb_total) splits = p.kb_total;
   if (splits > 1) splits = fit_cluster_splits(splits, tiles, bn, NUM_THREADS);
   p.splits = splits;
@@ -1514,6 +1540,25 @@ extern "C" int b200_gemm_bf16_heads(const void* X, const void* W, void* Y, const
     case 128: return launch_gemm<128>(tmW, tmX, p, grid, stream);
     default: return launch_gemm<256>(tmW, tmX, p, grid, stream);
   }
+}
+
+extern "C" int b200_gemm_bf16_heads(const void* X, const void* W, void* Y, const void* gate, int T, int N, int K,
+                                    int batch, int ldx, int ldw, int ldy, int ldg, int xs, int ys, int act, float cap,
+                                    float out_scale, int* status, int num_sms, cudaStream_t stream) {
+  return gemm_bf16_heads(X, W, Y, gate, nullptr, 0, T, N, K, batch, ldx, ldw, ldy, ldg, xs, ys, act, cap, out_scale, status,
+                         num_sms, stream);
+}
+
+// Y[t, n] = gelu(X[t] . W[n]) * table[ids[t], n] (gelu in its tanh form; table rows ldg elements apart, count of them)
+extern "C" int b200_gemm_bf16_token_gate(const void* X, const void* W, void* Y, const void* table, int ldg, int count,
+                                         const int* ids, int T, int N, int K, int ldx, int ldw, int ldy, int* status,
+                                         int num_sms, cudaStream_t stream) {
+  if (table == nullptr || ids == nullptr || count <= 0) {
+    b200_set_last_error("gemm_token_gate: a table and the rows' token ids are needed", __FILE__, __LINE__);
+    return -3;
+  }
+  return gemm_bf16_heads(X, W, Y, table, ids, count, T, N, K, 1, ldx, ldw, ldy, ldg, 0, 0, 0, 0.f, 1.f, status, num_sms,
+                         stream);
 }
 
 // Row-parallel GEMM fused with the cross-rank reduction: Y = sum over ranks of X_r * W_r^T.
@@ -1625,10 +1670,9 @@ static void init_params(GemmParams& p, void* Y, int T, int N, int K, int ldy, in
 }
 }  // namespace b200
 
-// Y[T, I] = act(X * Wg^T) * (X * Wu^T) with W = [gate rows (I) ; up rows (I)] x K packed as [2I, K]; act: silu, or
-// gelu in its tanh form.
-extern "C" int b200_gemm_bf16_swiglu(const void* X, const void* W, void* Y, int T, int I, int K, int ldx,
-                                     int ldw, int ldy, int gelu_tanh, int* status, int num_sms, cudaStream_t stream) {
+// Y[T, I] = gated_pair<act>(X * Wg^T, X * Wu^T) with W = [gate rows (I) ; up rows (I)] x K packed as [2I, K].
+extern "C" int b200_gemm_bf16_swiglu(const void* X, const void* W, void* Y, int T, int I, int K, int ldx, int ldw, int ldy,
+                                     int act, float alpha, float limit, int* status, int num_sms, cudaStream_t stream) {
   using namespace b200;
   if (T <= 0 || I <= 0 || K <= 0) return 0;
   if (K % 8 || ldx % 8 || ldw % 8) {
@@ -1639,7 +1683,7 @@ extern "C" int b200_gemm_bf16_swiglu(const void* X, const void* W, void* Y, int 
   GemmParams p;
   init_params(p, Y, T, I, K, ldy, bn, status);
   p.up_row_off = I;
-  p.act = gelu_tanh ? 3 : 0;
+  p.act = act; p.out_scale = alpha; p.cap = limit;
   p.w_evict_first = (p.t_tiles == 1) ? 1 : 0;
   {
     // few output tiles (small I per rank under tensor parallelism): split K over a cluster so that
@@ -1679,10 +1723,10 @@ extern "C" int b200_gemm_bf16_swiglu(const void* X, const void* W, void* Y, int 
 //   rows [group_off[e], group_off[e+1]) of X use weight W[e] ([N, K], or [2N, K] gate/up when swiglu).
 // X: [R, K]; Y: [R, N].  group_off lives in device memory, so the launch is CUDA-graph safe; the
 // grid is one persistent CTA per SM and CTAs without work exit.  avg_rows_hint picks the token tile.
-// act (without swiglu): 0 none, 4 the square of relu.
+// act with swiglu: as in gated_pair, with its alpha and limit; without: 0 none, 4 the square of relu.
 extern "C" int b200_grouped_gemm_bf16(const void* X, const void* W, void* Y, const int* group_off,
-                                      int num_groups, int R, int N, int K, int swiglu, int act, int avg_rows_hint,
-                                      int* status, int num_sms, cudaStream_t stream) {
+                                      int num_groups, int R, int N, int K, int swiglu, int act, float alpha, float limit,
+                                      int avg_rows_hint, int* status, int num_sms, cudaStream_t stream) {
   using namespace b200;
   if (R <= 0 || N <= 0 || K <= 0 || num_groups <= 0) return 0;
   if (K % 8 || N % BM || num_groups > MAX_GROUPS) {
@@ -1695,7 +1739,7 @@ extern "C" int b200_grouped_gemm_bf16(const void* X, const void* W, void* Y, con
   init_params(p, Y, R, N, K, N, bn, status);
   p.group_off = group_off;
   p.num_groups = num_groups;
-  if (!swiglu) p.act = act;
+  p.act = act; p.out_scale = alpha; p.cap = limit;
   p.w_rows_per_group = swiglu ? 2 * N : N;
   p.up_row_off = N;
   p.w_evict_first = avg_rows_hint <= bn ? 1 : 0;

@@ -6,7 +6,7 @@
 //
 // and of blocks that normalise the INPUT of a sublayer (RMS norm, weight stored with an offset):
 //
-//   add_rms: r' = r (+ y),  o = r' / rms(r') * (offset + w)     (r' fp32)
+//   add_rms: r' = r (+ mult * y),  o = r' / rms(r') * (offset + w)     (r' fp32)
 //
 // and of blocks that do both: the output y is normalised and scaled first, r' = r + mult * y / rms(y) * post.
 //
@@ -157,7 +157,7 @@ __global__ void add_rms_norm_kernel(const TY* __restrict__ y, const TR* res, con
       float a[V];
       load<V>(y + base + i, a);
 #pragma unroll
-      for (int j = 0; j < V; ++j) v[j] += a[j];
+      for (int j = 0; j < V; ++j) v[j] = fmaf(mult, a[j], v[j]);
     }
     if (res_out != nullptr) store<V>(res_out + base + i, v);
 #pragma unroll
@@ -251,7 +251,7 @@ extern "C" int b200_layer_norm(const void* x, int x_elem, const void* w, int w_e
 }
 
 // y (or null): type of w; res: element bytes res_elem; w, post and out: w_elem (2 = bf16, 4 = fp32); res_out fp32 or null;
-// post (or null): weight of the norm y passes first, times mult.
+// post (or null): weight of the norm y passes first; mult: factor on what is added.
 extern "C" int b200_add_rms_norm(const void* y, const void* res, int res_elem, const void* w, const void* post, int w_elem,
                                  void* res_out, void* out, int T, int H, float eps, float offset, float mult,
                                  cudaStream_t stream) {

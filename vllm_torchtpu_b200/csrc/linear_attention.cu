@@ -1,7 +1,9 @@
-// Linear attention with a carried state per request and head (S is [dk, dv], fp32), two rules:
+// Linear attention with a carried state per request and head (S is [dk, dv], fp32), four rules:
 //
-//   fixed decay per head:           S <- decay_h S + k v^T
-//   delta rule, decay per channel:  S <- g S (rows);  u = beta (v - S^T k);  S <- S + k u^T
+//   FIXED, decay per head:       S <- decay_h S + k v^T
+//   CHANNEL, decay per channel:  S <- g S (rows) + k v^T
+//   DELTA, decay per channel:    S <- g S (rows);  u = beta (v - S^T k);  S <- S + k u^T
+//   REMOVAL, decay and rate per channel, both on the old state:  S <- g S + b (S^T n)^T + k v^T,  n = k / |k|, b = -a * n
 //
 //   o = S^T q;   y = o / rms(o) [* norm] * act(gate)
 //
@@ -20,8 +22,12 @@
 //        A_ij = beta_i sum_c k_ic k_jc 2^(G_ic - G_jc) (i > j),  Q_ij the same with q_i and i >= j;
 //        (I + A) U = beta v,  (I + A) W = beta k 2^G  by forward substitution;  q' = q 2^G,  k' = k 2^(G_last - G).
 //        Decay factors only ever appear as 2^(difference <= 0).
+//        REMOVAL, where M_i = S_(i-1)^T n_i:  with e_i = n_i / (decay of token i), a factor of at most 2 (exp(exp(-1/2))),
+//        A_ij = sum_c e_ic a_jc n_jc 2^(G_ic - G_jc),  (I + A) M0 = (the same with k_j in place of a_j n_j) V,
+//        (I + A) W = e 2^G;  Q_ij as above with b_j, K_ij with k_j;  b' = b 2^(G_last - G).
 //      lin_scan_kernel (sequential over chunks, one warp per 16 value columns, no exchange between warps):
-//        U' = U - W S,  O = q' S + Q U',  S <- 2^G_last S + k'^T U'.
+//        U' = U - W S,  O = q' S + Q U',  S <- 2^G_last S + k'^T U'
+//        (REMOVAL: M = M0 + W S,  O = q' S + Q M + K V,  S <- 2^G_last S + b'^T M + k'^T V).
 //        The warp keeps S^T as mma accumulators: they are at the same time the A operand of the two products with S
 //        (the contraction index is permuted alike in the B operand), and U'^T comes out in the layout that the update
 //        and Q U' take.  Every operand is a pair of tf32 numbers (three products), fp32 accumulation and state.
@@ -95,18 +101,21 @@ constexpr int C = 16;                 // tokens per chunk
 constexpr float UNIT_EPS = 1e-6f;
 constexpr float LOG2E = 1.4426950408889634f;
 constexpr int AQ_LD = 24;             // row stride of Q in the scratch
+constexpr float REMOVAL_DECAY = 0.6065306597126334f;      // exp(-1/2): decays are exp(-exp(-1/2) sigmoid(z))
+
+enum Rule { FIXED = 0, DELTA = 1, CHANNEL = 2, REMOVAL = 3 };
 
 struct Params {
   const void *row, *a, *gate, *conv_w;
   void *ring, *y;
   float* state;
-  const float *inv_freq, *decay, *A_log, *dt_bias, *norm_w;
+  const float *inv_freq, *decay, *A_log, *dt_bias, *rate_bias, *norm_w;
   const int *qsl, *seq_lens, *slots;
   int ldr, q_off, k_off, v_off, beta_off, lda, ldg, taps, pairs, unit, gate_silu;
-  int T, H, Hk, dk, dv, req_begin, zero_rows;
-  float eps, q_mult, k_mult;
+  int T, H, Hk, dk, dv, req_begin, zero_rows, rate_off, ldy, norm_stride;
+  float eps, q_mult, k_mult, inv_tau;
   // ---- chunked prompts
-  float *qd, *w, *kd, *u, *aq, *gl, *o;
+  float *qd, *w, *kd, *bd, *u, *v, *aq, *ak, *gl, *o;
   int dkp, dvp, slab, chunk_begin;
 };
 
@@ -163,19 +172,20 @@ __device__ __forceinline__ float conv_at(const Params& p, const Req& q, int pos,
 // Between the reads of a token they are in shared memory, where a CTA's whole state arrives by asynchronous copies while
 // q, k, v are prepared (SMEM), in registers, at most RPT rows (REGS), or nowhere: the pool is read twice (POOL).
 enum Hold { POOL, REGS, SMEM };
-template <typename E, bool DELTA, int VEC, int RPT, Hold HOLD>
+template <typename E, int RULE, int VEC, int RPT, Hold HOLD>
 __global__ void __launch_bounds__(HOLD == POOL ? 1024 : (HOLD == REGS ? 512 : 256), HOLD == SMEM ? 3 : 1)
 lin_step_kernel(const Params p) {
   pdl_launch_dependents();
   pdl_wait();
   extern __shared__ __align__(16) float sm[];
   __shared__ float red[32];
-  __shared__ float sc[3];
+  __shared__ float sc[4];
+  constexpr bool MEM = RULE == DELTA || RULE == REMOVAL;     // the state is read along the key before it is written
   const int h = blockIdx.x, r = p.req_begin + blockIdx.y, tid = threadIdx.x, NT = blockDim.x;
   const Req q = request(p, r);
   if (q.len <= 0 || q.slot < 0) {
     if (p.zero_rows && r < p.T)
-      for (int j = tid; j < p.dv; j += NT) put(reinterpret_cast<E*>(p.y) + (size_t)r * p.H * p.dv + h * p.dv + j, 0.f);
+      for (int j = tid; j < p.dv; j += NT) put(reinterpret_cast<E*>(p.y) + (size_t)r * p.ldy + h * p.dv + j, 0.f);
     return;
   }
   const int dk = p.dk, dv = p.dv, n = p.Hk * dk, group = p.H / p.Hk, hk = h / group;
@@ -184,8 +194,9 @@ lin_step_kernel(const Params p) {
   float* sq = sm;                       // [dk]
   float* sk = sq + dk;                  // [dk]
   float* sg = sk + dk;                  // [dk]
-  float* sv = sg + dk;                  // [dv]
-  float* su = sv + dv;                  // [dv]
+  float* sa = sg + dk;                  // [dk] (REMOVAL: rates)
+  float* sv = RULE == REMOVAL ? sa + dk : sa;               // [dv]
+  float* su = sv + dv;                  // [dv]: what is added along k; REMOVAL: S^T n
   float* pm = su + dv;                  // [RG][dv]
   float* po = pm + RG * dv;             // [RG][dv]
   float* st = p.state + ((size_t)q.slot * p.H + h) * dk * dv + VEC * cg;
@@ -221,16 +232,17 @@ lin_step_kernel(const Params p) {
       if (!fresh && x < rows) load_row(rg + x * RG, S[x]);
     }
   }
-  const float a_log = DELTA ? expf(p.A_log[h]) : 0.f;
-  const float decay = DELTA ? 0.f : p.decay[h];
+  const float a_log = RULE == DELTA ? expf(p.A_log[h]) : 0.f;
+  const float decay = RULE == FIXED ? p.decay[h] : 0.f;
+  const float* norm_w = p.norm_w != nullptr ? p.norm_w + (size_t)h * p.norm_stride : nullptr;
   for (int t = q.qs; t < q.qs + q.len; ++t) {
     const int pos = q.start + t - q.qs;
     // needed late, loaded early: step size, output gate and norm weight of this thread's first value column
-    const float b_raw = DELTA ? to_f(reinterpret_cast<const E*>(p.row)[(size_t)t * p.ldr + p.beta_off + h]) : 0.f;
+    const float b_raw = RULE == DELTA ? to_f(reinterpret_cast<const E*>(p.row)[(size_t)t * p.ldr + p.beta_off + h]) : 0.f;
     float g_raw = 0.f, nw = 1.f;
     if (tid < dv) {
       g_raw = to_f(reinterpret_cast<const E*>(p.gate)[(size_t)t * p.ldg + h * dv + tid]);
-      if (p.norm_w != nullptr) nw = p.norm_w[tid];
+      if (norm_w != nullptr) nw = norm_w[tid];
     }
     for (int x = tid; x < 2 * dk + dv; x += NT) {
       const int c = x < dk ? hk * dk + x : (x < 2 * dk ? n + hk * dk + x - dk : 2 * n + h * dv + x - 2 * dk);
@@ -249,10 +261,16 @@ lin_step_kernel(const Params p) {
       else if (x < 2 * dk) sk[x - dk] = v;
       else sv[x - 2 * dk] = v;
     }
-    if constexpr (DELTA) {
+    if constexpr (RULE != FIXED) {
       for (int i = tid; i < dk; i += NT) {
         const float z = to_f(reinterpret_cast<const E*>(p.a)[(size_t)t * p.lda + h * dk + i]) + p.dt_bias[h * dk + i];
-        sg[i] = expf(-a_log * softplus(z));
+        if constexpr (RULE == DELTA) sg[i] = expf(-a_log * softplus(z));
+        if constexpr (RULE == CHANNEL) sg[i] = expf(-softplus(-z) * p.inv_tau);
+        if constexpr (RULE == REMOVAL) {
+          sg[i] = expf(-REMOVAL_DECAY * sigmoid(z));
+          sa[i] = sigmoid(to_f(reinterpret_cast<const E*>(p.row)[(size_t)t * p.ldr + p.rate_off + h * dk + i]) +
+                          p.rate_bias[h * dk + i]);
+        }
       }
     }
     __syncthreads();
@@ -268,12 +286,12 @@ lin_step_kernel(const Params p) {
       }
       __syncthreads();
     }
-    if (tid < 96) {
+    if (tid < (RULE == REMOVAL ? 128 : 96)) {
       const int wq = tid >> 5, lane = tid & 31;
       const float* x = wq == 1 ? sk : sq;
       const float* y = wq == 0 ? sq : sk;
       float s = 0.f;
-      for (int i = lane; i < dk; i += 32) s += x[i] * y[i];
+      for (int i = lane; i < dk; i += 32) s += x[i] * y[i] * (wq == 3 ? sa[i] : 1.f);
       s = warp_sum(s);
       if (lane == 0) sc[wq] = s;
     }
@@ -281,16 +299,19 @@ lin_step_kernel(const Params p) {
     const float iq = p.q_mult * (p.unit ? 1.f / sqrtf(sc[0] + UNIT_EPS) : 1.f);
     const float ik = p.k_mult * (p.unit ? 1.f / sqrtf(sc[1] + UNIT_EPS) : 1.f);
     const float qk = sc[2] * iq * ik;
+    const float in = RULE == REMOVAL ? 1.f / sqrtf(sc[1] + UNIT_EPS) : 0.f;       // n = k * in (before k_mult)
+    const float qb = RULE == REMOVAL ? -sc[3] * iq * in : 0.f;
     float mem[VEC], os[VEC];
 #pragma unroll
     for (int e = 0; e < VEC; ++e) mem[e] = os[e] = 0.f;
     const bool zero = HOLD == POOL && fresh && t == q.qs;
     auto pass = [&](int i, float (&s)[VEC]) {
-      const float g = DELTA ? sg[i] : decay, kk = sk[i] * ik, qq = sq[i] * iq;
+      const float g = RULE == FIXED ? decay : sg[i], kk = sk[i] * (RULE == REMOVAL ? in : ik), qq = sq[i] * iq;
 #pragma unroll
       for (int e = 0; e < VEC; ++e) {
+        if (RULE == REMOVAL) mem[e] = fmaf(kk, s[e], mem[e]);
         s[e] *= g;
-        if (DELTA) mem[e] = fmaf(kk, s[e], mem[e]);
+        if (RULE == DELTA) mem[e] = fmaf(kk, s[e], mem[e]);
         os[e] = fmaf(qq, s[e], os[e]);
       }
     };
@@ -316,22 +337,23 @@ lin_step_kernel(const Params p) {
     if (act) {
 #pragma unroll
       for (int e = 0; e < VEC; ++e) {
-        if (DELTA) pm[rg * dv + VEC * cg + e] = mem[e];
+        if (MEM) pm[rg * dv + VEC * cg + e] = mem[e];
         po[rg * dv + VEC * cg + e] = os[e];
       }
     }
     __syncthreads();
-    const float beta = DELTA ? sigmoid(b_raw) : 1.f;
+    const float beta = RULE == DELTA ? sigmoid(b_raw) : 1.f;
     float ss = 0.f;
     for (int j = tid; j < dv; j += NT) {
       float m = 0.f, o = 0.f;
       for (int x = 0; x < RG; ++x) {
-        if (DELTA) m += pm[x * dv + j];
+        if (MEM) m += pm[x * dv + j];
         o += po[x * dv + j];
       }
-      const float u = DELTA ? beta * (sv[j] - m) : sv[j];
+      const float u = RULE == DELTA ? beta * (sv[j] - m) : sv[j];
       o = fmaf(qk, u, o);
-      su[j] = u;
+      if (RULE == REMOVAL) o = fmaf(qb, m, o);
+      su[j] = RULE == REMOVAL ? m : u;
       po[j] = o;                        // (row group 0; only this thread reads column j)
       ss += o * o;
     }
@@ -342,49 +364,59 @@ lin_step_kernel(const Params p) {
       if (j == tid) {
         v *= nw;
       } else {
-        if (p.norm_w != nullptr) v *= p.norm_w[j];
+        if (norm_w != nullptr) v *= norm_w[j];
         g = to_f(reinterpret_cast<const E*>(p.gate)[(size_t)t * p.ldg + h * dv + j]);
       }
       v *= p.gate_silu ? silu(g) : sigmoid(g);
-      put(reinterpret_cast<E*>(p.y) + (size_t)t * p.H * dv + h * dv + j, v);
+      put(reinterpret_cast<E*>(p.y) + (size_t)t * p.ldy + h * dv + j, v);
     }
-    float u[VEC];
+    float u[VEC], m[VEC];                // REMOVAL: value and -S^T n, otherwise what is added along k
 #pragma unroll
-    for (int e = 0; e < VEC; ++e) u[e] = act ? su[VEC * cg + e] : 0.f;
+    for (int e = 0; e < VEC; ++e) {
+      u[e] = act ? (RULE == REMOVAL ? sv : su)[VEC * cg + e] : 0.f;
+      m[e] = RULE == REMOVAL && act ? -su[VEC * cg + e] : 0.f;
+    }
+    // row i of the new state from the decayed old one
+    auto write = [&](int i, float (&s)[VEC]) {
+      const float kk = sk[i] * ik, an = RULE == REMOVAL ? sa[i] * sk[i] * in : 0.f;
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) {
+        s[e] = fmaf(kk, u[e], s[e]);
+        if (RULE == REMOVAL) s[e] = fmaf(an, m[e], s[e]);
+      }
+    };
     if constexpr (HOLD == SMEM) {
       const bool last = t + 1 == q.qs + q.len;
 #pragma unroll 4
       for (int x = 0; x < rows; ++x) {
         const int i = rg + x * RG;
-        const float g = DELTA ? sg[i] : decay, kk = sk[i] * ik;
+        const float g = RULE == FIXED ? decay : sg[i];
         float4* d = reinterpret_cast<float4*>(held + (size_t)i * dv);
         const float4 f = *d;
-        const float4 n4 = make_float4(fmaf(kk, u[0], f.x * g), fmaf(kk, u[1 % VEC], f.y * g),
-                                      fmaf(kk, u[2 % VEC], f.z * g), fmaf(kk, u[3 % VEC], f.w * g));
+        float s[4] = {f.x * g, f.y * g, f.z * g, f.w * g};
+        write(i, reinterpret_cast<float(&)[VEC]>(s));
+        const float4 n4 = make_float4(s[0], s[1], s[2], s[3]);
         if (last) *reinterpret_cast<float4*>(st + (size_t)i * dv) = n4;
         else *d = n4;
       }
     } else if constexpr (HOLD == REGS) {
 #pragma unroll
       for (int x = 0; x < RPT; ++x)
-        if (x < rows) {
-          const float kk = sk[rg + x * RG] * ik;
-#pragma unroll
-          for (int e = 0; e < VEC; ++e) S[x][e] = fmaf(kk, u[e], S[x][e]);
-        }
+        if (x < rows) write(rg + x * RG, S[x]);
     } else {
       for (int x = 0; x < rows; ++x) {
         const int i = rg + x * RG;
-        const float g = DELTA ? sg[i] : decay, kk = sk[i] * ik;
+        const float g = RULE == FIXED ? decay : sg[i];
         float s[VEC];
         if (zero) {
 #pragma unroll
-          for (int e = 0; e < VEC; ++e) s[e] = kk * u[e];
+          for (int e = 0; e < VEC; ++e) s[e] = 0.f;
         } else {
           load_row(i, s);
 #pragma unroll
-          for (int e = 0; e < VEC; ++e) s[e] = fmaf(kk, u[e], s[e] * g);
+          for (int e = 0; e < VEC; ++e) s[e] *= g;
         }
+        write(i, s);
         store_row(i, s);
       }
     }
@@ -465,14 +497,16 @@ __device__ __forceinline__ void chunk_column(const Params& p, const Req& q, int 
 }
 
 // grid (requests * slab, H), 256 threads
-template <bool DELTA, int KM, int DKP>
-__global__ void __launch_bounds__(256, 3) lin_chunk_kernel(const Params p) {
+template <int RULE, int KM, int DKP>
+__global__ void __launch_bounds__(256, RULE == REMOVAL ? 2 : 3) lin_chunk_kernel(const Params p) {
   constexpr int dkp = DKP, ds = DKP + 4;
   pdl_launch_dependents();
   pdl_wait();
   extern __shared__ __align__(16) float sm[];
   __shared__ float beta[C], power[C + 1];
   __shared__ __align__(16) float sa[C][C + 4];
+  __shared__ __align__(16) float sx[RULE == REMOVAL ? C : 1][C + 4];       // REMOVAL: A with k_j, and |k| of every token
+  __shared__ float len[C];
   const int slot = blockIdx.x, h = blockIdx.y, tid = threadIdx.x;
   const Req q = request(p, p.req_begin + slot / p.slab);
   const int t0 = (p.chunk_begin + slot % p.slab) * C, n = min(C, q.len - t0);
@@ -481,7 +515,9 @@ __global__ void __launch_bounds__(256, 3) lin_chunk_kernel(const Params p) {
   const int dk = p.dk, dv = p.dv, nk = p.Hk * dk, hk = h / (p.H / p.Hk);
   float* sq = sm;                       // [C][ds]
   float* sk = sq + C * ds;
-  float* sg = sk + C * ds;              // decays accumulated from the chunk's first token on, log2 (delta rule)
+  float* sg = sk + C * ds;              // decays accumulated from the chunk's first token on, log2 (per channel)
+  float* se = sg + C * ds;              // REMOVAL: n over the decay of its own token
+  float* sr = se + C * ds;              // REMOVAL: rates
   // ---- q, k and the accumulated decays
 #pragma unroll 1
   for (int x = tid; x < 2 * dkp; x += 256) {
@@ -497,8 +533,8 @@ __global__ void __launch_bounds__(256, 3) lin_chunk_kernel(const Params p) {
 #pragma unroll
     for (int i = 0; i < C; ++i) d[i * ds + i0] = v[i];
   }
-  if constexpr (DELTA) {
-    const float a_log = expf(p.A_log[h]) * LOG2E;
+  if constexpr (RULE != FIXED) {
+    const float a_log = RULE == DELTA ? expf(p.A_log[h]) * LOG2E : (RULE == CHANNEL ? p.inv_tau : REMOVAL_DECAY) * LOG2E;
 #pragma unroll 1
     for (int c = tid; c < dkp; c += 256) {
       float g = 0.f;
@@ -511,11 +547,26 @@ __global__ void __launch_bounds__(256, 3) lin_chunk_kernel(const Params p) {
 #pragma unroll
       for (int i = 0; i < C; ++i) {
         // a factor below 2^-64 leaves nothing of the state in fp32: the sum keeps its digits
-        if (c < dk && i < n) g -= fminf(a_log * softplus_fast(z[i] + b), 64.f);
+        if (c < dk && i < n) {
+          const float x = z[i] + b;
+          const float step = RULE == REMOVAL ? __fdividef(1.f, 1.f + __expf(-x)) : softplus_fast(RULE == DELTA ? x : -x);
+          g -= fminf(a_log * step, 64.f);
+          if constexpr (RULE == REMOVAL) se[i * ds + c] = ex2(a_log * step);
+        } else if constexpr (RULE == REMOVAL) {
+          se[i * ds + c] = 0.f;
+        }
         sg[i * ds + c] = g;
       }
+      if constexpr (RULE == REMOVAL) {
+        const float rb = p.rate_bias[h * dk + cc];
+        const bf16* rr = reinterpret_cast<const bf16*>(p.row) + (size_t)row0 * p.ldr + p.rate_off + h * dk + cc;
+#pragma unroll
+        for (int i = 0; i < C; ++i) z[i] = to_f(rr[(size_t)min(i, n - 1) * p.ldr]);
+#pragma unroll
+        for (int i = 0; i < C; ++i) sr[i * ds + c] = c < dk && i < n ? __fdividef(1.f, 1.f + __expf(-(z[i] + rb))) : 0.f;
+      }
     }
-    if (tid < C)
+    if (RULE == DELTA && tid < C)
       beta[tid] = tid < n ? sigmoid(to_f(reinterpret_cast<const bf16*>(p.row)[(size_t)(row0 + tid) * p.ldr + p.beta_off + h]))
                           : 0.f;
   }
@@ -546,9 +597,17 @@ __global__ void __launch_bounds__(256, 3) lin_chunk_kernel(const Params p) {
         for (int i = lane; i < dk; i += 32) s += d[i] * d[i];
         m /= sqrtf(warp_sum(s) + UNIT_EPS);
       }
+      if (RULE == REMOVAL && x >= C) {   // k becomes n, its length is kept; e = n over the token's decay
+        float s = 0.f;
+        for (int i = lane; i < dk; i += 32) s += d[i] * d[i];
+        const float l = sqrtf(warp_sum(s) + UNIT_EPS);
+        if (lane == 0) len[x - C] = l * m;
+        m = 1.f / l;
+        for (int i = lane; i < dk; i += 32) se[(x - C) * ds + i] *= d[i] * m;
+      }
       for (int i = lane; i < dk; i += 32) d[i] *= m;
     }
-    if (!DELTA && tid <= C) power[tid] = exp2f(fmaxf(log2f(p.decay[h]), -64.f) * (float)tid);
+    if (RULE == FIXED && tid <= C) power[tid] = exp2f(fmaxf(log2f(p.decay[h]), -64.f) * (float)tid);
   }
   __syncthreads();
   const size_t unit = (size_t)slot * p.H + h;
@@ -566,11 +625,25 @@ __global__ void __launch_bounds__(256, 3) lin_chunk_kernel(const Params p) {
       j = x < 15 - r ? r + 1 + x : x + 1;
     }
     if (tid < 8 * 17) {
-      float qk = 0.f, kk = 0.f;
+      float qk = 0.f, kk = 0.f, qb = 0.f, kb = 0.f;
       const float *qi = sq + i * ds, *ki = sk + i * ds, *kj = sk + j * ds, *gi = sg + i * ds, *gj = sg + j * ds;
       for (int c = 0; c < dkp; c += 4) {
         const float4 a = *reinterpret_cast<const float4*>(qi + c), b = *reinterpret_cast<const float4*>(kj + c);
-        if constexpr (DELTA) {
+        if constexpr (RULE == REMOVAL) {
+          const float4 e = *reinterpret_cast<const float4*>(se + i * ds + c), r = *reinterpret_cast<const float4*>(sr + j * ds + c),
+                       x = *reinterpret_cast<const float4*>(gi + c), y = *reinterpret_cast<const float4*>(gj + c);
+          const float d0 = b.x * ex2(x.x - y.x), d1 = b.y * ex2(x.y - y.y), d2 = b.z * ex2(x.z - y.z),
+                      d3 = b.w * ex2(x.w - y.w);
+          const float f0 = d0 * r.x, f1 = d1 * r.y, f2 = d2 * r.z, f3 = d3 * r.w;
+          qk = fmaf(a.x, d0, qk); qk = fmaf(a.y, d1, qk); qk = fmaf(a.z, d2, qk); qk = fmaf(a.w, d3, qk);
+          kk = fmaf(e.x, d0, kk); kk = fmaf(e.y, d1, kk); kk = fmaf(e.z, d2, kk); kk = fmaf(e.w, d3, kk);
+          qb = fmaf(a.x, f0, qb); qb = fmaf(a.y, f1, qb); qb = fmaf(a.z, f2, qb); qb = fmaf(a.w, f3, qb);
+          kb = fmaf(e.x, f0, kb); kb = fmaf(e.y, f1, kb); kb = fmaf(e.z, f2, kb); kb = fmaf(e.w, f3, kb);
+        } else if constexpr (RULE == CHANNEL) {
+          const float4 x = *reinterpret_cast<const float4*>(gi + c), y = *reinterpret_cast<const float4*>(gj + c);
+          qk = fmaf(a.x, b.x * ex2(x.x - y.x), qk); qk = fmaf(a.y, b.y * ex2(x.y - y.y), qk);
+          qk = fmaf(a.z, b.z * ex2(x.z - y.z), qk); qk = fmaf(a.w, b.w * ex2(x.w - y.w), qk);
+        } else if constexpr (RULE == DELTA) {
           const float4 e = *reinterpret_cast<const float4*>(ki + c), x = *reinterpret_cast<const float4*>(gi + c),
                        y = *reinterpret_cast<const float4*>(gj + c);
           const float d0 = b.x * ex2(x.x - y.x), d1 = b.y * ex2(x.y - y.y), d2 = b.z * ex2(x.z - y.z),
@@ -581,14 +654,22 @@ __global__ void __launch_bounds__(256, 3) lin_chunk_kernel(const Params p) {
           qk = fmaf(a.x, b.x, qk); qk = fmaf(a.y, b.y, qk); qk = fmaf(a.z, b.z, qk); qk = fmaf(a.w, b.w, qk);
         }
       }
-      if constexpr (!DELTA) qk *= power[i - j];
-      p.aq[(unit * C + i) * AQ_LD + j] = qk;
-      if constexpr (DELTA) sa[i][j] = j < i ? beta[i] * kk : 0.f;
+      if constexpr (RULE == FIXED) qk *= power[i - j];
+      if constexpr (RULE == REMOVAL) {
+        p.aq[(unit * C + i) * AQ_LD + j] = -qb;
+        p.ak[(unit * C + i) * AQ_LD + j] = qk * len[j];
+        sa[i][j] = j < i ? kb : 0.f;
+        sx[i][j] = j < i ? kk * len[j] : 0.f;
+      } else {
+        p.aq[(unit * C + i) * AQ_LD + j] = qk;
+      }
+      if constexpr (RULE == DELTA) sa[i][j] = j < i ? beta[i] * kk : 0.f;
     } else if (j < C) {
       p.aq[(unit * C + i) * AQ_LD + j] = 0.f;
+      if constexpr (RULE == REMOVAL) p.ak[(unit * C + i) * AQ_LD + j] = 0.f;
     }
   }
-  if constexpr (DELTA) __syncthreads();
+  if constexpr (RULE == DELTA || RULE == REMOVAL) __syncthreads();
   // ---- columns of W and U (forward substitution), q', k', last decay
 #pragma unroll 1
   for (int x = tid; x < dkp + p.dvp; x += 256) {
@@ -596,14 +677,20 @@ __global__ void __launch_bounds__(256, 3) lin_chunk_kernel(const Params p) {
     asm volatile("" ::: "memory");       // values that do not depend on the column stay in shared memory
     if (x < dkp) {
       float *qd = p.qd + unit * C * (dkp + 8) + x, *kd = p.kd + unit * C * (dkp + 4) + x;
-      if constexpr (DELTA) {
+      if constexpr (RULE != FIXED) {
         const float last = sg[(C - 1) * ds + x];
 #pragma unroll
         for (int i = 0; i < C; ++i) {
-          const float g = sg[i * ds + x], e = ex2(g), k = sk[i * ds + x];
+          const float g = sg[i * ds + x], e = ex2(g), k = sk[i * ds + x], left = ex2(last - g);
           qd[i * (dkp + 8)] = sq[i * ds + x] * e;
-          kd[i * (dkp + 4)] = k * ex2(last - g);
-          v[i] = beta[i] * k * e;
+          if constexpr (RULE == REMOVAL) {
+            kd[i * (dkp + 4)] = k * len[i] * left;
+            p.bd[unit * C * (dkp + 4) + x + i * (dkp + 4)] = -(k * sr[i * ds + x]) * left;
+            v[i] = se[i * ds + x] * e;
+          } else {
+            kd[i * (dkp + 4)] = k * left;
+          }
+          if constexpr (RULE == DELTA) v[i] = beta[i] * k * e;
         }
         p.gl[unit * dkp + x] = ex2(last);
       } else {
@@ -622,12 +709,31 @@ __global__ void __launch_bounds__(256, 3) lin_chunk_kernel(const Params p) {
 #pragma unroll
         for (int i = 0; i < C; ++i) v[i] = 0.f;
       }
-      if constexpr (DELTA) {
+      if constexpr (RULE == DELTA) {
 #pragma unroll
         for (int i = 0; i < C; ++i) v[i] *= beta[i];
       }
+      if constexpr (RULE == REMOVAL) {   // the values go to the scan as they are; M0 starts from their products with A
+        float* d = p.v + (unit * (p.dvp / 64) + j / 64) * C * 64 + j % 64;
+#pragma unroll
+        for (int i = 0; i < C; ++i) d[i * 64] = v[i];
+#pragma unroll
+        for (int i = C - 1; i >= 0; --i) {
+          asm volatile("" ::: "memory");
+          float s = 0.f;
+#pragma unroll
+          for (int l = 0; l < i; l += 4) {
+            const float4 a = *reinterpret_cast<const float4*>(&sx[RULE == REMOVAL ? i : 0][l]);      // zeros from column i on
+            s = fmaf(a.x, v[l], s);
+            if (l + 1 < i) s = fmaf(a.y, v[l + 1], s);
+            if (l + 2 < i) s = fmaf(a.z, v[l + 2], s);
+            if (l + 3 < i) s = fmaf(a.w, v[l + 3], s);
+          }
+          v[i] = s;
+        }
+      }
     }
-    if constexpr (DELTA) {
+    if constexpr (RULE == DELTA || RULE == REMOVAL) {
 #pragma unroll
       for (int i = 1; i < C; ++i) {
         asm volatile("" ::: "memory");   // one row of A in registers at a time
@@ -643,7 +749,7 @@ __global__ void __launch_bounds__(256, 3) lin_chunk_kernel(const Params p) {
       if (x < dkp) {
         float* w = p.w + unit * C * (dkp + 8) + x;
 #pragma unroll
-        for (int i = 0; i < C; ++i) w[i * (dkp + 8)] = -v[i];
+        for (int i = 0; i < C; ++i) w[i * (dkp + 8)] = RULE == REMOVAL ? v[i] : -v[i];
       }
     }
     if (x >= dkp) {
@@ -656,20 +762,23 @@ __global__ void __launch_bounds__(256, 3) lin_chunk_kernel(const Params p) {
 }
 
 // grid (H * dvp / 64, requests), 128 threads: warp w owns value columns 16 w .. 16 w + 15 of the CTA's 64
-template <bool DELTA, int NT>
+template <int RULE, int NT>
 struct Scan {
-  static constexpr int DKP = 8 * NT;
-  static constexpr int QD = 0, W = C * (DKP + 8), KD = W + (DELTA ? C * (DKP + 8) : 0), U = KD + C * (DKP + 4);
-  static constexpr int U_LD = 68, AQ = U + C * U_LD, GL = AQ + C * AQ_LD, WORDS = GL + DKP;
-  static constexpr int STAGES = 3;
+  static constexpr bool MEM = RULE == DELTA || RULE == REMOVAL, TWO = RULE == REMOVAL;
+  static constexpr int DKP = 8 * NT, U_LD = 68;
+  static constexpr int QD = 0, W = C * (DKP + 8), KD = W + (MEM ? C * (DKP + 8) : 0), BD = KD + C * (DKP + 4);
+  static constexpr int U = BD + (TWO ? C * (DKP + 4) : 0), V = U + C * U_LD, AQ = V + (TWO ? C * U_LD : 0);
+  static constexpr int AK = AQ + C * AQ_LD, GL = AK + (TWO ? C * AQ_LD : 0), WORDS = GL + DKP;
+  static constexpr int STAGES = 3 * WORDS * 4 > 220 * 1024 ? 2 : 3;
   static constexpr int BYTES = STAGES * WORDS * 4;
 };
 
-template <bool DELTA, int NT>
+template <int RULE, int NT>
 __global__ void __launch_bounds__(128) lin_scan_kernel(const Params p) {
   pdl_launch_dependents();
   pdl_wait();
-  using L = Scan<DELTA, NT>;
+  using L = Scan<RULE, NT>;
+  constexpr bool MEM = L::MEM, TWO = L::TWO;
   constexpr int DKP = L::DKP;
   extern __shared__ __align__(16) float sm[];
   const int splits = p.dvp / 64, h = blockIdx.x / splits, col0 = (blockIdx.x % splits) * 64;
@@ -686,14 +795,19 @@ __global__ void __launch_bounds__(128) lin_scan_kernel(const Params p) {
       for (int i = tid * 4; i < words; i += 128 * 4) cp_async16(d + (word + i) * 4, src + i);
     };
     copy(L::QD, p.qd + unit * C * (DKP + 8), C * (DKP + 8));
-    if constexpr (DELTA) copy(L::W, p.w + unit * C * (DKP + 8), C * (DKP + 8));
+    if constexpr (MEM) copy(L::W, p.w + unit * C * (DKP + 8), C * (DKP + 8));
     copy(L::KD, p.kd + unit * C * (DKP + 4), C * (DKP + 4));
     copy(L::AQ, p.aq + unit * C * AQ_LD, C * AQ_LD);
+    if constexpr (TWO) {
+      copy(L::BD, p.bd + unit * C * (DKP + 4), C * (DKP + 4));
+      copy(L::AK, p.ak + unit * C * AQ_LD, C * AQ_LD);
+    }
     copy(L::GL, p.gl + unit * DKP, DKP);
 #pragma unroll
     for (int i = tid; i < C * 16; i += 128) {
       const int r = i >> 4, s = (i & 15) * 4;
       cp_async16(d + (L::U + r * L::U_LD + s) * 4, p.u + ((unit * splits + col0 / 64) * C + r) * 64 + s);
+      if constexpr (TWO) cp_async16(d + (L::V + r * L::U_LD + s) * 4, p.v + ((unit * splits + col0 / 64) * C + r) * 64 + s);
     }
   };
   float* st = p.state + ((size_t)q.slot * p.H + h) * dk * dv;
@@ -735,7 +849,7 @@ __global__ void __launch_bounds__(128) lin_scan_kernel(const Params p) {
       const SplitA a = split_tile(S[x]);
 #pragma unroll
       for (int y = 0; y < 2; ++y) {
-        if constexpr (DELTA) {
+        if constexpr (MEM) {
           const float2 bw = *reinterpret_cast<const float2*>(w + 8 * y * (DKP + 8) + 8 * x);
           mma_split(U[y], U2[y], a, bw.x, bw.y);
         }
@@ -743,12 +857,17 @@ __global__ void __launch_bounds__(128) lin_scan_kernel(const Params p) {
         mma_split(O[y], O2[y], a, bq.x, bq.y);
       }
     }
-    SplitA ua[2];
+    SplitA ua[2], va[2];
 #pragma unroll
     for (int x = 0; x < 2; ++x) {
 #pragma unroll
       for (int e = 0; e < 4; ++e) U[x][e] += U2[x][e];
       ua[x] = split_tile(U[x]);
+      if constexpr (TWO) {
+        const float* v = b + L::V + (8 * x + 2 * t) * L::U_LD + warp * 16 + g;
+        const float f[4] = {v[0], v[L::U_LD], v[8], v[L::U_LD + 8]};
+        va[x] = split_tile(f);
+      }
     }
 #pragma unroll
     for (int y = 0; y < 2; ++y) {
@@ -757,6 +876,10 @@ __global__ void __launch_bounds__(128) lin_scan_kernel(const Params p) {
         if (x > y) continue;             // Q is lower triangular
         const float2 bq = *reinterpret_cast<const float2*>(b + L::AQ + (8 * y + g) * AQ_LD + 8 * x + 2 * t);
         mma_split(O[y], O2[y], ua[x], bq.x, bq.y);
+        if constexpr (TWO) {
+          const float2 bk = *reinterpret_cast<const float2*>(b + L::AK + (8 * y + g) * AQ_LD + 8 * x + 2 * t);
+          mma_split(O[y], O2[y], va[x], bk.x, bk.y);
+        }
       }
 #pragma unroll
       for (int e = 0; e < 4; ++e) O[y][e] += O2[y][e];
@@ -770,7 +893,13 @@ __global__ void __launch_bounds__(128) lin_scan_kernel(const Params p) {
 #pragma unroll
       for (int y = 0; y < 2; ++y) {
         const float* k = kd + 8 * y * (DKP + 4) + 8 * x;
-        mma_split(S[x], S[x], ua[y], k[0], k[DKP + 4]);
+        if constexpr (TWO) {
+          const float* m = k + (L::BD - L::KD);
+          mma_split(S[x], S[x], va[y], k[0], k[DKP + 4]);
+          mma_split(S[x], S[x], ua[y], m[0], m[DKP + 4]);
+        } else {
+          mma_split(S[x], S[x], ua[y], k[0], k[DKP + 4]);
+        }
       }
     }
     const int rows = min(C, q.len - (p.chunk_begin + c) * C);
@@ -810,41 +939,41 @@ __global__ void __launch_bounds__(256) lin_finish_kernel(const Params p) {
   const float inv = 1.f / sqrtf(warp_sum(ss) / (float)dv + p.eps);
   const size_t t = q.qs + i;
   const bf16* gate = reinterpret_cast<const bf16*>(p.gate) + t * p.ldg + h * dv;
-  bf16* y = reinterpret_cast<bf16*>(p.y) + t * p.H * dv + h * dv;
+  bf16* y = reinterpret_cast<bf16*>(p.y) + t * p.ldy + h * dv;
   for (int j = lane; j < dv; j += 32) {
     float v = o[j] * inv;
-    if (p.norm_w != nullptr) v *= p.norm_w[j];
+    if (p.norm_w != nullptr) v *= p.norm_w[(size_t)h * p.norm_stride + j];
     const float g = to_f(gate[j]);
     put(y + j, v * (p.gate_silu ? silu(g) : sigmoid(g)));
   }
 }
 
 // ------------------------------------------------------------------------------------------- host
-template <typename E, bool DELTA, int VEC, int RPT, Hold HOLD>
+template <typename E, int RULE, int VEC, int RPT, Hold HOLD>
 static int launch_step_as(const Params& p, int R, int threads, cudaStream_t stream) {
   const int RG = threads / (p.dv / VEC);
-  const int smem = (3 * p.dk + 2 * p.dv + 2 * RG * p.dv + (HOLD == SMEM ? p.dk * p.dv : 0)) * (int)sizeof(float);
+  const int smem = ((RULE == REMOVAL ? 4 : 3) * p.dk + 2 * p.dv + 2 * RG * p.dv + (HOLD == SMEM ? p.dk * p.dv : 0)) * (int)sizeof(float);
   static unsigned long long seen = 0;
   if (smem > 46 * 1024)
-    B200_CUDA_CHECK(ensure_dynamic_smem(lin_step_kernel<E, DELTA, VEC, RPT, HOLD>, 220 * 1024, &seen));
-  B200_CUDA_CHECK(launch_pdl(lin_step_kernel<E, DELTA, VEC, RPT, HOLD>, dim3(p.H, R), dim3(threads), (size_t)smem,
+    B200_CUDA_CHECK(ensure_dynamic_smem(lin_step_kernel<E, RULE, VEC, RPT, HOLD>, 220 * 1024, &seen));
+  B200_CUDA_CHECK(launch_pdl(lin_step_kernel<E, RULE, VEC, RPT, HOLD>, dim3(p.H, R), dim3(threads), (size_t)smem,
                              stream, p));
   return 0;
 }
 
-template <typename E, bool DELTA, int VEC>
+template <typename E, int RULE, int VEC>
 static int launch_step_v(const Params& p, int R, cudaStream_t stream) {
   const int ncg = p.dv / VEC;
   if constexpr (VEC == 4) {
     // q, k and the decays are read as floats: the state behind them starts on 16 bytes when 3 dk is a multiple of 4
     if (p.dk % 4 == 0 && ncg <= 256 && p.dk * p.dv <= 48 * 1024)
-      return launch_step_as<E, DELTA, VEC, 1, SMEM>(p, R, p.dk * p.dv <= 2048 && ncg <= 128 ? 128 : 256, stream);
+      return launch_step_as<E, RULE, VEC, 1, SMEM>(p, R, p.dk * p.dv <= 2048 && ncg <= 128 ? 128 : 256, stream);
   } else {
     for (int threads = 128; threads <= 512; threads *= 2) {
       if (threads < ncg) continue;
       const int RG = threads / ncg, rows = (p.dk + RG - 1) / RG;
-      if (rows <= 4) return launch_step_as<E, DELTA, VEC, 4, REGS>(p, R, threads, stream);
-      if (rows <= 16) return launch_step_as<E, DELTA, VEC, 16, REGS>(p, R, threads, stream);
+      if (rows <= 4) return launch_step_as<E, RULE, VEC, 4, REGS>(p, R, threads, stream);
+      if (rows <= 16) return launch_step_as<E, RULE, VEC, 16, REGS>(p, R, threads, stream);
     }
   }
   int threads = 512;
@@ -853,73 +982,81 @@ static int launch_step_v(const Params& p, int R, cudaStream_t stream) {
     b200_set_last_error("linear attention: at most 1024 value columns per thread group", __FILE__, __LINE__);
     return -1;
   }
-  return launch_step_as<E, DELTA, VEC, 1, POOL>(p, R, threads, stream);
+  return launch_step_as<E, RULE, VEC, 1, POOL>(p, R, threads, stream);
 }
 
 template <typename E>
-static int launch_step(const Params& p, int R, cudaStream_t stream) {
-  const bool delta = p.decay == nullptr;
-  if (p.dv % 4 == 0)
-    return delta ? launch_step_v<E, true, 4>(p, R, stream) : launch_step_v<E, false, 4>(p, R, stream);
-  return delta ? launch_step_v<E, true, 1>(p, R, stream) : launch_step_v<E, false, 1>(p, R, stream);
+static int launch_step(const Params& p, int rule, int R, cudaStream_t stream) {
+  const bool v4 = p.dv % 4 == 0;
+  switch (rule) {
+    case FIXED: return v4 ? launch_step_v<E, FIXED, 4>(p, R, stream) : launch_step_v<E, FIXED, 1>(p, R, stream);
+    case DELTA: return v4 ? launch_step_v<E, DELTA, 4>(p, R, stream) : launch_step_v<E, DELTA, 1>(p, R, stream);
+    case CHANNEL: return v4 ? launch_step_v<E, CHANNEL, 4>(p, R, stream) : launch_step_v<E, CHANNEL, 1>(p, R, stream);
+    default: return v4 ? launch_step_v<E, REMOVAL, 4>(p, R, stream) : launch_step_v<E, REMOVAL, 1>(p, R, stream);
+  }
 }
 
-template <bool DELTA, int NT>
+template <int RULE, int NT>
 static int launch_scan(const Params& p, int R, cudaStream_t stream) {
   static unsigned long long seen = 0;
-  using L = Scan<DELTA, NT>;
-  B200_CUDA_CHECK(ensure_dynamic_smem(lin_scan_kernel<DELTA, NT>, L::BYTES, &seen));
-  B200_CUDA_CHECK(launch_pdl(lin_scan_kernel<DELTA, NT>, dim3(p.H * (p.dvp / 64), R), dim3(128), (size_t)L::BYTES,
+  using L = Scan<RULE, NT>;
+  B200_CUDA_CHECK(ensure_dynamic_smem(lin_scan_kernel<RULE, NT>, L::BYTES, &seen));
+  B200_CUDA_CHECK(launch_pdl(lin_scan_kernel<RULE, NT>, dim3(p.H * (p.dvp / 64), R), dim3(128), (size_t)L::BYTES,
                              stream, p));
   return 0;
 }
 
-template <bool DELTA, int KM, int DKP>
+template <int RULE, int KM, int DKP>
 static int launch_chunk_as(const Params& p, int R, cudaStream_t stream) {
-  constexpr int smem = (DELTA ? 3 : 2) * C * (DKP + 4) * (int)sizeof(float);
+  constexpr int smem = (RULE == REMOVAL ? 5 : (RULE == FIXED ? 2 : 3)) * C * (DKP + 4) * (int)sizeof(float);
   static unsigned long long seen = 0;
-  if (smem > 44 * 1024) B200_CUDA_CHECK(ensure_dynamic_smem(lin_chunk_kernel<DELTA, KM, DKP>, smem, &seen));
-  B200_CUDA_CHECK(launch_pdl(lin_chunk_kernel<DELTA, KM, DKP>, dim3(R * p.slab, p.H), dim3(256), (size_t)smem, stream, p));
+  if (smem > 44 * 1024) B200_CUDA_CHECK(ensure_dynamic_smem(lin_chunk_kernel<RULE, KM, DKP>, smem, &seen));
+  B200_CUDA_CHECK(launch_pdl(lin_chunk_kernel<RULE, KM, DKP>, dim3(R * p.slab, p.H), dim3(256), (size_t)smem, stream, p));
   return 0;
 }
-template <bool DELTA, int KM>
+template <int RULE, int KM>
 static int launch_chunk(const Params& p, int R, cudaStream_t stream) {
   switch (p.dkp) {
-    case 32: return launch_chunk_as<DELTA, KM, 32>(p, R, stream);
-    case 64: return launch_chunk_as<DELTA, KM, 64>(p, R, stream);
-    case 128: return launch_chunk_as<DELTA, KM, 128>(p, R, stream);
-    default: return launch_chunk_as<DELTA, KM, 256>(p, R, stream);
+    case 32: return launch_chunk_as<RULE, KM, 32>(p, R, stream);
+    case 64: return launch_chunk_as<RULE, KM, 64>(p, R, stream);
+    case 128: return launch_chunk_as<RULE, KM, 128>(p, R, stream);
+    default: return launch_chunk_as<RULE, KM, 256>(p, R, stream);
   }
 }
 
 static int padded_dk(int dk) { return dk <= 32 ? 32 : (dk <= 64 ? 64 : (dk <= 128 ? 128 : 256)); }
 
 // floats of scratch per chunk and head
-static size_t chunk_words(int dk, int dv, bool delta) {
-  const int dkp = padded_dk(dk), dvp = (dv + 63) / 64 * 64;
-  return (size_t)C * ((delta ? 2 : 1) * (dkp + 8) + dkp + 4 + dvp + AQ_LD + dv) + dkp;
+static size_t chunk_words(int dk, int dv, int rule) {
+  const int dkp = padded_dk(dk), dvp = (dv + 63) / 64 * 64, two = rule == REMOVAL ? 2 : 1;
+  return (size_t)C * ((rule == DELTA || rule == REMOVAL ? 2 : 1) * (dkp + 8) + two * (dkp + 4 + dvp + AQ_LD) + dv) + dkp;
 }
 
 // one of the three kernels of a slab of chunks
-template <bool DELTA>
+template <int RULE>
 static int launch_chunks(Params& p, int R, float* scratch, int mode, cudaStream_t stream) {
   const size_t units = (size_t)R * p.slab * p.H;
   p.qd = scratch;
   p.w = p.qd + units * C * (p.dkp + 8);
-  p.kd = p.w + (DELTA ? units * C * (p.dkp + 8) : 0);
-  p.u = p.kd + units * C * (p.dkp + 4);
-  p.aq = p.u + units * C * p.dvp;
-  p.gl = p.aq + units * C * AQ_LD;
+  constexpr bool mem = RULE == DELTA || RULE == REMOVAL, two = RULE == REMOVAL;
+  p.kd = p.w + (mem ? units * C * (p.dkp + 8) : 0);
+  p.bd = p.kd + units * C * (p.dkp + 4);
+  p.u = p.bd + (two ? units * C * (p.dkp + 4) : 0);
+  p.v = p.u + units * C * p.dvp;
+  p.aq = p.v + (two ? units * C * p.dvp : 0);
+  p.ak = p.aq + units * C * AQ_LD;
+  p.gl = p.ak + (two ? units * C * AQ_LD : 0);
   p.o = p.gl + units * p.dkp;
   if (mode == 1)
-    return p.taps == 0 ? launch_chunk<DELTA, 0>(p, R, stream)
-                       : (p.taps <= 4 ? launch_chunk<DELTA, 4>(p, R, stream) : launch_chunk<DELTA, 8>(p, R, stream));
+    return p.taps == 0 ? launch_chunk<RULE, 0>(p, R, stream)
+                       : (p.taps <= 4 && (RULE == FIXED || RULE == DELTA) ? launch_chunk<RULE, RULE < CHANNEL ? 4 : 8>(p, R, stream)
+                                                                          : launch_chunk<RULE, 8>(p, R, stream));
   if (mode == 3) {
     switch (p.dkp) {
-      case 32: return launch_scan<DELTA, 4>(p, R, stream);
-      case 64: return launch_scan<DELTA, 8>(p, R, stream);
-      case 128: return launch_scan<DELTA, 16>(p, R, stream);
-      default: return launch_scan<DELTA, 32>(p, R, stream);
+      case 32: return launch_scan<RULE, 4>(p, R, stream);
+      case 64: return launch_scan<RULE, 8>(p, R, stream);
+      case 128: return launch_scan<RULE, 16>(p, R, stream);
+      default: return launch_scan<RULE, 32>(p, R, stream);
     }
   }
   B200_CUDA_CHECK(launch_pdl(lin_finish_kernel, dim3(R * p.slab * C, (p.H + 7) / 8), dim3(256), (size_t)0, stream, p));
@@ -930,29 +1067,37 @@ static int launch_chunks(Params& p, int R, float* scratch, int mode, cudaStream_
 }  // namespace b200
 
 // Bytes of scratch per (chunk of 16 tokens, head) of b200_linear_attention in mode 1.
-extern "C" size_t b200_linear_attention_chunk_bytes(int dk, int dv, int delta) {
-  return b200::lin::chunk_words(dk, dv, delta != 0) * sizeof(float);
+extern "C" size_t b200_linear_attention_chunk_bytes(int dk, int dv, int rule) {
+  return b200::lin::chunk_words(dk, dv, rule) * sizeof(float);
 }
 
 // Requests [req_begin, req_end) of the batch.  mode 0: token by token (any sizes; the ring takes portions of more than
 // one token through mode 2); mode 1: products of chunks [chunk_begin, chunk_begin + slab) of every request (bf16, dk <=
 // 256, taps <= 8; into scratch for (req_end - req_begin) * slab * H chunks), mode 3: their recurrence, mode 4: their
-// norm and gate; mode 2: the ring of a prompt.  decay != null: fixed decay per head, otherwise the delta rule with a, A_log, dt_bias and the step sizes in
-// column beta_off of the row.  elem: 2 = bf16, 4 = fp32.
-extern "C" int b200_linear_attention(int mode, const void* row, int ldr, int q_off, int k_off, int v_off, int beta_off,
-                                     const void* a, int lda, const void* gate, int ldg, const void* conv_w, void* ring,
-                                     int taps, const float* inv_freq, int pairs, const float* decay, const float* A_log,
-                                     const float* dt_bias, const float* norm_w, float* state, void* y, const int* qsl,
-                                     const int* seq_lens, const int* slots, int req_begin, int req_end, int T, int H,
-                                     int Hk, int dk, int dv, int unit, int gate_silu, float eps, float q_mult,
-                                     float k_mult, int zero_rows, void* scratch, int chunk_begin, int slab, int elem,
-                                     cudaStream_t stream) {
+// norm and gate; mode 2: the ring of a prompt.  rule: 0 fixed decay per head (decay), 1 delta rule (a, A_log, dt_bias and
+// the step sizes in column beta_off of the row), 2 decay per channel (a, dt_bias, tau), 3 removal (a, dt_bias, the rates in
+// column rate_off with rate_bias).  norm_w: heads are norm_stride elements apart; y: rows are ldy apart.
+// elem: 2 = bf16, 4 = fp32.
+extern "C" int b200_linear_attention(int mode, int rule, const void* row, int ldr, int q_off, int k_off, int v_off,
+                                     int beta_off, int rate_off, const void* a, int lda, const void* gate, int ldg,
+                                     const void* conv_w, void* ring, int taps, const float* inv_freq, int pairs,
+                                     const float* decay, const float* A_log, const float* dt_bias, const float* rate_bias,
+                                     float tau, const float* norm_w, int norm_stride, float* state, void* y, int ldy,
+                                     const int* qsl, const int* seq_lens, const int* slots, int req_begin, int req_end,
+                                     int T, int H, int Hk, int dk, int dv, int unit, int gate_silu, float eps,
+                                     float q_mult, float k_mult, int zero_rows, void* scratch, int chunk_begin, int slab,
+                                     int elem, cudaStream_t stream) {
   using namespace b200;
   const int R = req_end - req_begin;
   if (R <= 0 || T <= 0) return 0;
   if (Hk <= 0 || H % Hk || 2 * pairs > dk || R > 65535 || dk <= 0 || dv <= 0) {
     b200_set_last_error("linear attention: heads must be a multiple of the q / k heads, pairs at most dk / 2", __FILE__,
                         __LINE__);
+    return -1;
+  }
+  if (rule < 0 || rule > 3 || (rule == 0 && decay == nullptr) || (rule != 0 && (a == nullptr || dt_bias == nullptr)) ||
+      (rule == 1 && A_log == nullptr) || (rule == 2 && !(tau > 0.f)) || (rule == 3 && (rate_bias == nullptr || unit))) {
+    b200_set_last_error("linear attention: parameters of the rule are missing", __FILE__, __LINE__);
     return -1;
   }
   lin::Params p;
@@ -963,17 +1108,23 @@ extern "C" int b200_linear_attention(int mode, const void* row, int ldr, int q_o
   p.ldr = ldr; p.q_off = q_off; p.k_off = k_off; p.v_off = v_off; p.beta_off = beta_off; p.lda = lda; p.ldg = ldg;
   p.taps = taps; p.pairs = pairs; p.unit = unit; p.gate_silu = gate_silu;
   p.T = T; p.H = H; p.Hk = Hk; p.dk = dk; p.dv = dv; p.req_begin = req_begin; p.zero_rows = zero_rows;
-  p.eps = eps; p.q_mult = q_mult; p.k_mult = k_mult;
+  p.eps = eps; p.q_mult = q_mult; p.k_mult = k_mult; p.inv_tau = rule == 2 ? 1.f / tau : 0.f;
+  p.rate_off = rate_off; p.rate_bias = rate_bias; p.norm_stride = norm_stride; p.ldy = ldy;
   p.dkp = lin::padded_dk(dk); p.dvp = (dv + 63) / 64 * 64;
   p.slab = slab; p.chunk_begin = chunk_begin;
-  if (mode == 0) return elem == 4 ? lin::launch_step<float>(p, R, stream) : lin::launch_step<__nv_bfloat16>(p, R, stream);
+  if (mode == 0) return elem == 4 ? lin::launch_step<float>(p, rule, R, stream)
+                                  : lin::launch_step<__nv_bfloat16>(p, rule, R, stream);
   if (mode == 1 || mode == 3 || mode == 4) {
     if (elem != 2 || dk > 256 || taps > 8 || slab <= 0 || scratch == nullptr) {
       b200_set_last_error("linear attention in chunks: bf16, dk of at most 256, at most 8 taps", __FILE__, __LINE__);
       return -1;
     }
-    return decay == nullptr ? lin::launch_chunks<true>(p, R, (float*)scratch, mode, stream)
-                            : lin::launch_chunks<false>(p, R, (float*)scratch, mode, stream);
+    switch (rule) {
+      case lin::FIXED: return lin::launch_chunks<lin::FIXED>(p, R, (float*)scratch, mode, stream);
+      case lin::DELTA: return lin::launch_chunks<lin::DELTA>(p, R, (float*)scratch, mode, stream);
+      case lin::CHANNEL: return lin::launch_chunks<lin::CHANNEL>(p, R, (float*)scratch, mode, stream);
+      default: return lin::launch_chunks<lin::REMOVAL>(p, R, (float*)scratch, mode, stream);
+    }
   }
   const dim3 grid((2 * Hk * dk + H * dv + 255) / 256, R);
   if (elem == 4) B200_CUDA_CHECK(launch_pdl(lin::lin_ring_kernel<float>, grid, dim3(256), (size_t)0, stream, p));

@@ -68,7 +68,7 @@ __global__ void moe_route_kernel(const T* __restrict__ logits, int ld, int Tn, i
         const float v = choice[lane * per + i];
         if (v > a) { b = a; a = v; } else if (v > b) { b = v; }
       }
-      s_group[warp][lane] = bias != nullptr ? a + b : a;
+      s_group[warp][lane] = bias != nullptr && per > 1 ? a + b : a;
     }
     __syncwarp();
     // keep the topk_group best groups (lowest index wins ties)
@@ -208,6 +208,76 @@ __global__ void moe_unpermute_any_kernel(const E* __restrict__ y, int ldy, const
   }
 }
 
+// The last step of an expert block on a 32-bit residual stream: r += sum_j w[t,j] * y[inv_pos[t,j]] (+ sigmoid(g_t) * shared[t]),
+// in place, and its rounded copy.  shared rows are H elements, gates ldg apart.  V elements per thread and pass.
+template <typename E, int V>
+__global__ void moe_unpermute_add_kernel(const E* __restrict__ y, int ldy, const int* __restrict__ inv_pos,
+                                         const float* __restrict__ w, const E* __restrict__ shared,
+                                         const float* __restrict__ gate, int ldg, float* __restrict__ res,
+                                         E* __restrict__ out, int H, int top_k, int rows_cap) {
+  __shared__ int s_pos[32];
+  __shared__ float s_w[32], s_gate;
+  const int t = blockIdx.x;
+  if (threadIdx.x < top_k) {
+    const int pos = inv_pos[(size_t)t * top_k + threadIdx.x];
+    s_pos[threadIdx.x] = pos < rows_cap ? pos : -1;
+    s_w[threadIdx.x] = w[(size_t)t * top_k + threadIdx.x];
+  }
+  if (threadIdx.x == 32) s_gate = shared != nullptr ? 1.f / (1.f + expf(-gate[(size_t)t * ldg])) : 0.f;
+  __syncthreads();
+  auto load = [](const E* p, float (&v)[V]) {
+    if constexpr (V == 1) {
+      v[0] = to_f(p[0]);
+    } else {
+      const bf16x8 a = *reinterpret_cast<const bf16x8*>(p);
+#pragma unroll
+      for (int q = 0; q < 4; ++q) {
+        const float2 f = __bfloat1622float2(a.v[q]);
+        v[2 * q] = f.x;
+        v[2 * q + 1] = f.y;
+      }
+    }
+  };
+  for (int i = threadIdx.x * V; i < H; i += blockDim.x * V) {
+    float acc[V], x[V];
+    float* r = res + (size_t)t * H + i;
+    if constexpr (V == 1) {
+      acc[0] = 0.f;
+    } else {
+#pragma unroll
+      for (int e = 0; e < V; ++e) acc[e] = 0.f;
+    }
+    for (int j = 0; j < top_k; ++j) {
+      if (s_pos[j] < 0) continue;
+      load(y + (size_t)s_pos[j] * ldy + i, x);
+#pragma unroll
+      for (int e = 0; e < V; ++e) acc[e] = fmaf(s_w[j], x[e], acc[e]);
+    }
+    if (shared != nullptr) {
+      load(shared + (size_t)t * H + i, x);
+#pragma unroll
+      for (int e = 0; e < V; ++e) acc[e] = fmaf(s_gate, x[e], acc[e]);
+    }
+    E* o = out + (size_t)t * H + i;
+    if constexpr (V == 1) {
+      acc[0] += r[0];
+      r[0] = acc[0];
+      if constexpr (sizeof(E) == 2) o[0] = __float2bfloat16(acc[0]);
+      else o[0] = acc[0];
+    } else {
+      float4 a = reinterpret_cast<float4*>(r)[0], b = reinterpret_cast<float4*>(r)[1];
+      a.x += acc[0]; a.y += acc[1]; a.z += acc[2]; a.w += acc[3];
+      b.x += acc[4]; b.y += acc[5]; b.z += acc[6]; b.w += acc[7];
+      reinterpret_cast<float4*>(r)[0] = a;
+      reinterpret_cast<float4*>(r)[1] = b;
+      bf16x8 c;
+      c.v[0] = __floats2bfloat162_rn(a.x, a.y); c.v[1] = __floats2bfloat162_rn(a.z, a.w);
+      c.v[2] = __floats2bfloat162_rn(b.x, b.y); c.v[3] = __floats2bfloat162_rn(b.z, b.w);
+      *reinterpret_cast<bf16x8*>(o) = c;
+    }
+  }
+}
+
 }  // namespace b200
 
 namespace b200 {
@@ -344,6 +414,34 @@ extern "C" int b200_moe_unpermute(const void* y, int ldy, const int* inv_pos, co
   else
     moe_unpermute_kernel<<<T, 128, 0, stream>>>((const __nv_bfloat16*)y, ldy, inv_pos, w, (__nv_bfloat16*)out, H,
                                                 top_k, rows_cap);
+  B200_CUDA_CHECK(cudaGetLastError());
+  return 0;
+}
+
+// shared (or null) [T, H] with the gate of token t at gate[t * ldg]; res [T, H] fp32 in place, out [T, H]; elem: 2 = bf16,
+// 4 = fp32.
+extern "C" int b200_moe_unpermute_add(const void* y, int ldy, const int* inv_pos, const float* w, const void* shared,
+                                      const float* gate, int ldg, float* res, void* out, int T, int H, int top_k,
+                                      int rows_cap, int elem, cudaStream_t stream) {
+  if (T == 0) return 0;
+  if (top_k > 32) {
+    b200_set_last_error("moe_unpermute_add: top_k <= 32 required", __FILE__, __LINE__);
+    return -1;
+  }
+  const uintptr_t a = (uintptr_t)y | (uintptr_t)shared | (uintptr_t)res | (uintptr_t)out;
+  int threads = (H / 8 + 31) / 32 * 32;
+  threads = threads < 64 ? 64 : (threads > 256 ? 256 : threads);
+  if (elem == 4)
+    moe_unpermute_add_kernel<float, 1><<<T, 128, 0, stream>>>((const float*)y, ldy, inv_pos, w, (const float*)shared, gate,
+                                                              ldg, res, (float*)out, H, top_k, rows_cap);
+  else if (H % 8 || ldy % 8 || a % 16)
+    moe_unpermute_add_kernel<__nv_bfloat16, 1><<<T, 128, 0, stream>>>(
+        (const __nv_bfloat16*)y, ldy, inv_pos, w, (const __nv_bfloat16*)shared, gate, ldg, res, (__nv_bfloat16*)out, H, top_k,
+        rows_cap);
+  else
+    moe_unpermute_add_kernel<__nv_bfloat16, 8><<<T, threads, 0, stream>>>(
+        (const __nv_bfloat16*)y, ldy, inv_pos, w, (const __nv_bfloat16*)shared, gate, ldg, res, (__nv_bfloat16*)out, H, top_k,
+        rows_cap);
   B200_CUDA_CHECK(cudaGetLastError());
   return 0;
 }

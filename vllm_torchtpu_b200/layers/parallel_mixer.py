@@ -17,17 +17,22 @@ import torch.nn.functional as F
 from .. import ops
 from ..config import ModelConfig
 from ..layer_specs import ParallelMixerSpec
+from ..parallel.state import get_state
 from .conv_attention import ConvAttention
 from .linear import RowParallelLinear
 from .linear_attention import RemovalDelta
+from .packed import ALIGN
 
 
 class JoinedRowLinear(RowParallelLinear):
-    """Output projections of several mixers as one: columns of (heads, size, padded size) each, side by side."""
+    """Output projections of several mixers as one: columns of (heads, size, padded size) each, side by side, and zero
+    columns up to a multiple of 8."""
 
     def __init__(self, name, sides: list, out_features: int, **kw):
         self.sides = sides
-        super().__init__(name, sum(h * padded for h, _, padded in sides), out_features, **kw)
+        tp = get_state().tp.size
+        width = sum(h * padded for h, _, padded in sides) // tp
+        super().__init__(name, (width + ALIGN - 1) // ALIGN * ALIGN * tp, out_features, **kw)
         self.full_in = sum(h * size for h, size, _ in sides)
 
     def shard_of(self, full_weight):
@@ -38,7 +43,8 @@ class JoinedRowLinear(RowParallelLinear):
             n = heads // self.tp_size
             w = F.pad(w[:, self.tp_rank * n:(self.tp_rank + 1) * n], (0, padded - size))
             out.append(w.reshape(full_weight.shape[0], n * padded))
-        return torch.cat(out, 1)
+        w = torch.cat(out, 1)
+        return F.pad(w, (0, self.in_features - w.shape[1]))
 
 
 class ParallelMixer:

@@ -110,7 +110,7 @@ class LlamaMLP:
 
     def forward(self, x):
         gu = self.gate_up
-        if self.act == "gelu_tanh" and gu.bias is None and not gu.lora_targets \
+        if self.act.split(":")[0] in ("gelu_tanh", "swigluoai") and gu.bias is None and not gu.lora_targets \
                 and type(gu.method) is UnquantizedLinearMethod:
             return self.down(ops.gemm_gated(x, gu.weight, self.act))
         if self.act != "silu":

@@ -275,6 +275,66 @@ def add_rms_norm(y, residual, weight, eps, offset: float = 0.0, update: bool = T
     return h, r
 
 
+def add_rms_norm_shift(y, residual, weight, eps, offset, shift, state, meta, post=None, mult: float = 1.0,
+                       keep: bool = False):
+    """See ``ops.token_shift.add_rms_norm_shift``; the sum goes to a buffer of its own."""
+    T, H = residual.shape
+    assert residual.is_contiguous() and (y is None or y.dtype == weight.dtype) and shift.dtype == weight.dtype
+    assert state.dtype == torch.float32 and state.is_contiguous() and state.shape[1] == H
+    assert post is None or post.dtype == weight.dtype
+    y = y.contiguous() if y is not None else None
+    new = lambda dtype: torch.empty((T, H), dtype=dtype, device=residual.device)       # noqa: E731
+    r, h, rows = new(torch.float32), new(weight.dtype), new(torch.float32) if keep else None
+    R = meta.padded_num_reqs if meta.padded_num_reqs is not None else meta.num_reqs
+    _check(lib().b200_norm_shift(
+        _p(y), _p(residual), c_int(_mixed(residual)), _p(weight), _p(post), _p(shift), c_int(_mixed(weight)), _p(r),
+        _p(state), _p(rows), _p(h), _p(meta.query_start_loc), _p(meta.seq_lens), _p(meta.state_slots), c_int(T), c_int(H),
+        c_int(R), c_float(eps), c_float(offset), c_float(mult), c_int(int(meta.num_decode_reqs == meta.num_reqs)),
+        _stream()), "norm_shift")
+    count_launch()
+    return h, r, rows
+
+
+def residual_add(y, residual, mult: float = 1.0, dtype=None):
+    """See ``ops.reference.residual_add``; an fp32 residual is updated in place."""
+    assert y.is_contiguous() and residual.is_contiguous() and residual.dtype == torch.float32
+    assert dtype is None or dtype == y.dtype
+    out = torch.empty_like(y)
+    _check(lib().b200_residual_add(_p(y), _p(residual), _p(residual), _p(out), c_longlong(y.numel()), c_float(mult),
+                                   c_int(_mixed(y)), _stream()), "residual_add")
+    count_launch()
+    return out, residual
+
+
+def add_gated(y, z, gate):
+    """y + sigmoid(gate)[:, None] * z."""
+    T, H = y.shape
+    assert y.is_contiguous() and z.is_contiguous() and z.dtype == y.dtype and gate.dtype == torch.float32
+    out = torch.empty_like(y)
+    _check(lib().b200_add_gated(_p(y), _p(z), _p(gate), c_int(gate.stride(0)), _p(out), c_int(T), c_int(H), c_int(_mixed(y)),
+                                _stream()), "add_gated")
+    count_launch()
+    return out
+
+
+def tanh_(x):
+    """In place over the columns of (strided) rows."""
+    assert x.dim() == 2 and x.stride(1) == 1
+    _check(lib().b200_tanh_columns(_p(x), c_int(x.stride(0)), c_int(x.shape[0]), c_int(x.shape[1]), c_int(_mixed(x)),
+                                   _stream()), "tanh_columns")
+    count_launch()
+    return x
+
+
+def resolve_tokens(ids, token_src, last_tokens):
+    out = torch.empty_like(ids)
+    assert ids.dtype == token_src.dtype == last_tokens.dtype == torch.int32
+    _check(lib().b200_resolve_tokens(_p(ids), _p(token_src), _p(last_tokens), _p(out), c_int(ids.numel()), _stream()),
+           "resolve_tokens")
+    count_launch()
+    return out
+
+
 def softcap(x, cap: float):
     """cap * tanh(x / cap) in fp32 (in place when x is fp32)."""
     x = x.contiguous()
@@ -379,12 +439,14 @@ def _tma_ready(t, stride: int) -> bool:
     return t.dtype == torch.bfloat16 and stride % 8 == 0 and t.data_ptr() % 16 == 0
 
 
-def gemm_simt(x, w, y, T, N, K, ldx, ldy, *, bias=None, gate=None, ldg=0, batch=1, xs=0, ys=0, act=0, cap=0.0, scale=1.0):
+def gemm_simt(x, w, y, T, N, K, ldx, ldy, *, bias=None, gate=None, ldg=0, batch=1, xs=0, ys=0, act=0, cap=0.0, scale=1.0,
+              gate_rows=None):
     """CUDA-core GEMM (``csrc/gemm_simt.cu``): fp32 operands, or bf16 ones without the TMA's alignment."""
     elem = _mixed(x)
     assert all(t is None or t.dtype == x.dtype for t in (w, bias, gate)), "operands of one dtype"
     assert y.dtype == (torch.float32 if act == 2 else x.dtype)
-    _check(lib().b200_gemm_simt(_p(x), _p(w), _p(y), _p(bias), _p(gate), c_int(T), c_int(N), c_int(K), c_int(batch),
+    _check(lib().b200_gemm_simt(_p(x), _p(w), _p(y), _p(bias), _p(gate), _p(gate_rows),
+                                c_int(gate.shape[0] if gate_rows is not None else 0), c_int(T), c_int(N), c_int(K), c_int(batch),
                                 c_longlong(ldx), c_longlong(K), c_longlong(ldy), c_longlong(ldg), c_longlong(xs),
                                 c_longlong(ys), c_int(act), c_float(cap), c_float(scale), c_int(elem), _stream()), "gemm_simt")
     count_launch()
@@ -416,12 +478,30 @@ def gemm_gelu(x, w):
 
 
 def gemm_gated(x, w, act: str):
-    """act(x @ w[:I].T) * (x @ w[I:].T), w [2I, K]: in the GEMM's epilogue for bf16 silu and gelu_tanh."""
-    if act in ("silu", "gelu_tanh") and x.shape[-1] % 8 == 0 and _tma_ready(x, x.stride(-2)) and _tma_ready(w, w.shape[1]):
-        from .cuda_moe import gemm_swiglu
-        return gemm_swiglu(x, w, gelu_tanh=act == "gelu_tanh")
+    """act(x @ w[:I].T, x @ w[I:].T), w [2I, K]: in the GEMM's epilogue for bf16 and the activations it has."""
+    from .cuda_moe import fused_act, gemm_swiglu
+    if fused_act(act) is not None and x.shape[-1] % 8 == 0 and _tma_ready(x, x.stride(-2)) and _tma_ready(w, w.shape[1]):
+        return gemm_swiglu(x, w, act=act)
     h = gemm(x, w)
     return gated_act_and_mul(h.reshape(-1, h.shape[-1]), act).reshape(*x.shape[:-1], w.shape[0] // 2)
+
+
+def gemm_token_gate(x, w, table, first: int, ids):
+    """See ``ops.reference.gemm_token_gate``."""
+    (T, K), N = x.shape, w.shape[0]
+    assert table.dtype == x.dtype == w.dtype and table.stride(1) == 1 and ids.dtype == torch.int32
+    gate = table[:, first:first + N]
+    y = torch.empty((T, N), dtype=x.dtype, device=x.device)
+    if T == 0:
+        return y
+    if not (_tma_ready(x, x.stride(0)) and _tma_ready(w, K)):
+        return gemm_simt(x, w, y, T, N, K, x.stride(0), N, gate=gate, ldg=table.stride(0), gate_rows=ids)
+    ws = Workspace.get(x.device)
+    _check(lib().b200_gemm_bf16_token_gate(
+        _p(x), _p(w), _p(y), _p(gate), c_int(table.stride(0)), c_int(table.shape[0]), _p(ids), c_int(T), c_int(N), c_int(K),
+        c_int(x.stride(0)), c_int(K), c_int(N), _p(ws.status), c_int(_sms), _stream()), "gemm_token_gate")
+    count_launch()
+    return y
 
 
 def gemm_softcap(x, w, cap: float = 0.0, scale: float = 1.0):
@@ -529,12 +609,12 @@ def decode_splits(num_reqs: int, num_kv_heads: int) -> int:
 
 
 def paged_attention(q, kv_cache, meta, scale, *, sliding_window=None, softcap=None, sinks=None,
-                    k_scale=1.0, v_scale=1.0, return_lse=False):
-    """Ragged paged attention over [decode | prefill/mixed] request ranges of the batch."""
+                    k_scale=1.0, v_scale=1.0, return_lse=False, out=None):
+    """Ragged paged attention over [decode | prefill/mixed] request ranges of the batch; see ``ops.paged_attention``."""
     if kv_cache.dtype == q.dtype and (q.dtype == torch.float32 or q.shape[2] not in (64, 128)):
         if return_lse or meta.dcp_size > 1:
             raise NotImplementedError("log-sum-exp and position-sharded caches: bf16, heads of 64 or 128")
-        return attention_simt(q, kv_cache, meta, scale, sliding_window, softcap, sinks)
+        return attention_simt(q, kv_cache, meta, scale, sliding_window, softcap, sinks, out)
     _require_bf16(q)
     # an e4m3 cache is expanded to bf16 in shared memory by the mma.sync kernels; k_scale joins the
     # logit scale and v_scale the output normalisation (reference: layers/adapter/quantization.py:91)
@@ -544,7 +624,12 @@ def paged_attention(q, kv_cache, meta, scale, *, sliding_window=None, softcap=No
     T, Hq, D = q.shape
     nb, _, Hkv, bs, _ = kv_cache.shape
     ws = Workspace.get(q.device)
-    if return_lse:
+    ldo = 0
+    if out is not None:
+        if return_lse or kv_fp8 or meta.dcp_size > 1:
+            raise NotImplementedError("output rows of the caller: bf16 cache, no log-sum-exp")
+        ldo, lse = _out_rows(q, out), None
+    elif return_lse:
         # callers that merge partial results keep several outputs alive: fresh, fully defined tensors
         out = torch.zeros_like(q)
         lse = torch.full((T, Hq), float("-inf"), dtype=torch.float32, device=q.device)
@@ -575,7 +660,7 @@ def paged_attention(q, kv_cache, meta, scale, *, sliding_window=None, softcap=No
             _check(L.b200_attn_decode_fp8kv(*args, c_float(k_scale), c_float(v_scale), _stream()),
                    "attn_decode_fp8kv")
         else:
-            _check(L.b200_attn_decode(*args, _stream()), "attn_decode")
+            _check(L.b200_attn_decode(*args, c_int(ldo), _stream()), "attn_decode")
         count_launch()
     else:
         nd = 0
@@ -602,7 +687,7 @@ def paged_attention(q, kv_cache, meta, scale, *, sliding_window=None, softcap=No
                 _p(q), _p(kv_cache), _p(out), _p(lse), _p(meta.block_tables), _p(meta.seq_lens),
                 _p(meta.query_start_loc), c_int(nd), c_int(R), c_int(tiles), c_int(T), c_int(max_blocks),
                 c_int(bs), c_longlong(nb), c_int(Hq), c_int(Hkv), c_int(D), c_float(scale), c_int(window),
-                c_float(cap), _p(sinks), _p(ws.status), _stream()), "attn_prefill_tc")
+                c_float(cap), _p(sinks), c_int(ldo), _p(ws.status), _stream()), "attn_prefill_tc")
         else:
             args = (_p(q), _p(kv_cache), _p(out), _p(lse), _p(meta.block_tables), _p(meta.seq_lens),
                     _p(meta.query_start_loc), c_int(nd), c_int(R), c_int(tiles), c_int(max_blocks), c_int(bs),
@@ -612,25 +697,36 @@ def paged_attention(q, kv_cache, meta, scale, *, sliding_window=None, softcap=No
                 _check(L.b200_attn_prefill_fp8kv(*args, c_float(k_scale), c_float(v_scale), _stream()),
                        "attn_prefill_fp8kv")
             else:
-                _check(L.b200_attn_prefill(*args, _stream()), "attn_prefill")
+                _check(L.b200_attn_prefill(*args, c_int(ldo), _stream()), "attn_prefill")
         count_launch()
     if return_lse:
         return out, lse
     return out
 
 
-def attention_simt(q, kv_cache, meta, scale, sliding_window=None, softcap=None, sinks=None):
+def _out_rows(q, out) -> int:
+    """Distance of output rows that hold the heads of q side by side."""
+    T, Hq, D = q.shape
+    if out.shape[0] != T or out.shape[1] < Hq * D or out.stride(1) != 1 or out.dtype != q.dtype:
+        raise ValueError("output rows do not fit the queries")
+    if q.dtype == torch.bfloat16 and (out.stride(0) % 8 or out.data_ptr() % 16):
+        raise ValueError("output rows must begin on 16 bytes")
+    return out.stride(0)
+
+
+def attention_simt(q, kv_cache, meta, scale, sliding_window=None, softcap=None, sinks=None, out=None):
     """Paged attention on the CUDA cores (``csrc/attention_simt.cu``): fp32, or head sizes the tensor-core kernels are
     not built for."""
     T, Hq, D = q.shape
     nb, _, Hkv, bs, _ = kv_cache.shape
     R = meta.padded_num_reqs if meta.padded_num_reqs is not None else meta.num_reqs
-    out = torch.empty_like(q)
+    ldo = _out_rows(q, out) if out is not None else 0
+    out = torch.empty_like(q) if out is None else out
     _check(lib().b200_attn_simt(
         _p(q), _p(kv_cache), _p(out), _p(meta.block_tables), _p(meta.seq_lens), _p(meta.query_start_loc), c_int(T),
         c_int(R), c_int(Hq), c_int(Hkv), c_int(D), c_int(meta.block_tables.shape[1]), c_int(bs), c_longlong(nb),
-        c_float(scale), c_int(int(sliding_window or 0)), c_float(float(softcap or 0.0)), _p(sinks), c_int(_mixed(q)),
-        _stream()), "attn_simt")
+        c_float(scale), c_int(int(sliding_window or 0)), c_float(float(softcap or 0.0)), _p(sinks), c_int(ldo),
+        c_int(_mixed(q)), _stream()), "attn_simt")
     count_launch()
     return out
 
@@ -959,7 +1055,7 @@ def p2p_all_reduce(x, heap):
 # Kernels of the sub-modules under this module's name (``cuda.moe_experts`` ...), resolved on first use: the
 # sub-modules import this module, so importing them here would make ``import ops.cuda_fp4`` depend on who came first.
 _SUBMODULE_EXPORTS = {
-    "cuda_moe": ("EpState", "gemm_swiglu", "group_bias_add", "grouped_gemm", "moe_experts", "moe_experts_ep",
+    "cuda_moe": ("EpState", "gemm_swiglu", "group_bias_add", "grouped_gemm", "moe_experts", "moe_experts_ep", "moe_unpermute_add",
                  "moe_route_post", "moe_permute", "moe_route", "moe_unpermute"),
     "cuda_fp8": ("fp8_block_gemm", "fp8_block_gemm_push", "fp8_block_gemm_push_quantised", "fp8_block_gemm_quantised",
                  "fp8_per_tensor_gemm", "fp8_rowwise_gemm", "grouped_fp8_gemm", "int8_gemm", "moe_experts_ep_fp8",

@@ -16,7 +16,7 @@ def _call(p, row, q, kv_cache, ring, meta, R, ring_from, single, only_ring):
     inv = p.inv_freq
     _c._check(_c.lib().b200_conv_cache(
         _c._p(row), c_int(row.stride(0)), *(c_int(o) for o in p.offsets), _c._p(p.conv_w), c_int(p.taps), _c._p(ring),
-        _c._p(inv), c_int(inv.numel() if inv is not None else 0), c_float(p.rot_mult), _c._p(q),
+        _c._p(inv), c_int(inv.numel() if inv is not None else 0), c_float(p.rot_mult), _c._p(p.q_scale), _c._p(q),
         _c._p(kv_cache) if p.kv_heads else c_void_p(0), _c._p(meta.slot_mapping), _c._p(meta.query_start_loc),
         _c._p(meta.seq_lens), _c._p(meta.state_slots), c_int(row.shape[0]), c_int(R), c_int(p.heads), c_int(p.kv_heads),
         c_int(p.dim), c_int(p.vdim), c_int(p.maps), c_int(p.width), c_int(bs), c_longlong(nb), c_int(ring_from),

@@ -7,6 +7,7 @@ import torch
 
 from . import count_launch
 from . import cuda as _c
+from .linear_attention import RULES
 
 STEP, CHUNKS, RING, SCAN, FINISH = 0, 1, 2, 3, 4
 CHUNK = 16
@@ -38,8 +39,9 @@ def _side_stream(device):
     return _side[i]
 
 
-def carried_state_attention(plan, row, decay_in, gate, meta, cache):
-    """See ``ops.linear_attention``: rows [T, ...] of the packed projection -> y [T, heads * vdim]."""
+def carried_state_attention(plan, row, decay_in, gate, meta, cache, out=None):
+    """See ``ops.linear_attention``: rows [T, ...] of the packed projection -> y [T, heads * vdim] (``out``, whose rows may
+    be strided; rows that belong to no request are left as they are in a step with prompts)."""
     elem = _c._mixed(row)
     p = plan
     T = row.shape[0]
@@ -54,17 +56,20 @@ def carried_state_attention(plan, row, decay_in, gate, meta, cache):
         qsl = meta.query_start_loc_cpu if meta.query_start_loc_cpu is not None else meta.query_start_loc.cpu()
         lens = (qsl[nd + 1:R + 1] - qsl[nd:R]).tolist()
     whole = decode_only or int(qsl[R]) == T                   # every row belongs to a request
-    y = (torch.empty if whole else torch.zeros)((T, p.heads * p.vdim), dtype=row.dtype, device=row.device)
+    y = out if out is not None else (torch.empty if whole else torch.zeros)((T, p.heads * p.vdim), dtype=row.dtype,
+                                                                            device=row.device)
+    assert y.stride(1) == 1 and y.dtype == row.dtype and y.shape[0] == T and y.shape[1] >= p.heads * p.vdim
+    rule = RULES.index(p.rule)
     L = _c.lib()
 
     def call(mode, lo, hi, scratch=None, chunk=0, slab=0, stream=None):
         _c._check(L.b200_linear_attention(
-            c_int(mode), _c._p(row), c_int(row.stride(0)), *(c_int(o) for o in p.offsets), c_int(p.beta_offset),
-            _c._p(decay_in), c_int(decay_in.stride(0) if decay_in is not None else 0), _c._p(gate),
+            c_int(mode), c_int(rule), _c._p(row), c_int(row.stride(0)), *(c_int(o) for o in p.offsets),
+            c_int(p.beta_offset), c_int(p.rate_offset), _c._p(decay_in), c_int(decay_in.stride(0) if decay_in is not None else 0), _c._p(gate),
             c_int(gate.stride(0)), _c._p(p.conv_w), _c._p(ring), c_int(p.taps), _c._p(p.inv_freq),
             c_int(p.inv_freq.numel() if p.inv_freq is not None else 0), _c._p(p.decay), _c._p(p.A_log),
-            _c._p(p.dt_bias), _c._p(p.norm_w), _c._p(state), _c._p(y), _c._p(meta.query_start_loc),
-            _c._p(meta.seq_lens), _c._p(meta.state_slots), c_int(lo), c_int(hi), c_int(T), c_int(p.heads),
+            _c._p(p.dt_bias), _c._p(p.rate_bias), c_float(p.tau), _c._p(p.norm_w), c_int(p.norm_stride), _c._p(state),
+            _c._p(y), c_int(y.stride(0)), _c._p(meta.query_start_loc), _c._p(meta.seq_lens), _c._p(meta.state_slots), c_int(lo), c_int(hi), c_int(T), c_int(p.heads),
             c_int(p.k_heads), c_int(p.dim), c_int(p.vdim), c_int(int(p.unit_norm)), c_int(int(p.gate_act == "silu")),
             c_float(p.eps), c_float(p.q_mult), c_float(p.k_mult), c_int(int(decode_only)), _c._p(scratch),
             c_int(chunk), c_int(slab), c_int(elem),
@@ -75,7 +80,7 @@ def carried_state_attention(plan, row, decay_in, gate, meta, cache):
         call(STEP, 0, n_dec)
     if lens:
         if elem == 2 and p.dim <= 256 and p.taps <= 8:
-            per = int(L.b200_linear_attention_chunk_bytes(c_int(p.dim), c_int(p.vdim), c_int(int(p.delta))))
+            per = int(L.b200_linear_attention_chunk_bytes(c_int(p.dim), c_int(p.vdim), c_int(rule)))
             parts = slabs(lens, p.heads, per)
             room = max((j - i) * n for i, j, _, n in parts) * p.heads * per
             scratch = torch.empty((min(2, len(parts)), room), dtype=torch.uint8, device=row.device)

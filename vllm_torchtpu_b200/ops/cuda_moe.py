@@ -8,11 +8,19 @@ import torch
 from .. import envs
 from . import count_launch
 from . import cuda as _c
-from .reference import UNGATED_ACTS
+from .reference import UNGATED_ACTS, parse_gated_act
 
 
-def gemm_swiglu(x, w, out=None, gelu_tanh: bool = False):
-    """silu(x @ w[:I].T) * (x @ w[I:].T) in one tcgen05 kernel; w is [2I, K].  ``gelu_tanh``: that activation instead."""
+def fused_act(act: str):
+    """(code, alpha, limit) of a gated activation that the GEMMs' epilogues have (``gated_pair``), None for others."""
+    name, a, b = parse_gated_act(act)
+    code = {0: 0, 2: 3, 3: 5}.get(name)
+    return None if code is None else (code, a, b)
+
+
+def gemm_swiglu(x, w, out=None, act: str = "silu"):
+    """act(x @ w[:I].T, x @ w[I:].T) in one tcgen05 kernel; w is [2I, K]; act: one of ``fused_act``."""
+    code, alpha, limit = fused_act(act)
     _c._require_bf16(x, w)
     if x.stride(-1) != 1:
         x = x.contiguous()
@@ -26,21 +34,23 @@ def gemm_swiglu(x, w, out=None, gelu_tanh: bool = False):
     if 0 < envs.B200_GEMM_2SM_MIN_T <= T:
         _c._check(_c.lib().b200_gemm_bf16_swiglu_2sm(
             _c._p(x2), _c._p(w), _c._p(y), c_int(T), c_int(I), c_int(K), c_int(x2.stride(0)), c_int(w.stride(0)),
-            c_int(y.stride(0)), c_int(gelu_tanh), _c._p(ws.status), c_int(_c._sms), _c._stream()), "gemm_swiglu_2sm")
+            c_int(y.stride(0)), c_int(code), c_float(alpha), c_float(limit), _c._p(ws.status), c_int(_c._sms),
+            _c._stream()), "gemm_swiglu_2sm")
         count_launch()
         return y
     _c._check(_c.lib().b200_gemm_bf16_swiglu(
         _c._p(x2), _c._p(w), _c._p(y), c_int(T), c_int(I), c_int(K), c_int(x2.stride(0)), c_int(w.stride(0)),
-        c_int(y.stride(0)), c_int(gelu_tanh), _c._p(ws.status), c_int(_c._sms), _c._stream()), "gemm_swiglu")
+        c_int(y.stride(0)), c_int(code), c_float(alpha), c_float(limit), _c._p(ws.status), c_int(_c._sms), _c._stream()),
+        "gemm_swiglu")
     count_launch()
     return y
 
 
 def grouped_gemm(x_perm, w, group_off, swiglu: bool, avg_rows: int, out=None, act: str = ""):
-    """Rows [group_off[e], group_off[e+1]) of x_perm times w[e] ([N,K] or [2N,K] when swiglu); ``act`` (without swiglu)
-    "relu2": the square of relu in the epilogue.  32-bit operands, and sizes a tensor map cannot describe, run on the
-    CUDA cores."""
-    code = {"": 0, "relu2": 4}[act]
+    """Rows [group_off[e], group_off[e+1]) of x_perm times w[e] ([N,K] or [2N,K] when swiglu); ``act`` in the epilogue:
+    with swiglu one of ``fused_act``, without it "relu2", the square of relu.  32-bit operands, and sizes a tensor map
+    cannot describe, run on the CUDA cores (without swiglu)."""
+    code, alpha, limit = fused_act(act or "silu") if swiglu else ({"": 0, "relu2": 4}[act], 0.0, 0.0)
     if not swiglu and (x_perm.dtype == torch.float32 or x_perm.shape[1] % 8 or w.shape[1] % 128):
         assert x_perm.is_contiguous() and w.is_contiguous() and x_perm.dtype == w.dtype and out is None
         y = torch.empty((x_perm.shape[0], w.shape[1]), dtype=x_perm.dtype, device=x_perm.device)
@@ -59,8 +69,8 @@ def grouped_gemm(x_perm, w, group_off, swiglu: bool, avg_rows: int, out=None, ac
     ws = _c.Workspace.get(x_perm.device)
     _c._check(_c.lib().b200_grouped_gemm_bf16(
         _c._p(x_perm), _c._p(w), _c._p(y), _c._p(group_off), c_int(E), c_int(R), c_int(N), c_int(K),
-        c_int(1 if swiglu else 0), c_int(code), c_int(max(1, avg_rows)), _c._p(ws.status), c_int(_c._sms), _c._stream()),
-        "grouped_gemm")
+        c_int(1 if swiglu else 0), c_int(code), c_float(alpha), c_float(limit), c_int(max(1, avg_rows)), _c._p(ws.status),
+        c_int(_c._sms), _c._stream()), "grouped_gemm")
     count_launch()
     return y
 
@@ -129,16 +139,37 @@ def group_bias_add(y, bias, group_off):
     return y
 
 
-def moe_experts(x, w13, w2, topk_ids, topk_w, expert_offset: int = 0, act: str = "silu", b13=None, b2=None):
+def moe_unpermute_add(y, inv_pos, topk_w, shared, residual):
+    """In place on the fp32 ``residual`` [T, H]: plus the weighted sums of the rows of y, plus the shared expert's output
+    times the sigmoid of its gate (``shared`` = (output, gate column fp32) or None).  Returns (rounded, fp32)."""
+    T, H = residual.shape
+    sh, gate = shared if shared is not None else (None, None)
+    assert residual.is_contiguous() and residual.dtype == torch.float32
+    assert sh is None or (sh.is_contiguous() and sh.dtype == y.dtype and gate.dtype == torch.float32)
+    out = torch.empty((T, H), dtype=y.dtype, device=y.device)
+    _c._check(_c.lib().b200_moe_unpermute_add(
+        _c._p(y), c_int(y.stride(0)), _c._p(inv_pos), _c._p(topk_w), _c._p(sh), _c._p(gate),
+        c_int(gate.stride(0) if gate is not None else 0), _c._p(residual), _c._p(out), c_int(T), c_int(H),
+        c_int(topk_w.shape[1]), c_int(y.shape[0]), c_int(_c._mixed(y)), _c._stream()), "moe_unpermute_add")
+    count_launch()
+    return out, residual
+
+
+def moe_experts(x, w13, w2, topk_ids, topk_w, expert_offset: int = 0, act: str = "silu", b13=None, b2=None, shared=None,
+                residual=None):
     """Σ_k w_k · FFN_e(x) over the local experts: permute → grouped SwiGLU GEMM → grouped GEMM →
-    weighted un-permute.  w13: [E_local, 2I, H] (gate rows first), w2: [E_local, H, I]."""
+    weighted un-permute.  w13: [E_local, 2I, H] (gate rows first), w2: [E_local, H, I].  With ``residual`` the last step is
+    ``moe_unpermute_add``."""
     T, H = x.shape
     E_local = w13.shape[0]
     k = topk_ids.shape[1]
     x_perm, group_off, _, inv_pos = moe_permute(x.contiguous(), topk_ids.contiguous(), expert_offset, E_local)
     avg = (T * k + E_local - 1) // E_local
-    if act == "silu" and b13 is None:
+    fused = act not in UNGATED_ACTS and b13 is None and fused_act(act) is not None
+    if act == "silu" and b13 is None and residual is None:
         h = grouped_gemm(x_perm, w13, group_off, True, avg)          # SiLU * mul in the GEMM epilogue
+    elif fused and x.dtype == torch.bfloat16 and H % 8 == 0 and w13.shape[1] % 256 == 0:
+        h = grouped_gemm(x_perm, w13, group_off, True, avg, act=act)
     elif act in UNGATED_ACTS:
         h = grouped_gemm(x_perm, w13, group_off, False, avg, act=act)
     else:
@@ -151,6 +182,8 @@ def moe_experts(x, w13, w2, topk_ids, topk_w, expert_offset: int = 0, act: str =
     y = grouped_gemm(h, w2, group_off, False, avg)
     if b2 is not None:
         group_bias_add(y, b2, group_off)
+    if residual is not None:
+        return moe_unpermute_add(y, inv_pos, topk_w.contiguous(), shared, residual)
     return moe_unpermute(y, inv_pos, topk_w.contiguous(), T, H)      # (y: down projection padded to the tile width)
 
 
