@@ -104,9 +104,9 @@ class ParallelMixer:
         """y / ``mult``."""
         ring, pages, state = cache
         row = self.inp(x)
-        n, k = self.left.Hq * self.left.D, self.o.in_features
-        z = ops.mixer_rows(x, k)
+        n, m = self.left.Hq * self.left.D, self.right.H * self.right.spec.dim
+        z = ops.mixer_rows(x, self.o.in_features)
         q = self.left.queries(row, (ring, pages), meta)
         self.left.attend(q, row, pages, meta, out=z[:, :n])
-        self.right.advance((row, self.right.decays(row)), (state,), meta, out=z[:, n:])
+        self.right.advance((row, self.right.decays(row)), (state,), meta, out=z[:, n:n + m])
         return self.o(z)

@@ -108,8 +108,13 @@ class UnquantizedMoEMethod:
         w13 = []
         w2 = []
         for e in range(lo, hi):
-            w13.append(seeded_normal(f"{moe.name}.experts.{e}.w13", (2 * I, H), std, moe.dtype, moe.device, seed))
-            w2.append(seeded_normal(f"{moe.name}.experts.{e}.w2", (H, I), std, moe.dtype, moe.device, seed))
+            # drawn in full, so that every rank holds its part of the same expert
+            full = I * moe.tp_size
+            up = seeded_normal(f"{moe.name}.experts.{e}.w13", (2 * full, H), std, moe.dtype, moe.device, seed)
+            down = seeded_normal(f"{moe.name}.experts.{e}.w2", (H, full), std, moe.dtype, moe.device, seed)
+            gate, up, down = expert_tp_shard(moe, up[:full], up[full:], down)
+            w13.append(torch.cat([gate, up]))
+            w2.append(down)
         moe.w13 = torch.stack(w13).contiguous()
         moe.w2 = torch.stack(w2).contiguous()
         if padded_hidden(moe) != H:
