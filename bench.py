@@ -72,7 +72,7 @@ def parse_args():
     ap.add_argument("--enforce-eager", action="store_true")
     ap.add_argument("--warmup-requests", type=int, default=0,
                     help="requests per warm-up serve (0 = the full workload)")
-    ap.add_argument("--layer-bench", default="", choices=["", "mazivik", "popanex", "zeganex"],
+    ap.add_argument("--layer-bench", default="", choices=["", "mazivik", "popanex", "zeganex", "vipolix"],
                     help="instead of the serving workload: layer throughput and kernels of this model beside its "
                          "closest neighbour, one JSON line per measurement")
     ap.add_argument("--layer-size", default="2048x16,4096x32,7168x128", help="--layer-bench: width x heads, ...")
@@ -174,7 +174,8 @@ def main():
         return 0
     if args.layer_bench:
         from importlib import import_module
-        module = {"mazivik": "bench_latent", "popanex": "bench_linear", "zeganex": "bench_window"}[args.layer_bench]
+        module = {"mazivik": "bench_latent", "popanex": "bench_linear", "zeganex": "bench_window",
+                  "vipolix": "bench_parallel"}[args.layer_bench]
         run = import_module(f"vllm_torchtpu_b200.ops.{module}").run
         for row in run(args.layer_size, args.layer_parts):
             print(json.dumps(row))

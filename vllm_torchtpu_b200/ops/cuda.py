@@ -628,7 +628,7 @@ def paged_attention(q, kv_cache, meta, scale, *, sliding_window=None, softcap=No
     if out is not None:
         if return_lse or kv_fp8 or meta.dcp_size > 1:
             raise NotImplementedError("output rows of the caller: bf16 cache, no log-sum-exp")
-        ldo, lse = _out_rows(q, out), None
+        ldo, lse = _out_rows(q, out, True), None
     elif return_lse:
         # callers that merge partial results keep several outputs alive: fresh, fully defined tensors
         out = torch.zeros_like(q)
@@ -704,12 +704,12 @@ def paged_attention(q, kv_cache, meta, scale, *, sliding_window=None, softcap=No
     return out
 
 
-def _out_rows(q, out) -> int:
+def _out_rows(q, out, tensor_cores: bool = False) -> int:
     """Distance of output rows that hold the heads of q side by side."""
     T, Hq, D = q.shape
     if out.shape[0] != T or out.shape[1] < Hq * D or out.stride(1) != 1 or out.dtype != q.dtype:
         raise ValueError("output rows do not fit the queries")
-    if q.dtype == torch.bfloat16 and (out.stride(0) % 8 or out.data_ptr() % 16):
+    if tensor_cores and (out.stride(0) % 8 or out.data_ptr() % 16):
         raise ValueError("output rows must begin on 16 bytes")
     return out.stride(0)
 
