@@ -551,7 +551,7 @@ def test_mixed_batches_reused_pages_and_slots_match_each_request_alone(tmp_path,
 def test_far_keys_chunk_edges_states_sinks_and_shifts_decide_logits(tmp_path, dev):
     """Each mistake that is planted in the plain model moves its logits far; the engine stays with the unspoilt model, in
     prompts, in portions and in decoding."""
-    cfg = config([(par(chunk=120, conv=4, scale=0.6), moe()), (gla(tau=30.0), None),
+    cfg = config([(par(chunk=110, conv=4, scale=0.6), moe()), (gla(tau=30.0), None),
                   (par(chunk=41, scale=0.6, conv=2, ls=0.5, rs=0.6), None)])
     w = write_model(str(tmp_path), cfg, seed=2)
     toks = tokens_of(130, cfg["vocab"], 3)
@@ -559,7 +559,7 @@ def test_far_keys_chunk_edges_states_sinks_and_shifts_decide_logits(tmp_path, de
     rep = make_replay(str(tmp_path), "float32", 192, dev)
     for cuts in ([97, 2] + [1] * 31, portions(130, [2, 5]), [130], portions(130, [33, 37, 1])):
         assert logit_error(replay_logits(rep, toks, cuts), want) < LIMIT["float32"] * 5, cuts
-    left = [{"lost_key": k} for k in (0, 1, 15, 16, 31, 32, 63, 64, 96, 97)] + [{"edge": 1}, {"edge": 119}]
+    left = [{"lost_key": k} for k in (0, 1, 15, 16, 31, 32, 63, 64, 96, 97)] + [{"edge": 1}, {"edge": 109}]
     left += [{"no_sink": True}, {"no_temp": True}] + [{"conv_cut": p} for p in (1, 16, 97, 99, 100)]
     plants = [{0: {"left": x}} for x in left] + [{2: {"left": {"edge": e}}} for e in (1, 40)]
     plants += [{i: {"right": x}} for i in (0, 2) for x in ({"no_removal": True}, {"forget_at": 1}, {"forget_at": 97}, {"forget_at": 120})]

@@ -32,7 +32,7 @@ def vipolix_config(width: int, heads: int, kind: str, layers: int = 4) -> ModelC
                           "right_scale": 0.7},
              "gla": {"heads": heads, "dim": D, "vdim": D, "tau": 16.0, "decay_rank": RANK}}[kind]
     mlp = {"kind": "moe", "expert": {"ff": FF, "limit": 7.0}, "shared": {"ff": FF, "limit": 7.0},
-           "router": {"experts": EXPERTS, "top": TOP, "scale": 1.5, "groups": {"count": 8, "keep": 4}}}
+           "router": {"experts": EXPERTS, "top": TOP, "scale": 2.0, "groups": {"count": 8, "keep": 4}}}
     return ModelConfig.from_layer_list({
         "architecture": "Vipolix", "width": width, "vocab": 1024, "norm": {"eps": 1e-6}, "token_side": {"dim": SIDE},
         "layers": [{"type": kind, "mixer": mixer, "mlp": mlp}] * layers}, "vipolix-bench")
